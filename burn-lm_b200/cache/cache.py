@@ -6,7 +6,7 @@ many pages as its length needs, listed in its row of the block table, so `max_to
 over live sequences of their lengths rounded up to 64, whatever their number.  Runs of the schedule
 whose mixers need the same thing (all keys of n heads of size d; a window; a state of some shape)
 form a group with storage, page allocator and block table of its own.  A group whose mixers look
-back over a window only gives a sequence's pages back as soon as every key in them lies before the
+back over a window, or to the start of a chunk, only gives a sequence's pages back as soon as every key in them lies before the
 window of every token still to come, so a long sequence holds about window / 64 + 2 of its pages.
 Pages and slots are given back when a sequence ends and are used again without being cleared: a
 kernel never reads a position at or beyond a sequence's length, nor one before the window.  State
@@ -57,7 +57,7 @@ class _KVGroup:
             self.pool = torch.empty((len(runs), n_pages, need.n_kv_heads * PAGE * (need.head_dim + need.value_dim)),
                                     dtype=dtype, device=device)
         # leading pages that hold some of the first `keep_first` positions: a windowed group never gives them back
-        self.kept_pages = (need.keep_first + PAGE - 1) // PAGE if need.window else 0
+        self.kept_pages = (need.keep_first + PAGE - 1) // PAGE if need.window or need.chunk else 0
         self.pages = IdAllocator(n_pages, "cache page")
         self.block_table = torch.zeros((max_seqs, max_pages_per_seq), dtype=torch.int32, device=device)
         # pages_of[slot][i]: the page that holds positions 64 i .. 64 i + 63 of the slot's sequence, or None once a
@@ -70,10 +70,10 @@ class _KVGroup:
 
     def drop_before_window(self, slot: int, length: int) -> None:
         """`length`: how long the slot's sequence is now; the tokens still to come sit at positions >= length and see
-        the keys from length - window + 1 on.  Pages that lie wholly before that are given back."""
-        if not self.need.window:
+        the keys from length - window + 1 on, or those of their chunk.  Pages that lie wholly before that are given back."""
+        if not self.need.window and not self.need.chunk:
             return
-        first_needed = max(0, length - self.need.window + 1) // PAGE
+        first_needed = self.need.first_needed(length) // PAGE
         last = min(first_needed, len(self.pages_of[slot]))
         start = max(self.dropped[slot], self.kept_pages)
         if last > start:

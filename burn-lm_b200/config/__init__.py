@@ -5,6 +5,7 @@ from .fobilorn import FobilornConfig
 from .nufolix import NufolixConfig
 from .ridopel import RidopelConfig
 from .marinex import MarinexConfig
+from .tomalix import TomalixConfig
 from .presets import preset, preset_names
 
-__all__ = ["ConfigError", "KeyReader", "read_config_json", "LlamaConfig", "Llama3RopeScaling", "FobilornConfig", "NufolixConfig", "RidopelConfig", "MarinexConfig", "preset", "preset_names"]
+__all__ = ["ConfigError", "KeyReader", "read_config_json", "LlamaConfig", "Llama3RopeScaling", "FobilornConfig", "NufolixConfig", "RidopelConfig", "MarinexConfig", "TomalixConfig", "preset", "preset_names"]

@@ -7,8 +7,13 @@
 //   out[n, h] = gate(n, h) * sum_j p_j v_j,  gate = sigmoid(g[n, h]) or 1
 // Options of the scores (ScoreOpts): a number per query head that multiplies its scores, s_j = scale t_h q.k_j; a cap,
 // s_j <- cap tanh(s_j / cap); and a score z_h of the sink other than 0, p_j = exp(s_j) / (exp(z_h) + sum exp(s_j)).
+// Instead of a window the mask may be a chunk: visible(i, j) = j <= i and j / chunk == i / chunk (Mask).  The gate may have a
+// number per value lane instead of one per head, and the result may be scaled and written as columns of wider rows (RowOut).
+// Differential attention (maps 2): every head has two queries and every key/value head two keys, [head][map][dk], over one
+// value; the kernels run the 2 n heads on 2 n_kv key heads and leave their sums, and a last kernel forms
+//   o = a_1 - lambda a_2,   out = o / sqrt(mean(o^2) + eps) * c   per head.
 //
-// The cache page of this family holds the keys [n_kv, page, dk] followed by the values [n_kv, page, dv].
+// The cache page of this family holds the keys [n_kv, page, dk] followed by the values [n_kv / maps, page, dv].
 // Scores, softmax and sums are fp32; q, keys and values are read in the cache's dtype.
 #include "common.cuh"
 
@@ -106,6 +111,28 @@ BLM_API int blm_qk_norm_append(const float* proj, long long proj_stride, int n_t
 // portions, 32-bit prompts and every head size.  With several splits each block leaves (max, sum, unnormalised
 // output) of its share of the keys and attention_sink_combine_kernel puts them together; the sink belongs to split 0.
 // ---------------------------------------------------------------------------------------------
+// which keys a position sees behind it: a window of the latest, or (chunk > 0) those of its own chunk of the sequence
+struct Mask {
+    int window, chunk;
+    __device__ __forceinline__ int first(int pos) const { return chunk > 0 ? pos - pos % chunk : max(0, pos - window + 1); }
+};
+
+// how a row's result leaves: times `scale`, times sigmoid(gate) (a number per head, or per lane when gate_lanes > 0: the number
+// of a head's lane d is gate[n * gate_stride + head * gate_lanes + d]), to out[n * stride + head * dv + d]
+struct RowOut {
+    const float* gate;
+    long long gate_stride;
+    int gate_lanes;
+    long long stride;
+    float scale;
+    __device__ __forceinline__ float head_gate(size_t n, int head) const {
+        return gate != nullptr && gate_lanes == 0 ? scale / (1.0f + expf(-gate[n * gate_stride + head])) : scale;
+    }
+    __device__ __forceinline__ float lane_gate(size_t n, int head, int d) const {
+        return gate != nullptr && gate_lanes > 0 ? 1.0f / (1.0f + expf(-gate[n * gate_stride + (size_t)head * gate_lanes + d])) : 1.f;
+    }
+};
+
 constexpr int kChunk = 32;
 constexpr int kMaxVRegs = 16;     // value lanes per thread: dv <= 32 * kMaxVRegs
 
@@ -142,7 +169,7 @@ __device__ __forceinline__ void stage_row<__nv_bfloat16>(float* dst, const __nv_
 // After the fused projection [q | k | v | ...] (fp32 rows), head by head:
 //   q_h <- q_h / rms(q_h) * wq   (wq [dk], the same for every head; null: as it is), k_h likewise with wk;
 //   the first rot_dims lanes of q_h and k_h turn by pos * freq[i]: lanes (2i, 2i + 1) when `halves` is 0, lanes
-//   (i, i + rot_dims / 2) when it is 1; the other lanes pass;
+//   (i, i + rot_dims / 2) when it is 1, cosine and sine both times `turn_scale`; the other lanes pass;
 //   v_h <- v_h / rms(v_h) when `value_norm` (no weight);
 // q goes to q_out, k and v to the token's place in the paged cache.  rms(x) = sqrt(mean(x^2) + eps).  A warp a head;
 // the angle, its sine and cosine in fp64, everything else fp32.
@@ -159,9 +186,9 @@ __device__ __forceinline__ float turned_lane(const float* src, const float* w, f
 }
 
 template <typename T>
-__global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, long long proj_stride, int n_heads, int n_kv, int dk,
-                                             int dv, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
-                                             int value_norm, const double* __restrict__ freq, int rot_dims, int halves,
+__global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, long long proj_stride, int n_heads, int n_kv, int n_v,
+                                             int dk, int dv, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
+                                             int value_norm, const double* __restrict__ freq, int rot_dims, int halves, float turn_scale,
                                              T* __restrict__ q_out, T* __restrict__ pool, long long page_elems, int page_size,
                                              const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                                              const int* __restrict__ slot_of_seq, const int* __restrict__ block_table,
@@ -175,7 +202,7 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
     for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
         double sn, cs;
         sincos((double)pos * freq[i], &sn, &cs);
-        turn[i] = make_float2((float)cs, (float)sn);
+        turn[i] = make_float2(turn_scale * (float)cs, turn_scale * (float)sn);
     }
     __syncthreads();
     T* kpage = nullptr;
@@ -187,7 +214,7 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
         kpage = pool + (size_t)page * page_elems;
         vpage = kpage + (size_t)n_kv * page_size * dk;
     }
-    const int n_vectors = n_heads + 2 * n_kv;          // the heads of q, then of k, then of v
+    const int n_vectors = n_heads + n_kv + n_v;        // the heads of q, then of k, then of v
     for (int item = warp; item < n_vectors; item += n_warps) {
         const bool is_q = item < n_heads, is_k = !is_q && item < n_heads + n_kv;
         const int head = is_q ? item : (is_k ? item - n_heads : item - n_heads - n_kv);
@@ -217,21 +244,24 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
     }
 }
 
-BLM_API int blm_head_norm_rope_append(const float* proj, long long proj_stride, int n_tokens, int n_heads, int n_kv, int dk, int dv,
-                                      const float* wq, const float* wk, float eps, int value_norm, const double* freq, int rot_dims,
-                                      int halves, void* q_out, void* pool, int dtype, long long page_elems, int page_size,
+BLM_API int blm_head_norm_rope_append(const float* proj, long long proj_stride, int n_tokens, int n_heads, int n_kv, int maps, int dk,
+                                      int dv, const float* wq, const float* wk, float eps, int value_norm, const double* freq, int rot_dims,
+                                      int halves, float turn_scale, void* q_out, void* pool, int dtype, long long page_elems, int page_size,
                                       const int* token_seq, const int* token_pos, const int* slot_of_seq, const int* block_table,
                                       int table_stride, cudaStream_t stream) {
     if (n_tokens == 0) return BLM_OK;
     BLM_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv > 0 && dk > 0 && dv > 0 && page_size > 0, "head_norm_rope_append: bad sizes");
-    BLM_REQUIRE(page_elems == (long long)n_kv * page_size * (dk + dv), "head_norm_rope_append: a page holds n_kv * page * (dk + dv) elements");
+    BLM_REQUIRE(maps >= 1 && n_kv % maps == 0, "head_norm_rope_append: %d maps of %d key heads", maps, n_kv);
+    const int n_v = n_kv / maps;                       // n_heads and n_kv count every map
+    BLM_REQUIRE(page_elems == (long long)page_size * ((long long)n_kv * dk + (long long)n_v * dv),
+                "head_norm_rope_append: a page holds page * (n_kv * dk + n_kv / maps * dv) elements");
     BLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || freq != nullptr),
                 "head_norm_rope_append: %d turning lanes of %d", rot_dims, dk);
-    const int vectors = n_heads + 2 * n_kv;
+    const int vectors = n_heads + n_kv + n_v;
     const int threads = vectors >= 8 ? 256 : 32 * vectors;
 #define BLM_HNRA(T)                                                                                                              \
-    head_norm_rope_append_kernel<T><<<n_tokens, threads, (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream>>>(proj, proj_stride, n_heads, n_kv, dk, dv, wq, wk, eps, value_norm, \
-        freq, rot_dims, halves, (T*)q_out, (T*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride)
+    head_norm_rope_append_kernel<T><<<n_tokens, threads, (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream>>>(proj, proj_stride, n_heads, n_kv, n_v, dk, dv, wq, wk, eps, value_norm, \
+        freq, rot_dims, halves, turn_scale, (T*)q_out, (T*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride)
     if (dtype == BLM_F32) BLM_HNRA(float);
     else if (dtype == BLM_BF16) BLM_HNRA(__nv_bfloat16);
     else return blm_fail(BLM_BAD_ARGUMENT, "head_norm_rope_append: dtype %d", dtype);
@@ -260,9 +290,8 @@ template <typename T>
 __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __restrict__ pool, long long page_elems,
                                            const int* __restrict__ block_table, int table_stride, const int* __restrict__ token_seq,
                                            const int* __restrict__ token_pos, const int* __restrict__ slot_of_seq,
-                                           const float* __restrict__ gate, long long gate_stride, T* __restrict__ out,
-                                           float* __restrict__ partial, int n_heads, int n_kv, int dk, int dv, int page_size,
-                                           int window, int keep_first, float scale, int sink, ScoreOpts so) {
+                                           RowOut ro, T* __restrict__ out, float* __restrict__ partial, int n_heads, int n_kv, int maps,
+                                           int dk, int dv, int page_size, Mask mask, int keep_first, float scale, int sink, ScoreOpts so) {
     extern __shared__ float smem[];
     const int n = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z, n_splits = gridDim.z;
     const int group = n_heads / n_kv;
@@ -272,20 +301,22 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
     float* vs = ks + kChunk * kstride;                 // [kChunk][dv]
     float* qs = vs + kChunk * dv;                      // [n_warps][dk]
     const int seq = token_seq[n];
-    T* orow = out + (size_t)n * n_heads * dv;
+    T* orow = out + (size_t)n * ro.stride;
+    const int vh = kvh / maps;
+    const int head_base = vh * group * maps + kvh % maps;      // query heads of this key head: head_base, head_base + maps, ...
     if (seq < 0) {                                     // a row of no sequence: zeros, nothing read
-        if (split == 0)
+        if (partial == nullptr)
             for (int c = threadIdx.x; c < group * dv; c += blockDim.x) orow[(size_t)kvh * group * dv + c] = from_f32<T>(0.f);
-        if (n_splits > 1)
+        else
             for (int c = threadIdx.x; c < group * (dv + 2); c += blockDim.x) {
-                const int head = kvh * group + c / (dv + 2), e = c % (dv + 2);
+                const int head = head_base + c / (dv + 2) * maps, e = c % (dv + 2);
                 partial[(((size_t)n * n_heads + head) * n_splits + split) * (dv + 2) + e] = e == 0 ? -INFINITY : 0.f;
             }
         return;
     }
     const int pos = token_pos[n];
     const int* pages = block_table + (size_t)slot_of_seq[seq] * table_stride;
-    const int lo = max(0, pos - window + 1);           // first key of the window
+    const int lo = mask.first(pos);                    // first key of the window or chunk
     const int n_first = min(keep_first, lo);           // kept first keys that lie before the window
     const int total = n_first + (pos - lo + 1);
     const int n_chunks = (total + kChunk - 1) / kChunk;
@@ -295,7 +326,7 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
     const int kstep = kvec ? 8 : 1, vstep = vvec ? 8 : 1;
     const bool with_sink = sink && split == 0;
     for (int h0 = 0; h0 < group; h0 += n_warps) {
-        const int head = kvh * group + h0 + warp;
+        const int head = head_base + (h0 + warp) * maps;
         const bool active = h0 + warp < group;
         __syncthreads();                               // the chunk buffers and qs of the heads before are done with
         if (active)
@@ -320,7 +351,7 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
                 if (i < c_end) {
                     const int j = i < n_first ? i : lo + (i - n_first);
                     const T* vpage = pool + (size_t)pages[j / page_size] * page_elems + (size_t)n_kv * page_size * dk;
-                    stage_row<T>(vs + row * dv, vpage + ((size_t)kvh * page_size + j % page_size) * dv, d, vvec);
+                    stage_row<T>(vs + row * dv, vpage + ((size_t)vh * page_size + j % page_size) * dv, d, vvec);
                 }
             }
             __syncthreads();
@@ -352,7 +383,7 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
                 }
             }
         }
-        if (active && n_splits > 1) {
+        if (active && partial != nullptr) {
             float* part = partial + (((size_t)n * n_heads + head) * n_splits + split) * (dv + 2);
             if (lane == 0) {
                 part[0] = m;
@@ -364,13 +395,11 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
                 if (d < dv) part[2 + d] = acc[i];
             }
         } else if (active) {
-            float g = 1.f;
-            if (gate != nullptr) g = 1.0f / (1.0f + expf(-gate[(size_t)n * gate_stride + head]));
-            const float inv = l > 0.f ? g / l : 0.f;
+            const float inv = l > 0.f ? ro.head_gate(n, head) / l : 0.f;
 #pragma unroll
             for (int i = 0; i < kMaxVRegs; ++i) {
                 const int d = lane + 32 * i;
-                if (d < dv) orow[(size_t)head * dv + d] = from_f32<T>(acc[i] * inv);
+                if (d < dv) orow[(size_t)head * dv + d] = from_f32<T>(acc[i] * inv * ro.lane_gate(n, head, d));
             }
         }
     }
@@ -378,8 +407,7 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
 
 // out[n, head] = gate * sum_z acc_z e^(m_z - M) / sum_z l_z e^(m_z - M),  M = max_z m_z: one warp per (row, head)
 template <typename T>
-__global__ void attention_sink_combine_kernel(const float* __restrict__ partial, const float* __restrict__ gate, long long gate_stride,
-                                              T* __restrict__ out, int n_rows, int n_heads, int dv, int n_splits) {
+__global__ void attention_sink_combine_kernel(const float* __restrict__ partial, RowOut ro, T* __restrict__ out, int n_rows, int n_heads, int dv, int n_splits) {
     const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (item >= n_rows * n_heads) return;
     const int n = item / n_heads, head = item % n_heads;
@@ -391,24 +419,79 @@ __global__ void attention_sink_combine_kernel(const float* __restrict__ partial,
         const float mz = part[(size_t)z * (dv + 2)];
         if (mz > -INFINITY) l += part[(size_t)z * (dv + 2) + 1] * expf(mz - big);
     }
-    float g = 1.f;
-    if (gate != nullptr) g = 1.0f / (1.0f + expf(-gate[(size_t)n * gate_stride + head]));
-    const float inv = l > 0.f ? g / l : 0.f;
+    const float inv = l > 0.f ? ro.head_gate(n, head) / l : 0.f;
     for (int d = lane; d < dv; d += 32) {
         float a = 0.f;
         for (int z = 0; z < n_splits; ++z) {
             const float mz = part[(size_t)z * (dv + 2)];
             if (mz > -INFINITY) a += part[(size_t)z * (dv + 2) + 2 + d] * expf(mz - big);
         }
-        out[((size_t)n * n_heads + head) * dv + d] = from_f32<T>(a * inv);
+        out[(size_t)n * ro.stride + (size_t)head * dv + d] = from_f32<T>(a * inv * ro.lane_gate(n, head, d));
     }
+}
+
+// Differential attention's end, a warp per (row, head): the two maps' shares put together as above, then
+// o = a_1 - lambda a_2, o / sqrt(mean(o^2) + eps) * c.  partial [rows][heads][2 maps][n_splits][max, sum, dv lanes].
+struct DiffOpts {
+    float lambda, c, eps;
+};
+template <typename T>
+__global__ void attention_difference_kernel(const float* __restrict__ partial, RowOut ro, T* __restrict__ out, int n_rows, int n_heads, int dv,
+                                            int n_splits, DiffOpts df) {
+    const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= n_rows * n_heads) return;
+    const int n = item / n_heads, head = item % n_heads;
+    float o[kMaxVRegs];
+#pragma unroll
+    for (int i = 0; i < kMaxVRegs; ++i) o[i] = 0.f;
+    for (int m = 0; m < 2; ++m) {
+        const float* part = partial + ((size_t)item * 2 + m) * n_splits * (dv + 2);
+        float big = -INFINITY, l = 0.f;
+        for (int z = 0; z < n_splits; ++z) big = fmaxf(big, part[(size_t)z * (dv + 2)]);
+        for (int z = 0; z < n_splits; ++z) {
+            const float mz = part[(size_t)z * (dv + 2)];
+            if (mz > -INFINITY) l += part[(size_t)z * (dv + 2) + 1] * expf(mz - big);
+        }
+        const float w = l > 0.f ? (m == 0 ? 1.f : -df.lambda) / l : 0.f;
+        for (int z = 0; z < n_splits; ++z) {
+            const float mz = part[(size_t)z * (dv + 2)];
+            if (!(mz > -INFINITY)) continue;
+            const float f = w * expf(mz - big);
+#pragma unroll
+            for (int i = 0; i < kMaxVRegs; ++i) {
+                const int d = lane + 32 * i;
+                if (d < dv) o[i] = fmaf(f, part[(size_t)z * (dv + 2) + 2 + d], o[i]);
+            }
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMaxVRegs; ++i) ss += o[i] * o[i];
+    ss = warp_sum(ss);
+    const float inv = df.c / sqrtf(ss / (float)dv + df.eps) * ro.head_gate(n, head);
+#pragma unroll
+    for (int i = 0; i < kMaxVRegs; ++i) {
+        const int d = lane + 32 * i;
+        if (d < dv) out[(size_t)n * ro.stride + (size_t)head * dv + d] = from_f32<T>(o[i] * inv * ro.lane_gate(n, head, d));
+    }
+}
+
+// what follows the kernels that left shares: one launch either way
+template <typename T>
+static void finish_shares(const float* partial, RowOut ro, void* out, int n_tokens, int n_heads, int maps, int dv, int n_splits, DiffOpts df,
+                          cudaStream_t stream) {
+    const int items = n_tokens * (n_heads / maps);
+    if (maps == 2)
+        attention_difference_kernel<T><<<(items + 3) / 4, 128, 0, stream>>>(partial, ro, (T*)out, n_tokens, n_heads / 2, dv, n_splits, df);
+    else
+        attention_sink_combine_kernel<T><<<(items + 3) / 4, 128, 0, stream>>>(partial, ro, (T*)out, n_tokens, n_heads, dv, n_splits);
 }
 
 template <typename T>
 static int launch_rows(const void* q, const void* pool, long long page_elems, const int* block_table, int table_stride,
-                       const int* token_seq, const int* token_pos, const int* slot_of_seq, const float* gate, long long gate_stride,
-                       void* out, float* partial, int n_splits, int n_tokens, int n_heads, int n_kv, int dk, int dv, int page_size,
-                       int window, int keep_first, float scale, int sink, ScoreOpts so, cudaStream_t stream) {
+                       const int* token_seq, const int* token_pos, const int* slot_of_seq, RowOut ro, void* out, float* partial,
+                       int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, int page_size, Mask mask,
+                       int keep_first, float scale, int sink, ScoreOpts so, DiffOpts df, cudaStream_t stream) {
     const int group = n_heads / n_kv;
     const int warps = group < 8 ? group : 8;
     const size_t smem = ((size_t)kChunk * (dk + 1) + (size_t)kChunk * dv + (size_t)warps * dk) * sizeof(float);
@@ -418,13 +501,9 @@ static int launch_rows(const void* q, const void* pool, long long page_elems, co
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "attention_sink: %s", cudaGetErrorString(e));
     }
     attention_sink_rows_kernel<T><<<dim3(n_tokens, n_kv, n_splits), warps * 32, smem, stream>>>(
-        (const T*)q, (const T*)pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, gate, gate_stride,
-        (T*)out, partial, n_heads, n_kv, dk, dv, page_size, window, keep_first, scale, sink, so);
-    if (n_splits > 1) {
-        const int items = n_tokens * n_heads;
-        attention_sink_combine_kernel<T><<<(items + 3) / 4, 128, 0, stream>>>(partial, gate, gate_stride, (T*)out, n_tokens, n_heads, dv,
-                                                                              n_splits);
-    }
+        (const T*)q, (const T*)pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro,
+        (T*)out, partial, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink, so);
+    if (partial != nullptr) finish_shares<T>(partial, ro, out, n_tokens, n_heads, maps, dv, n_splits, df, stream);
     return blm_check_launch("attention_sink");
 }
 
@@ -495,8 +574,7 @@ constexpr int kTileQ = 64, kTileK = 64;
 // The pages a query tile walks: `kept` pages from the sequence's start, then pages wp0 .. wp1.
 struct PageWalk {
     int kept, wp0, n_tiles;
-    __device__ __forceinline__ PageWalk(int p_first, int p_last, int window, int keep_first) {
-        const int lo = max(0, p_first - window + 1);
+    __device__ __forceinline__ PageWalk(int lo, int p_last, int keep_first) {      // lo: the first key the first query sees
         wp0 = lo / kTileK;
         kept = min((keep_first + kTileK - 1) / kTileK, wp0);
         n_tiles = kept + (p_last / kTileK - wp0 + 1);
@@ -517,11 +595,11 @@ struct GroupWalk {
 };
 
 // one page's keys and values of one kv head into a buffer pair (every thread of the block takes its share)
-__device__ __forceinline__ void stage_page(__nv_bfloat16* kbuf, __nv_bfloat16* vbuf, const __nv_bfloat16* page, int n_kv, int kvh, int dk,
-                                           int dv, int qstride, int vstride, int first_pos, int p_last, const GroupWalk& kw,
+__device__ __forceinline__ void stage_page(__nv_bfloat16* kbuf, __nv_bfloat16* vbuf, const __nv_bfloat16* page, int n_kv, int kvh, int vh,
+                                           int dk, int dv, int qstride, int vstride, int first_pos, int p_last, const GroupWalk& kw,
                                            const GroupWalk& vw) {
     const __nv_bfloat16* kpage = page + (size_t)kvh * kTileK * dk;
-    const __nv_bfloat16* vpage = page + (size_t)n_kv * kTileK * dk + (size_t)kvh * kTileK * dv;
+    const __nv_bfloat16* vpage = page + (size_t)n_kv * kTileK * dk + (size_t)vh * kTileK * dv;
     for (int r = kw.r, c = kw.c; r < kTileK;) {
         cp_async16(kbuf + r * qstride + c * 8, kpage + r * dk + c * 8, true);
         r += kw.dr;
@@ -546,8 +624,8 @@ template <int NV, int HB>
 __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool, long long page_elems,
     const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ start_pos,
-    const int* __restrict__ slot_of_seq, int n_seqs, int n_tokens, const float* __restrict__ gate, long long gate_stride,
-    __nv_bfloat16* __restrict__ out, int n_heads, int n_kv, int dk, int dv, int window, int keep_first, float scale, int sink,
+    const int* __restrict__ slot_of_seq, int n_seqs, int n_tokens, RowOut ro, __nv_bfloat16* __restrict__ out,
+    float* __restrict__ partial, int n_heads, int n_kv, int maps, int dk, int dv, Mask mask, int keep_first, float scale, int sink,
     ScoreOpts so) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ int found[3];
@@ -578,12 +656,16 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     if (found[0] < 0) {
         // a block without a tile: the rows after the last sequence (padding up to a captured step's size) get zeros
         const int end = cu_seqlens[n_seqs];
-        for (int idx = tid & 127; idx < (n_tokens - end) * dv; idx += 128)
-            out[((size_t)(end + idx / dv) * n_heads + head) * dv + idx % dv] = __float2bfloat16_rn(0.f);
+        if (partial == nullptr)
+            for (int idx = tid & 127; idx < (n_tokens - end) * dv; idx += 128)
+                out[(size_t)(end + idx / dv) * ro.stride + (size_t)head * dv + idx % dv] = __float2bfloat16_rn(0.f);
+        else
+            for (int idx = tid & 127; idx < (n_tokens - end) * (dv + 2); idx += 128)
+                partial[((size_t)(end + idx / (dv + 2)) * n_heads + head) * (dv + 2) + idx % (dv + 2)] = idx % (dv + 2) == 0 ? -INFINITY : 0.f;
         return;
     }
     const int seq = found[0], t0 = found[1], len = found[2];
-    const int kvh = head / (n_heads / n_kv);
+    const int vh = head / maps / (n_heads / n_kv), kvh = vh * maps + head % maps;
     const int row0 = cu_seqlens[seq] + t0;             // the tile's first token row
     const int rows = min(kTileQ, len - t0);
     const int p0 = start_pos[seq] + t0;                // its position
@@ -594,7 +676,7 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     for (int i = 0; i < HB; ++i) zero_unwritten(Qs + i * kTileQ * qstride, kTileQ, qstride, rows, dk);
     zero_unwritten(Kb, kPromptStages * kTileK, qstride, kPromptStages * kTileK, dk);
     zero_unwritten(Vb, kPromptStages * kTileK, vstride, kPromptStages * kTileK, dv);
-    const PageWalk walk(p0, p_last, window, keep_first);
+    const PageWalk walk(mask.first(p0), p_last, keep_first);
     for (int idx = tid & 127; idx < rows * (dk / 8); idx += 128) {       // every group of four warps brings its head's queries
         const int r = idx / (dk / 8), c = (idx % (dk / 8)) * 8;
         cp_async16(Qs + (hb * kTileQ + r) * qstride + c, q + ((size_t)(row0 + r) * n_heads + head) * dk + c, true);
@@ -602,7 +684,7 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     const GroupWalk kw(dk / 8), vw(dv / 8);
     auto fetch = [&](int it) {                         // page `it` of the walk into its place in the ring
         const int pg = walk.page(it), b = it % kPromptStages;
-        stage_page(Kb + b * kTileK * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, dk, dv, qstride,
+        stage_page(Kb + b * kTileK * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
                    vstride, pg * kTileK, p_last, kw, vw);
     };
 #pragma unroll
@@ -613,6 +695,7 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     const int quad = lane >> 2, pair = (lane & 3) * 2;
     const int lrow = lane & 7, lmat = lane >> 3;
     const int pr0 = p0 + warp * 16 + quad, pr1 = pr0 + 8;        // positions of this thread's two rows
+    const int lo0 = mask.first(pr0), lo1 = mask.first(pr1), lo_last = mask.first(p0 + warp * 16 + 15);     // the first keys they see, and the warp's last row
     // scores in units of log 2: the exponentials are exp2.  A cap (or a head's multiplier that is not positive, under which
     // the largest raw score is not the largest score) is applied to the raw scores first, which are then in natural units.
     const float pre = scale * (so.head_scale ? so.head_scale[head] : 1.f);
@@ -658,8 +741,8 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
         float mx0 = -INFINITY, mx1 = -INFINITY;
         // every row of this warp sees every key of the page when the page lies behind the warp's first row and inside
         // the window of its last (or among the kept first tokens): then nothing is masked (most pages of a long window)
-        const int w_first = p0 + warp * 16, w_last = w_first + 15, key0 = pg * kTileK;
-        if (key0 + kTileK - 1 <= w_first && (w_last - key0 < window || key0 + kTileK <= keep_first)) {
+        const int w_first = p0 + warp * 16, key0 = pg * kTileK;
+        if (key0 + kTileK - 1 <= w_first && (key0 >= lo_last || key0 + kTileK <= keep_first)) {
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
                 mx0 = fmaxf(mx0, fmaxf(s[j][0], s[j][1]));
@@ -672,7 +755,7 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
                 for (int e = 0; e < 4; ++e) {
                     const int key = key0 + 8 * j + pair + (e & 1);
                     const int pr = e < 2 ? pr0 : pr1;
-                    const bool sees = key <= pr && (pr - key < window || key < keep_first);
+                    const bool sees = key <= pr && (key >= (e < 2 ? lo0 : lo1) || key < keep_first);
                     const float v = sees ? s[j][e] : -INFINITY;
                     s[j][e] = v;
                     if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
@@ -725,31 +808,54 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     l[1] += __shfl_xor_sync(0xffffffffu, l[1], 2);
     const int r0 = warp * 16 + quad, r1 = r0 + 8;
     float inv0 = 0.f, inv1 = 0.f;
-    if (r0 < rows) {
-        const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)(row0 + r0) * gate_stride + head])) : 1.f;
-        inv0 = l[0] > 0.f ? g / l[0] : 0.f;
+    if (partial != nullptr) {                          // (one share: normalised, with a sum of 1 at a maximum of 0)
+        if (l[0] > 0.f) inv0 = 1.f / l[0];
+        if (l[1] > 0.f) inv1 = 1.f / l[1];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int r = half ? r1 : r0;
+            if (r >= rows) continue;
+            float* part = partial + ((size_t)(row0 + r) * n_heads + head) * (dv + 2);      // dv even: pairs are 8-byte aligned
+            const float inv = half ? inv1 : inv0;
+            if (pair == 0) *reinterpret_cast<float2*>(part) = make_float2(0.f, 1.f);
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int d = 8 * j + pair;
+                if (d < dv) *reinterpret_cast<float2*>(part + 2 + d) = make_float2(o[j][2 * half] * inv, o[j][2 * half + 1] * inv);
+            }
+        }
+        return;
     }
-    if (r1 < rows) {
-        const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)(row0 + r1) * gate_stride + head])) : 1.f;
-        inv1 = l[1] > 0.f ? g / l[1] : 0.f;
-    }
+    if (r0 < rows) inv0 = l[0] > 0.f ? ro.head_gate(row0 + r0, head) / l[0] : 0.f;
+    if (r1 < rows) inv1 = l[1] > 0.f ? ro.head_gate(row0 + r1, head) / l[1] : 0.f;
+    const bool by_lane = ro.gate != nullptr && ro.gate_lanes > 0;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
         const int d = 8 * j + pair;
         if (d < dv) {
+            if (by_lane) {
+                if (r0 < rows) {
+                    o[j][0] *= ro.lane_gate(row0 + r0, head, d);
+                    o[j][1] *= ro.lane_gate(row0 + r0, head, d + 1);
+                }
+                if (r1 < rows) {
+                    o[j][2] *= ro.lane_gate(row0 + r1, head, d);
+                    o[j][3] *= ro.lane_gate(row0 + r1, head, d + 1);
+                }
+            }
             if (r0 < rows)
-                *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + r0) * n_heads + head) * dv + d) = pack_bf16(o[j][0] * inv0, o[j][1] * inv0);
+                *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + r0) * ro.stride + (size_t)head * dv + d) = pack_bf16(o[j][0] * inv0, o[j][1] * inv0);
             if (r1 < rows)
-                *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + r1) * n_heads + head) * dv + d) = pack_bf16(o[j][2] * inv1, o[j][3] * inv1);
+                *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + r1) * ro.stride + (size_t)head * dv + d) = pack_bf16(o[j][2] * inv1, o[j][3] * inv1);
         }
     }
 }
 
 template <int NV, int HB>
 static int launch_prompt(const void* q, const void* pool, long long page_elems, const int* block_table, int table_stride,
-                         const int* cu_seqlens, const int* start_pos, const int* slot_of_seq, int n_seqs, const float* gate,
-                         long long gate_stride, void* out, int n_tokens, int n_heads, int n_kv, int dk, int dv, int window,
-                         int keep_first, float scale, int sink, ScoreOpts so, cudaStream_t stream) {
+                         const int* cu_seqlens, const int* start_pos, const int* slot_of_seq, int n_seqs, RowOut ro, void* out,
+                         float* partial, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, Mask mask, int keep_first,
+                         float scale, int sink, ScoreOpts so, DiffOpts df, cudaStream_t stream) {
     const int dkp = (dk + 15) & ~15;
     const size_t smem = ((size_t)(HB + kPromptStages) * kTileQ * (dkp + 8) + (size_t)kPromptStages * kTileK * (8 * NV + 8)) * sizeof(__nv_bfloat16);
     if (smem > 48 * 1024) {
@@ -760,7 +866,8 @@ static int launch_prompt(const void* q, const void* pool, long long page_elems, 
     const unsigned tiles = (unsigned)((n_tokens + kTileQ - 1) / kTileQ + n_seqs);     // every sequence may end in a tile that is not full
     attention_sink_prompt_kernel<NV, HB><<<dim3(tiles, n_heads / HB), 128 * HB, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq,
-        n_seqs, n_tokens, gate, gate_stride, (__nv_bfloat16*)out, n_heads, n_kv, dk, dv, window, keep_first, scale, sink, so);
+        n_seqs, n_tokens, ro, (__nv_bfloat16*)out, partial, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so);
+    if (partial != nullptr) finish_shares<__nv_bfloat16>(partial, ro, out, n_tokens, n_heads, maps, dv, 1, df, stream);
     return blm_check_launch("attention_sink (prompt)");
 }
 
@@ -772,9 +879,8 @@ template <int NV, int kDecodeStages>
 __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool, long long page_elems,
     const int* __restrict__ block_table, int table_stride, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
-    const int* __restrict__ slot_of_seq, const float* __restrict__ gate, long long gate_stride, __nv_bfloat16* __restrict__ out,
-    float* __restrict__ partial, int n_heads, int n_kv, int dk, int dv, int window, int keep_first, float scale, int sink,
-    ScoreOpts so) {
+    const int* __restrict__ slot_of_seq, RowOut ro, __nv_bfloat16* __restrict__ out, float* __restrict__ partial, int n_heads, int n_kv,
+    int maps, int dk, int dv, Mask mask, int keep_first, float scale, int sink, ScoreOpts so) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int n = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z, n_splits = gridDim.z;
@@ -786,13 +892,13 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     __nv_bfloat16* Kb = Qs + 16 * qstride;                               // kDecodeStages x [64][qstride]
     __nv_bfloat16* Vb = Kb + kDecodeStages * kTileK * qstride;           // kDecodeStages x [64][vstride]
     const int seq = token_seq[n];
-    const int head0 = kvh * group;
+    const int vh = kvh / maps, head0 = vh * group * maps + kvh % maps;      // this key head's query heads: head0, head0 + maps, ...
     if (seq < 0) {                                     // a row of no sequence: zeros, nothing read
-        if (split == 0)
-            for (int c = tid; c < group * dv; c += 128) out[((size_t)n * n_heads + head0) * dv + c] = __float2bfloat16_rn(0.f);
-        if (n_splits > 1)
+        if (partial == nullptr)
+            for (int c = tid; c < group * dv; c += 128) out[(size_t)n * ro.stride + (size_t)head0 * dv + c] = __float2bfloat16_rn(0.f);
+        else
             for (int c = tid; c < group * (dv + 2); c += 128) {
-                const int head = head0 + c / (dv + 2), e = c % (dv + 2);
+                const int head = head0 + c / (dv + 2) * maps, e = c % (dv + 2);
                 partial[(((size_t)n * n_heads + head) * n_splits + split) * (dv + 2) + e] = e == 0 ? -INFINITY : 0.f;
             }
         return;
@@ -802,17 +908,18 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     zero_unwritten(Qs, 16, qstride, group, dk);
     zero_unwritten(Kb, kDecodeStages * kTileK, qstride, kDecodeStages * kTileK, dk);
     zero_unwritten(Vb, kDecodeStages * kTileK, vstride, kDecodeStages * kTileK, dv);
-    const PageWalk walk(pos, pos, window, keep_first);
+    const int lo = mask.first(pos);
+    const PageWalk walk(lo, pos, keep_first);
     const int per_split = (walk.n_tiles + n_splits - 1) / n_splits;
     const int it_begin = split * per_split, it_end = min(walk.n_tiles, it_begin + per_split);
     for (int idx = tid; idx < group * (dk / 8); idx += 128) {
         const int r = idx / (dk / 8), c = (idx % (dk / 8)) * 8;
-        cp_async16(Qs + r * qstride + c, q + ((size_t)n * n_heads + head0 + r) * dk + c, true);
+        cp_async16(Qs + r * qstride + c, q + ((size_t)n * n_heads + head0 + r * maps) * dk + c, true);
     }
     const GroupWalk kw(dk / 8), vw(dv / 8);
     auto fetch = [&](int it) {                         // page `it` of the walk into its place in the ring
         const int pg = walk.page(it), b = (it - it_begin) % kDecodeStages;
-        stage_page(Kb + b * kTileK * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, dk, dv, qstride,
+        stage_page(Kb + b * kTileK * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
                    vstride, pg * kTileK, pos, kw, vw);
     };
 #pragma unroll
@@ -829,8 +936,8 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
 #pragma unroll
     for (int half = 0; half < 2; ++half) {                       // this thread's two rows are two heads of the group
         const int r = quad + 8 * half;
-        pre[half] = scale * (so.head_scale && r < group ? so.head_scale[head0 + r] : 1.f);
-        m[half] = with_sink ? (so.sink_logit && r < group ? so.sink_logit[head0 + r] * log2e : 0.f) : -INFINITY;
+        pre[half] = scale * (so.head_scale && r < group ? so.head_scale[head0 + r * maps] : 1.f);
+        m[half] = with_sink ? (so.sink_logit && r < group ? so.sink_logit[head0 + r * maps] * log2e : 0.f) : -INFINITY;
         l[half] = with_sink ? 0.25f : 0.f;
     }
 #pragma unroll
@@ -862,7 +969,7 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = pg * kTileK + 16 * warp + 8 * j + pair + (e & 1);
-                const bool sees = key <= pos && (pos - key < window || key < keep_first);
+                const bool sees = key <= pos && (key >= lo || key < keep_first);
                 s[j][e] = sees ? capped_fast(s[j][e] * pre[e >> 1], so.cap, inv_cap) * log2e : -INFINITY;
             }
         float mx0 = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
@@ -936,8 +1043,8 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
                 acc += src[2 + d] * f;
             }
         }
-        const int head = head0 + r;
-        if (n_splits > 1) {
+        const int head = head0 + r * maps;
+        if (partial != nullptr) {
             float* part = partial + (((size_t)n * n_heads + head) * n_splits + split) * (dv + 2);
             if (d == 0) {
                 part[0] = big * 0.6931471805599453f;       // the splits are put together in natural units
@@ -945,17 +1052,17 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
             }
             part[2 + d] = acc;
         } else {
-            const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)n * gate_stride + head])) : 1.f;
-            out[((size_t)n * n_heads + head) * dv + d] = __float2bfloat16_rn(lsum > 0.f ? acc * g / lsum : 0.f);
+            const float g = ro.head_gate(n, head) * ro.lane_gate(n, head, d);
+            out[(size_t)n * ro.stride + (size_t)head * dv + d] = __float2bfloat16_rn(lsum > 0.f ? acc * g / lsum : 0.f);
         }
     }
 }
 
 template <int NV, int kDecodeStages>
 static int launch_decode(const void* q, const void* pool, long long page_elems, const int* block_table, int table_stride,
-                         const int* token_seq, const int* token_pos, const int* slot_of_seq, const float* gate, long long gate_stride,
-                         void* out, float* partial, int n_splits, int n_tokens, int n_heads, int n_kv, int dk, int dv, int window,
-                         int keep_first, float scale, int sink, ScoreOpts so, cudaStream_t stream) {
+                         const int* token_seq, const int* token_pos, const int* slot_of_seq, RowOut ro, void* out, float* partial,
+                         int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, Mask mask, int keep_first,
+                         float scale, int sink, ScoreOpts so, DiffOpts df, cudaStream_t stream) {
     const int dkp = (dk + 15) & ~15;
     size_t smem = ((size_t)16 * (dkp + 8) + (size_t)kDecodeStages * kTileK * ((dkp + 8) + (8 * NV + 8))) * sizeof(__nv_bfloat16);
     const size_t merge = (size_t)16 * (dkp + 8) * sizeof(__nv_bfloat16) + (size_t)4 * 16 * (8 * NV + 2) * sizeof(float);
@@ -966,13 +1073,9 @@ static int launch_decode(const void* q, const void* pool, long long page_elems, 
     }
     cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
     attention_sink_decode_kernel<NV, kDecodeStages><<<dim3(n_tokens, n_kv, n_splits), 128, smem, stream>>>(
-        (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, gate,
-        gate_stride, (__nv_bfloat16*)out, partial, n_heads, n_kv, dk, dv, window, keep_first, scale, sink, so);
-    if (n_splits > 1) {
-        const int items = n_tokens * n_heads;
-        attention_sink_combine_kernel<__nv_bfloat16><<<(items + 3) / 4, 128, 0, stream>>>(partial, gate, gate_stride, (__nv_bfloat16*)out,
-                                                                                         n_tokens, n_heads, dv, n_splits);
-    }
+        (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro,
+        (__nv_bfloat16*)out, partial, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so);
+    if (partial != nullptr) finish_shares<__nv_bfloat16>(partial, ro, out, n_tokens, n_heads, maps, dv, n_splits, df, stream);
     return blm_check_launch("attention_sink (decode)");
 }
 
@@ -1000,7 +1103,7 @@ static int launch_prompt_heads(int hb, Args... args) {
 // Whether a step of this shape runs the prompt kernel (else the row kernel): bfloat16, pages of 64, sizes it takes,
 // and portions long enough to fill some of a tile's rows.
 BLM_API int blm_attention_sink_prompt_takes(int dtype, int dk, int dv, int page_size, int max_q_len, int n_heads) {
-    return dtype == BLM_BF16 && page_size == kTileK && dk % 8 == 0 && dv % 8 == 0 && dk >= 8 && dk <= 256 && dv >= 8 && dv <= 128 &&
+    return dtype == BLM_BF16 && page_size == kTileK && dk % 8 == 0 && dv % 8 == 0 && dk >= 8 && dk <= 256 && dv >= 8 && dv <= 256 &&
            max_q_len >= 8 && n_heads <= 65535;
 }
 
@@ -1008,16 +1111,19 @@ BLM_API int blm_attention_sink_prompt_takes(int dtype, int dk, int dv, int page_
 // same sizes, and a group of query heads that fits the 16 rows of a tile.  The keys are then cut by pages: a split
 // should have a page at least.
 BLM_API int blm_attention_sink_decode_takes(int dtype, int dk, int dv, int page_size, int n_heads, int n_kv) {
-    return dtype == BLM_BF16 && page_size == kTileK && dk % 8 == 0 && dv % 8 == 0 && dk >= 8 && dk <= 256 && dv >= 8 && dv <= 128 &&
+    return dtype == BLM_BF16 && page_size == kTileK && dk % 8 == 0 && dv % 8 == 0 && dk >= 8 && dk <= 256 && dv >= 8 && dv <= 256 &&
            n_kv > 0 && n_heads % n_kv == 0 && n_heads / n_kv <= 16;
 }
 
 BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long long page_elems, const int* block_table,
                                int table_stride, const int* token_seq, const int* token_pos, const int* slot_of_seq,
                                const int* cu_seqlens, const int* start_pos, int n_seqs, int max_q_len, const float* gate,
-                               long long gate_stride, void* out, float* partial, int n_splits, int n_tokens, int n_heads, int n_kv,
-                               int dk, int dv, int page_size, int window, int keep_first, float scale, int sink,
-                               const float* head_scale, const float* sink_logit, float softcap, cudaStream_t stream) {
+                               long long gate_stride, int gate_lanes, void* out, long long out_stride, float out_scale, float* partial,
+                               int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, int page_size, int window,
+                               int chunk, int keep_first, float scale, int sink, const float* head_scale, const float* sink_logit,
+                               float softcap, float diff_lambda, float diff_scale, float diff_eps, cudaStream_t stream) {
+    // maps 2: n_heads and n_kv count every map, and diff_* are the difference's numbers (DiffOpts); partial is then needed
+    // chunk > 0: the mask is by chunks and `window` is not looked at; gate_lanes 0: a gate per head, dv: one per lane
     // head_scale, sink_logit: float32 [n_heads] or null; softcap: 0 for none (see ScoreOpts)
     if (n_tokens == 0) return BLM_OK;
     const ScoreOpts so{head_scale, sink_logit, softcap};
@@ -1025,37 +1131,49 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
     BLM_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv > 0 && n_heads % n_kv == 0 && dk > 0 && dv > 0 && page_size > 0,
                 "attention_sink: bad sizes");
     BLM_REQUIRE(dv <= 32 * kMaxVRegs, "attention_sink: values of %d lanes; at most %d", dv, 32 * kMaxVRegs);
-    BLM_REQUIRE(window >= 1 && keep_first >= 0, "attention_sink: window %d, kept first %d", window, keep_first);
-    BLM_REQUIRE(page_elems == (long long)n_kv * page_size * (dk + dv), "attention_sink: a page holds n_kv * page * (dk + dv) elements");
+    BLM_REQUIRE(window >= 1 && chunk >= 0 && keep_first >= 0, "attention_sink: window %d, chunk %d, kept first %d", window, chunk, keep_first);
+    BLM_REQUIRE(maps == 1 || (maps == 2 && n_kv % 2 == 0 && partial != nullptr), "attention_sink: %d maps of %d key heads", maps, n_kv);
+    BLM_REQUIRE(page_elems == (long long)page_size * ((long long)n_kv * dk + (long long)(n_kv / maps) * dv),
+                "attention_sink: a page holds page * (n_kv * dk + n_kv / maps * dv) elements");
+    BLM_REQUIRE(gate_lanes == 0 || gate_lanes == dv, "attention_sink: a gate of %d lanes for values of %d", gate_lanes, dv);
+    BLM_REQUIRE(out_stride >= (long long)(n_heads / maps) * dv, "attention_sink: output rows of %lld elements", out_stride);
     BLM_REQUIRE(n_kv <= 65535 && n_splits >= 1 && n_splits <= 65535, "attention_sink: %d kv heads, %d splits", n_kv, n_splits);
     BLM_REQUIRE(n_splits == 1 || partial != nullptr, "attention_sink: %d splits need scratch", n_splits);
+    if (n_splits == 1 && maps == 1) partial = nullptr;      // shares are left only where something puts them together
+    const Mask mask{window, chunk};
+    const RowOut ro{gate, gate_stride, gate_lanes, out_stride, out_scale};
+    const DiffOpts df{diff_lambda, diff_scale, diff_eps};
     if (cu_seqlens != nullptr && start_pos != nullptr && n_seqs > 0 &&
-        blm_attention_sink_prompt_takes(dtype, dk, dv, page_size, max_q_len, n_heads)) {
-#define BLM_PROMPT(NV) launch_prompt_heads<NV>(hb, q, pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq, n_seqs, gate, \
-                                         gate_stride, out, n_tokens, n_heads, n_kv, dk, dv, window, keep_first, scale, sink, so, stream)
+        blm_attention_sink_prompt_takes(dtype, dk, dv, page_size, max_q_len, n_heads) &&
+        out_stride % 2 == 0 && ((size_t)out & 3) == 0) {
+#define BLM_PROMPT(NV) launch_prompt_heads<NV>(hb, q, pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq, n_seqs, ro, \
+                                         out, partial, n_tokens, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df, stream)
         const int group = n_heads / n_kv;
-        int hb = BLM_PROMPT_HEADS;
+        int hb = maps == 1 && dv <= 128 ? BLM_PROMPT_HEADS : 1;
         while (hb > 1 && (group % hb != 0 || (hb == 4 && dv > 64))) hb /= 2;    // four heads of 128 lanes would not fit the registers
         if (dv <= 32) return BLM_PROMPT(4);
         if (dv <= 64) return BLM_PROMPT(8);
-        return BLM_PROMPT(16);
+        if (dv <= 128) return BLM_PROMPT(16);
+        if (dv <= 192) return BLM_PROMPT(24);
+        return BLM_PROMPT(32);
 #undef BLM_PROMPT
     }
     if (blm_attention_sink_decode_takes(dtype, dk, dv, page_size, n_heads, n_kv)) {
-#define BLM_DECODE(NV, STAGES) launch_decode<NV, STAGES>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, gate, gate_stride, \
-                                         out, partial, n_splits, n_tokens, n_heads, n_kv, dk, dv, window, keep_first, scale, sink, so, stream)
+#define BLM_DECODE(NV, STAGES) launch_decode<NV, STAGES>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, \
+                                         out, partial, n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df, stream)
         if (dv <= 32) return BLM_DECODE(4, 2);
         if (dv <= 64) return BLM_DECODE(8, 2);
-        return BLM_DECODE(16, 3);
+        if (dv <= 128) return BLM_DECODE(16, 3);
+        if (dv <= 192) return BLM_DECODE(24, 2);
+        return BLM_DECODE(32, 2);
 #undef BLM_DECODE
     }
     if (dtype == BLM_F32)
-        return launch_rows<float>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, gate, gate_stride,
-                                  out, partial, n_splits, n_tokens, n_heads, n_kv, dk, dv, page_size, window, keep_first, scale, sink,
-                                  so, stream);
+        return launch_rows<float>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, out, partial,
+                                  n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink, so, df, stream);
     if (dtype == BLM_BF16)
-        return launch_rows<__nv_bfloat16>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, gate,
-                                          gate_stride, out, partial, n_splits, n_tokens, n_heads, n_kv, dk, dv, page_size, window,
-                                          keep_first, scale, sink, so, stream);
+        return launch_rows<__nv_bfloat16>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, out,
+                                          partial, n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink,
+                                          so, df, stream);
     return blm_fail(BLM_BAD_ARGUMENT, "attention_sink: dtype %d", dtype);
 }

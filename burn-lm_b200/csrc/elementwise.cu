@@ -204,7 +204,7 @@ __global__ void rope_append_kernel(T* __restrict__ qkv, const int* __restrict__ 
                                    const int* __restrict__ block_table, int table_stride,
                                    const double* __restrict__ inv_freq, int rot, int pairing,
                                    T* __restrict__ pool, int n_heads, int n_kv, int hd, int page_size,
-                                   int write_cache, const float2* __restrict__ table, int table_len) {
+                                   int write_cache, const float2* __restrict__ table, int table_len, float turn_scale) {
     // one item per thread: a rotated pair of q or k, a lane of k beyond the rotated ones, or two lanes of v
     const int n = blockIdx.y;
     const int item = blockIdx.x * blockDim.x + threadIdx.x;
@@ -237,8 +237,8 @@ __global__ void rope_append_kernel(T* __restrict__ qkv, const int* __restrict__ 
         } else {
             double sd, cd;
             sincos((double)pos * inv_freq[i], &sd, &cd);
-            c = (float)cd;
-            s = (float)sd;
+            c = turn_scale * (float)cd;
+            s = turn_scale * (float)sd;
         }
         const int la = pairing == 1 ? 2 * i : (pairing == 2 ? 16 * (i >> 3) + (i & 7) : i);
         const int lb = pairing == 1 ? la + 1 : (pairing == 2 ? la + 8 : i + half);
@@ -325,7 +325,8 @@ BLM_API int blm_rope_append(void* qkv, int dtype, const int* token_seq, const in
                             const int* slot_of_seq, const int* block_table, int table_stride,
                             const double* inv_freq, int rot, int pairing, void* pool, int n_tokens,
                             int n_heads, int n_kv, int hd, int page_size, int write_cache,
-                            const float2* table, int table_len, int table_covers_step, cudaStream_t stream) {
+                            const float2* table, int table_len, int table_covers_step, float turn_scale, cudaStream_t stream) {
+    // turn_scale: what cosine and sine are multiplied by (the table's numbers already are)
     if (n_tokens == 0) return BLM_OK;
     BLM_REQUIRE(rot >= 0 && rot <= hd && rot % 2 == 0, "rotary: %d rotated lanes of a head of %d", rot, hd);
     BLM_REQUIRE(rot == 0 || inv_freq != nullptr, "rotary: no frequencies");
@@ -352,29 +353,29 @@ BLM_API int blm_rope_append(void* qkv, int dtype, const int* token_seq, const in
         }
     }
     if (dtype == BLM_F32)
-        rope_append_kernel<float><<<grid, threads, smem, stream>>>((float*)qkv, token_seq, token_pos, slot_of_seq, block_table, table_stride, inv_freq, rot, pairing, (float*)pool, n_heads, n_kv, hd, page_size, write_cache, table, table_len);
+        rope_append_kernel<float><<<grid, threads, smem, stream>>>((float*)qkv, token_seq, token_pos, slot_of_seq, block_table, table_stride, inv_freq, rot, pairing, (float*)pool, n_heads, n_kv, hd, page_size, write_cache, table, table_len, turn_scale);
     else if (dtype == BLM_BF16)
-        rope_append_kernel<__nv_bfloat16><<<grid, threads, smem, stream>>>((__nv_bfloat16*)qkv, token_seq, token_pos, slot_of_seq, block_table, table_stride, inv_freq, rot, pairing, (__nv_bfloat16*)pool, n_heads, n_kv, hd, page_size, write_cache, table, table_len);
+        rope_append_kernel<__nv_bfloat16><<<grid, threads, smem, stream>>>((__nv_bfloat16*)qkv, token_seq, token_pos, slot_of_seq, block_table, table_stride, inv_freq, rot, pairing, (__nv_bfloat16*)pool, n_heads, n_kv, hd, page_size, write_cache, table, table_len, turn_scale);
     else
         return blm_fail(BLM_BAD_ARGUMENT, "rotary: dtype %d", dtype);
     return blm_check_launch("rope_append");
 }
 
-// (cos, sin) of pos * inv_freq[i] for pos < n_pos, in fp64, rounded to fp32: what rope_append_kernel
+// (cos, sin) of pos * inv_freq[i] for pos < n_pos, in fp64, rounded to fp32, times turn_scale: what rope_append_kernel
 // computes on the fly, once for all steps
-__global__ void rope_table_kernel(const double* __restrict__ inv_freq, float2* __restrict__ table, int n_pos, int half) {
+__global__ void rope_table_kernel(const double* __restrict__ inv_freq, float2* __restrict__ table, int n_pos, int half, float turn_scale) {
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= (size_t)n_pos * half) return;
     const int pos = (int)(idx / half), i = (int)(idx % half);
     double s, c;
     sincos((double)pos * inv_freq[i], &s, &c);
-    table[idx] = make_float2((float)c, (float)s);
+    table[idx] = make_float2(turn_scale * (float)c, turn_scale * (float)s);
 }
 
-BLM_API int blm_rope_table(const double* inv_freq, float* table, int n_pos, int half, cudaStream_t stream) {
+BLM_API int blm_rope_table(const double* inv_freq, float* table, int n_pos, int half, float turn_scale, cudaStream_t stream) {
     if (n_pos == 0 || half == 0) return BLM_OK;
     const size_t total = (size_t)n_pos * half;
-    rope_table_kernel<<<(unsigned)((total + 255) / 256), 256, 0, stream>>>(inv_freq, (float2*)table, n_pos, half);
+    rope_table_kernel<<<(unsigned)((total + 255) / 256), 256, 0, stream>>>(inv_freq, (float2*)table, n_pos, half, turn_scale);
     return blm_check_launch("rope_table");
 }
 

@@ -20,7 +20,7 @@
 // expert with every expert's share starting at a multiple of 128 rows, and W is the experts' weights one below the other
 // ([experts x N, K]).  A table on the device names the expert of every tile of 128 rows (-1: a tile no expert owns); a block
 // looks its tile's expert up and fetches W's tiles from that expert's rows.  The tensor maps cover the whole buffers, so they
-// depend on sizes and addresses only and a step can be captured.  Its epilogues: the exact GELU (an expert without a gate),
+// depend on sizes and addresses only and a step can be captured.  Its epilogues: the exact GELU or the squared relu (an expert without a gate),
 // and fp32 sums stored as they are.
 //
 // Every mbarrier wait is bounded; a wait that runs out records a code in the caller's status word and
@@ -43,7 +43,7 @@ constexpr int kTmemCols = 512;                  // two fp32 accumulators of 256 
 constexpr unsigned kABytes = BM * BK * 2, kBBytes = BN * BK * 2;
 constexpr unsigned kSpinLimit = 1u << 22;
 
-enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESID_ADD = 2, EPI_GELU = 3, EPI_STORE_F32 = 4 };
+enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESID_ADD = 2, EPI_GELU = 3, EPI_STORE_F32 = 4, EPI_RELU2 = 5 };
 enum { TC_OK = 0, TC_TIMEOUT_FULL = 11, TC_TIMEOUT_EMPTY = 12, TC_TIMEOUT_ACCUM = 13, TC_TIMEOUT_DRAIN = 14 };
 
 struct TcArgs {
@@ -197,6 +197,11 @@ __device__ __forceinline__ void store_columns(const TcArgs& a, const float (&v)[
             if (EPI == EPI_GELU) {           // the exact form: z (1 + erf(z / sqrt 2)) / 2
                 lo = 0.5f * lo * (1.0f + erff(lo * 0.70710678118654752f));
                 hi = 0.5f * hi * (1.0f + erff(hi * 0.70710678118654752f));
+            } else if (EPI == EPI_RELU2) {   // relu(z)^2
+                lo = fmaxf(lo, 0.f);
+                hi = fmaxf(hi, 0.f);
+                lo *= lo;
+                hi *= hi;
             }
             const __nv_bfloat162 p = __floats2bfloat162_rn(lo, hi);
             packed[e] = *reinterpret_cast<const unsigned*>(&p);
@@ -395,7 +400,7 @@ int make_map(const void* base, long long ld, int rows, int K, int box_rows, bool
 BLM_API int blm_gemm_tc_supported(int M, int N, int K) { return M >= 1 && N >= 16 && K >= 64 && K % 8 == 0; }
 
 // y[M, N] = x[M, K] . w[N, K]^T (epi 0), or y[M, N / 2] = silu(gate) * up for a weight in tiles of 8 gate rows
-// followed by their 8 up rows (epi 1), or y[M, N] += x . w^T with y fp32 (epi 2: the residual stream).  x, w
+// followed by their 8 up rows (epi 1), or y[M, N] += x . w^T with y fp32 (epi 2: the residual stream), or y = relu(x . w^T)^2 (epi 5).  x, w
 // bfloat16, y bfloat16 but for epi 2; ldx, ldw, ldy in elements.
 BLM_API int blm_gemm_tc(const void* x, long long ldx, const void* w, long long ldw, void* y, long long ldy, int M, int N, int K,
                         int epi, int* status, cudaStream_t stream) {
@@ -403,7 +408,7 @@ BLM_API int blm_gemm_tc(const void* x, long long ldx, const void* w, long long l
     BLM_REQUIRE(blm_gemm_tc_supported(M, N, K), "gemm_tc: shape %d x %d x %d (K a multiple of 8, at least 64)", M, N, K);
     BLM_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0 && ((size_t)x & 15) == 0 && ((size_t)w & 15) == 0,
                 "gemm_tc: operand rows must be 16-byte aligned");
-    BLM_REQUIRE(epi == EPI_STORE || epi == EPI_RESID_ADD || (epi == EPI_SWIGLU && N % 16 == 0), "gemm_tc: epilogue %d with %d weight rows", epi, N);
+    BLM_REQUIRE(epi == EPI_STORE || epi == EPI_RESID_ADD || epi == EPI_RELU2 || (epi == EPI_SWIGLU && N % 16 == 0), "gemm_tc: epilogue %d with %d weight rows", epi, N);
     BLM_REQUIRE(epi != EPI_RESID_ADD || ((size_t)y & 15) == 0, "gemm_tc: the stream must be 16-byte aligned");
     BLM_REQUIRE(status != nullptr, "gemm_tc: no status word");
     CUtensorMap xmap, wmap;
@@ -420,6 +425,7 @@ BLM_API int blm_gemm_tc(const void* x, long long ldx, const void* w, long long l
         cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_STORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_SWIGLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_RESID_ADD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_RELU2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "gemm_tc: %s", cudaGetErrorString(e));
         opted_in = true;
     }
@@ -427,6 +433,7 @@ BLM_API int blm_gemm_tc(const void* x, long long ldx, const void* w, long long l
     const int grid = (int)(tiles < blm_sm_count() ? tiles : blm_sm_count());        // persistent: one block per SM
     if (epi == EPI_SWIGLU) gemm_tc_kernel<EPI_SWIGLU><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     else if (epi == EPI_RESID_ADD) gemm_tc_kernel<EPI_RESID_ADD><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
+    else if (epi == EPI_RELU2) gemm_tc_kernel<EPI_RELU2><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     else gemm_tc_kernel<EPI_STORE><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     return blm_check_launch("gemm_tc");
 }
@@ -435,14 +442,14 @@ BLM_API int blm_gemm_tc(const void* x, long long ldx, const void* w, long long l
 // The grouped form.  x bfloat16 [M, K] (row stride ldx): the pairs' rows expert by expert, every expert's share starting at a
 // multiple of 128 rows, M a multiple of 128 (rows no pair owns hold zeros); w bfloat16 [n_experts x N, K] (row stride ldw);
 // tile_expert int32 [M / 128] on the device: the expert of every tile of rows, -1 for a tile no expert owns.
-// epi 3: y bfloat16 [M, N] = gelu(x . w_e^T), the exact form; epi 4: y float32 [M, N] = x . w_e^T.
+// epi 3: y bfloat16 [M, N] = gelu(x . w_e^T), the exact form; epi 5: relu(x . w_e^T)^2; epi 4: y float32 [M, N] = x . w_e^T.
 BLM_API int blm_gemm_tc_grouped(const void* x, long long ldx, const void* w, long long ldw, void* y, long long ldy, int M, int N, int K,
                                 int n_experts, const int* tile_expert, int epi, int* status, cudaStream_t stream) {
     if (M == 0 || N == 0) return BLM_OK;
     BLM_REQUIRE(blm_gemm_tc_supported(M, N, K) && M % BM == 0 && n_experts >= 1, "gemm_tc_grouped: shape %d x %d x %d, %d experts", M, N, K, n_experts);
     BLM_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0 && ((size_t)x & 15) == 0 && ((size_t)w & 15) == 0,
                 "gemm_tc_grouped: operand rows must be 16-byte aligned");
-    BLM_REQUIRE(epi == EPI_GELU || epi == EPI_STORE_F32, "gemm_tc_grouped: epilogue %d", epi);
+    BLM_REQUIRE(epi == EPI_GELU || epi == EPI_RELU2 || epi == EPI_STORE_F32, "gemm_tc_grouped: epilogue %d", epi);
     BLM_REQUIRE(status != nullptr && tile_expert != nullptr, "gemm_tc_grouped: no status word or no table of tiles");
     BLM_REQUIRE((long long)n_experts * N < (1ll << 31), "gemm_tc_grouped: %d experts of %d rows", n_experts, N);
     CUtensorMap xmap, wmap;
@@ -457,6 +464,7 @@ BLM_API int blm_gemm_tc_grouped(const void* x, long long ldx, const void* w, lon
     static bool opted_in = false;
     if (!opted_in) {
         cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_GELU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_RELU2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_STORE_F32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "gemm_tc_grouped: %s", cudaGetErrorString(e));
         opted_in = true;
@@ -464,6 +472,7 @@ BLM_API int blm_gemm_tc_grouped(const void* x, long long ldx, const void* w, lon
     const long long tiles = (long long)((N + BN - 1) / BN) * (M / BM);
     const int grid = (int)(tiles < blm_sm_count() ? tiles : blm_sm_count());        // persistent: one block per SM
     if (epi == EPI_GELU) gemm_tc_kernel<EPI_GELU><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
+    else if (epi == EPI_RELU2) gemm_tc_kernel<EPI_RELU2><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     else gemm_tc_kernel<EPI_STORE_F32><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     return blm_check_launch("gemm_tc_grouped");
 }

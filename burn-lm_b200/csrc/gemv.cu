@@ -47,7 +47,7 @@ constexpr int kGemvThreads = (kConsumerWarps + 1) * 32;   // + the producer warp
 // bytes], swizzled
 constexpr unsigned kSpinLimit = 1u << 20;   // polls of a wait before it gives up (seconds; a real wait is microseconds)
 
-enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESID_ADD = 2, EPI_ROPE = 3 };
+enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESID_ADD = 2, EPI_ROPE = 3, EPI_RELU2 = 4 };     // EPI_RELU2: stores relu(sum)^2
 
 // EPI_ROPE: the product is a step's q, k and v (heads in that order); q and k are rotated by their token's
 // position and the rotated k and the v go straight to the token's place in the paged cache, q to y.  The
@@ -650,8 +650,13 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvArgs a,
                     for (int bb = 0; bb < 2; ++bb) {
                         const int b = b0 + bb;
                         if (b >= a.N) continue;
-                        if (a.y_f32) reinterpret_cast<float*>(a.y)[(size_t)b * a.ldy + m] = v[rr][bb];
-                        else reinterpret_cast<__nv_bfloat16*>(a.y)[(size_t)b * a.ldy + m] = __float2bfloat16_rn(v[rr][bb]);
+                        float val = v[rr][bb];
+                        if (a.epi == EPI_RELU2) {
+                            val = fmaxf(val, 0.f);
+                            val *= val;
+                        }
+                        if (a.y_f32) reinterpret_cast<float*>(a.y)[(size_t)b * a.ldy + m] = val;
+                        else reinterpret_cast<__nv_bfloat16*>(a.y)[(size_t)b * a.ldy + m] = __float2bfloat16_rn(val);
                     }
                 }
             }
@@ -790,7 +795,7 @@ BLM_API int blm_gemv(const void* w, long long ldw, int M, int K, const void* x, 
     BLM_REQUIRE((x != nullptr) != (resid != nullptr), "gemv: give either x or the stream to normalise");
     BLM_REQUIRE(x == nullptr || (ldx % 8 == 0 && ((size_t)x & 15) == 0), "gemv: x rows must be 16-byte aligned");
     BLM_REQUIRE(ldw % 8 == 0 && ((size_t)w & 15) == 0, "gemv: weight rows must be 16-byte aligned");
-    BLM_REQUIRE(epi == EPI_STORE || epi == EPI_SWIGLU || epi == EPI_RESID_ADD || epi == EPI_ROPE, "gemv: epilogue %d", epi);
+    BLM_REQUIRE(epi == EPI_STORE || epi == EPI_SWIGLU || epi == EPI_RESID_ADD || epi == EPI_ROPE || epi == EPI_RELU2, "gemv: epilogue %d", epi);
     if (epi == EPI_ROPE) {
         BLM_REQUIRE(rope != nullptr && rope->token_pos && rope->table && y_f32 == 0, "gemv: the rotary epilogue needs positions, a table and a bfloat16 q");
         BLM_REQUIRE(rope->hd % 16 == 0 && rope->hd >= 16, "gemv: the rotary epilogue takes head sizes in steps of 16, got %d", rope->hd);

@@ -9,8 +9,11 @@
 //   A choice limited to groups: the experts form `n_groups` equal groups of neighbours, a group's mark is the sum of its
 //   two largest choice scores (with the correction), and only experts of the `keep_groups` groups of largest mark (ties:
 //   the lower index) can be chosen; the others' choice scores count as minus infinity.
+//   The logits may get a bias, z = W_router h + b, and decide the choice themselves, the weights a softmax over the chosen
+//   logits only (scores 2).
 //   Option of the experts: the clamped gated unit, g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit),
-//   g * sigmoid(alpha g) * (u + 1).  Or a unit without a gate, W_down act(W_up x), act the exact (erf) GELU or its tanh form.
+//   g * sigmoid(alpha g) * (u + 1).  Or a unit without a gate, W_down act(W_up x), act the exact (erf) GELU, its tanh form or the
+//   squared relu.
 //
 // Everything runs on the device with sizes that depend on the step's token count only, so a step can be captured
 // in a CUDA graph: the grids cover the worst case (every expert's share padded to a tile) and blocks beyond the
@@ -24,8 +27,9 @@ BLM_API const char* blm_moe_last_error() { return g_blm_error; }
 // ---------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, int width, int n_experts, int top,
-                                 int* __restrict__ ids, float* __restrict__ weights, int softmax, const float* __restrict__ correction,
-                                 int renorm, int n_groups, int keep_groups) {
+                                 int* __restrict__ ids, float* __restrict__ weights, int scores, const float* __restrict__ bias,
+                                 const float* __restrict__ correction, int renorm, int n_groups, int keep_groups) {
+    const bool softmax = scores == 1, by_logit = scores == 2;      // else sigmoids
     extern __shared__ __align__(16) float smem[];
     float* x = smem;                     // [width]
     float* score = smem + width;         // [n_experts]: what a chosen expert is weighted by
@@ -52,8 +56,9 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
             for (int d = lane; d < width; d += 32) z = fmaf(w[d], x[d], z);
         }
         z = warp_sum(z);
+        if (bias) z += bias[e];
         // (a row of no sequence may hold anything, a NaN too: its score is 0, so that it still names experts that exist)
-        if (lane == 0) score[e] = softmax ? (z == z ? z : 0.f) : (z == z ? 1.0f / (1.0f + expf(-z)) : 0.f);
+        if (lane == 0) score[e] = softmax || by_logit ? (z == z ? z : 0.f) : (z == z ? 1.0f / (1.0f + expf(-z)) : 0.f);
     }
     __syncthreads();
     if (warp == 0) {
@@ -92,7 +97,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
             }
             __syncwarp();
         }
-        float total = 0.f;
+        float total = 0.f, first = 0.f;
         for (int k = 0; k < top; ++k) {
             float best = -INFINITY;
             int arg = 0x7fffffff;
@@ -107,7 +112,11 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
                 if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
             }
             if (arg == 0x7fffffff) arg = k;              // (scores that compare with nothing: still an expert that exists)
-            const float wgt = score[arg];
+            float wgt = score[arg];
+            if (by_logit) {                              // without a correction the first chosen logit is the largest
+                if (k == 0) first = wgt;
+                wgt = expf(wgt - first);
+            }
             total += wgt;
             if (lane == 0) {
                 ids[(size_t)n * top + k] = arg;
@@ -116,17 +125,22 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
             }
             __syncwarp();
         }
-        if (renorm)
-            for (int k = lane; k < top; k += 32) weights[(size_t)n * top + k] = weights[(size_t)n * top + k] / (total + 1e-20f);
+        if (renorm || by_logit) {
+            const float inv_of = by_logit ? total : total + 1e-20f;
+            for (int k = lane; k < top; k += 32) weights[(size_t)n * top + k] = weights[(size_t)n * top + k] / inv_of;
+        }
     }
 }
 
 BLM_API int blm_moe_route(const void* h, int dtype, const float* router, int n_tokens, int width, int n_experts, int top, int* ids,
-                          float* weights, int softmax, const float* correction, int renorm, int n_groups, int keep_groups,
-                          cudaStream_t stream) {
+                          float* weights, int scores, const float* bias, const float* correction, int renorm, int n_groups,
+                          int keep_groups, cudaStream_t stream) {
+    // scores 0: sigmoids; 1: a softmax over all experts; 2: the logits decide, the weights a softmax over the chosen (no
+    // correction then: the first chosen logit must be the largest).  bias float32 [experts] or null
     // n_groups <= 1: the choice is among all experts
     if (n_tokens == 0) return BLM_OK;
     BLM_REQUIRE(n_tokens > 0 && width > 0 && n_experts > 0 && top > 0 && top <= n_experts, "moe_route: bad sizes");
+    BLM_REQUIRE(scores >= 0 && scores <= 2 && (scores != 2 || correction == nullptr), "moe_route: scores of kind %d", scores);
     if (n_groups < 1) n_groups = 1;
     BLM_REQUIRE(n_experts % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups &&
                 (long long)keep_groups * (n_experts / n_groups) >= top,
@@ -136,11 +150,11 @@ BLM_API int blm_moe_route(const void* h, int dtype, const float* router, int n_t
     // a warp an expert where the experts are few (the warps' dot products wait for memory side by side), sixteen warps at most
     const int threads = n_experts <= 4 ? 128 : (n_experts >= 16 ? 512 : 32 * n_experts);
     if (dtype == BLM_F32)
-        moe_route_kernel<float><<<n_tokens, threads, smem, stream>>>((const float*)h, router, width, n_experts, top, ids, weights, softmax,
+        moe_route_kernel<float><<<n_tokens, threads, smem, stream>>>((const float*)h, router, width, n_experts, top, ids, weights, scores, bias,
                                                                  correction, renorm, n_groups, keep_groups);
     else if (dtype == BLM_BF16)
         moe_route_kernel<__nv_bfloat16><<<n_tokens, threads, smem, stream>>>((const __nv_bfloat16*)h, router, width, n_experts, top, ids,
-                                                                         weights, softmax, correction, renorm, n_groups, keep_groups);
+                                                                         weights, scores, bias, correction, renorm, n_groups, keep_groups);
     else
         return blm_fail(BLM_BAD_ARGUMENT, "moe_route: dtype %d", dtype);
     return blm_check_launch("moe_route");
@@ -219,7 +233,7 @@ template <typename T> __device__ __forceinline__ float as_input(float v) { retur
 
 // The unit of an expert.  plain 0, the gated units: limit <= 0: silu(g) * u; limit > 0, the clamped unit: g = min(g, limit),
 // u = clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + 1).  plain 1 and 2, the units without a gate (the weight then
-// holds the up rows only, and u is not computed): the exact GELU, g (1 + erf(g / sqrt 2)) / 2, and its tanh form.
+// holds the up rows only, and u is not computed): the exact GELU, g (1 + erf(g / sqrt 2)) / 2, and its tanh form.  plain 3: relu(g)^2.
 struct GluAct {
     float limit, alpha;
     int plain;
@@ -227,6 +241,10 @@ struct GluAct {
 __device__ __forceinline__ float glu_act(float g, float u, GluAct a) {
     if (a.plain == 1) return 0.5f * g * (1.0f + erff(g * 0.70710678118654752f));
     if (a.plain == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+    if (a.plain == 3) {
+        g = fmaxf(g, 0.f);
+        return g * g;
+    }
     if (a.limit <= 0.f) return g / (1.0f + expf(-g)) * u;
     g = fminf(g, a.limit);
     u = fminf(fmaxf(u, -a.limit), a.limit);
@@ -949,10 +967,10 @@ BLM_API int blm_moe_experts(const void* h, int dtype, const float* weights, cons
                             int scale_input, float act_limit, float act_alpha, int plain_unit, int down_splits, cudaStream_t stream) {
     // down_splits: blm_moe_down_splits(...) of the same sizes; y holds that many planes [places][width]
     // plain_unit 0: the gated units, w_gu [experts][2 ff][width]; act_limit <= 0: silu(gate) * up; > 0: the clamped unit with
-    // that limit and act_alpha.  plain_unit 1 (exact GELU) or 2 (tanh GELU): no gate, w_gu [experts][ff][width]
+    // that limit and act_alpha.  plain_unit 1 (exact GELU), 2 (tanh GELU) or 3 (squared relu): no gate, w_gu [experts][ff][width]
     if (n_tokens == 0) return BLM_OK;
     BLM_REQUIRE(n_tokens > 0 && width > 0 && ff > 0 && n_experts > 0 && top > 0, "moe_experts: bad sizes");
-    BLM_REQUIRE(plain_unit >= 0 && plain_unit <= 2, "moe_experts: unit %d", plain_unit);
+    BLM_REQUIRE(plain_unit >= 0 && plain_unit <= 3, "moe_experts: unit %d", plain_unit);
     const GluAct glu{act_limit, act_alpha, plain_unit};
     const long long pairs = (long long)n_tokens * top;
     const long long tiles = (pairs + kBM - 1) / kBM + n_experts;      // every expert's share may end in a tile that is not full

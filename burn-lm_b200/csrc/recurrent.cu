@@ -1,5 +1,5 @@
 // Recurrent mixers over the packed tokens of a step: the short causal convolution with its carried inputs, the
-// state-space scan (a scalar decay per head), the gated delta rule (a decay per key channel, an error-correcting
+// state-space scan (a scalar decay per head), the selective scan (a decay per channel and state), the gated delta rule (a decay per key channel, an error-correcting
 // write), and the group-wise RMS norm with a gate that follows either.  Everything here is fp32.
 //
 // What a sequence carries lives in a fixed-size block per cache slot, twice: a step that starts at position p reads
@@ -658,4 +658,177 @@ BLM_API int blm_gated_group_norm(const float* y, long long y_stride, const float
     else
         return blm_fail(BLM_BAD_ARGUMENT, "gated_group_norm: out dtype %d", out_dtype);
     return blm_check_launch("gated_group_norm");
+}
+
+// ---------------------------------------------------------------------------------------------
+// Selective scan (Mamba).  Per channel c and state n:
+//     S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B[n],   y_c = sum_n S[c, n] C[n] + D_c x_c,
+//     out_c = scale y_c silu(z_c),   dt_c = softplus(dt_raw_c + dt_bias_c),   A = -exp(A_log)
+// x float32 [T, *] (after convolution and silu), B and C columns of low [T, *], z columns of another row.  dt_raw is given
+// [T, C], or (dt_w) formed here from the first `rank` columns of low and dt_w [C, rank]: for single tokens, where a product
+// of its own would be a launch for a few kilobytes.  A block owns (sequence, kSelThreads / G channels); G lanes share a channel,
+// RN neighbouring states each in registers; tokens come in chunks of kChunk through shared memory, and a chunk's results
+// leave through shared memory too, gated and converted by rows.  The state is stored as [channel][state].  AT double: state
+// and sums in float64 inside a step (the 32-bit path), else float with exp2 of A scaled by log2 e.
+// ---------------------------------------------------------------------------------------------
+constexpr int kSelThreads = 128, kSelLanes = 4, kSelChannels = kSelThreads / kSelLanes;
+
+struct SelArgs {
+    const float* x; long long x_stride;
+    const float* low; long long low_stride; int b_col0, c_col0;
+    const float* dt_raw; long long dt_stride;
+    const void* dt_w; int dt_w_bf16, rank;
+    const float* dt_bias; const float* A_log; const float* D;
+    const float* z; long long z_stride;
+    void* out; long long out_stride; float scale;
+    int channels, n_states;
+};
+
+template <int RN, typename AT, typename TO>
+__global__ void __launch_bounds__(kSelThreads)
+    selective_scan_kernel(SelArgs a, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
+                          const int* __restrict__ start_pos, float* __restrict__ state, long long slot_stride, long long copy_stride,
+                          long long state_off) {
+    constexpr int NP = RN * kSelLanes, CH = kSelChannels;
+    __shared__ __align__(16) float Bs[kChunk][NP], Cs[kChunk][NP];
+    __shared__ float dts[kChunk][CH], xs[kChunk][CH], ys[kChunk][CH];
+    const int seq = blockIdx.x, c0 = blockIdx.y * CH;
+    const ScanSeq sq = scan_seq(seq, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off);
+    if (sq.n_new <= 0) return;
+    const int tid = threadIdx.x, ch = tid / kSelLanes, g = tid % kSelLanes;
+    const int c = c0 + ch, n0 = g * RN;
+    const bool live = c < a.channels;
+    AT s[RN], A[RN];
+#pragma unroll
+    for (int r = 0; r < RN; ++r) {
+        const bool in = live && n0 + r < a.n_states;
+        const size_t at = (size_t)c * a.n_states + n0 + r;
+        s[r] = in && sq.read ? (AT)sq.read[at] : (AT)0;
+        if (sizeof(AT) == 8) A[r] = in ? (AT)-exp((double)a.A_log[at]) : (AT)0;
+        else A[r] = in ? (AT)(-expf(a.A_log[at]) * 1.4426950408889634f) : (AT)0;
+    }
+    for (int t0 = 0; t0 < sq.n_new; t0 += kChunk) {
+        const int nt = min(kChunk, sq.n_new - t0);
+        const size_t row0 = (size_t)(sq.first + t0);
+        __syncthreads();
+        for (int e = tid; e < nt * NP; e += kSelThreads) {
+            const int t = e / NP, n = e % NP;
+            const float* low = a.low + (row0 + t) * a.low_stride;
+            Bs[t][n] = n < a.n_states ? low[a.b_col0 + n] : 0.f;
+            Cs[t][n] = n < a.n_states ? low[a.c_col0 + n] : 0.f;
+        }
+        for (int e = tid; e < nt * CH; e += kSelThreads) {
+            const int t = e / CH, k = e % CH, cc = c0 + k;
+            float dt = 0.f, x = 0.f;
+            if (cc < a.channels) {
+                x = a.x[(row0 + t) * a.x_stride + cc];
+                float raw = a.dt_bias[cc];
+                if (a.dt_w != nullptr) {
+                    const float* low = a.low + (row0 + t) * a.low_stride;
+                    float sum = 0.f;
+                    if (a.dt_w_bf16) {
+                        const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.dt_w) + (size_t)cc * a.rank;
+#pragma unroll 8
+                        for (int k2 = 0; k2 < a.rank; ++k2) sum = fmaf(__bfloat162float(w[k2]), low[k2], sum);
+                    } else {
+                        const float* w = reinterpret_cast<const float*>(a.dt_w) + (size_t)cc * a.rank;
+#pragma unroll 8
+                        for (int k2 = 0; k2 < a.rank; ++k2) sum = fmaf(w[k2], low[k2], sum);
+                    }
+                    raw += sum;
+                } else {
+                    raw += a.dt_raw[(row0 + t) * a.dt_stride + cc];
+                }
+                dt = softplus_r(raw);
+            }
+            dts[t][k] = dt;
+            xs[t][k] = x;
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int t = 0; t < nt; ++t) {
+            const AT dt = (AT)dts[t][ch], dx = dt * (AT)xs[t][ch];
+            AT part[2] = {0, 0};
+#pragma unroll
+            for (int r = 0; r < RN; ++r) {
+                AT dec;
+                if (sizeof(AT) == 8) dec = (AT)exp((double)(dt * A[r]));
+                else dec = (AT)exp2f((float)(dt * A[r]));
+                s[r] = dec * s[r] + dx * (AT)Bs[t][n0 + r];
+                part[r & 1] += s[r] * (AT)Cs[t][n0 + r];
+            }
+            const AT y = group_sum<kSelLanes>(part[0] + part[1]);
+            if (g == 0) ys[t][ch] = (float)(y + (AT)(live ? a.D[c] : 0.f) * (AT)xs[t][ch]);
+        }
+        __syncthreads();
+        for (int e = tid; e < nt * CH; e += kSelThreads) {
+            const int t = e / CH, k = e % CH, cc = c0 + k;
+            if (cc < a.channels) {
+                const float z = a.z[(row0 + t) * a.z_stride + cc];
+                reinterpret_cast<TO*>(a.out)[(row0 + t) * a.out_stride + cc] = from_f32<TO>(a.scale * ys[t][k] * silu_f(z));
+            }
+        }
+    }
+    if (live) {
+#pragma unroll
+        for (int r = 0; r < RN; ++r)
+            if (n0 + r < a.n_states) sq.write[(size_t)c * a.n_states + n0 + r] = (float)s[r];
+    }
+}
+
+template <typename AT, typename TO>
+static int launch_selective(const SelArgs& a, int n_seqs, const int* cu_seqlens, const int* slot_of_seq, const int* start_pos, float* state,
+                            long long slot_stride, long long copy_stride, long long state_off, cudaStream_t stream) {
+    dim3 grid(n_seqs, (a.channels + kSelChannels - 1) / kSelChannels);
+#define BLM_SEL(RN)                                                                                                                      \
+    if (a.n_states <= RN * kSelLanes) {                                                                                                  \
+        selective_scan_kernel<RN, AT, TO><<<grid, kSelThreads, 0, stream>>>(a, cu_seqlens, slot_of_seq, start_pos, state, slot_stride,    \
+                                                                            copy_stride, state_off);                                     \
+        return blm_check_launch("selective_scan");                                                                                       \
+    }
+    BLM_SEL(2) BLM_SEL(4) BLM_SEL(6) BLM_SEL(8) BLM_SEL(16) BLM_SEL(32)
+#undef BLM_SEL
+    return blm_fail(BLM_BAD_ARGUMENT, "selective_scan: %d states a channel; this kernel takes up to %d", a.n_states, 32 * kSelLanes);
+}
+
+BLM_API int blm_selective_scan(const float* x, long long x_stride, const float* low, long long low_stride, int b_col0, int c_col0,
+                               const float* dt_raw, long long dt_stride, const void* dt_w, int dt_w_dtype, int rank, const float* dt_bias,
+                               const float* A_log, const float* D, const float* z, long long z_stride, void* out, int out_dtype,
+                               long long out_stride, float scale, int channels, int n_states, const int* cu_seqlens, const int* slot_of_seq,
+                               const int* start_pos, int n_seqs, float* state, long long slot_stride,
+                               long long copy_stride, long long state_off, cudaStream_t stream) {
+    // dt_raw [T, dt_stride], or null and dt_w [channels, rank] (the step sizes' projection of low's first columns).
+    // out float32: the 32-bit path (sums in float64).  Rows of no sequence are left as they are.
+    if (n_seqs == 0) return BLM_OK;
+    BLM_REQUIRE(channels > 0 && n_states > 0 && n_seqs > 0, "selective_scan: bad sizes");
+    BLM_REQUIRE((dt_raw == nullptr) != (dt_w == nullptr) && (dt_w == nullptr || rank > 0), "selective_scan: give step sizes or their projection");
+    BLM_REQUIRE((channels + kSelChannels - 1) / kSelChannels <= 65535, "selective_scan: %d channels", channels);
+    SelArgs a;
+    a.x = x; a.x_stride = x_stride; a.low = low; a.low_stride = low_stride; a.b_col0 = b_col0; a.c_col0 = c_col0;
+    a.dt_raw = dt_raw; a.dt_stride = dt_stride; a.dt_w = dt_w; a.dt_w_bf16 = dt_w_dtype == BLM_BF16; a.rank = rank;
+    a.dt_bias = dt_bias; a.A_log = A_log; a.D = D; a.z = z; a.z_stride = z_stride;
+    a.out = out; a.out_stride = out_stride; a.scale = scale; a.channels = channels; a.n_states = n_states;
+#define BLM_SEL_ARGS a, n_seqs, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off, stream
+    if (out_dtype == BLM_F32) return launch_selective<double, float>(BLM_SEL_ARGS);
+    if (out_dtype == BLM_BF16) return launch_selective<float, __nv_bfloat16>(BLM_SEL_ARGS);
+#undef BLM_SEL_ARGS
+    return blm_fail(BLM_BAD_ARGUMENT, "selective_scan: out dtype %d", out_dtype);
+}
+
+// out[n, d] = src[n, col0 + d] in out's type: some columns of a wider fp32 row as a product's operand
+template <typename TO>
+__global__ void take_cols_kernel(const float* __restrict__ src, long long stride, int col0, TO* __restrict__ out, int width, int total) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < total) out[i] = from_f32<TO>(src[(size_t)(i / width) * stride + col0 + i % width]);
+}
+
+BLM_API int blm_take_cols(const float* src, long long stride, int col0, void* out, int out_dtype, int n_rows, int width, cudaStream_t stream) {
+    if (n_rows == 0) return BLM_OK;
+    BLM_REQUIRE(width > 0 && col0 >= 0 && (long long)n_rows * width < (1ll << 31), "take_cols: bad sizes");
+    const int total = n_rows * width;
+    if (out_dtype == BLM_F32) take_cols_kernel<float><<<(total + 255) / 256, 256, 0, stream>>>(src, stride, col0, (float*)out, width, total);
+    else if (out_dtype == BLM_BF16)
+        take_cols_kernel<__nv_bfloat16><<<(total + 255) / 256, 256, 0, stream>>>(src, stride, col0, (__nv_bfloat16*)out, width, total);
+    else return blm_fail(BLM_BAD_ARGUMENT, "take_cols: out dtype %d", out_dtype);
+    return blm_check_launch("take_cols");
 }

@@ -121,7 +121,7 @@ BLM_API int blm_sandwich_norm(float* resid, const void* delta, const void* delta
 }
 
 // ---------------------------------------------------------------------------------------------
-// out = act(x + bias).  kind 0: identity.  kind 1: xIELU with the two numbers params = (p, q):
+// out = act(x + bias).  kind 0: identity.  kind 2: tanh.  kind 3: relu(z)^2.  kind 1: xIELU with the two numbers params = (p, q):
 //     z > 0:  softplus(p) z^2 + z / 2;     z <= 0:  (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2
 // ---------------------------------------------------------------------------------------------
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
@@ -140,6 +140,10 @@ __global__ void bias_act_kernel(const TI* __restrict__ x, const float* __restric
         if (bias) z += bias[c];
         if (kind == 1) z = z > 0.f ? ap * z * z + 0.5f * z : an * (expm1f(z) - z) + 0.5f * z;
         else if (kind == 2) z = tanhf(z);
+        else if (kind == 3) {
+            z = fmaxf(z, 0.f);
+            z *= z;
+        }
         out[row + c] = from_f32<TA>(z);
     }
 }
@@ -147,7 +151,7 @@ __global__ void bias_act_kernel(const TI* __restrict__ x, const float* __restric
 BLM_API int blm_bias_act(const void* x, int x_dtype, const float* bias, const float* params, void* out, int out_dtype, int n,
                          int width, int kind, cudaStream_t stream) {
     if (n == 0) return BLM_OK;
-    BLM_REQUIRE(n > 0 && width > 0 && (kind == 0 || kind == 1 || kind == 2), "bias_act: bad sizes or kind");
+    BLM_REQUIRE(n > 0 && width > 0 && kind >= 0 && kind <= 3, "bias_act: bad sizes or kind");
     BLM_REQUIRE(kind != 1 || params != nullptr, "bias_act: the activation needs its two numbers");
     BLM_REQUIRE(n <= 65535, "bias_act: %d rows; this kernel takes 65,535", n);
     const int threads = 256;
@@ -231,4 +235,33 @@ BLM_API int blm_softcap(float* x, float cap, size_t total, cudaStream_t stream) 
     const int blocks = (int)(want < 65535u * 16u ? want : 65535u * 16u);
     softcap_kernel<<<blocks, threads, 0, stream>>>(x, cap, total);
     return blm_check_launch("softcap");
+}
+
+// ---------------------------------------------------------------------------------------------
+// The stream at the start of a pass over looped layers: x <- x (+ delta, a pending output) (+ again, the embedding's output)
+// + step [D] for every row, fp32 in place.
+// ---------------------------------------------------------------------------------------------
+template <typename TD>
+__global__ void pass_entry_kernel(float* __restrict__ x, const TD* __restrict__ delta, const float* __restrict__ again,
+                                  const float* __restrict__ step, int width) {
+    const size_t row = (size_t)blockIdx.y * width;
+    const int d = blockIdx.x * blockDim.x + threadIdx.x;
+    if (d >= width) return;
+    float v = x[row + d];
+    if (delta) v += to_f32(delta[row + d]);
+    if (again) v += again[row + d];
+    x[row + d] = v + step[d];
+}
+
+BLM_API int blm_pass_entry(float* x, const void* delta, int delta_dtype, const float* again, const float* step, int n_rows, int width,
+                           cudaStream_t stream) {
+    if (n_rows == 0) return BLM_OK;
+    BLM_REQUIRE(n_rows > 0 && n_rows <= 65535 && width > 0 && step != nullptr, "pass_entry: bad sizes");
+    const int threads = 256;
+    dim3 grid((width + threads - 1) / threads, n_rows);
+    if (delta_dtype == BLM_F32) pass_entry_kernel<float><<<grid, threads, 0, stream>>>(x, (const float*)delta, again, step, width);
+    else if (delta_dtype == BLM_BF16)
+        pass_entry_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>(x, (const __nv_bfloat16*)delta, again, step, width);
+    else return blm_fail(BLM_BAD_ARGUMENT, "pass_entry: dtype %d", delta_dtype);
+    return blm_check_launch("pass_entry");
 }

@@ -76,8 +76,8 @@ _protos = {
         "blm_add_rmsnorm": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int,
                             c_float, c_void_p],
         "blm_rope_append": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
-                            c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
-        "blm_rope_table": [c_void_p, c_void_p, c_int, c_int, c_void_p],
+                            c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p],
+        "blm_rope_table": [c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
         "blm_swiglu": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "blm_convert": [c_void_p, c_int, c_void_p, c_int, c_size_t, c_void_p],
         "blm_decode_advance": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
@@ -93,10 +93,11 @@ _protos = {
                                c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p, c_void_p,
                                c_void_p, c_int, c_void_p],
         "blm_attention_sink": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                               c_void_p, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                               c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_float, c_void_p],
-        "blm_head_norm_rope_append": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
-                                      c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
+                               c_void_p, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_float, c_void_p, c_int, c_int,
+                               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_float,
+                               c_float, c_float, c_float, c_void_p],
+        "blm_head_norm_rope_append": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
+                                      c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
                                       c_void_p, c_void_p, c_int, c_void_p],
         "blm_attention_sink_prompt_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
         "blm_attention_sink_decode_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
@@ -108,6 +109,7 @@ _protos = {
         "blm_bias_act": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "blm_weighted_sum": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_size_t, c_void_p],
         "blm_pack_cols": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p],
+        "blm_pass_entry": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "blm_softcap": [c_void_p, c_float, c_size_t, c_void_p],
     },
     "recurrent": {
@@ -126,6 +128,10 @@ _protos = {
                            c_longlong, c_int, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int,
                            c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_longlong,
                            c_void_p],
+        "blm_selective_scan": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int,
+                               c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_float, c_int, c_int,
+                               c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p],
+        "blm_take_cols": [c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
         "blm_gated_group_norm": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                  c_float, c_void_p, c_int, c_longlong, c_int, c_void_p],
     },
@@ -152,8 +158,8 @@ _protos = {
         "blm_sigmoid_gate": [c_void_p, c_int, c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p],
     },
     "moe": {
-        "blm_moe_route": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                          c_void_p],
+        "blm_moe_route": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                          c_int, c_int, c_void_p],
         "blm_moe_group": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
         "blm_moe_experts": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                             c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p],
@@ -363,8 +369,9 @@ def kv_page_elems(n_kv, key_dim, value_dim) -> int:
     return n_kv * PAGE * (key_dim + value_dim)
 
 
-def _flat_pool(pool, n_kv, key_dim, value_dim):
-    elems = kv_page_elems(n_kv, key_dim, value_dim)
+def _flat_pool(pool, n_kv, key_dim, value_dim, maps=1):
+    """Elements of a page of n_kv key heads (every map counted) and n_kv / maps value heads."""
+    elems = kv_page_elems(n_kv // maps, maps * key_dim, value_dim)
     if not pool.is_contiguous() or pool.numel() != pool.shape[0] * elems:
         raise KernelError(f"the cache pool must hold pages of {elems} elements ({n_kv} kv heads, keys of {key_dim}, values of {value_dim})")
     return elems
@@ -394,17 +401,21 @@ def qk_norm_append(proj, step, pool, block_table, q_out, n_heads, n_kv, key_dim,
 
 
 def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, key_dim, value_dim, q_weight=None, k_weight=None,
-                          eps=0.0, value_norm=False, freq=None, rotary_dims=0, halves=False):
+                          eps=0.0, value_norm=False, freq=None, rotary_dims=0, halves=False, turn_scale=1.0, maps=1):
     """What follows a fused projection [q | k | v | ...] (float32 [N, >= (n_heads + n_kv) key_dim + n_kv value_dim]), head by
     head: every head of q is divided by its root mean square (eps inside the root) and multiplied by `q_weight` (float32
     [key_dim], the same for all heads; None: q stays as it is), every head of k likewise with `k_weight`; the first
     `rotary_dims` lanes of every q and k head turn by position * freq[i] (freq float64 [rotary_dims / 2]), lanes (2i, 2i + 1)
-    together, or (i, i + rotary_dims / 2) with `halves`; with `value_norm` every head of v is divided by its root mean square
-    (no weight).  q goes to `q_out` [N, n_heads key_dim], k and v to the token's place in the paged cache."""
-    _need_cuda(proj, pool, block_table, q_out, q_weight, k_weight, freq)
+    together, or (i, i + rotary_dims / 2) with `halves`, cosine and sine both times `turn_scale`; with `value_norm` every head
+    of v is divided by its root mean square (no weight).  q goes to `q_out` [N, n_heads key_dim], k and v to the token's place
+    in the paged cache.  `maps` 2: a head has two queries and two keys, [head][map][key_dim], over one value; n_heads and
+    n_kv count every map.  `proj` may be a column range of a wider tensor."""
+    _need_cuda(pool, block_table, q_out, q_weight, k_weight, freq)
     _f32(proj, q_weight, k_weight)
+    if not proj.is_cuda:
+        raise KernelError("burn-lm_b200 kernels run on a CUDA device only; got a CPU tensor")
     n = proj.shape[0]
-    qc, kc, vc = n_heads * key_dim, n_kv * key_dim, n_kv * value_dim
+    qc, kc, vc = n_heads * key_dim, n_kv * key_dim, n_kv // maps * value_dim
     if proj.dim() != 2 or proj.shape[1] < qc + kc + vc or proj.stride(1) != 1:
         raise KernelError("head_norm_rope_append: the projection is float32 [N, q + k + v (+ more)]")
     if tuple(q_out.shape) != (n, qc) or q_out.dtype != pool.dtype or not q_out.is_contiguous():
@@ -414,14 +425,15 @@ def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, k
             raise KernelError("head_norm_rope_append: the norms' weights are float32 [key_dim]")
     if rotary_dims and (freq is None or freq.dtype != torch.float64 or freq.numel() != rotary_dims // 2):
         raise KernelError("head_norm_rope_append: freq must be float64 [rotary_dims / 2]")
-    _call("attention_sink", "blm_head_norm_rope_append", _ptr(proj), c_longlong(proj.stride(0)), n, n_heads, n_kv, key_dim, value_dim,
-          _ptr(q_weight), _ptr(k_weight), c_float(eps), 1 if value_norm else 0, _ptr(freq), int(rotary_dims), 1 if halves else 0,
-          _ptr(q_out), _ptr(pool), _code(pool.dtype), c_longlong(_flat_pool(pool, n_kv, key_dim, value_dim)), PAGE, _ptr(step.token_seq),
+    _call("attention_sink", "blm_head_norm_rope_append", _ptr(proj), c_longlong(proj.stride(0)), n, n_heads, n_kv, int(maps), key_dim,
+          value_dim, _ptr(q_weight), _ptr(k_weight), c_float(eps), 1 if value_norm else 0, _ptr(freq), int(rotary_dims), 1 if halves else 0,
+          c_float(turn_scale), _ptr(q_out), _ptr(pool), _code(pool.dtype), c_longlong(_flat_pool(pool, n_kv, key_dim, value_dim, maps)), PAGE, _ptr(step.token_seq),
           _ptr(step.token_pos), _ptr(step.slot_of_seq), _ptr(block_table), block_table.shape[1], _stream())
 
 
-def attention_sink_scratch_floats(n_tokens, n_heads, value_dim, n_splits) -> int:
-    return 0 if n_splits <= 1 else n_tokens * n_heads * n_splits * (value_dim + 2)
+def attention_sink_scratch_floats(n_tokens, n_heads, value_dim, n_splits, maps=1) -> int:
+    """(n_heads counts every map; with two maps the kernels always leave their sums for the one that forms the difference)"""
+    return 0 if n_splits <= 1 and maps == 1 else n_tokens * n_heads * n_splits * (value_dim + 2)
 
 
 def attention_sink_prompt_takes(dtype, key_dim, value_dim, max_q_len, n_heads) -> bool:
@@ -436,7 +448,8 @@ def attention_sink_decode_takes(dtype, key_dim, value_dim, n_heads, n_kv) -> boo
 
 
 def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, value_dim, scale, window, keep_first=0, sink=True,
-                   gate=None, gate_stride=0, max_q_len=1, n_splits=1, scratch=None, head_scale=None, sink_logit=None, softcap=0.0):
+                   gate=None, gate_stride=0, max_q_len=1, n_splits=1, scratch=None, head_scale=None, sink_logit=None, softcap=0.0,
+                   chunk=0, gate_lanes=0, out_scale=1.0, maps=1, difference=(0.0, 1.0, 0.0)):
     """Attention of the step's tokens over the paged cache (after the append) where the query at position i sees the
     key at j when j <= i and (i - j < window or j < keep_first); softmax with `sink` added to its denominator (one more
     entry of score 0 without a value); keys of `key_dim` and values of `value_dim` lanes; `gate`: a float32 tensor
@@ -445,19 +458,27 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
     `head_scale` float32 [n_heads]: head h's scores are scale * head_scale[h] * q.k; `softcap` > 0: a score s becomes
     softcap * tanh(s / softcap) before the softmax; `sink_logit` float32 [n_heads]: the sink's score is that number instead
     of 0 (exp(sink_logit[h]) joins the denominator).
+    `chunk` > 0: instead of a window, a position sees the keys of its own chunk of the sequence (j // chunk == i // chunk).
+    `gate_lanes` = value_dim: the gate has a number per lane, at n * gate_stride + h * value_dim + d.  The result is multiplied
+    by `out_scale`; `out` may be a column range of a wider tensor.
+    `maps` 2, differential attention: a head has two queries and a key/value head two keys, [head][map][key_dim], over one
+    value; n_heads and n_kv count every map, out is [N, n_heads / 2 value_dim], and `difference` = (lambda, c, eps) gives
+    o = a_1 - lambda a_2, out = o / sqrt(mean(o^2) + eps) * c per head; it needs `scratch` for any n_splits.
 
     `max_q_len`: the longest run of new tokens of one sequence (a bound is enough): bfloat16 steps of 8 or more run
     the tensor-core prompt kernel, 64 query rows a block (it reads step.cu_seqlens and step.start_pos); shorter ones
     the tensor-core decode kernel (bfloat16, up to 16 query heads a kv head) or else the row kernel, a block per (row,
     kv head) either, whose keys `n_splits` > 1 cuts over that many blocks (it then needs `scratch`:
     attention_sink_scratch_floats(...) float32)."""
-    _need_cuda(q, pool, block_table, out, scratch, head_scale, sink_logit)
+    _need_cuda(q, pool, block_table, scratch, head_scale, sink_logit)
     _f32(head_scale, sink_logit)
+    if not out.is_cuda or out.stride(1) != 1:
+        raise KernelError("attention_sink: out is a CUDA tensor with unit stride along its rows")
     for t in (head_scale, sink_logit):
         if t is not None and t.numel() != n_heads:
             raise KernelError("attention_sink: head_scale and sink_logit have a number per query head")
     n = q.shape[0]
-    if tuple(q.shape) != (n, n_heads * key_dim) or tuple(out.shape) != (n, n_heads * value_dim) or q.dtype != pool.dtype \
+    if tuple(q.shape) != (n, n_heads * key_dim) or tuple(out.shape) != (n, n_heads // maps * value_dim) or q.dtype != pool.dtype \
             or out.dtype != pool.dtype:
         raise KernelError("attention_sink: q [N, heads * key_dim] and out [N, heads * value_dim] in the cache's dtype")
     if gate is not None and (not gate.is_cuda or gate.dtype != torch.float32):
@@ -465,28 +486,38 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
     prompt = attention_sink_prompt_takes(pool.dtype, key_dim, value_dim, max_q_len, n_heads) and getattr(step, "cu_seqlens", None) is not None
     if prompt:
         n_splits = 1
-    if n_splits > 1:
-        need = attention_sink_scratch_floats(n, n_heads, value_dim, n_splits)
+    need = attention_sink_scratch_floats(n, n_heads, value_dim, n_splits, maps)
+    if need:
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"attention_sink: {n_splits} splits need {need} float32 of scratch")
     cu = step.cu_seqlens if prompt else None
-    _call("attention_sink", "blm_attention_sink", _ptr(q), _ptr(pool), _code(pool.dtype), _flat_pool(pool, n_kv, key_dim, value_dim),
+    _call("attention_sink", "blm_attention_sink", _ptr(q), _ptr(pool), _code(pool.dtype), _flat_pool(pool, n_kv, key_dim, value_dim, maps),
           _ptr(block_table), block_table.shape[1], _ptr(step.token_seq), _ptr(step.token_pos), _ptr(step.slot_of_seq), _ptr(cu),
           _ptr(step.start_pos if prompt else None), (cu.numel() - 1) if prompt else 0, int(max_q_len), _ptr(gate), int(gate_stride),
-          _ptr(out), _ptr(scratch), int(n_splits), n, n_heads, n_kv, key_dim, value_dim, PAGE, int(window), int(keep_first),
-          c_float(scale), 1 if sink else 0, _ptr(head_scale), _ptr(sink_logit if sink else None), c_float(softcap or 0.0), _stream(),
-          kernels=2 if n_splits > 1 else 1)
+          int(gate_lanes), _ptr(out), c_longlong(out.stride(0)), c_float(out_scale), _ptr(scratch if need else None), int(n_splits), n, n_heads,
+          n_kv, int(maps), key_dim, value_dim, PAGE, int(window), int(chunk), int(keep_first), c_float(scale), 1 if sink else 0,
+          _ptr(head_scale), _ptr(sink_logit if sink else None), c_float(softcap or 0.0), *(c_float(v) for v in difference), _stream(),
+          kernels=2 if need else 1)
 
 
-def moe_route(h, router, top, softmax=False, correction=None, renormalise=False, n_groups=1, keep_groups=1):
+SCORES_SIGMOID, SCORES_SOFTMAX, SCORES_CHOSEN_SOFTMAX = 0, 1, 2
+
+
+def moe_route(h, router, top, softmax=False, correction=None, renormalise=False, n_groups=1, keep_groups=1, scores=None, bias=None):
     """(ids int32 [N, top], weights float32 [N, top]): every token's `top` experts of largest sigmoid(router h), in
     falling order (the lower index on a tie), with those scores.  router float32 [experts, D]; sums in float32.
     `softmax`: the scores are softmax(router h) over all experts.  `correction` float32 [experts]: added to the scores for
     the choice only; the weights stay the scores.  `renormalise`: the chosen weights are divided by their sum + 1e-20.
     `n_groups` > 1: the experts form that many equal groups of neighbours, a group's mark is the sum of its two largest
-    choice scores (correction included), and only experts of the `keep_groups` groups of largest mark can be chosen."""
-    _need_cuda(h, router, correction)
-    _f32(correction)
+    choice scores (correction included), and only experts of the `keep_groups` groups of largest mark can be chosen.
+    `bias` float32 [experts] joins the logits.  `scores` (SCORES_*; None: what `softmax` says): SCORES_CHOSEN_SOFTMAX chooses
+    by the logits, and the weights are the softmax over the chosen logits only."""
+    if scores is None:
+        scores = SCORES_SOFTMAX if softmax else SCORES_SIGMOID
+    _need_cuda(h, router, correction, bias)
+    _f32(correction, bias)
+    if bias is not None and bias.numel() != router.shape[0]:
+        raise KernelError("moe_route: the bias has a number per expert")
     if correction is not None and correction.numel() != router.shape[0]:
         raise KernelError("moe_route: the correction has a number per expert")
     n, d = h.shape
@@ -495,11 +526,13 @@ def moe_route(h, router, top, softmax=False, correction=None, renormalise=False,
     ids = torch.empty((n, top), dtype=torch.int32, device=h.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=h.device)
     _call("moe", "blm_moe_route", _ptr(h), _code(h.dtype), _ptr(router), n, d, router.shape[0], top, _ptr(ids), _ptr(weights),
-          1 if softmax else 0, _ptr(correction), 1 if renormalise else 0, int(n_groups), int(keep_groups if n_groups > 1 else 1), _stream())
+          int(scores), _ptr(bias), _ptr(correction), 1 if renormalise else 0, int(n_groups), int(keep_groups if n_groups > 1 else 1), _stream())
     return ids, weights
 
 
-UNIT_GATED, UNIT_GELU, UNIT_GELU_TANH = 0, 1, 2      # an expert's unit: gated (silu or clamped); W_down gelu(W_up x), exact or tanh form
+# an expert's unit: gated (silu or clamped); W_down gelu(W_up x), exact or tanh form; W_down relu(W_up x)^2
+UNIT_GATED, UNIT_GELU, UNIT_GELU_TANH, UNIT_RELU2 = 0, 1, 2, 3
+MOE_TC_UNITS = {UNIT_GELU: 3, UNIT_RELU2: 5}         # units the grouped tcgen05 product takes, and its epilogue for each
 
 
 def moe_experts(h, ids, weights, gate_up, down, extra=None, weight_on_input=True, clamp_limit=0.0, clamp_alpha=1.702, out_dtype=None,
@@ -508,8 +541,8 @@ def moe_experts(h, ids, weights, gate_up, down, extra=None, weight_on_input=True
     [N, D] when given; expert(x) = down[e] (silu(gate[e] x) * (up[e] x)).  gate_up [experts, 2 ff, D] (an expert's
     gate rows, then its up rows) and down [experts, D, ff] in h's dtype.  Returns [N, D] in h's dtype, or in float32
     (`out_dtype`).  `clamp_limit` > 0: the experts' unit is the clamped one, g = min(gate x, limit), u = clamp(up x, -limit,
-    limit), g sigmoid(clamp_alpha g) (u + 1).  `unit` UNIT_GELU or UNIT_GELU_TANH: the experts have no gate,
-    expert(x) = down[e] gelu(up[e] x), and `gate_up` is [experts, ff, D], the up rows alone."""
+    limit), g sigmoid(clamp_alpha g) (u + 1).  `unit` UNIT_GELU, UNIT_GELU_TANH or UNIT_RELU2: the experts have no gate,
+    expert(x) = down[e] act(up[e] x), and `gate_up` is [experts, ff, D], the up rows alone."""
     _need_cuda(h, ids, weights, gate_up, down, extra)
     n, d = h.shape
     top = ids.shape[1]
@@ -524,9 +557,9 @@ def moe_experts(h, ids, weights, gate_up, down, extra=None, weight_on_input=True
         raise KernelError("moe_experts: extra must be [N, D] in the activations' dtype")
     dev = h.device
     pairs = n * top
-    if (unit == UNIT_GELU and not weight_on_input and h.dtype == torch.bfloat16 and pairs >= MOE_TC_PAIRS * e and d % 8 == 0 and ff % 8 == 0
+    if (unit in MOE_TC_UNITS and not weight_on_input and h.dtype == torch.bfloat16 and pairs >= MOE_TC_PAIRS * e and d % 8 == 0 and ff % 8 == 0
             and d >= 64 and ff >= 64 and e * max(d, ff) < (1 << 31)):
-        return _moe_experts_tc(h, ids, weights, gate_up, down, extra, out_dtype or h.dtype)
+        return _moe_experts_tc(h, ids, weights, gate_up, down, extra, out_dtype or h.dtype, unit)
     offsets = torch.empty(e + 1, dtype=torch.int32, device=dev)
     order = torch.empty(pairs, dtype=torch.int32, device=dev)
     place_of = torch.empty(pairs, dtype=torch.int32, device=dev)
@@ -550,11 +583,11 @@ MOE_TC_PAIRS = int(os.environ.get("BURN_LM_B200_MOE_TC_PAIRS", "16"))
 MOE_TC_ROWS = 128       # rows of a tile of the tcgen05 product: an expert's share of the pairs starts at a multiple of it
 
 
-def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype):
+def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype, unit=UNIT_GELU):
     """Experts without a gate for prompts, both products on the tcgen05 tensor cores: the pairs' token rows are gathered expert
     by expert, every expert's share starting at a multiple of 128 places (a place no pair owns holds zeros), and one grouped
     product runs over all experts at once (kernels of gemm_tc.cu: a table names the expert of every tile of places); the
-    first product's epilogue applies the exact GELU, the second leaves fp32 sums, and the sum over a token's experts weighs
+    first product's epilogue applies the unit's activation, the second leaves fp32 sums, and the sum over a token's experts weighs
     them as ever.  Everything is sized by the token count alone, so a step can be captured."""
     n, d = h.shape
     e, ff, _ = up.shape
@@ -573,7 +606,7 @@ def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype):
     _call("moe", "blm_moe_group_padded", _ptr(ids), pairs, e, MOE_TC_ROWS, _ptr(place_of), _ptr(pair_of_place), _ptr(tile_expert), stream)
     _call("moe", "blm_moe_gather_rows", _ptr(h), _ptr(pair_of_place), _ptr(xs), places, d, top, stream)
     _call("gemm_tc", "blm_gemm_tc_grouped", _ptr(xs), c_longlong(d), _ptr(up), c_longlong(d), _ptr(act), c_longlong(ff), places, ff, d, e,
-          _ptr(tile_expert), 3, _ptr(status), stream)
+          _ptr(tile_expert), MOE_TC_UNITS[unit], _ptr(status), stream)
     _call("gemm_tc", "blm_gemm_tc_grouped", _ptr(act), c_longlong(ff), _ptr(down), c_longlong(ff), _ptr(y), c_longlong(d), places, d, ff, e,
           _ptr(tile_expert), 4, _ptr(status), stream)
     _call("moe", "blm_moe_combine", _ptr(y), _ptr(place_of), _ptr(weights), _ptr(extra), _ptr(out), _code(h.dtype), n, d, top,
@@ -581,13 +614,14 @@ def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype):
     return out
 
 
-def rope_table(inv_freq, n_positions):
+def rope_table(inv_freq, n_positions, turn_scale=1.0):
     """(cos, sin) of position * inv_freq for positions below n_positions: float32 [n_positions, half, 2],
-    computed in float64 on the device; rope_append reads it instead of computing angles per token."""
+    computed in float64 on the device; rope_append reads it instead of computing angles per token.
+    `turn_scale`: what cosine and sine are multiplied by."""
     _need_cuda(inv_freq)
     half = inv_freq.numel()
     table = torch.empty((n_positions, half, 2), dtype=torch.float32, device=inv_freq.device)
-    _call("elementwise", "blm_rope_table", _ptr(inv_freq), _ptr(table), n_positions, half, _stream())
+    _call("elementwise", "blm_rope_table", _ptr(inv_freq), _ptr(table), n_positions, half, c_float(turn_scale), _stream())
     return table
 
 
@@ -595,7 +629,7 @@ PAIRS_HALVES, PAIRS_INTERLEAVED, PAIRS_TILED = 0, 1, 2
 
 
 def rope_append(qkv, token_seq, token_pos, slot_of_seq, block_table, inv_freq, rotary_dim, interleaved,
-                pool, n_heads, n_kv, head_dim, write_cache=True, table=None, max_position=None):
+                pool, n_heads, n_kv, head_dim, write_cache=True, table=None, max_position=None, turn_scale=1.0):
     """Rotate q (in place) and k of every token by its position, and append k, v to the paged cache.
 
     `interleaved`: False or PAIRS_HALVES: pair i is lanes (i, i + rotary_dim / 2); True or
@@ -605,7 +639,8 @@ def rope_append(qkv, token_seq, token_pos, slot_of_seq, block_table, inv_freq, r
     qkv [N, (n_heads + 2 n_kv) * head_dim]; pool [pages, 2, n_kv, PAGE, head_dim] of one cache line;
     inv_freq float64 [rotary_dim / 2] or None when rotary_dim == 0; `table` (from rope_table) spares
     the per-token angles for positions it covers.  `max_position`: an upper bound of the step's
-    positions known on the host; when the table covers it, the vector kernel may run."""
+    positions known on the host; when the table covers it, the vector kernel may run.  `turn_scale`: what cosine
+    and sine are multiplied by (a table holds them multiplied)."""
     _need_cuda(qkv, token_seq, token_pos, slot_of_seq, block_table, inv_freq, pool, table)
     if table is not None and (table.dtype != torch.float32 or tuple(table.shape[1:]) != (rotary_dim // 2, 2)):
         raise KernelError("rope_append: table must be float32 [positions, rotary_dim / 2, 2]")
@@ -622,7 +657,7 @@ def rope_append(qkv, token_seq, token_pos, slot_of_seq, block_table, inv_freq, r
           _ptr(slot_of_seq), _ptr(block_table), block_table.shape[1], _ptr(inv_freq), rotary_dim,
           int(interleaved), _ptr(pool), n, n_heads, n_kv, head_dim, PAGE, 1 if write_cache else 0,
           _ptr(table), table.shape[0] if table is not None else 0,
-          1 if (table is not None and max_position is not None and max_position < table.shape[0]) else 0, _stream())
+          1 if (table is not None and max_position is not None and max_position < table.shape[0]) else 0, c_float(turn_scale), _stream())
 
 
 def tiled_pair_order(head_dim: int) -> list:
@@ -764,7 +799,7 @@ def batched_product(x, w, out=None, out_dtype=None):
     return torch.bmm(x, w.transpose(1, 2))
 
 
-EPI_STORE, EPI_SWIGLU, EPI_RESID_ADD, EPI_ROPE = 0, 1, 2, 3
+EPI_STORE, EPI_SWIGLU, EPI_RESID_ADD, EPI_ROPE, EPI_RELU2 = 0, 1, 2, 3, 4
 
 
 class _GemvRope(ctypes.Structure):
@@ -783,19 +818,19 @@ def gemm_tc_supported(m, n, k) -> bool:
     return bool(_lib("gemm_tc").blm_gemm_tc_supported(m, n, k))
 
 
-def gemm_tc(x, w, out=None, swiglu=False, add_into=None):
+def gemm_tc(x, w, out=None, swiglu=False, add_into=None, relu2=False):
     """x [M, K] times w [N, K] transposed on the tcgen05 tensor cores (bfloat16, fp32 accumulation in
     tensor memory).  out [M, N]; with `swiglu`, w is a fused gate/up weight in tiles of GATE_TILE gate
     rows followed by their up rows and out [M, N / 2] = silu(gate) * up, formed in the epilogue; with
     `add_into` (float32 [M, N], the residual stream) the product is added into it in the epilogue and
-    nothing else is written."""
+    nothing else is written; with `relu2` out = relu(product)^2."""
     _need_cuda(x, w, out, add_into)
     m, k = x.shape
     n = w.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != k:
         raise KernelError("gemm_tc: bfloat16 x [M, K] and w [N, K]")
     if add_into is not None:
-        if swiglu or out is not None or add_into.dtype != torch.float32 or tuple(add_into.shape) != (m, n) or add_into.stride(1) != 1:
+        if swiglu or relu2 or out is not None or add_into.dtype != torch.float32 or tuple(add_into.shape) != (m, n) or add_into.stride(1) != 1:
             raise KernelError("gemm_tc: add_into must be float32 [M, N], alone")
         _call("gemm_tc", "blm_gemm_tc", _ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(add_into), add_into.stride(0), m, n, k,
               2, _ptr(status_word(x.device)), _stream())
@@ -803,7 +838,7 @@ def gemm_tc(x, w, out=None, swiglu=False, add_into=None):
     if out is None or out.dtype != torch.bfloat16 or tuple(out.shape) != (m, n // 2 if swiglu else n):
         raise KernelError("gemm_tc: out must be bfloat16 [M, N] (or [M, N / 2] with the gated epilogue)")
     _call("gemm_tc", "blm_gemm_tc", _ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(out), out.stride(0), m, n, k,
-          1 if swiglu else 0, _ptr(status_word(x.device)), _stream())
+          1 if swiglu else (5 if relu2 else 0), _ptr(status_word(x.device)), _stream())
 
 
 SK_SQUARES_ROWS = 64     # row length of the sums of squares that go with a norm handed over between gemm_sk products
@@ -939,14 +974,14 @@ SQUARES_ROWS = 16     # row length of the sums of squares that go with a handed-
 
 
 def gemv(w, n_tokens, x=None, stream_rows=None, gamma=None, eps=0.0, rows=None, out=None, add_into=None, swiglu=False,
-         squares=None, hand_over=None, rope=None):
+         squares=None, hand_over=None, rope=None, relu2=False):
     """Skinny product of n_tokens <= 16 tokens with a bfloat16 weight [M, K], with fused ends.
 
     Input: `x` bfloat16 [N, K], or the fp32 residual stream `stream_rows` [*, K] to be RMS-normalised
     with `gamma`, `eps` (optionally gathering `rows`), or a norm that the writer of the stream handed
     over: `x` = bfloat16(stream * gamma) with `squares` (fp32 [parts, SQUARES_ROWS], the stream rows'
     sums of squares in parts) and `eps`; the result is then divided by the rows' root mean square.
-    Output: `out` [N, M] bfloat16 or float32;
+    Output: `out` [N, M] bfloat16 or float32 (with `relu2`: relu of the product, squared);
     with `swiglu` the weight is [2 I, K] in tiles of GATE_TILE gate rows followed by the up rows of the
     same outputs, and out [N, I] = silu(gate) * up; with
     `add_into` (fp32 [N, M]) the product is added into it and nothing else is written, unless
@@ -963,7 +998,9 @@ def gemv(w, n_tokens, x=None, stream_rows=None, gamma=None, eps=0.0, rows=None, 
     if w.dtype != torch.bfloat16:
         raise KernelError("gemv: the weight must be bfloat16")
     m = m_rows // 2 if swiglu else m_rows
-    epi = EPI_SWIGLU if swiglu else (EPI_RESID_ADD if add_into is not None else (EPI_ROPE if rope is not None else EPI_STORE))
+    epi = EPI_SWIGLU if swiglu else (EPI_RESID_ADD if add_into is not None else (EPI_ROPE if rope is not None else (EPI_RELU2 if relu2 else EPI_STORE)))
+    if relu2 and (swiglu or add_into is not None or rope is not None):
+        raise KernelError("gemv: one epilogue at a time")
     rope_arg = None
     if rope is not None:
         if swiglu or add_into is not None:
@@ -1094,6 +1131,9 @@ def uniform32(seed, stream_id, counter) -> int:
 # ------------------------------------------------------------------------------------------------
 # blocks that norm a sublayer's output before it is added to the stream
 # ------------------------------------------------------------------------------------------------
+ACT_NONE, ACT_XIELU, ACT_TANH, ACT_RELU2 = 0, 1, 2, 3
+
+
 def _f32(*tensors):
     for t in tensors:
         if t is not None and t.dtype != torch.float32:
@@ -1140,13 +1180,12 @@ def sandwich_norm(resid, delta, post_weight, mult, eps_post, pre_weight, eps_pre
           c_float(eps_pre), _ptr(out), _code(out.dtype) if out is not None else F32, _ptr(rows), n_out, d, _stream())
 
 
-ACT_NONE, ACT_XIELU, ACT_TANH = 0, 1, 2
 
 
 def bias_act(x, bias, out, kind=ACT_NONE, params=None):
     """out = act(x + bias) row by row; x, out [N, D] (float32 or bfloat16), bias float32 [D] or None.  ACT_XIELU with
     params = float32 [2] (p, q): z > 0: softplus(p) z^2 + z / 2; else (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2.
-    ACT_TANH: tanh(z)."""
+    ACT_TANH: tanh(z).  ACT_RELU2: relu(z)^2."""
     _need_cuda(x, bias, out, params)
     _f32(bias, params)
     n, d = x.shape
@@ -1304,6 +1343,47 @@ def decay_scan(q, q_col0, k, k_col0, v, v_col0, a, a_col0, bias, extra, out, hea
 
 
 GATE_FIRST, GATE_LAST, GATE_SILU_LAST, GATE_NONE = 0, 1, 2, 3
+
+
+SELECTIVE_STATES = 128      # states a channel the selective scan takes at most
+
+
+def selective_scan(x, low, rank, n_state, dt_bias, a_log, d_skip, z, out, step, state, state_offset, dt=None, dt_weight=None, scale=1.0):
+    """The selective scan per channel c with `n_state` states: S <- exp(dt A) S + dt x B, y = S C + D x, out = scale y silu(z),
+    dt = softplus(. + dt_bias), A = -exp(a_log).  x float32 [N, channels]; low float32 [N, rank + 2 n_state] = [dt | B | C];
+    the step sizes before bias and softplus are `dt` float32 [N, channels], or dt_weight [channels, rank] times low's first
+    columns, formed by the kernel; z float32 [N, channels], possibly a column range; out [N, channels] bfloat16, or float32 in
+    the 32-bit path (sums in float64), possibly a column range.  The state (fp32) lies in `state` at state_offset,
+    [channels, n_state]."""
+    channels = x.shape[1]
+    _need_cuda(x, low, dt, dt_weight, dt_bias, a_log, d_skip, state)
+    _f32(x, low, dt, dt_bias, a_log, d_skip, z)
+    n = step.n_tokens
+    if n_state > SELECTIVE_STATES:
+        raise KernelError(f"selective_scan: {n_state} states a channel; at most {SELECTIVE_STATES}")
+    if (x.shape[0] != n or tuple(low.shape) != (n, rank + 2 * n_state) or tuple(a_log.shape) != (channels, n_state)
+            or dt_bias.numel() != channels or d_skip.numel() != channels):
+        raise KernelError("selective_scan: x [N, C], low [N, rank + 2 n_state], a_log [C, n_state], a bias and a skip per channel")
+    if (dt is None) == (dt_weight is None) or (dt is not None and tuple(dt.shape) != (n, channels)) \
+            or (dt_weight is not None and tuple(dt_weight.shape) != (channels, rank)):
+        raise KernelError("selective_scan: step sizes [N, C], or their projection [C, rank]")
+    for t in (z, out):
+        if not t.is_cuda or tuple(t.shape) != (n, channels) or t.stride(1) != 1:
+            raise KernelError("selective_scan: z and out are CUDA tensors [N, C] with unit stride along their rows")
+    _call("recurrent", "blm_selective_scan", _ptr(x), c_longlong(x.stride(0)), _ptr(low), c_longlong(low.stride(0)), int(rank),
+          int(rank + n_state), _ptr(dt), c_longlong(channels), _ptr(dt_weight), _code(dt_weight.dtype) if dt_weight is not None else F32,
+          int(rank), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), _ptr(z), c_longlong(z.stride(0)), _ptr(out), _code(out.dtype),
+          c_longlong(out.stride(0)), c_float(scale), channels, int(n_state), _ptr(step.cu_seqlens), _ptr(step.slot_of_seq),
+          _ptr(step.start_pos), step.n_seqs, *_state_args(state, state_offset), _stream())
+
+
+def take_cols(src, col0, out):
+    """out = src[:, col0 : col0 + out's columns] in out's dtype: src float32 [N, *], out contiguous."""
+    _need_cuda(out)
+    p, stride, at = _cols(src, col0, out.shape[1])
+    if not src.is_cuda or src.shape[0] != out.shape[0]:
+        raise KernelError("take_cols: a row of out per row of a CUDA src")
+    _call("recurrent", "blm_take_cols", p, stride, at, _ptr(out), _code(out.dtype), out.shape[0], out.shape[1], _stream())
 
 
 def gated_group_norm(y, gate, gate_col0, weight, group, mode, eps, out):
@@ -1511,3 +1591,15 @@ def softcap(x, cap: float):
     _need_cuda(x)
     _f32(x)
     _call("stream_ops", "blm_softcap", _ptr(x), c_float(cap), c_size_t(x.numel()), _stream())
+
+
+def pass_entry(resid, delta, embedded, step):
+    """resid += delta (a pending output, or None) + embedded (the embedding's output, or None) + step, in place: resid and
+    embedded float32 [N, D], delta float32 or bfloat16 [N, D], step float32 [D]."""
+    _need_cuda(resid, delta, embedded, step)
+    _f32(resid, embedded, step)
+    n, d = resid.shape
+    if step.numel() != d or any(t is not None and t.shape != resid.shape for t in (delta, embedded)):
+        raise KernelError("pass_entry: resid, delta and embedded [N, D], step [D]")
+    _call("stream_ops", "blm_pass_entry", _ptr(resid), _ptr(delta), _code(delta.dtype) if delta is not None else F32, _ptr(embedded),
+          _ptr(step), n, d, _stream())

@@ -3,13 +3,14 @@ embedding and head.  Importing this package registers the built-in kinds."""
 from .base import CacheNeed, Part, Runtime, StepContext
 from .linear import Linear
 from .norm import DynamicTanh, DynamicTanhSpec, PostNormed, PostRMSNorm, PostRMSNormSpec, RMSNorm, RMSNormSpec
-from .position import Llama3Scaling, NoPosition, NoPositionSpec, Rotary, RotarySpec, rotary_inverse_frequencies
+from .position import LinearScaling, Llama3Scaling, NoPosition, NoPositionSpec, YarnScaling, rotary_multiplier, Rotary, RotarySpec, rotary_inverse_frequencies
 from .attention import Attention, AttentionSpec
-from .feed_forward import BiasedMLP, BiasedMLPSpec, SwiGLU, SwiGLUSpec
+from .feed_forward import MLP, MLPSpec, BiasedMLP, BiasedMLPSpec, SwiGLU, SwiGLUSpec
 from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
 from .sink_attention import SinkAttention, SinkAttentionSpec
 from .moe import SigmoidMoE, SigmoidMoESpec
 from .embedding import Embedding, EmbeddingSpec, Head, HeadSpec, PairEmbedding, PairEmbeddingSpec, ScaledEmbedding, ScaledEmbeddingSpec
+from .mamba import Mamba, MambaSpec
 from .mamba2 import Mamba2, Mamba2Spec
 from .gated_delta import GatedDelta, GatedDeltaSpec
 from .sigmoid_attention import SigmoidAttention, SigmoidAttentionSpec
@@ -18,7 +19,7 @@ from .filter import ShortConv, ShortConvSpec
 from .latent_attention import LatentAttention, LatentAttentionSpec
 from .hgrn2 import Hgrn2, Hgrn2Spec
 from .wkv import Wkv, WkvSpec
-from .stream import ConcatProjection, ConcatProjectionSpec
+from .stream import ConcatProjection, ConcatProjectionSpec, PassEntry, PassEntrySpec
 from .normed_attention import NormedAttention, NormedAttentionSpec
 
 __all__ = ["CacheNeed", "Part", "Runtime", "StepContext", "Linear", "RMSNorm", "RMSNormSpec", "Llama3Scaling",
@@ -29,4 +30,5 @@ __all__ = ["CacheNeed", "Part", "Runtime", "StepContext", "Linear", "RMSNorm", "
            "ScaledEmbeddingSpec", "Mamba2", "Mamba2Spec", "GatedDelta", "GatedDeltaSpec", "SigmoidAttention", "SigmoidAttentionSpec",
            "ParallelMixers", "ParallelMixersSpec", "ShortConv", "ShortConvSpec", "LatentAttention", "LatentAttentionSpec", "Hgrn2",
            "Hgrn2Spec", "Wkv", "WkvSpec", "ConcatProjection", "ConcatProjectionSpec", "NormedAttention", "NormedAttentionSpec",
-           "PostNormBlock"]
+           "PostNormBlock", "Mamba", "MambaSpec", "PassEntry", "PassEntrySpec", "LinearScaling", "YarnScaling", "rotary_multiplier", "MLP",
+           "MLPSpec"]

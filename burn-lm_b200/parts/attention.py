@@ -23,6 +23,7 @@ from .base import CacheNeed, Part
 from .linear import Linear
 
 BLOCKS_PER_SM = 2     # blocks a decode step should offer every multiprocessor
+TUNED_HEADS = (64, 128)   # head sizes with kernels of their own (tcgen05 prompts, streaming decode); the others run the general one
 
 
 @dataclass(frozen=True)
@@ -152,7 +153,8 @@ class Attention(Part):
             qkv = product(x, out_dtype=rt.dtype)
             K.rope_append(qkv, step.token_seq, step.token_pos, step.slot_of_seq, cache.block_table, inv_freq, rot,
                           self.pairs, cache.pool, s.n_heads, s.n_kv_heads if cache.writes else 0, s.head_dim,
-                          write_cache=cache.writes, table=table, max_position=step.max_kv_len - 1)
+                          write_cache=cache.writes, table=table, max_position=step.max_kv_len - 1,
+                          turn_scale=getattr(self.position, "turn_scale", 1.0))
         out = torch.empty((n, s.n_heads * s.head_dim), dtype=rt.dtype, device=qkv.device)
         n_splits = self._splits(step)
         scratch = None

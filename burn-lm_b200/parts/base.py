@@ -48,7 +48,8 @@ class CacheNeed:
 
     kind "kv":    keys and values per position: n_kv_heads x head_dim each (values of `value_dim` lanes when
                   that is set and differs); `window` None keeps all positions, a number keeps that many of the
-                  latest, and beside them the first `keep_first` positions of the sequence.
+                  latest, and beside them the first `keep_first` positions of the sequence; `chunk`: a position looks back to the
+                  start of its own chunk of that many positions, counted from the sequence's start.
     kind "rows":  one row of `head_dim` lanes per position in the compute dtype, shared by all heads (a latent that keys
                   and values are made from), paged like keys and values; `window` as above.
     kind "ids":   one int32 per position (a token id, say), paged like keys and values; `window` as above.
@@ -63,6 +64,13 @@ class CacheNeed:
     state_dtype: str = "float32"
     value_dim: Optional[int] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
+
+    def first_needed(self, length: int) -> int:
+        """The first position that tokens at positions >= length look back to (what the sequence keeps from its start aside)."""
+        if self.chunk:
+            return length - length % self.chunk
+        return max(0, length - self.window + 1) if self.window else 0
 
 
 @dataclass

@@ -1,7 +1,7 @@
 """How a layer's parts stand around the residual stream: one after the other behind norms of their own
 (pre-norm), or side by side behind one norm (parallel).
 
-Pre-norm: h = x + mixer(norm(x)); out = h + feed_forward(norm(h))
+Pre-norm: h = x + mixer(norm(x)); out = h + feed_forward(norm(h)), the latter if the layer has one
 (crates/burn-lm-llama/src/nn/transformer.rs:241-256).  The residual stream is fp32; a part's
 output is added into it by the next norm's fused kernel, so a block takes the pending output of
 the block before it (`delta`) and returns its own.
@@ -27,10 +27,10 @@ class PreNormBlock:
     NAMES = ("mixer_norm", "mixer", "feed_forward_norm", "feed_forward")
 
     def __init__(self, parts: dict):
-        if set(parts) != set(self.NAMES):
-            raise ValueError(f"the prenorm block arranges parts named {self.NAMES}; the layer has {sorted(parts)}")
+        if not set(self.NAMES[:2]) <= set(parts) <= set(self.NAMES) or len(parts) not in (2, 4):
+            raise ValueError(f"the prenorm block arranges parts named {self.NAMES} (the last two may be absent); the layer has {sorted(parts)}")
         self.mixer_norm, self.mixer = parts["mixer_norm"], parts["mixer"]
-        self.feed_forward_norm, self.feed_forward = parts["feed_forward_norm"], parts["feed_forward"]
+        self.feed_forward_norm, self.feed_forward = parts.get("feed_forward_norm"), parts.get("feed_forward")
 
     def first_norm(self):
         """The norm that reads the stream first in this block: the block before may prepare its input."""
@@ -48,10 +48,12 @@ class PreNormBlock:
         handoff = step.handoff
         x = _add_norm(self.mixer_norm, resid, delta, getattr(mixer, "takes_pending_norm", False), handoff)
         if getattr(mixer, "adds_to_stream", False):
-            handoff.expect(self.feed_forward_norm)
+            handoff.expect(self.feed_forward_norm if ff is not None else next_norm)
             a = mixer.forward(x, step, cache_view, stream=resid)
         else:
             a = mixer.forward(x, step, cache_view)
+        if ff is None:
+            return a
         x = _add_norm(self.feed_forward_norm, resid, a, getattr(ff, "takes_pending_norm", False), handoff)
         if getattr(ff, "adds_to_stream", False):
             handoff.expect(next_norm)

@@ -98,3 +98,40 @@ class BiasedMLP(Part):
         act = torch.empty(z.shape, dtype=self.runtime.dtype, device=z.device)
         K.bias_act(z, self.up_bias, act, K.ACT_XIELU, self.params)
         return self.down(act, out_dtype=torch.float32), self.down_bias
+
+
+@dataclass(frozen=True)
+class MLPSpec:
+    hidden_size: int
+    intermediate_size: int
+    activation: str = "relu2"     # "relu2": the square of relu
+
+
+@register_part("feed_forward", "mlp")
+class MLP(Part):
+    """W_down act(W_up h), without biases and without a gate.  The activation is taken in fp32 on the up product's sums."""
+    family = "feed_forward"
+    graph_safe = True
+    roles = ("up", "down")
+    kernel_modules = ("elementwise", "stream_ops")
+    takes_pending_norm = True
+    adds_to_stream = True
+
+    ACTIVATIONS = {"relu2": K.ACT_RELU2}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        if spec.activation not in self.ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r}; this feed-forward knows {sorted(self.ACTIVATIONS)}")
+
+    def tensor_specs(self):
+        s, t = self.spec, self.tensor_names
+        return [TensorSpec(t["up"], (s.intermediate_size, s.hidden_size)), TensorSpec(t["down"], (s.hidden_size, s.intermediate_size))]
+
+    def bind(self, loaded):
+        t = self.tensor_names
+        self.up, self.down = Linear(loaded[t["up"]]), Linear(loaded[t["down"]])
+
+    def forward(self, x, step, stream=None):
+        act = self.up.activated(x, self.runtime.dtype, self.ACTIVATIONS[self.spec.activation])
+        return self.down.into_stream(act, stream, torch.float32, handoff=getattr(step, "handoff", None))

@@ -247,6 +247,26 @@ class Linear:
         K.swiglu(self(x, out_dtype), act, tile=self.gate_tile)
         return act
 
+    def activated(self, x, out_dtype: torch.dtype, act: int) -> torch.Tensor:
+        """act(x W^T), the activation (kernels.ACT_*) taken in fp32 on the product's sums; the skinny and the tcgen05 product
+        square a relu in their own epilogue."""
+        n = self._tokens(x)
+        if act == K.ACT_RELU2 and out_dtype == torch.bfloat16 and self.weight.dtype == torch.bfloat16:
+            out = torch.empty((n, self.out_features), dtype=out_dtype, device=self.weight.device)
+            if self._skinny(n, self.out_features, x):
+                K.gemv(self.weight, n, out=out, relu2=True, **self._source(x))
+                return out
+            if n >= TENSOR_CORE_TOKENS and K.gemm_tc_supported(n, self.out_features, self.in_features):
+                if isinstance(x, NormedStream):
+                    x = x.materialize()
+                if x.dtype == torch.bfloat16 and x.is_contiguous():
+                    K.gemm_tc(x, self.weight, out, relu2=True)
+                    return out
+        z = self(x, out_dtype=torch.float32)
+        out = torch.empty(z.shape, dtype=out_dtype, device=z.device)
+        K.bias_act(z, None, out, act)
+        return out
+
     def _library(self, x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
         w = self.weight
         if w.dtype == torch.float32:

@@ -93,7 +93,9 @@ class RoutedMoESpec:
     n_experts: int
     top: int
     expert_size: int
-    scores: str = "softmax"                # "softmax" over all experts, or "sigmoid" of every logit
+    scores: str = "softmax"                # "softmax" over all experts, "sigmoid" of every logit, or "chosen_softmax": the logits
+                                           # decide the choice and the weights are a softmax over the chosen ones
+    bias: bool = False                     # a stored number per expert joins the router's logits
     correction: bool = False               # a stored number per expert joins the scores for the choice only
     renormalise: bool = True               # the chosen weights are divided by their sum + 1e-20
     clamp_limit: Optional[float] = None    # the experts' clamped unit: g = min(Wgate x, limit), u = clamp(Wup x, -limit, limit),
@@ -101,7 +103,8 @@ class RoutedMoESpec:
     n_groups: int = 1                      # the experts form this many equal groups of neighbours; only experts of the
     keep_groups: int = 1                   # `keep_groups` best groups can be chosen (a group's mark: its two largest choice scores)
     unit: str = "gated"                    # "gated": W_down (act(W_gate x) * W_up x); "gelu" / "gelu_tanh": W_down gelu(W_up x),
-                                           # the exact (erf) form or the tanh one; such experts store no gate
+                                           # the exact (erf) form or the tanh one; "relu2": W_down relu(W_up h)^2; such
+                                           # experts store no gate
 
 
 @register_part("feed_forward", "routed_moe")
@@ -110,15 +113,15 @@ class RoutedMoE(SigmoidMoE):
     sigmoids), the `top` experts of largest s (+ a stored correction that the weights do not see), weights s of the chosen,
     optionally divided by their sum; out = sum weight_k expert_k(h), with the plain or the clamped gated unit, or a unit
     without a gate.  The choice may be limited to the experts of the best groups.  Router logits, scores and weights are
-    fp32.  tensors: "router", "correction" (when the spec says so); "gate" (gated units), "up", "down" with {} where the
+    fp32.  tensors: "router", "bias" and "correction" (when the spec says so); "gate" (gated units), "up", "down" with {} where the
     expert's number stands."""
-    roles = ("router", "correction", "gate", "up", "down")
+    roles = ("router", "bias", "correction", "gate", "up", "down")
     adds_to_stream = False
 
     def __init__(self, spec, tensors, runtime):
         Part.__init__(self, spec, tensors, runtime)
-        if spec.scores not in ("softmax", "sigmoid"):
-            raise ValueError(f"scores are 'softmax' or 'sigmoid', not {spec.scores!r}")
+        if spec.scores not in self.SCORES:
+            raise ValueError(f"scores are one of {sorted(self.SCORES)}, not {spec.scores!r}")
         if not 1 <= spec.top <= spec.n_experts:
             raise ValueError(f"top {spec.top} of {spec.n_experts} experts")
         if spec.unit not in self.UNITS:
@@ -129,10 +132,11 @@ class RoutedMoE(SigmoidMoE):
                 or spec.keep_groups * (spec.n_experts // spec.n_groups) < spec.top):
             raise ValueError(f"{spec.n_experts} experts in {spec.n_groups} groups of which {spec.keep_groups} are kept, for {spec.top} chosen")
         self.shared = None
-        if spec.unit == "gelu" and runtime.dtype == torch.bfloat16:
+        if self.UNITS[spec.unit] in K.MOE_TC_UNITS and runtime.dtype == torch.bfloat16:
             self.kernel_modules = ("elementwise", "moe", "gemm_tc")       # prompts run these experts' products on tcgen05
 
-    UNITS = {"gated": K.UNIT_GATED, "gelu": K.UNIT_GELU, "gelu_tanh": K.UNIT_GELU_TANH}
+    UNITS = {"gated": K.UNIT_GATED, "gelu": K.UNIT_GELU, "gelu_tanh": K.UNIT_GELU_TANH, "relu2": K.UNIT_RELU2}
+    SCORES = {"sigmoid": K.SCORES_SIGMOID, "softmax": K.SCORES_SOFTMAX, "chosen_softmax": K.SCORES_CHOSEN_SOFTMAX}
 
     def tensor_specs(self):
         s = self.spec
@@ -142,6 +146,8 @@ class RoutedMoE(SigmoidMoE):
             specs = [TensorSpec(self.tensor_names["router"], (s.n_experts, s.hidden_size), init="normal:0.1")]
             for u, d in zip(self._names("up"), self._names("down")):
                 specs += [TensorSpec(u, (s.expert_size, s.hidden_size)), TensorSpec(d, (s.hidden_size, s.expert_size))]
+        if self.spec.bias:
+            specs.insert(1, TensorSpec(self.tensor_names["bias"], (self.spec.n_experts,), init="normal:0.5"))
         if self.spec.correction:
             specs.insert(1, TensorSpec(self.tensor_names["correction"], (self.spec.n_experts,), init="normal:0.05"))
         return specs
@@ -154,13 +160,15 @@ class RoutedMoE(SigmoidMoE):
             self.router = loaded[self.tensor_names["router"]].to(torch.float32).contiguous()
             self.gate_up = torch.stack([loaded[n].to(dt) for n in self._names("up")]).contiguous()
             self.down = torch.stack([loaded[n].to(dt) for n in self._names("down")]).contiguous()
-        self.correction = None
+        self.correction = self.bias = None
+        if self.spec.bias:
+            self.bias = loaded[self.tensor_names["bias"]].to(torch.float32).contiguous()
         if self.spec.correction:
             self.correction = loaded[self.tensor_names["correction"]].to(torch.float32).contiguous()
 
     def forward(self, x, step):
         s = self.spec
-        ids, weights = K.moe_route(x, self.router, s.top, softmax=s.scores == "softmax", correction=self.correction,
+        ids, weights = K.moe_route(x, self.router, s.top, scores=self.SCORES[s.scores], bias=self.bias, correction=self.correction,
                                    renormalise=s.renormalise, n_groups=s.n_groups, keep_groups=s.keep_groups)
         return K.moe_experts(x, ids, weights, self.gate_up, self.down, weight_on_input=False, clamp_limit=s.clamp_limit or 0.0,
                              clamp_alpha=s.clamp_alpha, out_dtype=torch.float32, unit=self.UNITS[s.unit])

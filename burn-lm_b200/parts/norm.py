@@ -23,6 +23,7 @@ from .linear import NormedStream
 class RMSNormSpec:
     size: int
     eps: float
+    around_zero: bool = False     # the stored weight is what the multiplier exceeds 1 by: gamma = 1 + weight (fp32)
 
 
 @dataclass
@@ -46,10 +47,12 @@ class RMSNorm(Part):
     roles = ("weight",)
 
     def tensor_specs(self):
-        return [TensorSpec(self.tensor_names["weight"], (self.spec.size,), init="one_plus_normal:0.1")]
+        return [TensorSpec(self.tensor_names["weight"], (self.spec.size,), init="normal:0.1" if self.spec.around_zero else "one_plus_normal:0.1")]
 
     def bind(self, loaded):
         self.gamma = loaded[self.tensor_names["weight"]]
+        if self.spec.around_zero:
+            self.gamma = (1.0 + self.gamma.to(torch.float32)).contiguous()
 
     takes_handed_norm = True      # a product that writes the stream may leave this norm's input (parts.linear.NormHandoff)
     takes_post_normed = True      # `delta` may be a PostNormed: normed, scaled and added by this norm's kernel

@@ -1,21 +1,28 @@
-"""Grouped-query attention whose queries, keys and values are normed head by head, with a number per head on the
-scores, capped scores and a sink in the softmax.
+"""Grouped-query attention with options on its queries, keys, values, scores, mask and output: normed heads, a turn of some
+lanes, a number per head on the scores, capped scores, a sink in the softmax, a window or chunks, two maps a head whose
+difference is taken, a gate on every lane.
 
-q = Wq h, k = Wk h, v = Wv h without biases.  Every head of q and of k is divided by its root mean square and
-multiplied by a weight of the head's size that all heads share (`qk_norm`); the first `rotary_dims` lanes of every q
-and k head then turn by position * base^(-2i / rotary_dims), lanes (2i, 2i + 1) together (`rotary_halves`: lanes
-(i, i + rotary_dims / 2)); every head of v is divided by its root mean square (`value_norm`, no weight) and cached so.
-Query head h reads key/value head h // (heads / kv heads); keys have `head_dim` lanes, values `value_dim`.
-s = scale * t_h * q.k (`head_temperature`: t a stored number per query head), then s <- cap tanh(s / cap)
-(`softcap`); position i sees j <= i, or only 0 <= i - j < window; p_j = exp(s_j) / (sink + sum exp(s_j)) with `sink`
-one more entry of score 0 that carries no value.  The heads' outputs are concatenated and projected by Wo.
+q = Wq h, k = Wk h, v = Wv h without biases.  With `qk_norm` every head of q and of k is divided by its root mean square and
+multiplied by a weight of the head's size that all heads share; the first `rotary_dims` lanes of every q and k head then turn
+by position * f_i, f_i = base^(-2i / rotary_dims) or scaled as `rotary_scaling` says (parts.position), lanes (2i, 2i + 1)
+together (`rotary_halves`: lanes (i, i + rotary_dims / 2)); with `value_norm` every head of v is divided by its root mean
+square and cached so.  Query head h reads key/value head h // (heads / kv heads); keys have `head_dim` lanes, values `value_dim`.
+s = scale * t_h * q.k (`head_temperature`: t a stored number per query head), then s <- cap tanh(s / cap) (`softcap`);
+position i sees j <= i, or only 0 <= i - j < window, or only the j of its own chunk of the sequence; p_j = exp(s_j) / (sink +
+sum exp(s_j)) with `sink` one more entry of score 0 that carries no value.  With `output_gate` every lane of the heads' outputs
+is multiplied by sigmoid(Wg h).  The heads' outputs are concatenated and projected by Wo.
 
-Norms, rotation, scores, cap and softmax are fp32 in both dtypes.  The three projections run as one product with a
-fused [q; k; v] weight whose result stays in fp32 for the norms; the attention kernels are the windowed family's
-(`kernels.attention_sink`), which take the head's number, the cap and the sink as options.
+`diff` makes it differential attention: q has two queries and k two keys a head, [head][map][head_dim], each pair an attention
+of its own over the head's one value; with lambda = exp(lq1.lk1) - exp(lq2.lk2) + diff the head's output is a_1 - lambda a_2,
+divided by its root mean square and multiplied by 1 - diff.
+
+Norms, rotation, scores, cap, softmax and the difference are fp32 in both dtypes.  The projections run as one product with a
+fused [q; k; v; g] weight whose result stays in fp32; the attention kernels are the windowed family's
+(`kernels.attention_sink`), which take all of this as options.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Optional
 
@@ -26,6 +33,7 @@ from ..registry import register_part
 from ..weights.loader import TensorSpec
 from .base import CacheNeed, Part
 from .linear import Linear
+from .position import RotarySpec, rotary_inverse_frequencies, rotary_multiplier
 
 BLOCKS_PER_SM = 4          # blocks of the single-token kernels a step should offer every multiprocessor
 NO_WINDOW = 1 << 30        # what the kernels take for "every earlier key"
@@ -49,13 +57,17 @@ class NormedAttentionSpec:
     softcap: Optional[float] = None   # s <- cap tanh(s / cap)
     sink: bool = True                 # one more entry of score 0 in the softmax's denominator
     window: Optional[int] = None      # None: every earlier key
+    chunk: Optional[int] = None       # instead of a window: the keys of the position's own chunk of this many
+    rotary_scaling: object = None     # parts.position.LinearScaling, YarnScaling or Llama3Scaling
+    output_gate: bool = False         # sigmoid(Wg h) on every lane of the heads' outputs
+    diff: Optional[float] = None      # two maps a head, and this constant in the weight of the second
 
 
 @register_part("mixer", "normed_attention")
 class NormedAttention(Part):
     family = "mixer"
     graph_safe = True
-    roles = ("q", "k", "v", "o", "q_norm", "k_norm", "temperature")
+    roles = ("q", "k", "v", "o", "g", "q_norm", "k_norm", "temperature", "lq1", "lk1", "lq2", "lk2")
     kernel_modules = ("elementwise", "attention_sink")
 
     def __init__(self, spec, tensors, runtime):
@@ -68,13 +80,24 @@ class NormedAttention(Part):
             raise ValueError(f"{spec.rotary_dims} turning lanes of {spec.head_dim}: an even number, at most all of them")
         if spec.window is not None and spec.window < 1:
             raise ValueError(f"a window of {spec.window}")
+        if spec.chunk is not None and (spec.chunk < 1 or spec.window is not None):
+            raise ValueError(f"chunks of {spec.chunk} with a window of {spec.window}: one of the two, at least 1")
+        self.maps = 1 if spec.diff is None else 2
+        self.q_cols, self.k_cols = self.maps * spec.n_heads * spec.head_dim, self.maps * spec.n_kv_heads * spec.head_dim
+        self.v_cols = spec.n_kv_heads * spec.value_dim
+        self.out_width = spec.n_heads * spec.value_dim
+        self.proj_width = self.q_cols + self.k_cols + self.v_cols + (self.out_width if spec.output_gate else 0)
 
     def tensor_specs(self):
         s, t = self.spec, self.tensor_names
-        specs = [TensorSpec(t["q"], (s.n_heads * s.head_dim, s.hidden_size)),
-                 TensorSpec(t["k"], (s.n_kv_heads * s.head_dim, s.hidden_size)),
-                 TensorSpec(t["v"], (s.n_kv_heads * s.value_dim, s.hidden_size)),
-                 TensorSpec(t["o"], (s.hidden_size, s.n_heads * s.value_dim))]
+        specs = [TensorSpec(t["q"], (self.q_cols, s.hidden_size)),
+                 TensorSpec(t["k"], (self.k_cols, s.hidden_size)),
+                 TensorSpec(t["v"], (self.v_cols, s.hidden_size)),
+                 TensorSpec(t["o"], (s.hidden_size, self.out_width))]
+        if s.output_gate:
+            specs.append(TensorSpec(t["g"], (self.out_width, s.hidden_size)))
+        if s.diff is not None:
+            specs += [TensorSpec(t[r], (s.head_dim,), init="normal:0.1") for r in ("lq1", "lk1", "lq2", "lk2")]
         if s.qk_norm:
             specs += [TensorSpec(t["q_norm"], (s.head_dim,), init="one_plus_normal:0.1"),
                       TensorSpec(t["k_norm"], (s.head_dim,), init="one_plus_normal:0.1")]
@@ -84,7 +107,7 @@ class NormedAttention(Part):
 
     def bind(self, loaded):
         s, t = self.spec, self.tensor_names
-        ws = [loaded[t["q"]], loaded[t["k"]], loaded[t["v"]]]
+        ws = [loaded[t[r]] for r in (("q", "k", "v", "g") if s.output_gate else ("q", "k", "v"))]
         if len({w.dtype for w in ws}) != 1:
             raise ValueError(f"the projections of {t['q']} and its neighbours are stored in different dtypes")
         self.proj = Linear(torch.cat(ws, dim=0).contiguous())
@@ -93,23 +116,30 @@ class NormedAttention(Part):
         self.q_weight = f32(loaded[t["q_norm"]]) if s.qk_norm else None
         self.k_weight = f32(loaded[t["k_norm"]]) if s.qk_norm else None
         self.temperature = f32(loaded[t["temperature"]]) if s.head_temperature else None
-        self.freq = None
+        self.freq, self.turn_scale = None, 1.0
         if s.rotary_dims:
-            self.freq = torch.tensor([s.rotary_base ** (-2.0 * i / s.rotary_dims) for i in range(s.rotary_dims // 2)],
-                                     dtype=torch.float64).to(self.o.weight.device)
+            rot = RotarySpec(s.head_dim, s.rotary_base, rotary_dim=s.rotary_dims, scaling=s.rotary_scaling)
+            self.freq = torch.tensor(rotary_inverse_frequencies(rot), dtype=torch.float64).to(self.o.weight.device)
+            self.turn_scale = rotary_multiplier(rot)
+        self.difference = (0.0, 1.0, 0.0)
+        if s.diff is not None:
+            lq1, lk1, lq2, lk2 = (loaded[t[r]].to(torch.float64) for r in ("lq1", "lk1", "lq2", "lk2"))
+            lam = math.exp(float((lq1 * lk1).sum())) - math.exp(float((lq2 * lk2).sum())) + s.diff
+            self.difference = (lam, 1.0 - s.diff, s.eps)
 
     def cache_need(self) -> CacheNeed:
         s = self.spec
-        return CacheNeed("kv", n_kv_heads=s.n_kv_heads, head_dim=s.head_dim, window=s.window, value_dim=s.value_dim)
+        return CacheNeed("kv", n_kv_heads=s.n_kv_heads, head_dim=self.maps * s.head_dim, window=s.window, value_dim=s.value_dim,
+                         chunk=s.chunk)
 
     def _splits(self, step) -> int:
         """Over how many blocks the single-token kernels cut a row's keys: a few tokens with many keys leave most of the
         multiprocessors idle otherwise."""
         s = self.spec
-        if K.attention_sink_prompt_takes(self.runtime.dtype, s.head_dim, s.value_dim, step.max_q_len, s.n_heads):
+        if K.attention_sink_prompt_takes(self.runtime.dtype, s.head_dim, s.value_dim, step.max_q_len, self.maps * s.n_heads):
             return 1
-        seen = min(step.max_kv_len, s.window or step.max_kv_len)
-        blocks = step.n_tokens * s.n_kv_heads
+        seen = min(step.max_kv_len, s.window or s.chunk or step.max_kv_len)
+        blocks = step.n_tokens * self.maps * s.n_kv_heads
         want = BLOCKS_PER_SM * K.sm_count(self.runtime.device)
         if K.attention_sink_decode_takes(self.runtime.dtype, s.head_dim, s.value_dim, s.n_heads, s.n_kv_heads):
             pages = seen // K.PAGE + 1                       # that kernel cuts by pages, and its blocks hold several
@@ -117,22 +147,39 @@ class NormedAttention(Part):
             return max(1, min((want + blocks - 1) // blocks, pages // 4, 32))
         return max(1, min((want + blocks - 1) // blocks, seen // 128, 32))
 
-    def forward(self, x, step, cache):
-        s, rt = self.spec, self.runtime
+    takes_pending_norm = True
+    adds_to_stream = True
+
+    def forward(self, x, step, cache, stream=None):
+        rt = self.runtime
+        proj = self.proj(x, out_dtype=torch.float32)            # [N, q | k | v (| g)] in fp32
+        out = torch.empty((step.n_tokens, self.out_width), dtype=rt.dtype, device=proj.device)
+        self.core(proj, step, cache, out)
+        return self.o.into_stream(out, stream, torch.float32, handoff=getattr(step, "handoff", None) if stream is not None else None)
+
+    # what two mixers that run side by side with one product in front and one behind ask for (parts.parallel_mixers)
+    def input_weight(self):
+        return self.proj.weight
+
+    def output_weight(self):
+        return self.o.weight
+
+    def core(self, proj, step, cache, out, scale=1.0):
+        """What lies between the projections: proj float32 [N, proj_width], out [N, out_width] in the compute dtype, times
+        `scale`; either may be a column range of a wider tensor."""
+        s, rt, maps = self.spec, self.runtime, self.maps
         if not cache.writes:
             raise ValueError("this mixer appends to a cache line of its own; it cannot read another run's")
-        n = step.n_tokens
-        proj = self.proj(x, out_dtype=torch.float32)            # [N, q | k | v] in fp32
-        q = torch.empty((n, s.n_heads * s.head_dim), dtype=rt.dtype, device=proj.device)
-        K.head_norm_rope_append(proj, step, cache.pool, cache.block_table, q, s.n_heads, s.n_kv_heads, s.head_dim, s.value_dim,
+        n, heads, kv_heads = step.n_tokens, self.maps * s.n_heads, self.maps * s.n_kv_heads
+        q = torch.empty((n, self.q_cols), dtype=rt.dtype, device=proj.device)
+        K.head_norm_rope_append(proj, step, cache.pool, cache.block_table, q, heads, kv_heads, s.head_dim, s.value_dim,
                                 q_weight=self.q_weight, k_weight=self.k_weight, eps=s.eps, value_norm=s.value_norm, freq=self.freq,
-                                rotary_dims=s.rotary_dims, halves=s.rotary_halves)
-        out = torch.empty((n, s.n_heads * s.value_dim), dtype=rt.dtype, device=proj.device)
+                                rotary_dims=s.rotary_dims, halves=s.rotary_halves, turn_scale=self.turn_scale, maps=maps)
         n_splits = self._splits(step)
-        scratch = None
-        if n_splits > 1:
-            scratch = step.workspace.scratch("attention_sink", K.attention_sink_scratch_floats(n, s.n_heads, s.value_dim, n_splits))
-        K.attention_sink(q, step, cache.pool, cache.block_table, out, s.n_heads, s.n_kv_heads, s.head_dim, s.value_dim, s.scale,
-                         s.window or NO_WINDOW, 0, sink=s.sink, max_q_len=step.max_q_len, n_splits=n_splits, scratch=scratch,
-                         head_scale=self.temperature, softcap=s.softcap or 0.0)
-        return self.o(out, out_dtype=torch.float32)
+        floats = K.attention_sink_scratch_floats(n, heads, s.value_dim, n_splits, maps)
+        scratch = step.workspace.scratch("attention_sink", floats) if floats else None
+        gate = proj[:, self.proj_width - self.out_width:] if s.output_gate else None
+        K.attention_sink(q, step, cache.pool, cache.block_table, out, heads, kv_heads, s.head_dim, s.value_dim, s.scale,
+                         s.window or NO_WINDOW, 0, sink=s.sink, gate=gate, gate_stride=proj.stride(0), max_q_len=step.max_q_len,
+                         n_splits=n_splits, scratch=scratch, head_scale=self.temperature, softcap=s.softcap or 0.0, chunk=s.chunk or 0,
+                         gate_lanes=s.value_dim if s.output_gate else 0, out_scale=scale, maps=maps, difference=self.difference)

@@ -3,6 +3,11 @@
 The mixers are parts of the "mixer" family named by the spec; what a run keeps per sequence is what both keep (keys and
 values of the one beside the state of the other, say), so `cache_need()` gives both needs and the cache hands a view
 with the fields of both.
+
+With `joined` the two input projections run as one product and the two output projections as another: both mixers read the
+same rows, so their weights stand one below the other in front, and behind them scale_a Wa a + scale_b Wb b is the product
+of [Wa | Wb] with the mixers' outputs side by side, each scaled (in fp32) before it is rounded.  A mixer that can be joined
+has input_weight(), output_weight(), proj_width, out_width and core(proj, step, cache, out, scale).
 """
 from __future__ import annotations
 
@@ -14,6 +19,7 @@ from .. import kernels as K
 from ..plan import PartPlan
 from ..registry import part_class, register_part
 from .base import Part
+from .linear import Linear
 
 
 @dataclass(frozen=True)
@@ -22,6 +28,7 @@ class ParallelMixersSpec:
     right: PartPlan
     left_scale: float = 1.0
     right_scale: float = 1.0
+    joined: bool = False          # one product in front of both mixers and one behind
 
 
 @dataclass
@@ -37,10 +44,11 @@ class WeightedPair:
 class ParallelMixers(Part):
     family = "mixer"
     roles = ()
-    gives_pairs = True            # forward(..., as_pair=True) leaves the weighted sum to the caller's next kernel
 
     def __init__(self, spec, tensors, runtime):
         super().__init__(spec, tensors, runtime)
+        self.gives_pairs = not spec.joined      # forward(..., as_pair=True) leaves the weighted sum to the caller's next kernel
+        self.takes_pending_norm = self.adds_to_stream = spec.joined
         self.left = part_class("mixer", spec.left.kind)(spec.left.spec, spec.left.tensors, runtime)
         self.right = part_class("mixer", spec.right.kind)(spec.right.spec, spec.right.tensors, runtime)
         self.graph_safe = bool(getattr(self.left, "graph_safe", False) and getattr(self.right, "graph_safe", False))
@@ -53,6 +61,14 @@ class ParallelMixers(Part):
     def bind(self, loaded):
         self.left.bind(loaded)
         self.right.bind(loaded)
+        if self.spec.joined:
+            pair = (self.left, self.right)
+            if len({w.dtype for m in pair for w in (m.input_weight(), m.output_weight())}) != 1:
+                raise ValueError("the projections of two joined mixers are stored in different dtypes")
+            self.proj = Linear(torch.cat([m.input_weight() for m in pair], dim=0).contiguous())
+            self.o = Linear(torch.cat([m.output_weight() for m in pair], dim=1).contiguous())
+            for m in pair:                      # their own copies are not read any more
+                m.proj = m.o = None
 
     def prepare(self, max_positions: int) -> None:
         for m in (self.left, self.right):
@@ -66,8 +82,18 @@ class ParallelMixers(Part):
             needs.extend(need if isinstance(need, tuple) else [need])
         return tuple(n for n in needs if n.kind != "none")
 
-    def forward(self, x, step, cache, as_pair=False):
+    def _forward_joined(self, x, step, cache, stream):
+        left, right = self.left, self.right
+        proj = self.proj(x, out_dtype=torch.float32)
+        out = torch.empty((step.n_tokens, left.out_width + right.out_width), dtype=self.runtime.dtype, device=proj.device)
+        left.core(proj[:, :left.proj_width], step, cache, out[:, :left.out_width], scale=self.spec.left_scale)
+        right.core(proj[:, left.proj_width:], step, cache, out[:, left.out_width:], scale=self.spec.right_scale)
+        return self.o.into_stream(out, stream, torch.float32, handoff=getattr(step, "handoff", None) if stream is not None else None)
+
+    def forward(self, x, step, cache, as_pair=False, stream=None):
         """`as_pair`: the caller's next kernel takes the weighted sum itself; it gets a WeightedPair."""
+        if self.spec.joined:
+            return self._forward_joined(x, step, cache, stream)
         a = self.left.forward(x, step, cache)
         b = self.right.forward(x, step, cache)
         if a.dtype != torch.float32 or b.dtype != torch.float32:

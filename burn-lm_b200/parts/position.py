@@ -12,7 +12,7 @@ from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Union
 
 import torch
 
@@ -29,6 +29,23 @@ class Llama3Scaling:
 
 
 @dataclass(frozen=True)
+class LinearScaling:
+    """Every frequency divided by the factor."""
+    factor: float
+
+
+@dataclass(frozen=True)
+class YarnScaling:
+    """Frequencies scaled by lanes (YaRN).  A lane pair that turns `fast` times or more over the original positions keeps its
+    frequency, one that turns `slow` times or fewer has it divided by the factor, with a ramp over the pairs between; cosine
+    and sine are both multiplied by 0.1 ln(factor) + 1."""
+    factor: float
+    original_max_position: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     head_dim: int
     theta: float
@@ -36,7 +53,7 @@ class RotarySpec:
     interleaved: bool = False             # False: pairs (i, i + dim/2), the layout of weights stored
                                           # under Hugging Face names; True: pairs (2i, 2i + 1), the
                                           # reference's layout (nn/llama/import.rs:95-126 permutes)
-    scaling: Optional[Llama3Scaling] = None
+    scaling: Union[Llama3Scaling, LinearScaling, YarnScaling, None] = None
 
 
 def rotary_inverse_frequencies(spec: RotarySpec) -> list:
@@ -45,6 +62,13 @@ def rotary_inverse_frequencies(spec: RotarySpec) -> list:
     s = spec.scaling
     if s is None:
         return freqs
+    if isinstance(s, LinearScaling):
+        return [f / s.factor for f in freqs]
+    if isinstance(s, YarnScaling):
+        pair_of = lambda turns: dim * math.log(s.original_max_position / (2.0 * math.pi * turns)) / (2.0 * math.log(spec.theta))
+        lo, hi = max(math.floor(pair_of(s.fast)), 0), min(math.ceil(pair_of(s.slow)), dim - 1)
+        ramps = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(dim // 2)]
+        return [f / s.factor * r + f * (1.0 - r) for f, r in zip(freqs, ramps)]
     low_wavelen = s.original_max_position / s.low_freq_factor
     high_wavelen = s.original_max_position / s.high_freq_factor
     out = []
@@ -60,6 +84,11 @@ def rotary_inverse_frequencies(spec: RotarySpec) -> list:
     return out
 
 
+def rotary_multiplier(spec: RotarySpec) -> float:
+    """What cosine and sine are multiplied by."""
+    return 0.1 * math.log(spec.scaling.factor) + 1.0 if isinstance(spec.scaling, YarnScaling) else 1.0
+
+
 @register_part("position", "rotary")
 class Rotary(Part):
     family = "position"
@@ -70,6 +99,7 @@ class Rotary(Part):
         dim = spec.rotary_dim or spec.head_dim
         if dim % 2 or dim > spec.head_dim:
             raise ValueError(f"rotary_dim {dim} must be even and at most head_dim {spec.head_dim}")
+        self.turn_scale = rotary_multiplier(spec)      # what cosine and sine are multiplied by
         self.rotary_dim = dim
         self.inv_freq = torch.tensor(rotary_inverse_frequencies(spec), dtype=torch.float64, device=runtime.device)
         self._table = None
@@ -82,7 +112,7 @@ class Rotary(Part):
         positions beyond the table are still computed per token by the kernel."""
         from .. import kernels as K
         if self.inv_freq.is_cuda and self.rotary_dim and (self._table is None or self._table.shape[0] < max_positions):
-            self._table = K.rope_table(self.inv_freq, max_positions)
+            self._table = K.rope_table(self.inv_freq, max_positions, self.turn_scale)
 
     def table(self):
         return self._table

@@ -6,6 +6,9 @@ parts and names, per run of its schedule, the one that stands in front of it.
 
 Kind "concat_projection": x <- W [x; x0] with W [width, 2 width] (the stream's columns first) and x0 the embedding's
 output: a loop over some layers feeds the input in again at the start of every pass.
+
+Kind "pass_entry": x <- x + steps[t], and from the second pass on x <- x + x0 + steps[t]: pass t of a loop has a stored vector
+of its own, and the embedding's output joins again.
 """
 from __future__ import annotations
 
@@ -46,3 +49,32 @@ class ConcatProjection(Part):
         K.pack_cols(resid, delta, both, 0)          # the pending output joins the stream on the way (fp32)
         K.pack_cols(embedded, None, both, d)
         return self.linear(both, out_dtype=torch.float32)
+
+
+@dataclass(frozen=True)
+class PassEntrySpec:
+    hidden_size: int
+    passes: int                   # rows of the stored table
+    number: int                   # the pass this part stands in front of, from 0
+
+
+@register_part("stream", "pass_entry")
+class PassEntry(Part):
+    family = "stream"
+    graph_safe = True
+    roles = ("steps",)
+    kernel_modules = ("stream_ops",)
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.needs_embedding = spec.number > 0
+
+    def tensor_specs(self):
+        return [TensorSpec(self.tensor_names["steps"], (self.spec.passes, self.spec.hidden_size), init="normal:0.1")]
+
+    def bind(self, loaded):
+        self.step = loaded[self.tensor_names["steps"]][self.spec.number].to(torch.float32).contiguous()
+
+    def forward(self, resid, delta, embedded, step):
+        K.pass_entry(resid, delta, embedded if self.needs_embedding else None, self.step)
+        return resid
