@@ -802,10 +802,164 @@ def marinex_kernels(z, pk):
     return out
 
 
+def tomalix_configs(z):
+    """(llama, tomalix) of one size.  The new design's layers take turns: attention with scaled frequencies (Llama's head counts
+    and head size) and a dense feed-forward; differential attention (half of Llama's heads with two maps each of its head
+    size, values twice as wide: Llama's weights) and 8 experts of which a token uses 2; attention in chunks of 1,024 with a
+    gate a lane (Llama's heads) beside a selective scan of twice the width's channels with 16 states, and a dense feed-forward.
+    Feed-forwards have no gate: two matrices of 3/2 of the inner size where the dense decoder has three of it."""
+    llama = compare_configs(z)["llama"]
+    hd, d, H, G = z["hd"], z["width"], z["heads"], z["kv"]
+    dense = {"kind": "dense", "ff": 3 * z["inner"] // 2}
+    moe = {"kind": "moe", "expert": {"ff": 3 * z["inner"] // (2 * z["top"])}, "router": {"experts": z["experts"], "top": z["top"]}}
+    scaled = {"type": "attention_2", "mlp": dense,
+              "mixer": {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5,
+                        "rot": {"dims": hd, "base": 500000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    diff = {"type": "attention", "mlp": moe,
+            "mixer": {"heads": H // 2, "kv_heads": G // 2, "dim": hd, "vdim": 2 * hd, "scale": hd ** -0.5, "diff": 0.4,
+                      "rot": {"dims": hd, "base": 10000.0, "scaling": {"factor": 4.0}}}}
+    par = {"type": "parallel", "mlp": dense,
+           "mixer": {"left": {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": z["window"]},
+                              "rot": {"dims": hd // 2, "base": 500000.0}},
+                     "right": {"inner": 2 * d, "state": 16, "conv": 4, "dt_rank": d // 16}, "left_scale": 0.7, "right_scale": 0.6}}
+    tom = {"architecture": "Tomalix", "vocab": z["vocab"], "width": d, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+           "layers": [(scaled, diff, par)[i % 3] for i in range(z["layers"])]}
+    return {"llama": llama, "tomalix": tom}
+
+
+def tomalix_kernels(z, pk):
+    """The new design's kernels alone, CUDA events, back to back, beside the like kernel of another model: attention in chunks
+    with a gate a lane and differential attention (one 2,048-token prompt; 64 sequences of 1,088 tokens) beside the dense
+    decoder's attention, what stands between projection and attention, the selective scan beside the state-space scan of the
+    same channels, feed-forwards and experts with a squared relu beside the dense decoder's and the GELU experts."""
+    import torch
+    from types import SimpleNamespace
+    from burn_lm_b200 import kernels as K
+    from burn_lm_b200.parts.linear import Linear
+    dev, bf = "cuda", torch.bfloat16
+    H, G, hd, d, W = z["heads"], z["kv"], z["hd"], z["width"], z["window"]
+    out = {}
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    frac_bf16 = lambda flops, ms: round(flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12), 4)
+    frac_hbm = lambda nbytes, ms: round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4)
+
+    def step(n_seqs, new, cached):
+        seq = [s for s in range(n_seqs) for _ in range(new)]
+        pos = [cached + t for _ in range(n_seqs) for t in range(new)]
+        return SimpleNamespace(token_seq=i32(seq), token_pos=i32(pos), slot_of_seq=i32(list(range(n_seqs))),
+                               cu_seqlens=i32([new * s for s in range(n_seqs + 1)]), start_pos=i32([cached] * n_seqs),
+                               n_tokens=n_seqs * new, n_seqs=n_seqs, max_q_len=new, max_kv_len=cached + new)
+
+    for n_seqs, new, cached in ((1, 2048, 0), (64, 1, 1087)):
+        total, prompt = cached + new, new > 1
+        pages_each = -(-total // K.PAGE)
+        n = n_seqs * new
+        bt = torch.arange(n_seqs * pages_each, dtype=torch.int32, device=dev).reshape(n_seqs, pages_each)
+        st = step(n_seqs, new, cached)
+        pool5 = torch.randn((n_seqs * pages_each, 2, G, K.PAGE, hd), dtype=bf, device=dev)
+        pool = pool5.view(n_seqs * pages_each, -1)          # two key maps and one value of twice the size on half the heads: the same bytes
+        q = torch.randn((n, H * hd), dtype=bf, device=dev)
+        o = torch.empty_like(q)
+        gate = torch.randn((n, H * hd), dtype=torch.float32, device=dev)
+        llama = lambda w: _time(lambda: K.attention(q, q.shape[1], pool5, bt, st.cu_seqlens, st.slot_of_seq, st.start_pos, o, n, n_seqs, new,
+                                                    H, G, hd, hd ** -0.5, window=w, n_splits=1, max_kv_len=total))
+        ms_l, ms_lw = llama(0), llama(W)
+        windowed = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, hd, hd ** -0.5, W, 0, sink=False, max_q_len=new))
+        chunks = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, hd, hd ** -0.5, 1 << 30, 0, sink=False, max_q_len=new, chunk=W,
+                                                gate=gate, gate_stride=gate.stride(0), gate_lanes=hd))
+        plain = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, hd, hd ** -0.5, 1 << 30, 0, sink=False, max_q_len=new))
+        scratch = torch.empty(K.attention_sink_scratch_floats(n, H, 2 * hd, 1, 2), dtype=torch.float32, device=dev)
+        diff = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, 2 * hd, hd ** -0.5, 1 << 30, 0, sink=False, max_q_len=new, maps=2,
+                                              difference=(0.5, 0.6, 1e-6), scratch=scratch))
+        r = {"llama_ms": round(ms_l, 4), "llama_window_ms": round(ms_lw, 4), "windowed_family_no_mask_ms": round(plain, 4),
+             "windowed_family_window_ms": round(windowed, 4), "chunks_ms": round(chunks, 4), "difference_ms": round(diff, 4)}
+        if prompt:
+            full = new * (new + 1) / 2
+            in_window, in_chunk = sum(min(t + 1, W) for t in range(new)), sum(t % W + 1 for t in range(new))
+            r.update(llama_frac_bf16=frac_bf16(4.0 * H * hd * full, ms_l), llama_window_frac_bf16=frac_bf16(4.0 * H * hd * in_window, ms_lw),
+                     windowed_family_no_mask_frac_bf16=frac_bf16(4.0 * H * hd * full, plain),
+                     windowed_family_window_frac_bf16=frac_bf16(4.0 * H * hd * in_window, windowed),
+                     chunks_frac_bf16=frac_bf16(4.0 * H * hd * in_chunk, chunks), difference_frac_bf16=frac_bf16(6.0 * H * hd * full, diff))
+        else:
+            key_bytes = n * G * 2 * hd * 2.0
+            seen = (total - 1) % W + 1
+            r.update(keys_seen_in_the_chunk=seen, llama_frac_hbm=frac_hbm(key_bytes * total, ms_l),
+                     llama_window_frac_hbm=frac_hbm(key_bytes * min(total, W), ms_lw), windowed_family_no_mask_frac_hbm=frac_hbm(key_bytes * total, plain),
+                     windowed_family_window_frac_hbm=frac_hbm(key_bytes * min(total, W), windowed),
+                     chunks_frac_hbm=frac_hbm(key_bytes * seen, chunks), difference_frac_hbm=frac_hbm(key_bytes * total, diff))
+        out["attention_prefill_2048" if prompt else "attention_decode_b64"] = r
+        # between the projection and the attention
+        cols = (H + 2 * G) * hd
+        proj = torch.randn((n, cols), dtype=torch.float32, device=dev)
+        qkv = torch.randn((n, cols), dtype=bf, device=dev)
+        freq = torch.tensor([500000.0 ** (-2.0 * i / hd) for i in range(hd // 2)], dtype=torch.float64, device=dev)
+        ms_new = _time(lambda: K.head_norm_rope_append(proj, st, pool, bt, q, H, G, hd, 2 * hd, freq=freq, rotary_dims=hd, halves=True, maps=2))
+        ms_llama = _time(lambda: K.rope_append(qkv, st.token_seq, st.token_pos, st.slot_of_seq, bt, freq, hd, K.PAIRS_HALVES, pool5, H, G, hd,
+                                               write_cache=True, max_position=cached + new - 1))
+        out[f"between_{n_seqs}x{new}"] = {"turn_append_two_maps_ms": round(ms_new, 4), "llama_turn_append_ms": round(ms_llama, 4),
+                                          "frac_hbm": frac_hbm(n * cols * 6.0, ms_new), "llama_frac_hbm": frac_hbm(n * cols * 4.0, ms_llama)}
+        # the scan: rows in and out, and the states
+        C, S, R = 2 * d, 16, d // 16
+        state = torch.zeros((n_seqs, 2, C * S), dtype=torch.float32, device=dev)
+        x, dt = torch.randn((n, C), dtype=torch.float32, device=dev), torch.randn((n, C), dtype=torch.float32, device=dev)
+        xz = torch.randn((n, 2 * C), dtype=torch.float32, device=dev)
+        low = torch.randn((n, R + 2 * S), dtype=torch.float32, device=dev)
+        a_log, one = torch.zeros((C, S), dtype=torch.float32, device=dev), torch.ones(C, dtype=torch.float32, device=dev)
+        y = torch.empty((n, C), dtype=bf, device=dev)
+        ms_scan = _time(lambda: K.selective_scan(x, low, R, S, one, a_log, one, xz[:, C:], y, st, state, 0, dt=dt))
+        nbytes = n * C * (3 * 4.0 + 2.0) + 4.0 * n * 2 * S + (2.0 if not prompt else 1.0) * 4 * n_seqs * C * S
+        heads, groups, rows, dv = C // 64, 8, 128, 64
+        floats = K.scan_state_floats(heads, rows, dv)
+        state2 = torch.zeros((n_seqs, 2, floats), dtype=torch.float32, device=dev)
+        xbc = torch.randn((n, C + 2 * groups * rows), dtype=torch.float32, device=dev)
+        dth, zero, y2 = torch.randn((n, heads), dtype=torch.float32, device=dev), torch.zeros(heads, dtype=torch.float32, device=dev), torch.zeros((n, C), dtype=torch.float32, device=dev)
+        ms_ssm = _time(lambda: K.ssm_scan(xbc, 0, C, C + groups * rows, dth, 0, zero, zero, zero, y2, heads, groups, rows, dv, st, state2, 0), reps=3)
+        ssm_bytes = 4.0 * n * (2 * C + 2 * groups * rows + heads) + 2.0 * 4 * n_seqs * floats
+        taps = torch.randn((C, 4), dtype=torch.float32, device=dev)
+        hist = torch.zeros((n_seqs, 2, 3 * C), dtype=torch.float32, device=dev)
+        xb = torch.empty((n, C), dtype=bf, device=dev)
+        ms_conv = _time(lambda: K.causal_conv(xz, 0, C, taps, one, x, 0, st, hist, 0, silu=True, out_bf16=xb))
+        out[f"scan_{n_seqs}x{new}"] = {"selective_ms": round(ms_scan, 4), "selective_frac_hbm": frac_hbm(nbytes, ms_scan),
+                                       "exponentials_per_ns": round(n * C * S / (ms_scan * 1e6), 1), "state_space_ms": round(ms_ssm, 4),
+                                       "state_space_frac_hbm": frac_hbm(ssm_bytes, ms_ssm), "convolution_ms": round(ms_conv, 4),
+                                       "convolution_frac_hbm": frac_hbm(n * C * 10.0, ms_conv)}
+        resid, delta = torch.randn((n, d), dtype=torch.float32, device=dev), torch.randn((n, d), dtype=torch.float32, device=dev)
+        gamma, xo = torch.ones(d, dtype=torch.float32, device=dev), torch.empty((n, d), dtype=bf, device=dev)
+        ms_entry = _time(lambda: K.pass_entry(resid, delta, delta, gamma))
+        ms_norm = _time(lambda: K.add_rmsnorm(resid, delta, gamma, 1e-6, xo))
+        out[f"stream_{n_seqs}x{new}"] = {"pass_entry_ms": round(ms_entry, 4), "pass_entry_frac_hbm": frac_hbm(n * d * 16.0, ms_entry),
+                                         "add_norm_ms": round(ms_norm, 4), "add_norm_frac_hbm": frac_hbm(n * d * 14.0, ms_norm)}
+    # feed-forwards of a token's work
+    E, top = z["experts"], z["top"]
+    ff, each = 3 * z["inner"] // 2, 3 * z["inner"] // (2 * top)
+    w_up, w_down = Linear(torch.randn((ff, d), dtype=bf, device=dev) * 0.02), Linear(torch.randn((d, ff), dtype=bf, device=dev) * 0.02)
+    w1, w2 = Linear(torch.randn((2 * z["inner"], d), dtype=bf, device=dev) * 0.02, gate_tile=K.GATE_TILE), Linear(torch.randn((d, z["inner"]), dtype=bf, device=dev) * 0.02)
+    up, down = torch.randn((E, each, d), dtype=bf, device=dev) * 0.02, torch.randn((E, d, each), dtype=bf, device=dev) * 0.02
+    router, bias = torch.randn((E, d), dtype=torch.float32, device=dev), torch.randn(E, dtype=torch.float32, device=dev)
+    for n in (2048, 64, 8):
+        h = torch.randn((n, d), dtype=bf, device=dev)
+        ms_up = _time(lambda: w_up.activated(h, bf, K.ACT_RELU2))
+        ms_gated = _time(lambda: w1.gated(h, bf))
+        ms_mlp = _time(lambda: w_down(w_up.activated(h, bf, K.ACT_RELU2), out_dtype=torch.float32))
+        ms_llama = _time(lambda: w2(w1.gated(h, bf)))
+        ms_route = _time(lambda: K.moe_route(h, router, top, scores=K.SCORES_CHOSEN_SOFTMAX, bias=bias))
+        ids, weights = K.moe_route(h, router, top, scores=K.SCORES_CHOSEN_SOFTMAX, bias=bias)
+        run = lambda unit: _time(lambda: K.moe_experts(h, ids, weights, up, down, weight_on_input=False, out_dtype=torch.float32, unit=unit))
+        ms_moe, ms_gelu = run(K.UNIT_RELU2), run(K.UNIT_GELU)
+        flops, wbytes = 4.0 * n * ff * d, 2.0 * 2 * each * d * min(E, n * top)
+        out[f"feed_forward_{n}_tokens"] = {
+            "up_relu2_ms": round(ms_up, 4), "llama_gate_up_ms": round(ms_gated, 4), "mlp_ms": round(ms_mlp, 4), "llama_mlp_ms": round(ms_llama, 4),
+            "mlp_frac_bf16": frac_bf16(flops, ms_mlp), "llama_frac_bf16": frac_bf16(6.0 * n * z["inner"] * d, ms_llama),
+            "mlp_frac_hbm": frac_hbm(4.0 * ff * d, ms_mlp), "llama_frac_hbm": frac_hbm(6.0 * z["inner"] * d, ms_llama),
+            "route_ms": round(ms_route, 4), "experts_relu2_ms": round(ms_moe, 4), "experts_gelu_ms": round(ms_gelu, 4),
+            "experts_frac_bf16": frac_bf16(4.0 * n * top * each * d, ms_moe), "experts_frac_hbm": frac_hbm(wbytes, ms_moe)}
+    return out
+
+
 def run_compare(args):
     """One JSON line per size and model: prefill of one 2,048-token prompt and decode at batch 8 and 64 after 512-token
     prompts, for the dense Llama decoder and the named design (Fobilorn with dense feed-forwards and with experts, Nufolix,
-    Ridopel) at equal layer sizes with random weights; then a line with the kernels alone."""
+    Ridopel, Marinex, Tomalix) at equal layer sizes with random weights; then a line with the kernels alone."""
     import torch
     import burn_lm_b200 as blm
     if not torch.cuda.is_available():
@@ -815,9 +969,12 @@ def run_compare(args):
     for size, z in COMPARE_SIZES.items():
         if args.size and size != args.size:
             continue
-        if args.compare in ("ridopel", "marinex"):
+        if args.compare in ("ridopel", "marinex", "tomalix"):
             z = dict(z, experts=8)          # 8 experts of half the dense inner size each: four times the dense layer's weights
-        configs = {"nufolix": nufolix_configs, "ridopel": ridopel_configs, "marinex": marinex_configs}.get(args.compare, compare_configs)(z)
+        if args.compare == "tomalix":
+            z = dict(z, layers=3)           # one layer of every kind
+        configs = {"nufolix": nufolix_configs, "ridopel": ridopel_configs, "marinex": marinex_configs,
+                   "tomalix": tomalix_configs}.get(args.compare, compare_configs)(z)
         for name, cfg in configs.items():
             vocab = z["vocab"]
             lm = blm.load_random(cfg, seed=0, dtype="bfloat16", max_seq_len=4096, max_batch=64, max_tokens=64 * 1024)
@@ -834,7 +991,8 @@ def run_compare(args):
             print(json.dumps(line), flush=True)
             del lm, engine
             torch.cuda.empty_cache()
-        alone = {"nufolix": nufolix_kernels, "ridopel": ridopel_kernels, "marinex": marinex_kernels}.get(args.compare, compare_kernels)(z, pk)
+        alone = {"nufolix": nufolix_kernels, "ridopel": ridopel_kernels, "marinex": marinex_kernels,
+                 "tomalix": tomalix_kernels}.get(args.compare, compare_kernels)(z, pk)
         print(json.dumps({"compare": size, "kernels": alone, "peaks": pk["source"]}), flush=True)
     return 0
 
@@ -949,7 +1107,7 @@ def main():
     ap.add_argument("--only", default=None, choices=["decode", "prefill", "sweep"],
                     help="run one workload briefly (for profilers), or a sweep over batch sizes and context lengths")
     ap.add_argument("--prompt-tokens", type=int, default=0, help="with --only prefill: one prompt of this many tokens instead of the workload's")
-    ap.add_argument("--compare", default=None, choices=["fobilorn", "nufolix", "ridopel", "marinex"],
+    ap.add_argument("--compare", default=None, choices=["fobilorn", "nufolix", "ridopel", "marinex", "tomalix"],
                     help="instead of the workload: the named design beside the dense Llama decoder at equal layer sizes "
                          "(prefill and decode throughput, then its kernels alone), one JSON line each")
     ap.add_argument("--size", default=None, choices=sorted(COMPARE_SIZES), help="with --compare: one of the sizes only")

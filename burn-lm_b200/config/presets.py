@@ -169,6 +169,47 @@ _PRESETS["marinex_tiny"] = {
 }
 
 
+def _tomalix_experts(experts, top, ff):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+
+
+def _tomalix_difference(heads, kv_heads, dim, vdim, rot_dims, scale, diff, base, factor, mlp):
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "diff": diff,
+                      "rot": {"dims": rot_dims, "base": base, "scaling": {"factor": factor}}}}
+
+
+def _tomalix_scaled(heads, kv_heads, dim, vdim, rot_dims, scale, base, scaling, mlp):
+    return {"type": "attention_2", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale,
+                      "rot": {"dims": rot_dims, "base": base, "scaling": dict(zip(("factor", "original", "fast", "slow"), scaling))}}}
+
+
+def _tomalix_pair(heads, kv_heads, dim, vdim, rot_dims, scale, chunk, inner, state, conv, dt_rank, scales, mlp):
+    return {"type": "parallel", "mlp": mlp,
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": chunk},
+                               "rot": {"dims": rot_dims, "base": 20000.0}},
+                      "right": {"inner": inner, "state": state, "conv": conv, "dt_rank": dt_rank},
+                      "left_scale": scales[0], "right_scale": scales[1]}}
+
+
+# a small Tomalix decoder that uses every branch of the design: all three mixers, dense feed-forwards, experts and none,
+# several query heads a key/value head and one, values wider and narrower than the keys, some and all of a head's lanes
+# turning, chunks inside a cache page and across page borders, a loop over layers of two kinds
+_PRESETS["tomalix_tiny"] = {
+    "architecture": "Tomalix", "vocab": 272, "width": 96, "norm": {"eps": 1e-5}, "logit_softcap": 20.0,
+    "loop": {"start": 1, "stop": 4, "times": 2},
+    "layers": [
+        _tomalix_difference(4, 2, 16, 32, 16, 0.3, 0.35, 10000.0, 2.5, _tomalix_experts(6, 2, 48)),
+        _tomalix_pair(4, 2, 24, 40, 12, 0.25, 80, 128, 16, 4, 8, (0.8, 0.45), {"kind": "dense", "ff": 160}),
+        _tomalix_scaled(6, 3, 32, 16, 24, 0.2, 500000.0, (8.0, 256, 16.0, 1.0), None),
+        _tomalix_pair(2, 2, 16, 16, 16, 0.3, 24, 64, 8, 3, 6, (0.5, 0.9), _tomalix_experts(5, 3, 32)),
+        _tomalix_difference(3, 1, 24, 16, 8, 0.25, 0.6, 3000.0, 4.0, {"kind": "dense", "ff": 128}),
+        _tomalix_scaled(2, 1, 16, 16, 16, 0.25, 1000.0, (3.0, 64, 8.0, 2.0), {"kind": "dense", "ff": 64}),
+    ],
+}
+
+
 def preset_names() -> list:
     return sorted(_PRESETS)
 

@@ -189,7 +189,7 @@ template <typename T>
 __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, long long proj_stride, int n_heads, int n_kv, int n_v,
                                              int dk, int dv, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
                                              int value_norm, const double* __restrict__ freq, int rot_dims, int halves, float turn_scale,
-                                             T* __restrict__ q_out, T* __restrict__ pool, long long page_elems, int page_size,
+                                             const float2* __restrict__ table, int table_len, T* __restrict__ q_out, T* __restrict__ pool, long long page_elems, int page_size,
                                              const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                                              const int* __restrict__ slot_of_seq, const int* __restrict__ block_table,
                                              int table_stride) {
@@ -200,6 +200,10 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
     const bool real = seq >= 0;                        // a row of no sequence leaves zeros in q and reaches no cache
     const int pos = real ? token_pos[n] : 0;
     for (int i = threadIdx.x; i < rot_dims / 2; i += blockDim.x) {
+        if (pos < table_len) {                         // the same numbers, worked out once
+            turn[i] = table[(size_t)pos * (rot_dims / 2) + i];
+            continue;
+        }
         double sn, cs;
         sincos((double)pos * freq[i], &sn, &cs);
         turn[i] = make_float2(turn_scale * (float)cs, turn_scale * (float)sn);
@@ -246,7 +250,7 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
 
 BLM_API int blm_head_norm_rope_append(const float* proj, long long proj_stride, int n_tokens, int n_heads, int n_kv, int maps, int dk,
                                       int dv, const float* wq, const float* wk, float eps, int value_norm, const double* freq, int rot_dims,
-                                      int halves, float turn_scale, void* q_out, void* pool, int dtype, long long page_elems, int page_size,
+                                      int halves, float turn_scale, const float* table, int table_len, void* q_out, void* pool, int dtype, long long page_elems, int page_size,
                                       const int* token_seq, const int* token_pos, const int* slot_of_seq, const int* block_table,
                                       int table_stride, cudaStream_t stream) {
     if (n_tokens == 0) return BLM_OK;
@@ -257,11 +261,12 @@ BLM_API int blm_head_norm_rope_append(const float* proj, long long proj_stride, 
                 "head_norm_rope_append: a page holds page * (n_kv * dk + n_kv / maps * dv) elements");
     BLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || freq != nullptr),
                 "head_norm_rope_append: %d turning lanes of %d", rot_dims, dk);
+    if (table == nullptr) table_len = 0;               // [table_len][rot_dims / 2] (cosine, sine), already times turn_scale
     const int vectors = n_heads + n_kv + n_v;
     const int threads = vectors >= 8 ? 256 : 32 * vectors;
 #define BLM_HNRA(T)                                                                                                              \
     head_norm_rope_append_kernel<T><<<n_tokens, threads, (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream>>>(proj, proj_stride, n_heads, n_kv, n_v, dk, dv, wq, wk, eps, value_norm, \
-        freq, rot_dims, halves, turn_scale, (T*)q_out, (T*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride)
+        freq, rot_dims, halves, turn_scale, (const float2*)table, table_len, (T*)q_out, (T*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride)
     if (dtype == BLM_F32) BLM_HNRA(float);
     else if (dtype == BLM_BF16) BLM_HNRA(__nv_bfloat16);
     else return blm_fail(BLM_BAD_ARGUMENT, "head_norm_rope_append: dtype %d", dtype);
@@ -597,10 +602,11 @@ struct GroupWalk {
 // one page's keys and values of one kv head into a buffer pair (every thread of the block takes its share)
 __device__ __forceinline__ void stage_page(__nv_bfloat16* kbuf, __nv_bfloat16* vbuf, const __nv_bfloat16* page, int n_kv, int kvh, int vh,
                                            int dk, int dv, int qstride, int vstride, int first_pos, int p_last, const GroupWalk& kw,
-                                           const GroupWalk& vw) {
+                                           const GroupWalk& vw, int key_rows = kTileK) {
+    // key_rows: 2 kTileK brings the keys of the next key head as well (they lie behind these)
     const __nv_bfloat16* kpage = page + (size_t)kvh * kTileK * dk;
     const __nv_bfloat16* vpage = page + (size_t)n_kv * kTileK * dk + (size_t)vh * kTileK * dv;
-    for (int r = kw.r, c = kw.c; r < kTileK;) {
+    for (int r = kw.r, c = kw.c; r < key_rows;) {
         cp_async16(kbuf + r * qstride + c * 8, kpage + r * dk + c * 8, true);
         r += kw.dr;
         c += kw.dc;
@@ -875,52 +881,65 @@ static int launch_prompt(const void* q, const void* pool, long long page_elems, 
 // 1,088 tokens on 8 kv heads: heads of 64 lanes 45 us with two stages (five blocks to a multiprocessor), 60 with three,
 // 61 with four; heads of 128 lanes 84, 79 and 121 us.
 
-template <int NV, int kDecodeStages>
+//
+// PAIR: two maps a head, both in one block, so that a page's values are brought in once for both: a block per (token, value
+// head, split); rows 0 .. 7 of the tile are the group's first maps and rows 8 .. 15 their second maps; both key heads' keys
+// of a page lie in shared memory and the products with either give all sixteen rows, of which each keeps its own eight.
+// Without splits the block also forms the difference (DiffOpts) itself.
+
+template <int NV, int kDecodeStages, bool PAIR>
 __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool, long long page_elems,
     const int* __restrict__ block_table, int table_stride, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
     const int* __restrict__ slot_of_seq, RowOut ro, __nv_bfloat16* __restrict__ out, float* __restrict__ partial, int n_heads, int n_kv,
-    int maps, int dk, int dv, Mask mask, int keep_first, float scale, int sink, ScoreOpts so) {
+    int maps, int dk, int dv, Mask mask, int keep_first, float scale, int sink, ScoreOpts so, DiffOpts df) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int n = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z, n_splits = gridDim.z;
+    const int n = blockIdx.x, kvh = PAIR ? 2 * blockIdx.y : blockIdx.y, split = blockIdx.z, n_splits = gridDim.z;
     const int group = n_heads / n_kv;                  // <= 16: the rows of the tile
     const int dkp = (dk + 15) & ~15;
     const int qstride = dkp + 8;
     constexpr int vstride = 8 * NV + 8;
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [16][qstride]
-    __nv_bfloat16* Kb = Qs + 16 * qstride;                               // kDecodeStages x [64][qstride]
-    __nv_bfloat16* Vb = Kb + kDecodeStages * kTileK * qstride;           // kDecodeStages x [64][vstride]
+    constexpr int kKeyRows = PAIR ? 2 * kTileK : kTileK;
+    __nv_bfloat16* Kb = Qs + 16 * qstride;                               // kDecodeStages x [kKeyRows][qstride]
+    __nv_bfloat16* Vb = Kb + kDecodeStages * kKeyRows * qstride;         // kDecodeStages x [64][vstride]
     const int seq = token_seq[n];
     const int vh = kvh / maps, head0 = vh * group * maps + kvh % maps;      // this key head's query heads: head0, head0 + maps, ...
+    // rows of the tile that stand for a query, and its head (every map counted)
+    auto row_head = [&](int r) { return PAIR ? head0 + 2 * (r & 7) + (r >> 3) : head0 + r * maps; };
+    auto row_used = [&](int r) { return PAIR ? (r & 7) < group : r < group; };
     if (seq < 0) {                                     // a row of no sequence: zeros, nothing read
         if (partial == nullptr)
-            for (int c = tid; c < group * dv; c += 128) out[(size_t)n * ro.stride + (size_t)head0 * dv + c] = __float2bfloat16_rn(0.f);
+            for (int c = tid; c < group * dv; c += 128) out[(size_t)n * ro.stride + (size_t)(PAIR ? head0 / 2 : head0) * dv + c] = __float2bfloat16_rn(0.f);
         else
-            for (int c = tid; c < group * (dv + 2); c += 128) {
-                const int head = head0 + c / (dv + 2) * maps, e = c % (dv + 2);
+            for (int c = tid; c < (PAIR ? 2 : 1) * group * (dv + 2); c += 128) {
+                const int head = head0 + c / (dv + 2) * (PAIR ? 1 : maps), e = c % (dv + 2);
                 partial[(((size_t)n * n_heads + head) * n_splits + split) * (dv + 2) + e] = e == 0 ? -INFINITY : 0.f;
             }
         return;
     }
     const int pos = token_pos[n];
     const int* pages = block_table + (size_t)slot_of_seq[seq] * table_stride;
-    zero_unwritten(Qs, 16, qstride, group, dk);
-    zero_unwritten(Kb, kDecodeStages * kTileK, qstride, kDecodeStages * kTileK, dk);
+    for (int idx = tid; idx < 16 * (qstride / 8); idx += 128) {          // zeros where no copy will write
+        const int r = idx / (qstride / 8), c = (idx % (qstride / 8)) * 8;
+        if (!row_used(r) || c >= dk) *reinterpret_cast<uint4*>(Qs + r * qstride + c) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    zero_unwritten(Kb, kDecodeStages * kKeyRows, qstride, kDecodeStages * kKeyRows, dk);
     zero_unwritten(Vb, kDecodeStages * kTileK, vstride, kDecodeStages * kTileK, dv);
     const int lo = mask.first(pos);
     const PageWalk walk(lo, pos, keep_first);
     const int per_split = (walk.n_tiles + n_splits - 1) / n_splits;
     const int it_begin = split * per_split, it_end = min(walk.n_tiles, it_begin + per_split);
-    for (int idx = tid; idx < group * (dk / 8); idx += 128) {
+    for (int idx = tid; idx < 16 * (dk / 8); idx += 128) {
         const int r = idx / (dk / 8), c = (idx % (dk / 8)) * 8;
-        cp_async16(Qs + r * qstride + c, q + ((size_t)n * n_heads + head0 + r * maps) * dk + c, true);
+        if (row_used(r)) cp_async16(Qs + r * qstride + c, q + ((size_t)n * n_heads + row_head(r)) * dk + c, true);
     }
     const GroupWalk kw(dk / 8), vw(dv / 8);
     auto fetch = [&](int it) {                         // page `it` of the walk into its place in the ring
         const int pg = walk.page(it), b = (it - it_begin) % kDecodeStages;
-        stage_page(Kb + b * kTileK * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
-                   vstride, pg * kTileK, pos, kw, vw);
+        stage_page(Kb + b * kKeyRows * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
+                   vstride, pg * kTileK, pos, kw, vw, kKeyRows);
     };
 #pragma unroll
     for (int ahead = 0; ahead < kDecodeStages - 1; ++ahead) {
@@ -936,8 +955,8 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
 #pragma unroll
     for (int half = 0; half < 2; ++half) {                       // this thread's two rows are two heads of the group
         const int r = quad + 8 * half;
-        pre[half] = scale * (so.head_scale && r < group ? so.head_scale[head0 + r * maps] : 1.f);
-        m[half] = with_sink ? (so.sink_logit && r < group ? so.sink_logit[head0 + r * maps] * log2e : 0.f) : -INFINITY;
+        pre[half] = scale * (so.head_scale && row_used(r) ? so.head_scale[row_head(r)] : 1.f);
+        m[half] = with_sink ? (so.sink_logit && row_used(r) ? so.sink_logit[row_head(r)] * log2e : 0.f) : -INFINITY;
         l[half] = with_sink ? 0.25f : 0.f;
     }
 #pragma unroll
@@ -953,8 +972,9 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
         cp_async_wait_all_but<kDecodeStages - 1>();    // this page (and the queries) have landed; the others may be on their way
         __syncthreads();
         const int pg = walk.page(it);
-        const unsigned kb = kb0 + buf * kTileK * qstride * 2, vb = vb0 + buf * kTileK * vstride * 2;
-        float s[2][4];
+        const unsigned kb = kb0 + buf * kKeyRows * qstride * 2, vb = vb0 + buf * kTileK * vstride * 2;
+        float s[2][4], s2[2][4];
+        s2[0][0] = s2[0][1] = s2[0][2] = s2[0][3] = s2[1][0] = s2[1][1] = s2[1][2] = s2[1][3] = 0.f;
         s[0][0] = s[0][1] = s[0][2] = s[0][3] = s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.f;
         for (int kk = 0; kk < dkp; kk += 16) {
             uint32_t a[4], b[4];
@@ -962,6 +982,15 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
             ldsm_x4(b, kb + kk * 2);
             mma_bf16(s[0], a, b[0], b[1]);
             mma_bf16(s[1], a, b[2], b[3]);
+            if (PAIR) {
+                ldsm_x4(b, kb + (kTileK * qstride + kk) * 2);
+                mma_bf16(s2[0], a, b[0], b[1]);
+                mma_bf16(s2[1], a, b[2], b[3]);
+            }
+        }
+        if (PAIR) {                                    // rows 8 .. 15 look at the second map's keys
+            s[0][2] = s2[0][2]; s[0][3] = s2[0][3];
+            s[1][2] = s2[1][2]; s[1][3] = s2[1][3];
         }
         // every row (head) sees the same keys
 #pragma unroll
@@ -1028,8 +1057,53 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
         }
     }
     __syncthreads();
-    for (int idx = tid; idx < group * dv; idx += 128) {
-        const int r = idx / dv, d = idx % dv;
+    if (PAIR && partial == nullptr) {                  // the difference of the two maps, a warp a head
+        constexpr int kLanes = (NV + 3) / 4;           // value lanes of a thread
+        for (int r = warp; r < group; r += 4) {
+            float acc[kLanes];
+#pragma unroll
+            for (int i = 0; i < kLanes; ++i) acc[i] = 0.f;
+#pragma unroll
+            for (int m2 = 0; m2 < 2; ++m2) {
+                const float* src = sh + (size_t)(r + 8 * m2) * rstride;
+                float big = -INFINITY, lsum = 0.f, f[4];
+#pragma unroll
+                for (int w = 0; w < 4; ++w) big = fmaxf(big, src[(size_t)w * 16 * rstride]);
+#pragma unroll
+                for (int w = 0; w < 4; ++w) {
+                    const float mw = src[(size_t)w * 16 * rstride];
+                    f[w] = mw > -INFINITY ? fast_exp2(mw - big) : 0.f;
+                    lsum += src[(size_t)w * 16 * rstride + 1] * f[w];
+                }
+                const float wgt = lsum > 0.f ? (m2 == 0 ? 1.f : -df.lambda) / lsum : 0.f;
+#pragma unroll
+                for (int i = 0; i < kLanes; ++i) {
+                    const int d = lane + 32 * i;
+                    if (d < dv) {
+                        float v = 0.f;
+#pragma unroll
+                        for (int w = 0; w < 4; ++w) v = fmaf(f[w], src[(size_t)w * 16 * rstride + 2 + d], v);
+                        acc[i] = fmaf(wgt, v, acc[i]);
+                    }
+                }
+            }
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < kLanes; ++i) ss += acc[i] * acc[i];
+            ss = warp_sum(ss);
+            const int head = vh * group + r;
+            const float inv = df.c / sqrtf(ss / (float)dv + df.eps) * ro.head_gate(n, head);
+#pragma unroll
+            for (int i = 0; i < kLanes; ++i) {
+                const int d = lane + 32 * i;
+                if (d < dv) out[(size_t)n * ro.stride + (size_t)head * dv + d] = __float2bfloat16_rn(acc[i] * inv * ro.lane_gate(n, head, d));
+            }
+        }
+        return;
+    }
+    for (int idx = tid; idx < (PAIR ? 2 : 1) * group * dv; idx += 128) {
+        const int item = idx / dv, d = idx % dv;
+        const int r = PAIR ? (item % group) + 8 * (item / group) : item;
         float big = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) big = fmaxf(big, sh[((size_t)w * 16 + r) * rstride]);
@@ -1043,7 +1117,7 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
                 acc += src[2 + d] * f;
             }
         }
-        const int head = head0 + r * maps;
+        const int head = row_head(r);
         if (partial != nullptr) {
             float* part = partial + (((size_t)n * n_heads + head) * n_splits + split) * (dv + 2);
             if (d == 0) {
@@ -1058,23 +1132,23 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     }
 }
 
-template <int NV, int kDecodeStages>
+template <int NV, int kDecodeStages, bool PAIR>
 static int launch_decode(const void* q, const void* pool, long long page_elems, const int* block_table, int table_stride,
                          const int* token_seq, const int* token_pos, const int* slot_of_seq, RowOut ro, void* out, float* partial,
                          int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, Mask mask, int keep_first,
                          float scale, int sink, ScoreOpts so, DiffOpts df, cudaStream_t stream) {
     const int dkp = (dk + 15) & ~15;
-    size_t smem = ((size_t)16 * (dkp + 8) + (size_t)kDecodeStages * kTileK * ((dkp + 8) + (8 * NV + 8))) * sizeof(__nv_bfloat16);
+    size_t smem = ((size_t)16 * (dkp + 8) + (size_t)kDecodeStages * kTileK * ((PAIR ? 2 : 1) * (dkp + 8) + (8 * NV + 8))) * sizeof(__nv_bfloat16);
     const size_t merge = (size_t)16 * (dkp + 8) * sizeof(__nv_bfloat16) + (size_t)4 * 16 * (8 * NV + 2) * sizeof(float);
     if (merge > smem) smem = merge;
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "attention_sink: %s", cudaGetErrorString(e));
     }
-    cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
-    attention_sink_decode_kernel<NV, kDecodeStages><<<dim3(n_tokens, n_kv, n_splits), 128, smem, stream>>>(
+    cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages, PAIR>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    attention_sink_decode_kernel<NV, kDecodeStages, PAIR><<<dim3(n_tokens, PAIR ? n_kv / 2 : n_kv, n_splits), 128, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro,
-        (__nv_bfloat16*)out, partial, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so);
+        (__nv_bfloat16*)out, partial, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df);
     if (partial != nullptr) finish_shares<__nv_bfloat16>(partial, ro, out, n_tokens, n_heads, maps, dv, n_splits, df, stream);
     return blm_check_launch("attention_sink (decode)");
 }
@@ -1115,6 +1189,11 @@ BLM_API int blm_attention_sink_decode_takes(int dtype, int dk, int dv, int page_
            n_kv > 0 && n_heads % n_kv == 0 && n_heads / n_kv <= 16;
 }
 
+// Whether the decode kernel takes both maps of a head in one block (and, without splits, forms the difference there).
+BLM_API int blm_attention_sink_pairs(int dtype, int dk, int dv, int page_size, int n_heads, int n_kv, int maps) {
+    return maps == 2 && blm_attention_sink_decode_takes(dtype, dk, dv, page_size, n_heads, n_kv) && n_heads / n_kv <= 8 && dk <= 128;
+}
+
 BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long long page_elems, const int* block_table,
                                int table_stride, const int* token_seq, const int* token_pos, const int* slot_of_seq,
                                const int* cu_seqlens, const int* start_pos, int n_seqs, int max_q_len, const float* gate,
@@ -1132,7 +1211,10 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
                 "attention_sink: bad sizes");
     BLM_REQUIRE(dv <= 32 * kMaxVRegs, "attention_sink: values of %d lanes; at most %d", dv, 32 * kMaxVRegs);
     BLM_REQUIRE(window >= 1 && chunk >= 0 && keep_first >= 0, "attention_sink: window %d, chunk %d, kept first %d", window, chunk, keep_first);
-    BLM_REQUIRE(maps == 1 || (maps == 2 && n_kv % 2 == 0 && partial != nullptr), "attention_sink: %d maps of %d key heads", maps, n_kv);
+    const bool is_prompt = cu_seqlens != nullptr && start_pos != nullptr && n_seqs > 0 &&
+                           blm_attention_sink_prompt_takes(dtype, dk, dv, page_size, max_q_len, n_heads) && out_stride % 2 == 0 && ((size_t)out & 3) == 0;
+    const bool inside = !is_prompt && n_splits == 1 && blm_attention_sink_pairs(dtype, dk, dv, page_size, n_heads, n_kv, maps);
+    BLM_REQUIRE(maps == 1 || (maps == 2 && n_kv % 2 == 0 && (inside || partial != nullptr)), "attention_sink: %d maps of %d key heads", maps, n_kv);
     BLM_REQUIRE(page_elems == (long long)page_size * ((long long)n_kv * dk + (long long)(n_kv / maps) * dv),
                 "attention_sink: a page holds page * (n_kv * dk + n_kv / maps * dv) elements");
     BLM_REQUIRE(gate_lanes == 0 || gate_lanes == dv, "attention_sink: a gate of %d lanes for values of %d", gate_lanes, dv);
@@ -1143,9 +1225,7 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
     const Mask mask{window, chunk};
     const RowOut ro{gate, gate_stride, gate_lanes, out_stride, out_scale};
     const DiffOpts df{diff_lambda, diff_scale, diff_eps};
-    if (cu_seqlens != nullptr && start_pos != nullptr && n_seqs > 0 &&
-        blm_attention_sink_prompt_takes(dtype, dk, dv, page_size, max_q_len, n_heads) &&
-        out_stride % 2 == 0 && ((size_t)out & 3) == 0) {
+    if (is_prompt) {
 #define BLM_PROMPT(NV) launch_prompt_heads<NV>(hb, q, pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq, n_seqs, ro, \
                                          out, partial, n_tokens, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df, stream)
         const int group = n_heads / n_kv;
@@ -1159,13 +1239,20 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
 #undef BLM_PROMPT
     }
     if (blm_attention_sink_decode_takes(dtype, dk, dv, page_size, n_heads, n_kv)) {
-#define BLM_DECODE(NV, STAGES) launch_decode<NV, STAGES>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, \
+#define BLM_DECODE(NV, STAGES, PAIR) launch_decode<NV, STAGES, PAIR>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, \
                                          out, partial, n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df, stream)
-        if (dv <= 32) return BLM_DECODE(4, 2);
-        if (dv <= 64) return BLM_DECODE(8, 2);
-        if (dv <= 128) return BLM_DECODE(16, 3);
-        if (dv <= 192) return BLM_DECODE(24, 2);
-        return BLM_DECODE(32, 2);
+        if (blm_attention_sink_pairs(dtype, dk, dv, page_size, n_heads, n_kv, maps)) {
+            if (n_splits == 1) partial = nullptr;
+            if (dv <= 64) return BLM_DECODE(8, 2, true);
+            if (dv <= 128) return BLM_DECODE(16, 2, true);
+            if (dv <= 192) return BLM_DECODE(24, 2, true);
+            return BLM_DECODE(32, 2, true);
+        }
+        if (dv <= 32) return BLM_DECODE(4, 2, false);
+        if (dv <= 64) return BLM_DECODE(8, 2, false);
+        if (dv <= 128) return BLM_DECODE(16, 3, false);
+        if (dv <= 192) return BLM_DECODE(24, 2, false);
+        return BLM_DECODE(32, 2, false);
 #undef BLM_DECODE
     }
     if (dtype == BLM_F32)

@@ -1111,7 +1111,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
                                    const T* __restrict__ extra, TO* __restrict__ out, int width, int top, int scale_output, int n_planes,
                                    long long plane) {
     const int n = blockIdx.x;
-    for (int d = threadIdx.x; d < width; d += blockDim.x) {
+    for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < width; d += gridDim.y * blockDim.x) {
         float s = 0.f;
         for (int k = 0; k < top; ++k) {
             const size_t at = (size_t)place_of[(size_t)n * top + k] * width + d;
@@ -1130,15 +1130,18 @@ BLM_API int blm_moe_combine(const float* y, const int* place_of, const float* we
     if (n_tokens == 0) return BLM_OK;
     BLM_REQUIRE(n_tokens > 0 && width > 0 && top > 0 && n_planes >= 1, "moe_combine: bad sizes");
     const long long plane = (long long)n_tokens * top * width;
+    // few tokens: a row's columns over several blocks, so that the planes' sums of a token do not wait for one another
+    const unsigned parts = n_tokens >= 128 ? 1u : (unsigned)((width + 255) / 256 < 64 ? (width + 255) / 256 : 64);
+    const dim3 grid(n_tokens, parts);
     if (dtype == BLM_BF16 && out_dtype == BLM_F32)
-        moe_combine_kernel<__nv_bfloat16, float><<<n_tokens, 256, 0, stream>>>(y, place_of, weights, (const __nv_bfloat16*)extra,
+        moe_combine_kernel<__nv_bfloat16, float><<<grid, 256, 0, stream>>>(y, place_of, weights, (const __nv_bfloat16*)extra,
                                                                                (float*)out, width, top, scale_output, n_planes, plane);
     else if (dtype != out_dtype)
         return blm_fail(BLM_BAD_ARGUMENT, "moe_combine: dtype %d with out dtype %d", dtype, out_dtype);
     else if (dtype == BLM_F32)
-        moe_combine_kernel<float, float><<<n_tokens, 256, 0, stream>>>(y, place_of, weights, (const float*)extra, (float*)out, width, top, scale_output, n_planes, plane);
+        moe_combine_kernel<float, float><<<grid, 256, 0, stream>>>(y, place_of, weights, (const float*)extra, (float*)out, width, top, scale_output, n_planes, plane);
     else if (dtype == BLM_BF16)
-        moe_combine_kernel<__nv_bfloat16, __nv_bfloat16><<<n_tokens, 256, 0, stream>>>(y, place_of, weights, (const __nv_bfloat16*)extra,
+        moe_combine_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 256, 0, stream>>>(y, place_of, weights, (const __nv_bfloat16*)extra,
                                                                                        (__nv_bfloat16*)out, width, top, scale_output, n_planes, plane);
     else
         return blm_fail(BLM_BAD_ARGUMENT, "moe_combine: dtype %d", dtype);

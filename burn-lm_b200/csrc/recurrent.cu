@@ -109,6 +109,54 @@ __global__ void conv_carry_kernel(const float* __restrict__ x, long long x_strid
         if (m < K - 1) fresh[(size_t)m * channels + c] = keep[m];
 }
 
+// The same for portions and up to four taps: a thread owns a channel and kConvRows rows after one another, the taps in
+// registers and the inputs behind the current one in a sliding window (an input is read once a thread, not once a tap).
+constexpr int kConvRows = 16;
+template <int K>
+__global__ void conv_rows_kernel(const float* __restrict__ x, long long x_stride, int x_col0, int channels, const float* __restrict__ taps,
+                                 const float* __restrict__ bias, int act, float* __restrict__ out, long long out_stride, int out_col0,
+                                 const int* __restrict__ token_seq, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
+                                 const int* __restrict__ start_pos, const float* __restrict__ state, long long slot_stride,
+                                 long long copy_stride, long long hist_off, __nv_bfloat16* __restrict__ out_bf, long long out_bf_stride,
+                                 int n_tokens) {
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= channels) return;
+    const int first = blockIdx.y * kConvRows, last = min(n_tokens, first + kConvRows);
+    float w[K], past[K];                        // past[j]: the input j tokens back (past[0]: the current one)
+#pragma unroll
+    for (int j = 0; j < K; ++j) w[j] = taps[(size_t)c * K + (K - 1 - j)];
+    const float b = bias ? bias[c] : 0.f;
+    int held = -1;                              // the sequence the window belongs to
+    const float* in = x + x_col0 + c;
+#pragma unroll 4
+    for (int n = first; n < last; ++n) {
+        const int seq = token_seq[n];
+        float res = 0.f;
+        if (seq >= 0) {
+            if (seq != held) {                  // the window's inputs before this row: the step's, the carried ones, or zeros
+                held = seq;
+                const int i = n - cu_seqlens[seq], start = start_pos[seq];
+                const float* hist = state + (size_t)slot_of_seq[seq] * slot_stride + hist_off + (size_t)(start & 1) * copy_stride;
+#pragma unroll
+                for (int j = 1; j < K; ++j) {
+                    const int back = i - j;
+                    past[j - 1] = back >= 0 ? in[(size_t)(n - j) * x_stride] : (start + back < 0 ? 0.f : hist[(size_t)(K - 1 + back) * channels + c]);
+                }
+            }
+#pragma unroll
+            for (int j = K - 1; j > 0; --j) past[j] = past[j - 1];
+            past[0] = in[(size_t)n * x_stride];
+            float acc = b;
+#pragma unroll
+            for (int j = K - 1; j >= 0; --j) acc += w[j] * past[j];
+            if (act == 2) acc += past[0];
+            res = act == 1 ? silu_f(acc) : acc;
+        }
+        out[(size_t)n * out_stride + out_col0 + c] = res;
+        if (out_bf) out_bf[(size_t)n * out_bf_stride + c] = __float2bfloat16(res);
+    }
+}
+
 BLM_API int blm_causal_conv(const float* x, long long x_stride, int x_col0, int channels, const float* taps, const float* bias,
                             int K, int act, float* out, long long out_stride, int out_col0, const int* token_seq,
                             const int* cu_seqlens, const int* slot_of_seq, const int* start_pos, int n_tokens, int n_seqs,
@@ -119,10 +167,18 @@ BLM_API int blm_causal_conv(const float* x, long long x_stride, int x_col0, int 
     BLM_REQUIRE(channels > 0 && K >= 1 && K <= kMaxTaps, "causal_conv: %d taps; this kernel takes 1 to %d", K, kMaxTaps);
     BLM_REQUIRE(n_tokens <= 65535 && n_seqs <= 65535, "causal_conv: a step of %d rows; this kernel takes 65,535", n_tokens);
     const int threads = 128;
-    dim3 grid((channels + threads - 1) / threads, n_tokens);
-    conv_kernel<<<grid, threads, 0, stream>>>(x, x_stride, x_col0, channels, taps, bias, K, act, out, out_stride, out_col0,
-                                              token_seq, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride,
-                                              hist_off, single_tokens && K > 1 ? 1 : 0, (__nv_bfloat16*)out_bf, out_bf_stride);
+    if (!single_tokens && K >= 2 && K <= 4 && n_tokens >= 4 * kConvRows) {
+        dim3 tiles((channels + threads - 1) / threads, (n_tokens + kConvRows - 1) / kConvRows);
+        auto kern = K == 2 ? conv_rows_kernel<2> : (K == 3 ? conv_rows_kernel<3> : conv_rows_kernel<4>);
+        kern<<<tiles, threads, 0, stream>>>(x, x_stride, x_col0, channels, taps, bias, act, out, out_stride, out_col0, token_seq, cu_seqlens,
+                                            slot_of_seq, start_pos, state, slot_stride, copy_stride, hist_off, (__nv_bfloat16*)out_bf,
+                                            out_bf_stride, n_tokens);
+    } else {
+        dim3 grid((channels + threads - 1) / threads, n_tokens);
+        conv_kernel<<<grid, threads, 0, stream>>>(x, x_stride, x_col0, channels, taps, bias, K, act, out, out_stride, out_col0,
+                                                  token_seq, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride,
+                                                  hist_off, single_tokens && K > 1 ? 1 : 0, (__nv_bfloat16*)out_bf, out_bf_stride);
+    }
     int rc = blm_check_launch("causal_conv");
     if (rc != BLM_OK || K == 1 || single_tokens) return rc;
     dim3 grid2((channels + threads - 1) / threads, n_seqs);
@@ -666,10 +722,15 @@ BLM_API int blm_gated_group_norm(const float* y, long long y_stride, const float
 //     out_c = scale y_c silu(z_c),   dt_c = softplus(dt_raw_c + dt_bias_c),   A = -exp(A_log)
 // x float32 [T, *] (after convolution and silu), B and C columns of low [T, *], z columns of another row.  dt_raw is given
 // [T, C], or (dt_w) formed here from the first `rank` columns of low and dt_w [C, rank]: for single tokens, where a product
-// of its own would be a launch for a few kilobytes.  A block owns (sequence, kSelThreads / G channels); G lanes share a channel,
-// RN neighbouring states each in registers; tokens come in chunks of kChunk through shared memory, and a chunk's results
-// leave through shared memory too, gated and converted by rows.  The state is stored as [channel][state].  AT double: state
-// and sums in float64 inside a step (the 32-bit path), else float with exp2 of A scaled by log2 e.
+// of its own would be a launch for a few kilobytes.  A block owns (sequence, kSelThreads / kSelLanes channels); kSelLanes lanes
+// share a channel, RN neighbouring states each in registers.  The state is stored as [channel][state].  Three kernels:
+//   selective_scan_kernel   portions, bfloat16 results: chunks of kChunk tokens come through cp.async into two buffers in
+//                           turn, one on its way while the other is worked on; a pass makes (dt, dt x) of the raw rows; four
+//                           tokens' sums over the states are reduced together, so that every lane ends with one token's
+//                           sum; results leave gated and converted by rows.  The exponentials are exp2 by the special
+//                           function unit with A scaled by log2 e: at 16 states a channel they are what the kernel takes longest for.
+//   selective_step_kernel   one token a sequence, bfloat16 results: nothing staged but the latents the step sizes are made of.
+//   selective_exact_kernel  the 32-bit path, any portion: state and sums in float64 inside a step.
 // ---------------------------------------------------------------------------------------------
 constexpr int kSelThreads = 128, kSelLanes = 4, kSelChannels = kSelThreads / kSelLanes;
 
@@ -684,11 +745,13 @@ struct SelArgs {
     int channels, n_states;
 };
 
-template <int RN, typename AT, typename TO>
+template <int RN>
 __global__ void __launch_bounds__(kSelThreads)
-    selective_scan_kernel(SelArgs a, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
+    selective_exact_kernel(SelArgs a, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
                           const int* __restrict__ start_pos, float* __restrict__ state, long long slot_stride, long long copy_stride,
                           long long state_off) {
+    typedef double AT;
+    typedef float TO;
     constexpr int NP = RN * kSelLanes, CH = kSelChannels;
     __shared__ __align__(16) float Bs[kChunk][NP], Cs[kChunk][NP];
     __shared__ float dts[kChunk][CH], xs[kChunk][CH], ys[kChunk][CH];
@@ -704,8 +767,7 @@ __global__ void __launch_bounds__(kSelThreads)
         const bool in = live && n0 + r < a.n_states;
         const size_t at = (size_t)c * a.n_states + n0 + r;
         s[r] = in && sq.read ? (AT)sq.read[at] : (AT)0;
-        if (sizeof(AT) == 8) A[r] = in ? (AT)-exp((double)a.A_log[at]) : (AT)0;
-        else A[r] = in ? (AT)(-expf(a.A_log[at]) * 1.4426950408889634f) : (AT)0;
+        A[r] = in ? -exp((double)a.A_log[at]) : 0.0;
     }
     for (int t0 = 0; t0 < sq.n_new; t0 += kChunk) {
         const int nt = min(kChunk, sq.n_new - t0);
@@ -751,10 +813,7 @@ __global__ void __launch_bounds__(kSelThreads)
             AT part[2] = {0, 0};
 #pragma unroll
             for (int r = 0; r < RN; ++r) {
-                AT dec;
-                if (sizeof(AT) == 8) dec = (AT)exp((double)(dt * A[r]));
-                else dec = (AT)exp2f((float)(dt * A[r]));
-                s[r] = dec * s[r] + dx * (AT)Bs[t][n0 + r];
+                s[r] = exp(dt * A[r]) * s[r] + dx * (AT)Bs[t][n0 + r];
                 part[r & 1] += s[r] * (AT)Cs[t][n0 + r];
             }
             const AT y = group_sum<kSelLanes>(part[0] + part[1]);
@@ -776,28 +835,287 @@ __global__ void __launch_bounds__(kSelThreads)
     }
 }
 
-template <typename AT, typename TO>
-static int launch_selective(const SelArgs& a, int n_seqs, const int* cu_seqlens, const int* slot_of_seq, const int* start_pos, float* state,
-                            long long slot_stride, long long copy_stride, long long state_off, cudaStream_t stream) {
-    dim3 grid(n_seqs, (a.channels + kSelChannels - 1) / kSelChannels);
-#define BLM_SEL(RN)                                                                                                                      \
-    if (a.n_states <= RN * kSelLanes) {                                                                                                  \
-        selective_scan_kernel<RN, AT, TO><<<grid, kSelThreads, 0, stream>>>(a, cu_seqlens, slot_of_seq, start_pos, state, slot_stride,    \
-                                                                            copy_stride, state_off);                                     \
-        return blm_check_launch("selective_scan");                                                                                       \
+__device__ __forceinline__ float ex2_approx(float x) {       // x <= 0 here: no overflow, and what underflows is zero
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+template <int BYTES>
+__device__ __forceinline__ void copy_async(float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], %2;\n" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src), "n"(BYTES) : "memory");
+}
+
+// states n0 .. n0 + RN of one row of B or C (shared memory): the widest loads RN allows
+template <int RN>
+__device__ __forceinline__ void load_states(float (&v)[RN], const float* p) {
+    if (RN % 4 == 0) {
+#pragma unroll
+        for (int r = 0; r < RN; r += 4) {
+            const float4 q = *reinterpret_cast<const float4*>(p + r);
+            v[r] = q.x; v[r + 1] = q.y; v[r + 2] = q.z; v[r + 3] = q.w;
+        }
+    } else {
+#pragma unroll
+        for (int r = 0; r < RN; r += 2) {
+            const float2 q = *reinterpret_cast<const float2*>(p + r);
+            v[r] = q.x; v[r + 1] = q.y;
+        }
     }
-    BLM_SEL(2) BLM_SEL(4) BLM_SEL(6) BLM_SEL(8) BLM_SEL(16) BLM_SEL(32)
-#undef BLM_SEL
-    return blm_fail(BLM_BAD_ARGUMENT, "selective_scan: %d states a channel; this kernel takes up to %d", a.n_states, 32 * kSelLanes);
+}
+
+template <int RN>
+struct SelSmem {        // two buffers of raw rows, then what is made of them
+    static constexpr int NP = RN * kSelLanes, CH = kSelChannels, YS = CH + 8;      // (YS: the four lanes of a channel write four rows' same column)
+    float B[2][kChunk][NP], C[2][kChunk][NP];
+    float x[2][kChunk][CH], dt[2][kChunk][CH], z[2][kChunk][CH];
+    float2 made[kChunk][CH];
+    float y[kChunk][YS];
+};
+
+template <int RN>
+__global__ void __launch_bounds__(kSelThreads)
+    selective_scan_kernel(SelArgs a, int rows16, int low16, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
+                          const int* __restrict__ start_pos, float* __restrict__ state, long long slot_stride, long long copy_stride,
+                          long long state_off) {
+    // rows16, low16: the rows of x, dt and z (of low) can be copied 16 bytes at a time
+    constexpr int NP = RN * kSelLanes, CH = kSelChannels;
+    extern __shared__ __align__(16) unsigned char sel_raw[];
+    SelSmem<RN>& sm = *reinterpret_cast<SelSmem<RN>*>(sel_raw);
+    const int seq = blockIdx.x, c0 = blockIdx.y * CH;
+    const ScanSeq sq = scan_seq(seq, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off);
+    if (sq.n_new <= 0) return;
+    const int tid = threadIdx.x, ch = tid / kSelLanes, g = tid % kSelLanes;
+    const int c = c0 + ch, n0 = g * RN;
+    const bool live = c < a.channels;
+    float s[RN], A[RN];
+#pragma unroll
+    for (int r = 0; r < RN; ++r) {
+        const bool in = live && n0 + r < a.n_states;
+        const size_t at = (size_t)c * a.n_states + n0 + r;
+        s[r] = in && sq.read ? sq.read[at] : 0.f;
+        A[r] = in ? -expf(a.A_log[at]) * 1.4426950408889634f : 0.f;
+    }
+    // the passes by rows: a thread always has the same column
+    const int col = tid % CH, row_of = tid / CH;
+    const float bias = c0 + col < a.channels ? a.dt_bias[c0 + col] : 0.f, skip = c0 + col < a.channels ? a.D[c0 + col] : 0.f;
+    // columns no copy writes stay zero: states beyond n_states, channels beyond the last
+    for (int e = tid; e < (int)(sizeof(SelSmem<RN>) / sizeof(float)); e += kSelThreads) reinterpret_cast<float*>(&sm)[e] = 0.f;
+    __syncthreads();
+    auto fetch = [&](int buf, int t0) {
+        const int nt = min(kChunk, sq.n_new - t0);
+        const size_t row0 = (size_t)(sq.first + t0);
+        if (rows16) {
+            constexpr int V = CH / 4;
+            for (int e = tid; e < nt * V; e += kSelThreads) {
+                const int t = e / V, k = (e % V) * 4;
+                if (c0 + k < a.channels) {              // channels is a multiple of 4
+                    copy_async<16>(&sm.x[buf][t][k], a.x + (row0 + t) * a.x_stride + c0 + k);
+                    copy_async<16>(&sm.dt[buf][t][k], a.dt_raw + (row0 + t) * a.dt_stride + c0 + k);
+                    copy_async<16>(&sm.z[buf][t][k], a.z + (row0 + t) * a.z_stride + c0 + k);
+                }
+            }
+        } else {
+            for (int t = row_of; t < nt; t += kSelThreads / CH)
+                if (c0 + col < a.channels) {
+                    copy_async<4>(&sm.x[buf][t][col], a.x + (row0 + t) * a.x_stride + c0 + col);
+                    copy_async<4>(&sm.dt[buf][t][col], a.dt_raw + (row0 + t) * a.dt_stride + c0 + col);
+                    copy_async<4>(&sm.z[buf][t][col], a.z + (row0 + t) * a.z_stride + c0 + col);
+                }
+        }
+        if (low16) {
+            constexpr int V = NP / 4;
+            for (int e = tid; e < nt * V; e += kSelThreads) {
+                const int t = e / V, n = (e % V) * 4;
+                if (n < a.n_states) {                   // n_states is a multiple of 4
+                    const float* low = a.low + (row0 + t) * a.low_stride;
+                    copy_async<16>(&sm.B[buf][t][n], low + a.b_col0 + n);
+                    copy_async<16>(&sm.C[buf][t][n], low + a.c_col0 + n);
+                }
+            }
+        } else {
+            for (int e = tid; e < nt * NP; e += kSelThreads) {
+                const int t = e / NP, n = e % NP;
+                if (n < a.n_states) {
+                    const float* low = a.low + (row0 + t) * a.low_stride;
+                    copy_async<4>(&sm.B[buf][t][n], low + a.b_col0 + n);
+                    copy_async<4>(&sm.C[buf][t][n], low + a.c_col0 + n);
+                }
+            }
+        }
+        asm volatile("cp.async.commit_group;\n" ::: "memory");
+    };
+    fetch(0, 0);
+    for (int t0 = 0, it = 0; t0 < sq.n_new; t0 += kChunk, ++it) {
+        const int buf = it & 1, nt = min(kChunk, sq.n_new - t0);
+        if (t0 + kChunk < sq.n_new) {                   // into the buffer the chunk before this one has left (the loop ends on a barrier)
+            fetch(buf ^ 1, t0 + kChunk);
+            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < kChunk * CH / kSelThreads; ++i) {
+            const int t = row_of + i * (kSelThreads / CH);
+            const float dt = t < nt ? softplus_r(sm.dt[buf][t][col] + bias) : 0.f;       // a token of no step size changes nothing
+            sm.made[t][col] = make_float2(dt, t < nt ? dt * sm.x[buf][t][col] : 0.f);
+        }
+        __syncthreads();
+        // (rows beyond the last token hold what an earlier chunk left, numbers, and meet a step size of zero)
+        for (int t = 0; t < nt; t += 4) {
+            float part[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const float2 d = sm.made[t + u][ch];
+                float b[RN], cc[RN];
+                load_states<RN>(b, &sm.B[buf][t + u][n0]);
+                load_states<RN>(cc, &sm.C[buf][t + u][n0]);
+                float p0 = 0.f, p1 = 0.f;
+#pragma unroll
+                for (int r = 0; r < RN; ++r) {
+                    s[r] = fmaf(ex2_approx(d.x * A[r]), s[r], d.y * b[r]);
+                    if (r & 1) p1 = fmaf(s[r], cc[r], p1);
+                    else p0 = fmaf(s[r], cc[r], p0);
+                }
+                part[u] = p0 + p1;
+            }
+            // over the channel's four lanes: two exchanges leave lane g with token t + g's sum
+            const bool odd = g & 1, high = g & 2;
+            float k0 = odd ? part[1] : part[0], k1 = odd ? part[3] : part[2];
+            k0 += __shfl_xor_sync(0xffffffffu, odd ? part[0] : part[1], 1);
+            k1 += __shfl_xor_sync(0xffffffffu, odd ? part[2] : part[3], 1);
+            float mine = high ? k1 : k0;
+            mine += __shfl_xor_sync(0xffffffffu, high ? k0 : k1, 2);
+            sm.y[t + g][ch] = mine;
+        }
+        __syncthreads();
+        if (c0 + col < a.channels) {
+#pragma unroll
+            for (int i = 0; i < kChunk * CH / kSelThreads; ++i) {
+                const int t = row_of + i * (kSelThreads / CH);
+                if (t < nt) {
+                    const float z = sm.z[buf][t][col], y = fmaf(skip, sm.x[buf][t][col], sm.y[t][col]);
+                    reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)(sq.first + t0 + t) * a.out_stride + c0 + col] =
+                        __float2bfloat16_rn(a.scale * y * __fdividef(z, 1.0f + __expf(-z)));
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (live) {
+#pragma unroll
+        for (int r = 0; r < RN; ++r)
+            if (n0 + r < a.n_states) sq.write[(size_t)c * a.n_states + n0 + r] = s[r];
+    }
+}
+
+template <int RN>
+__global__ void __launch_bounds__(kSelThreads)
+    selective_step_kernel(SelArgs a, int vec8, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
+                          const int* __restrict__ start_pos, float* __restrict__ state, long long slot_stride, long long copy_stride,
+                          long long state_off) {
+    // vec8: rows of dt_w are bfloat16 and can be read 16 bytes at a time
+    extern __shared__ __align__(16) unsigned char sel_raw[];
+    float* lat = reinterpret_cast<float*>(sel_raw);      // [rank]
+    const int seq = blockIdx.x;
+    const ScanSeq sq = scan_seq(seq, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off);
+    if (sq.n_new <= 0) return;
+    const int tid = threadIdx.x, ch = tid / kSelLanes, g = tid % kSelLanes, n0 = g * RN;
+    const int c = min(blockIdx.y * kSelChannels + ch, a.channels - 1);      // (lanes beyond the last channel work on it too and write nothing)
+    const bool live = blockIdx.y * kSelChannels + ch < a.channels;
+    const size_t row = (size_t)sq.first;
+    const float* low = a.low + row * a.low_stride;
+    float s[RN], A[RN], b[RN], cc[RN];
+#pragma unroll
+    for (int r = 0; r < RN; ++r) {
+        const bool in = n0 + r < a.n_states;
+        const size_t at = (size_t)c * a.n_states + n0 + r;
+        s[r] = in && sq.read ? sq.read[at] : 0.f;
+        A[r] = in ? a.A_log[at] : 0.f;
+        b[r] = in ? low[a.b_col0 + n0 + r] : 0.f;
+        cc[r] = in ? low[a.c_col0 + n0 + r] : 0.f;
+    }
+    const float x = a.x[row * a.x_stride + c], z = a.z[row * a.z_stride + c];
+    float raw = a.dt_bias[c];
+    if (a.dt_w != nullptr) {
+        for (int k = tid; k < a.rank; k += kSelThreads) lat[k] = low[k];
+        __syncthreads();
+        float sum = 0.f;
+        if (vec8) {
+            const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.dt_w) + (size_t)c * a.rank;
+#pragma unroll 4
+            for (int k = g * 8; k < a.rank; k += 8 * kSelLanes) {
+                const uint4 v = *reinterpret_cast<const uint4*>(w + k);
+                const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float2 f = __bfloat1622float2(p[e]);
+                    sum = fmaf(f.x, lat[k + 2 * e], fmaf(f.y, lat[k + 2 * e + 1], sum));
+                }
+            }
+        } else if (a.dt_w_bf16) {
+            const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.dt_w) + (size_t)c * a.rank;
+            for (int k = g; k < a.rank; k += kSelLanes) sum = fmaf(__bfloat162float(w[k]), lat[k], sum);
+        } else {
+            const float* w = reinterpret_cast<const float*>(a.dt_w) + (size_t)c * a.rank;
+            for (int k = g; k < a.rank; k += kSelLanes) sum = fmaf(w[k], lat[k], sum);
+        }
+        raw += group_sum<kSelLanes>(sum);
+    } else {
+        raw += a.dt_raw[row * a.dt_stride + c];
+    }
+    const float dt = softplus_r(raw), dx = dt * x;
+    float y = 0.f;
+#pragma unroll
+    for (int r = 0; r < RN; ++r) {
+        const float dec = n0 + r < a.n_states ? ex2_approx(-expf(A[r]) * 1.4426950408889634f * dt) : 0.f;
+        s[r] = fmaf(dec, s[r], dx * b[r]);
+        y = fmaf(s[r], cc[r], y);
+    }
+    y = group_sum<kSelLanes>(y);
+    if (!live) return;
+#pragma unroll
+    for (int r = 0; r < RN; ++r)
+        if (n0 + r < a.n_states) sq.write[(size_t)c * a.n_states + n0 + r] = s[r];
+    if (g == 0) reinterpret_cast<__nv_bfloat16*>(a.out)[row * a.out_stride + c] = __float2bfloat16_rn(a.scale * (y + a.D[c] * x) * silu_f(z));
+}
+
+static bool aligned16(const void* p, long long stride) { return ((size_t)p & 15) == 0 && stride % 4 == 0; }
+
+template <int RN>
+static int launch_selective(const SelArgs& a, int exact, int single, int n_seqs, const int* cu_seqlens, const int* slot_of_seq, const int* start_pos,
+                            float* state, long long slot_stride, long long copy_stride, long long state_off, cudaStream_t stream) {
+    const dim3 grid(n_seqs, (a.channels + kSelChannels - 1) / kSelChannels);
+    if (exact) {
+        selective_exact_kernel<RN><<<grid, kSelThreads, 0, stream>>>(a, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off);
+        return blm_check_launch("selective_scan (exact)");
+    }
+    if (single) {
+        const int vec8 = a.dt_w != nullptr && a.dt_w_bf16 && a.rank % 8 == 0 && ((size_t)a.dt_w & 15) == 0;
+        const size_t smem = a.dt_w != nullptr ? (size_t)a.rank * sizeof(float) : 0;
+        BLM_REQUIRE(smem <= 48 * 1024, "selective_scan: step sizes made of %d numbers", a.rank);
+        selective_step_kernel<RN><<<grid, kSelThreads, smem, stream>>>(a, vec8, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride,
+                                                                       state_off);
+        return blm_check_launch("selective_scan (single tokens)");
+    }
+    BLM_REQUIRE(a.dt_raw != nullptr, "selective_scan: portions bring their step sizes");
+    const int rows16 = a.channels % 4 == 0 && aligned16(a.x, a.x_stride) && aligned16(a.dt_raw, a.dt_stride) && aligned16(a.z, a.z_stride);
+    const int low16 = a.n_states % 4 == 0 && aligned16(a.low, a.low_stride) && a.b_col0 % 4 == 0 && a.c_col0 % 4 == 0;
+    const int rc = allow_smem(selective_scan_kernel<RN>, sizeof(SelSmem<RN>), "selective_scan");
+    if (rc != BLM_OK) return rc;
+    selective_scan_kernel<RN><<<grid, kSelThreads, sizeof(SelSmem<RN>), stream>>>(a, rows16, low16, cu_seqlens, slot_of_seq, start_pos, state,
+                                                                                  slot_stride, copy_stride, state_off);
+    return blm_check_launch("selective_scan");
 }
 
 BLM_API int blm_selective_scan(const float* x, long long x_stride, const float* low, long long low_stride, int b_col0, int c_col0,
                                const float* dt_raw, long long dt_stride, const void* dt_w, int dt_w_dtype, int rank, const float* dt_bias,
                                const float* A_log, const float* D, const float* z, long long z_stride, void* out, int out_dtype,
                                long long out_stride, float scale, int channels, int n_states, const int* cu_seqlens, const int* slot_of_seq,
-                               const int* start_pos, int n_seqs, float* state, long long slot_stride,
+                               const int* start_pos, int n_seqs, int single_tokens, float* state, long long slot_stride,
                                long long copy_stride, long long state_off, cudaStream_t stream) {
-    // dt_raw [T, dt_stride], or null and dt_w [channels, rank] (the step sizes' projection of low's first columns).
+    // dt_raw [T, dt_stride], or null and dt_w [channels, rank] (the step sizes' projection of low's first columns; single tokens
+    // and the 32-bit path only).  single_tokens: every sequence brings one token.
     // out float32: the 32-bit path (sums in float64).  Rows of no sequence are left as they are.
     if (n_seqs == 0) return BLM_OK;
     BLM_REQUIRE(channels > 0 && n_states > 0 && n_seqs > 0, "selective_scan: bad sizes");
@@ -808,11 +1126,14 @@ BLM_API int blm_selective_scan(const float* x, long long x_stride, const float* 
     a.dt_raw = dt_raw; a.dt_stride = dt_stride; a.dt_w = dt_w; a.dt_w_bf16 = dt_w_dtype == BLM_BF16; a.rank = rank;
     a.dt_bias = dt_bias; a.A_log = A_log; a.D = D; a.z = z; a.z_stride = z_stride;
     a.out = out; a.out_stride = out_stride; a.scale = scale; a.channels = channels; a.n_states = n_states;
-#define BLM_SEL_ARGS a, n_seqs, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off, stream
-    if (out_dtype == BLM_F32) return launch_selective<double, float>(BLM_SEL_ARGS);
-    if (out_dtype == BLM_BF16) return launch_selective<float, __nv_bfloat16>(BLM_SEL_ARGS);
-#undef BLM_SEL_ARGS
-    return blm_fail(BLM_BAD_ARGUMENT, "selective_scan: out dtype %d", out_dtype);
+    BLM_REQUIRE(out_dtype == BLM_F32 || out_dtype == BLM_BF16, "selective_scan: out dtype %d", out_dtype);
+#define BLM_SEL(RN)                                                                                                                      \
+    if (n_states <= RN * kSelLanes)                                                                                                      \
+        return launch_selective<RN>(a, out_dtype == BLM_F32, single_tokens, n_seqs, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, \
+                                    copy_stride, state_off, stream);
+    BLM_SEL(2) BLM_SEL(4) BLM_SEL(6) BLM_SEL(8) BLM_SEL(16) BLM_SEL(32)
+#undef BLM_SEL
+    return blm_fail(BLM_BAD_ARGUMENT, "selective_scan: %d states a channel; this kernel takes up to %d", n_states, 32 * kSelLanes);
 }
 
 // out[n, d] = src[n, col0 + d] in out's type: some columns of a wider fp32 row as a product's operand

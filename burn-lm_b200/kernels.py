@@ -97,10 +97,11 @@ _protos = {
                                c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_float,
                                c_float, c_float, c_float, c_void_p],
         "blm_head_norm_rope_append": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
-                                      c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
+                                      c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
                                       c_void_p, c_void_p, c_int, c_void_p],
         "blm_attention_sink_prompt_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
         "blm_attention_sink_decode_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
+        "blm_attention_sink_pairs": [c_int, c_int, c_int, c_int, c_int, c_int, c_int],
     },
     "stream_ops": {
         "blm_embed_scaled": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
@@ -130,7 +131,7 @@ _protos = {
                            c_void_p],
         "blm_selective_scan": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_float, c_int, c_int,
-                               c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p],
+                               c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p],
         "blm_take_cols": [c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
         "blm_gated_group_norm": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                  c_float, c_void_p, c_int, c_longlong, c_int, c_void_p],
@@ -401,7 +402,7 @@ def qk_norm_append(proj, step, pool, block_table, q_out, n_heads, n_kv, key_dim,
 
 
 def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, key_dim, value_dim, q_weight=None, k_weight=None,
-                          eps=0.0, value_norm=False, freq=None, rotary_dims=0, halves=False, turn_scale=1.0, maps=1):
+                          eps=0.0, value_norm=False, freq=None, rotary_dims=0, halves=False, turn_scale=1.0, maps=1, table=None):
     """What follows a fused projection [q | k | v | ...] (float32 [N, >= (n_heads + n_kv) key_dim + n_kv value_dim]), head by
     head: every head of q is divided by its root mean square (eps inside the root) and multiplied by `q_weight` (float32
     [key_dim], the same for all heads; None: q stays as it is), every head of k likewise with `k_weight`; the first
@@ -409,9 +410,12 @@ def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, k
     together, or (i, i + rotary_dims / 2) with `halves`, cosine and sine both times `turn_scale`; with `value_norm` every head
     of v is divided by its root mean square (no weight).  q goes to `q_out` [N, n_heads key_dim], k and v to the token's place
     in the paged cache.  `maps` 2: a head has two queries and two keys, [head][map][key_dim], over one value; n_heads and
-    n_kv count every map.  `proj` may be a column range of a wider tensor."""
-    _need_cuda(pool, block_table, q_out, q_weight, k_weight, freq)
-    _f32(proj, q_weight, k_weight)
+    n_kv count every map.  `table` (from rope_table, with the same turn_scale) spares the angles of the positions it covers.
+    `proj` may be a column range of a wider tensor."""
+    _need_cuda(pool, block_table, q_out, q_weight, k_weight, freq, table)
+    _f32(proj, q_weight, k_weight, table)
+    if table is not None and tuple(table.shape[1:]) != (rotary_dims // 2, 2):
+        raise KernelError("head_norm_rope_append: the table is float32 [positions, rotary_dims / 2, 2]")
     if not proj.is_cuda:
         raise KernelError("burn-lm_b200 kernels run on a CUDA device only; got a CPU tensor")
     n = proj.shape[0]
@@ -427,13 +431,19 @@ def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, k
         raise KernelError("head_norm_rope_append: freq must be float64 [rotary_dims / 2]")
     _call("attention_sink", "blm_head_norm_rope_append", _ptr(proj), c_longlong(proj.stride(0)), n, n_heads, n_kv, int(maps), key_dim,
           value_dim, _ptr(q_weight), _ptr(k_weight), c_float(eps), 1 if value_norm else 0, _ptr(freq), int(rotary_dims), 1 if halves else 0,
-          c_float(turn_scale), _ptr(q_out), _ptr(pool), _code(pool.dtype), c_longlong(_flat_pool(pool, n_kv, key_dim, value_dim, maps)), PAGE, _ptr(step.token_seq),
+          c_float(turn_scale), _ptr(table), table.shape[0] if table is not None else 0, _ptr(q_out), _ptr(pool), _code(pool.dtype), c_longlong(_flat_pool(pool, n_kv, key_dim, value_dim, maps)), PAGE, _ptr(step.token_seq),
           _ptr(step.token_pos), _ptr(step.slot_of_seq), _ptr(block_table), block_table.shape[1], _stream())
 
 
-def attention_sink_scratch_floats(n_tokens, n_heads, value_dim, n_splits, maps=1) -> int:
-    """(n_heads counts every map; with two maps the kernels always leave their sums for the one that forms the difference)"""
-    return 0 if n_splits <= 1 and maps == 1 else n_tokens * n_heads * n_splits * (value_dim + 2)
+def attention_sink_pairs(dtype, key_dim, value_dim, n_heads, n_kv, maps) -> bool:
+    """Whether the decode kernel takes both maps of a head in one block and, without splits, forms their difference itself."""
+    return bool(_lib("attention_sink").blm_attention_sink_pairs(_code(dtype), key_dim, value_dim, PAGE, n_heads, n_kv, maps))
+
+
+def attention_sink_scratch_floats(n_tokens, n_heads, value_dim, n_splits, maps=1, inside=False) -> int:
+    """n_heads counts every map; with two maps the kernels leave their sums for the one that forms the difference, unless
+    the decode kernel does (`inside`: a step of its own, attention_sink_pairs(...), without splits)."""
+    return 0 if n_splits <= 1 and (maps == 1 or inside) else n_tokens * n_heads * n_splits * (value_dim + 2)
 
 
 def attention_sink_prompt_takes(dtype, key_dim, value_dim, max_q_len, n_heads) -> bool:
@@ -486,7 +496,8 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
     prompt = attention_sink_prompt_takes(pool.dtype, key_dim, value_dim, max_q_len, n_heads) and getattr(step, "cu_seqlens", None) is not None
     if prompt:
         n_splits = 1
-    need = attention_sink_scratch_floats(n, n_heads, value_dim, n_splits, maps)
+    inside = maps == 2 and not prompt and attention_sink_pairs(pool.dtype, key_dim, value_dim, n_heads, n_kv, maps)
+    need = attention_sink_scratch_floats(n, n_heads, value_dim, n_splits, maps, inside)
     if need:
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"attention_sink: {n_splits} splits need {need} float32 of scratch")
@@ -1352,7 +1363,7 @@ def selective_scan(x, low, rank, n_state, dt_bias, a_log, d_skip, z, out, step, 
     """The selective scan per channel c with `n_state` states: S <- exp(dt A) S + dt x B, y = S C + D x, out = scale y silu(z),
     dt = softplus(. + dt_bias), A = -exp(a_log).  x float32 [N, channels]; low float32 [N, rank + 2 n_state] = [dt | B | C];
     the step sizes before bias and softplus are `dt` float32 [N, channels], or dt_weight [channels, rank] times low's first
-    columns, formed by the kernel; z float32 [N, channels], possibly a column range; out [N, channels] bfloat16, or float32 in
+    columns, formed by the kernel (steps of one token a sequence, and the 32-bit path); z float32 [N, channels], possibly a column range; out [N, channels] bfloat16, or float32 in
     the 32-bit path (sums in float64), possibly a column range.  The state (fp32) lies in `state` at state_offset,
     [channels, n_state]."""
     channels = x.shape[1]
@@ -1374,7 +1385,7 @@ def selective_scan(x, low, rank, n_state, dt_bias, a_log, d_skip, z, out, step, 
           int(rank + n_state), _ptr(dt), c_longlong(channels), _ptr(dt_weight), _code(dt_weight.dtype) if dt_weight is not None else F32,
           int(rank), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), _ptr(z), c_longlong(z.stride(0)), _ptr(out), _code(out.dtype),
           c_longlong(out.stride(0)), c_float(scale), channels, int(n_state), _ptr(step.cu_seqlens), _ptr(step.slot_of_seq),
-          _ptr(step.start_pos), step.n_seqs, *_state_args(state, state_offset), _stream())
+          _ptr(step.start_pos), step.n_seqs, 1 if getattr(step, "max_q_len", 0) == 1 else 0, *_state_args(state, state_offset), _stream())
 
 
 def take_cols(src, col0, out):

@@ -98,7 +98,7 @@ class Mamba(Part):
         K.causal_conv(proj, 0, s.inner, self.taps, self.conv_bias, x, 0, step, cache.state, cache.state_offset, silu=True, out_bf16=rounded)
         low = self.x(rounded if rounded is not None else x, out_dtype=torch.float32)            # [N, dt | B | C] in fp32
         dt = None
-        if n > FUSED_STEP_TOKENS:
+        if n > FUSED_STEP_TOKENS or step.max_q_len > 1:
             latent = torch.empty((n, s.dt_rank), dtype=self.dt.weight.dtype, device=proj.device)
             K.take_cols(low, 0, latent)
             dt = self.dt(latent, out_dtype=torch.float32)

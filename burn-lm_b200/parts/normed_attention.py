@@ -36,6 +36,7 @@ from .linear import Linear
 from .position import RotarySpec, rotary_inverse_frequencies, rotary_multiplier
 
 BLOCKS_PER_SM = 4          # blocks of the single-token kernels a step should offer every multiprocessor
+TABLE_BYTES = 64 << 20     # a layer's table of cosines and sines at most
 NO_WINDOW = 1 << 30        # what the kernels take for "every earlier key"
 
 
@@ -116,7 +117,7 @@ class NormedAttention(Part):
         self.q_weight = f32(loaded[t["q_norm"]]) if s.qk_norm else None
         self.k_weight = f32(loaded[t["k_norm"]]) if s.qk_norm else None
         self.temperature = f32(loaded[t["temperature"]]) if s.head_temperature else None
-        self.freq, self.turn_scale = None, 1.0
+        self.freq, self.turn_scale, self.table = None, 1.0, None
         if s.rotary_dims:
             rot = RotarySpec(s.head_dim, s.rotary_base, rotary_dim=s.rotary_dims, scaling=s.rotary_scaling)
             self.freq = torch.tensor(rotary_inverse_frequencies(rot), dtype=torch.float64).to(self.o.weight.device)
@@ -126,6 +127,13 @@ class NormedAttention(Part):
             lq1, lk1, lq2, lk2 = (loaded[t[r]].to(torch.float64) for r in ("lq1", "lk1", "lq2", "lk2"))
             lam = math.exp(float((lq1 * lk1).sum())) - math.exp(float((lq2 * lk2).sum())) + s.diff
             self.difference = (lam, 1.0 - s.diff, s.eps)
+
+    def prepare(self, max_positions: int) -> None:
+        """Cosines and sines of the positions the cache can hold, worked out once (beyond TABLE_BYTES: by the kernel, a token
+        at a time)."""
+        if self.freq is not None and self.freq.is_cuda and 8 * self.freq.numel() * max_positions <= TABLE_BYTES \
+                and (self.table is None or self.table.shape[0] < max_positions):
+            self.table = K.rope_table(self.freq, max_positions, self.turn_scale)
 
     def cache_need(self) -> CacheNeed:
         s = self.spec
@@ -140,6 +148,8 @@ class NormedAttention(Part):
             return 1
         seen = min(step.max_kv_len, s.window or s.chunk or step.max_kv_len)
         blocks = step.n_tokens * self.maps * s.n_kv_heads
+        if self.maps == 2 and K.attention_sink_pairs(self.runtime.dtype, s.head_dim, s.value_dim, 2 * s.n_heads, 2 * s.n_kv_heads, 2):
+            blocks //= 2                                     # both maps of a head share a block
         want = BLOCKS_PER_SM * K.sm_count(self.runtime.device)
         if K.attention_sink_decode_takes(self.runtime.dtype, s.head_dim, s.value_dim, s.n_heads, s.n_kv_heads):
             pages = seen // K.PAGE + 1                       # that kernel cuts by pages, and its blocks hold several
@@ -174,10 +184,16 @@ class NormedAttention(Part):
         q = torch.empty((n, self.q_cols), dtype=rt.dtype, device=proj.device)
         K.head_norm_rope_append(proj, step, cache.pool, cache.block_table, q, heads, kv_heads, s.head_dim, s.value_dim,
                                 q_weight=self.q_weight, k_weight=self.k_weight, eps=s.eps, value_norm=s.value_norm, freq=self.freq,
-                                rotary_dims=s.rotary_dims, halves=s.rotary_halves, turn_scale=self.turn_scale, maps=maps)
+                                rotary_dims=s.rotary_dims, halves=s.rotary_halves, turn_scale=self.turn_scale, maps=maps, table=self.table)
         n_splits = self._splits(step)
-        floats = K.attention_sink_scratch_floats(n, heads, s.value_dim, n_splits, maps)
-        scratch = step.workspace.scratch("attention_sink", floats) if floats else None
+        prompt = K.attention_sink_prompt_takes(rt.dtype, s.head_dim, s.value_dim, step.max_q_len, heads)
+        inside = maps == 2 and not prompt and K.attention_sink_pairs(rt.dtype, s.head_dim, s.value_dim, heads, kv_heads, maps)
+        floats = K.attention_sink_scratch_floats(n, heads, s.value_dim, n_splits, maps, inside)
+        scratch = None
+        if floats and step.max_q_len == 1:
+            scratch = step.workspace.scratch("attention_sink", floats)
+        elif floats:                            # (a prompt's shares: captured prompt steps share their memory)
+            scratch = torch.empty(floats, dtype=torch.float32, device=proj.device)
         gate = proj[:, self.proj_width - self.out_width:] if s.output_gate else None
         K.attention_sink(q, step, cache.pool, cache.block_table, out, heads, kv_heads, s.head_dim, s.value_dim, s.scale,
                          s.window or NO_WINDOW, 0, sink=s.sink, gate=gate, gate_stride=proj.stride(0), max_q_len=step.max_q_len,
