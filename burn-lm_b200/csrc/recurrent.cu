@@ -128,6 +128,24 @@ __global__ void conv_rows_kernel(const float* __restrict__ x, long long x_stride
     const float b = bias ? bias[c] : 0.f;
     int held = -1;                              // the sequence the window belongs to
     const float* in = x + x_col0 + c;
+    const int seq0 = token_seq[first];
+    if (last - first == kConvRows && seq0 >= 0 && token_seq[last - 1] == seq0 && first - cu_seqlens[seq0] >= K - 1) {
+        // all rows and what lies behind them are one sequence's rows of this step: every load at once
+        float v[kConvRows + K - 1];
+#pragma unroll
+        for (int i = 0; i < kConvRows + K - 1; ++i) v[i] = in[(size_t)(first - (K - 1) + i) * x_stride];
+#pragma unroll
+        for (int i = 0; i < kConvRows; ++i) {
+            float acc = b;
+#pragma unroll
+            for (int j = K - 1; j >= 0; --j) acc += w[j] * v[i + K - 1 - j];
+            if (act == 2) acc += v[i + K - 1];
+            const float res = act == 1 ? silu_f(acc) : acc;
+            out[(size_t)(first + i) * out_stride + out_col0 + c] = res;
+            if (out_bf) out_bf[(size_t)(first + i) * out_bf_stride + c] = __float2bfloat16(res);
+        }
+        return;
+    }
 #pragma unroll 4
     for (int n = first; n < last; ++n) {
         const int seq = token_seq[n];
@@ -724,11 +742,11 @@ BLM_API int blm_gated_group_norm(const float* y, long long y_stride, const float
 // [T, C], or (dt_w) formed here from the first `rank` columns of low and dt_w [C, rank]: for single tokens, where a product
 // of its own would be a launch for a few kilobytes.  A block owns (sequence, kSelThreads / kSelLanes channels); kSelLanes lanes
 // share a channel, RN neighbouring states each in registers.  The state is stored as [channel][state].  Three kernels:
-//   selective_scan_kernel   portions, bfloat16 results: chunks of kChunk tokens come through cp.async into two buffers in
-//                           turn, one on its way while the other is worked on; a pass makes (dt, dt x) of the raw rows; four
-//                           tokens' sums over the states are reduced together, so that every lane ends with one token's
-//                           sum; results leave gated and converted by rows.  The exponentials are exp2 by the special
-//                           function unit with A scaled by log2 e: at 16 states a channel they are what the kernel takes longest for.
+//   selective_scan_kernel   portions, bfloat16 results: chunks of kChunk tokens; four warps walk the tokens and four serve
+//                           them (rows through cp.async, what is made of them, results out), a chunk apart, so that the
+//                           walk waits for nothing but its own arithmetic; a lane leaves its share of a token's sum in
+//                           shared memory, so nothing is shuffled on the way.  The exponentials are exp2 by the special
+//                           function unit with A scaled by log2 e: at 16 states a channel 32 of its cycles a token and warp.
 //   selective_step_kernel   one token a sequence, bfloat16 results: nothing staged but the latents the step sizes are made of.
 //   selective_exact_kernel  the 32-bit path, any portion: state and sums in float64 inside a step.
 // ---------------------------------------------------------------------------------------------
@@ -863,17 +881,23 @@ __device__ __forceinline__ void load_states(float (&v)[RN], const float* p) {
     }
 }
 
-template <int RN>
-struct SelSmem {        // two buffers of raw rows, then what is made of them
-    static constexpr int NP = RN * kSelLanes, CH = kSelChannels, YS = CH + 8;      // (YS: the four lanes of a channel write four rows' same column)
-    float B[2][kChunk][NP], C[2][kChunk][NP];
-    float x[2][kChunk][CH], dt[2][kChunk][CH], z[2][kChunk][CH];
-    float2 made[kChunk][CH];
-    float y[kChunk][YS];
-};
+constexpr int kSelBlock = 2 * kSelThreads;      // threads of a block of the portions' kernel: four warps scan, four serve them
 
 template <int RN>
-__global__ void __launch_bounds__(kSelThreads)
+struct SelSmem {
+    static constexpr int NP = RN * kSelLanes, CH = kSelChannels;
+    float B[3][kChunk][NP], C[3][kChunk][NP];                                    // on their way, landed, read by the scan
+    float x[2][kChunk][CH], dt[2][kChunk][CH], z[2][kChunk][CH];                 // raw rows: on their way, landed
+    float2 made[2][kChunk][CH];                                                  // (dt, dt x)
+    float2 after[2][kChunk][CH];                                                 // (D x, scale silu(z)): what the results meet on their way out
+    float4 y[2][kChunk][CH];                                                     // a channel's four lanes' sums
+};
+
+// Chunk c of the sequence passes through the block in four turns, a barrier after each:
+//   turn c - 1  the serving warps ask for its rows;      turn c      they make (dt, dt x) and (D x, scale silu(z)) of them;
+//   turn c + 1  the scanning warps walk its tokens;      turn c + 2  the serving warps write its results out.
+template <int RN>
+__global__ void __launch_bounds__(kSelBlock)
     selective_scan_kernel(SelArgs a, int rows16, int low16, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
                           const int* __restrict__ start_pos, float* __restrict__ state, long long slot_stride, long long copy_stride,
                           long long state_off) {
@@ -884,39 +908,102 @@ __global__ void __launch_bounds__(kSelThreads)
     const int seq = blockIdx.x, c0 = blockIdx.y * CH;
     const ScanSeq sq = scan_seq(seq, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off);
     if (sq.n_new <= 0) return;
-    const int tid = threadIdx.x, ch = tid / kSelLanes, g = tid % kSelLanes;
-    const int c = c0 + ch, n0 = g * RN;
-    const bool live = c < a.channels;
-    float s[RN], A[RN];
-#pragma unroll
-    for (int r = 0; r < RN; ++r) {
-        const bool in = live && n0 + r < a.n_states;
-        const size_t at = (size_t)c * a.n_states + n0 + r;
-        s[r] = in && sq.read ? sq.read[at] : 0.f;
-        A[r] = in ? -expf(a.A_log[at]) * 1.4426950408889634f : 0.f;
-    }
-    // the passes by rows: a thread always has the same column
-    const int col = tid % CH, row_of = tid / CH;
-    const float bias = c0 + col < a.channels ? a.dt_bias[c0 + col] : 0.f, skip = c0 + col < a.channels ? a.D[c0 + col] : 0.f;
-    // columns no copy writes stay zero: states beyond n_states, channels beyond the last
-    for (int e = tid; e < (int)(sizeof(SelSmem<RN>) / sizeof(float)); e += kSelThreads) reinterpret_cast<float*>(&sm)[e] = 0.f;
+    // places no copy writes stay zero: states beyond n_states, channels beyond the last, rows beyond the last token
+    for (int e = threadIdx.x; e < (int)(sizeof(SelSmem<RN>) / sizeof(float)); e += kSelBlock) reinterpret_cast<float*>(&sm)[e] = 0.f;
     __syncthreads();
-    auto fetch = [&](int buf, int t0) {
-        const int nt = min(kChunk, sq.n_new - t0);
+    const int n_chunks = (sq.n_new + kChunk - 1) / kChunk;
+    auto turn_over = [] { asm volatile("bar.sync 2, %0;\n" ::"n"(kSelBlock) : "memory"); };     // both halves of the block, each from its own loop
+    if (threadIdx.x < kSelThreads) {
+        // ---------------- the scan: a channel's state in four lanes ----------------
+        const int ch = threadIdx.x / kSelLanes, g = threadIdx.x % kSelLanes, c = c0 + ch, n0 = g * RN;
+        const bool live = c < a.channels;
+        float s[RN], A[RN];
+#pragma unroll
+        for (int r = 0; r < RN; ++r) {
+            const bool in = live && n0 + r < a.n_states;
+            const size_t at = (size_t)c * a.n_states + n0 + r;
+            s[r] = in && sq.read ? sq.read[at] : 0.f;
+            A[r] = in ? -expf(a.A_log[at]) * 1.4426950408889634f : 0.f;
+        }
+        for (int turn = 0; turn < n_chunks + 2; ++turn) {
+            const int k = turn - 1;                     // the chunk this turn walks
+            if (k >= 0 && k < n_chunks) {
+                // (rows beyond the last token, up to a multiple of four, meet a step size of zero: nothing changes)
+                const int nt = min(kChunk, sq.n_new - k * kChunk);
+                const float2* made = &sm.made[k & 1][0][ch];
+                const float* Bs = &sm.B[k % 3][0][n0];
+                const float* Cs = &sm.C[k % 3][0][n0];
+                float* y = reinterpret_cast<float*>(&sm.y[k & 1][0][ch]) + g;
+                constexpr int U = RN <= 8 ? 4 : 1;      // tokens whose operands are fetched together, ahead of the ones worked on
+                float2 d[U];
+                float b[U][RN], cc[U][RN];
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    d[u] = made[u * CH];
+                    load_states<RN>(b[u], Bs + u * NP);
+                    load_states<RN>(cc[u], Cs + u * NP);
+                }
+                for (int t = 0; t < nt; t += U) {
+                    float2 dn[U];
+                    float bn[U][RN], cn[U][RN];
+                    const int tn = min(t + U, kChunk - U);      // (the last turn's fetch is not used)
+#pragma unroll
+                    for (int u = 0; u < U; ++u) {
+                        dn[u] = made[(tn + u) * CH];
+                        load_states<RN>(bn[u], Bs + (tn + u) * NP);
+                        load_states<RN>(cn[u], Cs + (tn + u) * NP);
+                    }
+#pragma unroll
+                    for (int u = 0; u < U; ++u) {
+                        float p0 = 0.f, p1 = 0.f;
+#pragma unroll
+                        for (int r = 0; r < RN; ++r) {
+                            s[r] = fmaf(ex2_approx(d[u].x * A[r]), s[r], d[u].y * b[u][r]);
+                            if (r & 1) p1 = fmaf(s[r], cc[u][r], p1);
+                            else p0 = fmaf(s[r], cc[u][r], p0);
+                        }
+                        y[(size_t)(t + u) * CH * kSelLanes] = p0 + p1;
+                    }
+#pragma unroll
+                    for (int u = 0; u < U; ++u) {
+                        d[u] = dn[u];
+#pragma unroll
+                        for (int r = 0; r < RN; ++r) {
+                            b[u][r] = bn[u][r];
+                            cc[u][r] = cn[u][r];
+                        }
+                    }
+                }
+            }
+            turn_over();
+        }
+        if (live) {
+#pragma unroll
+            for (int r = 0; r < RN; ++r)
+                if (n0 + r < a.n_states) sq.write[(size_t)c * a.n_states + n0 + r] = s[r];
+        }
+        return;
+    }
+    // ---------------- the serving warps: a thread always has the same column of the rows ----------------
+    const int tid = threadIdx.x - kSelThreads, col = tid % CH, row_of = tid / CH;
+    const bool mine = c0 + col < a.channels;
+    const float bias = mine ? a.dt_bias[c0 + col] : 0.f, skip = mine ? a.D[c0 + col] : 0.f;
+    auto fetch = [&](int k) {                           // the rows of chunk k
+        const int t0 = k * kChunk, nt = min(kChunk, sq.n_new - t0), buf = k & 1, low_buf = k % 3;
         const size_t row0 = (size_t)(sq.first + t0);
         if (rows16) {
             constexpr int V = CH / 4;
             for (int e = tid; e < nt * V; e += kSelThreads) {
-                const int t = e / V, k = (e % V) * 4;
-                if (c0 + k < a.channels) {              // channels is a multiple of 4
-                    copy_async<16>(&sm.x[buf][t][k], a.x + (row0 + t) * a.x_stride + c0 + k);
-                    copy_async<16>(&sm.dt[buf][t][k], a.dt_raw + (row0 + t) * a.dt_stride + c0 + k);
-                    copy_async<16>(&sm.z[buf][t][k], a.z + (row0 + t) * a.z_stride + c0 + k);
+                const int t = e / V, kk = (e % V) * 4;
+                if (c0 + kk < a.channels) {             // channels is a multiple of 4
+                    copy_async<16>(&sm.x[buf][t][kk], a.x + (row0 + t) * a.x_stride + c0 + kk);
+                    copy_async<16>(&sm.dt[buf][t][kk], a.dt_raw + (row0 + t) * a.dt_stride + c0 + kk);
+                    copy_async<16>(&sm.z[buf][t][kk], a.z + (row0 + t) * a.z_stride + c0 + kk);
                 }
             }
         } else {
             for (int t = row_of; t < nt; t += kSelThreads / CH)
-                if (c0 + col < a.channels) {
+                if (mine) {
                     copy_async<4>(&sm.x[buf][t][col], a.x + (row0 + t) * a.x_stride + c0 + col);
                     copy_async<4>(&sm.dt[buf][t][col], a.dt_raw + (row0 + t) * a.dt_stride + c0 + col);
                     copy_async<4>(&sm.z[buf][t][col], a.z + (row0 + t) * a.z_stride + c0 + col);
@@ -928,8 +1015,8 @@ __global__ void __launch_bounds__(kSelThreads)
                 const int t = e / V, n = (e % V) * 4;
                 if (n < a.n_states) {                   // n_states is a multiple of 4
                     const float* low = a.low + (row0 + t) * a.low_stride;
-                    copy_async<16>(&sm.B[buf][t][n], low + a.b_col0 + n);
-                    copy_async<16>(&sm.C[buf][t][n], low + a.c_col0 + n);
+                    copy_async<16>(&sm.B[low_buf][t][n], low + a.b_col0 + n);
+                    copy_async<16>(&sm.C[low_buf][t][n], low + a.c_col0 + n);
                 }
             }
         } else {
@@ -937,75 +1024,45 @@ __global__ void __launch_bounds__(kSelThreads)
                 const int t = e / NP, n = e % NP;
                 if (n < a.n_states) {
                     const float* low = a.low + (row0 + t) * a.low_stride;
-                    copy_async<4>(&sm.B[buf][t][n], low + a.b_col0 + n);
-                    copy_async<4>(&sm.C[buf][t][n], low + a.c_col0 + n);
+                    copy_async<4>(&sm.B[low_buf][t][n], low + a.b_col0 + n);
+                    copy_async<4>(&sm.C[low_buf][t][n], low + a.c_col0 + n);
                 }
             }
         }
-        asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
-    fetch(0, 0);
-    for (int t0 = 0, it = 0; t0 < sq.n_new; t0 += kChunk, ++it) {
-        const int buf = it & 1, nt = min(kChunk, sq.n_new - t0);
-        if (t0 + kChunk < sq.n_new) {                   // into the buffer the chunk before this one has left (the loop ends on a barrier)
-            fetch(buf ^ 1, t0 + kChunk);
-            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
-        }
-        __syncthreads();
+    fetch(0);
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+    constexpr int kPasses = kChunk * CH / kSelThreads;
+    for (int turn = 0; turn < n_chunks + 2; ++turn) {
+        if (turn >= 2 && mine) {                        // chunk turn - 2 goes out
+            const int k = turn - 2, nt = min(kChunk, sq.n_new - k * kChunk);
+            __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (size_t)(sq.first + k * kChunk) * a.out_stride + c0 + col;
 #pragma unroll
-        for (int i = 0; i < kChunk * CH / kSelThreads; ++i) {
-            const int t = row_of + i * (kSelThreads / CH);
-            const float dt = t < nt ? softplus_r(sm.dt[buf][t][col] + bias) : 0.f;       // a token of no step size changes nothing
-            sm.made[t][col] = make_float2(dt, t < nt ? dt * sm.x[buf][t][col] : 0.f);
-        }
-        __syncthreads();
-        // (rows beyond the last token hold what an earlier chunk left, numbers, and meet a step size of zero)
-        for (int t = 0; t < nt; t += 4) {
-            float part[4];
-#pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const float2 d = sm.made[t + u][ch];
-                float b[RN], cc[RN];
-                load_states<RN>(b, &sm.B[buf][t + u][n0]);
-                load_states<RN>(cc, &sm.C[buf][t + u][n0]);
-                float p0 = 0.f, p1 = 0.f;
-#pragma unroll
-                for (int r = 0; r < RN; ++r) {
-                    s[r] = fmaf(ex2_approx(d.x * A[r]), s[r], d.y * b[r]);
-                    if (r & 1) p1 = fmaf(s[r], cc[r], p1);
-                    else p0 = fmaf(s[r], cc[r], p0);
-                }
-                part[u] = p0 + p1;
-            }
-            // over the channel's four lanes: two exchanges leave lane g with token t + g's sum
-            const bool odd = g & 1, high = g & 2;
-            float k0 = odd ? part[1] : part[0], k1 = odd ? part[3] : part[2];
-            k0 += __shfl_xor_sync(0xffffffffu, odd ? part[0] : part[1], 1);
-            k1 += __shfl_xor_sync(0xffffffffu, odd ? part[2] : part[3], 1);
-            float mine = high ? k1 : k0;
-            mine += __shfl_xor_sync(0xffffffffu, high ? k0 : k1, 2);
-            sm.y[t + g][ch] = mine;
-        }
-        __syncthreads();
-        if (c0 + col < a.channels) {
-#pragma unroll
-            for (int i = 0; i < kChunk * CH / kSelThreads; ++i) {
+            for (int i = 0; i < kPasses; ++i) {
                 const int t = row_of + i * (kSelThreads / CH);
-                if (t < nt) {
-                    const float z = sm.z[buf][t][col], y = fmaf(skip, sm.x[buf][t][col], sm.y[t][col]);
-                    reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)(sq.first + t0 + t) * a.out_stride + c0 + col] =
-                        __float2bfloat16_rn(a.scale * y * __fdividef(z, 1.0f + __expf(-z)));
-                }
+                const float4 y = sm.y[k & 1][t][col];
+                const float2 f = sm.after[k & 1][t][col];
+                if (t < nt) out[(size_t)t * a.out_stride] = __float2bfloat16_rn(((y.x + y.y) + (y.z + y.w) + f.x) * f.y);
             }
         }
-        __syncthreads();
-    }
-    if (live) {
+        if (turn < n_chunks) {
+            asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+            // every serving thread's copies have landed when all of them have waited
+            asm volatile("bar.sync 1, %0;\n" ::"n"(kSelThreads) : "memory");
+            const int k = turn, nt = min(kChunk, sq.n_new - k * kChunk), buf = k & 1;
+            if (turn + 1 < n_chunks) fetch(turn + 1);
+            asm volatile("cp.async.commit_group;\n" ::: "memory");
 #pragma unroll
-        for (int r = 0; r < RN; ++r)
-            if (n0 + r < a.n_states) sq.write[(size_t)c * a.n_states + n0 + r] = s[r];
+            for (int i = 0; i < kPasses; ++i) {
+                const int t = row_of + i * (kSelThreads / CH);
+                const float x = sm.x[buf][t][col], z = sm.z[buf][t][col];
+                const float dt = t < nt ? softplus_r(sm.dt[buf][t][col] + bias) : 0.f;
+                sm.made[buf][t][col] = make_float2(dt, t < nt ? dt * x : 0.f);
+                // (the chunk two before this one has gone out: the same thread read its place above)
+                sm.after[buf][t][col] = make_float2(skip * x, a.scale * __fdividef(z, 1.0f + __expf(-z)));
+            }
+        }
+        turn_over();
     }
 }
 
@@ -1103,7 +1160,7 @@ static int launch_selective(const SelArgs& a, int exact, int single, int n_seqs,
     const int low16 = a.n_states % 4 == 0 && aligned16(a.low, a.low_stride) && a.b_col0 % 4 == 0 && a.c_col0 % 4 == 0;
     const int rc = allow_smem(selective_scan_kernel<RN>, sizeof(SelSmem<RN>), "selective_scan");
     if (rc != BLM_OK) return rc;
-    selective_scan_kernel<RN><<<grid, kSelThreads, sizeof(SelSmem<RN>), stream>>>(a, rows16, low16, cu_seqlens, slot_of_seq, start_pos, state,
+    selective_scan_kernel<RN><<<grid, kSelBlock, sizeof(SelSmem<RN>), stream>>>(a, rows16, low16, cu_seqlens, slot_of_seq, start_pos, state,
                                                                                   slot_stride, copy_stride, state_off);
     return blm_check_launch("selective_scan");
 }
