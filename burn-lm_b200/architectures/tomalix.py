@@ -40,7 +40,7 @@ def _scaling(s):
 
 def _attention(width: int, eps: float, m, a: str, gate: bool = False) -> PartPlan:
     tensors = {r: a + r for r in ("q", "k", "v", "o")}
-    if m.diff is None and m.chunk is None and not gate and m.dim == m.vdim and m.dim in TUNED_HEADS:
+    if m.diff is None and m.chunk is None and not gate and m.dim == m.vdim and m.dim in TUNED_HEADS and m.scale > 0:
         # nothing but full causal attention, at a head size the dense decoder's mixer has kernels for
         position = PartPlan("none", NoPositionSpec())
         if m.rot.dims:

@@ -370,7 +370,7 @@ BLM_API int blm_attention(const void* q, long long q_stride, const void* pool, i
         BLM_REQUIRE(q_stride % 8 == 0 && ((size_t)q & 15) == 0, "attention: q rows must be 16-byte aligned");
         if (max_q_len >= 64 && status != nullptr && n_pages > 0 && ((size_t)pool & 15) == 0) {
             // long prompts: the products on tcgen05, accumulators in tensor memory
-            AttnPrefillTcArgs t;
+            AttnPrefillTcArgs t = {};
             t.block_table = block_table; t.table_stride = table_stride; t.cu_seqlens = cu_seqlens; t.slot_of_seq = slot_of_seq;
             t.start_pos = start_pos; t.out = (__nv_bfloat16*)out; t.n_heads = n_heads; t.n_kv = n_kv; t.window = window;
             t.scale_log2e = f.scale_log2e; t.status = status;

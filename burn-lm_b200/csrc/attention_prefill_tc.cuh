@@ -27,6 +27,12 @@
 // softmax threads before the product: a probability of zero does not silence a NaN.  Every mbarrier wait
 // is bounded; one that runs out records a code in the status word and the block goes to its end, where
 // the tensor memory is given back.
+//
+// The kernel is a template of the keys' and the values' lanes (HDK, HDV: multiples of 64) and of GEN.  GEN false: keys and
+// values of one size, the dense decoder's use of it.  GEN true, the windowed family's: keys and values of any multiple of 8
+// lanes up to HDK and HDV (the TMA fills the lanes beyond with zeros: three-dimensional maps, lanes by rows by pages), a
+// window or chunks, two maps a head (a query head for each; their sums leave as shares for the kernel that forms the
+// difference), a gate per head or per lane, results scaled and written as columns of wider rows.
 #pragma once
 #include <cuda.h>
 
@@ -45,6 +51,14 @@ struct AttnPrefillTcArgs {
     int n_heads, n_kv, window;
     float scale_log2e;
     int* status;                 // 0, or 31..37 when a bounded wait ran out
+    // GEN only
+    int chunk, maps, dv;         // chunk > 0: a position sees the keys of its own chunk; n_heads and n_kv count every map
+    const float* gate;           // null, or sigmoids on the result: of gate[n * gate_stride + head] (gate_lanes 0), or of a number per lane
+    long long gate_stride;
+    int gate_lanes;
+    long long out_stride;
+    float out_scale;
+    float* partial;              // null, or where a row's share goes: [N][n_heads][max, sum, dv lanes]
 };
 
 namespace attn_tc {
@@ -53,8 +67,10 @@ constexpr int kThreads = 224;        // producer warp, two tensor-core warps (sc
 constexpr int BQ = 128, BKV = 64;    // query rows of a block, keys of a step (one cache page)
 constexpr int kVStages = 2;          // pages of values in shared memory
 // pages of keys in shared memory and score tiles in tensor memory: what lets two blocks share an SM
-__host__ __device__ constexpr int key_stages(int hd) { return hd == 64 ? 4 : 2; }
-__host__ __device__ constexpr int score_ring(int hd) { return hd == 64 ? 3 : 2; }
+// (values beyond 128 lanes leave room for one block only, with deeper rings)
+__host__ __device__ constexpr int key_stages(int hdk, int hdv) { return hdk == 64 || hdv > 128 ? 4 : 2; }
+__host__ __device__ constexpr int score_ring(int hdk, int hdv) { return (hdk == 64 && hdv == 64) || hdv > 128 ? 3 : 2; }
+__host__ __device__ constexpr int blocks_an_sm(int hdv) { return hdv > 128 ? 1 : 2; }
 enum { TC_ATTN_Q = 31, TC_ATTN_K = 32, TC_ATTN_V = 33, TC_ATTN_S = 34, TC_ATTN_P = 35, TC_ATTN_PV = 36, TC_ATTN_FREE = 37 };
 
 __device__ __forceinline__ unsigned smem_u32(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -97,6 +113,12 @@ __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, i
     asm volatile(
         "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];\n" ::"r"(smem_u32(dst)),
         "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar))
+        : "memory");
+}
+__device__ __forceinline__ void tma_load_3d(void* dst, const CUtensorMap* map, int x, int y, int z, unsigned long long* bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];\n" ::"r"(smem_u32(dst)),
+        "l"(map), "r"(x), "r"(y), "r"(z), "r"(smem_u32(bar))
         : "memory");
 }
 // Shared-memory operand descriptors; tiles are rows of 128 bytes with the 128-byte swizzle, eight rows
@@ -216,22 +238,24 @@ __device__ __forceinline__ void tmem_st32_bits(unsigned taddr, const unsigned (&
 constexpr float kLazy = 8.0f;     // the reference maximum of a row moves only when a block exceeds it by more than 2^kLazy
 }  // namespace attn_tc
 
-template <int HD>
-__global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(const AttnPrefillTcArgs a, const __grid_constant__ CUtensorMap qmap,
-                                                                            const __grid_constant__ CUtensorMap pool_map) {
+template <int HDK, int HDV, bool GEN>
+__global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
+    attn_prefill_tc_kernel(const AttnPrefillTcArgs a, const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap pool_map,
+                           const __grid_constant__ CUtensorMap value_map) {
+    // pool_map: the pool's rows (GEN: the keys of its pages); value_map: GEN only, the values of its pages
     using namespace attn_tc;
-    constexpr int SUB = HD / 64;                         // 64-lane sub-tiles of a row
-    constexpr int kKStages = key_stages(HD), kSRing = score_ring(HD);
+    constexpr int SUB = HDK / 64, SUBV = HDV / 64;       // 64-lane sub-tiles of a row
+    constexpr int kKStages = key_stages(HDK, HDV), kSRing = score_ring(HDK, HDV);
     constexpr unsigned kTile = 128 * 128;                // bytes of a sub-tile: 128 rows of 128 bytes
     constexpr unsigned kPage = 64 * 128;                 // bytes of a page's sub-tile: 64 keys of 128 bytes
-    constexpr unsigned kQBytes = SUB * kTile, kKBytes = SUB * kPage, kVBytes = SUB * kPage;
+    constexpr unsigned kQBytes = SUB * kTile, kKBytes = SUB * kPage, kVBytes = SUBV * kPage;
     constexpr int kOCol = kSRing * BKV;                  // S of step j: columns 64 (j % kSRing) ..; O: the columns behind the ring
-    constexpr int kTmemCols = kOCol + HD <= 256 ? 256 : 512;
+    constexpr int kTmemCols = kOCol + HDV <= 256 ? 256 : 512;
     extern __shared__ __align__(1024) unsigned char smem_tc_raw[];
     unsigned char* smem = smem_tc_raw + ((1024u - (smem_u32(smem_tc_raw) & 1023u)) & 1023u);
     unsigned char* Qs = smem;                            // [SUB][128 rows][128 bytes]
     unsigned char* Ks = Qs + kQBytes;                    // [kKStages][SUB][64 keys][128 bytes]
-    unsigned char* Vs = Ks + kKStages * kKBytes;         // [kVStages][SUB][64 keys][128 bytes]
+    unsigned char* Vs = Ks + kKStages * kKBytes;         // [kVStages][SUBV][64 keys][128 bytes]
     unsigned long long* q_full = reinterpret_cast<unsigned long long*>(Vs + kVStages * kVBytes);
     unsigned long long* k_full = q_full + 1;             // [kKStages] a page's keys have landed
     unsigned long long* k_empty = k_full + kKStages;     // [kKStages] the scores that read them are formed
@@ -255,9 +279,14 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
     const int kv_total = start + q_len;                           // keys of this sequence in the cache after the step's append
     const int rows = min(BQ, q_len - q0);
     const int key_hi = start + q0 + rows - 1;                     // the last key any row of the block sees
-    const int key_lo = a.window > 0 ? max(0, start + q0 - a.window + 1) : 0;
+    auto first_key = [&](int pos) -> int {                        // the first key a position sees
+        if (GEN && a.chunk > 0) return pos - pos % a.chunk;
+        return a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    };
+    const int key_lo = first_key(start + q0);
     const int kb_lo = key_lo / BKV, kb_hi = key_hi / BKV, n_blocks = kb_hi - kb_lo + 1;
-    const int kvh = head / (a.n_heads / a.n_kv);
+    const int vh = GEN ? head / a.maps / (a.n_heads / a.n_kv) : 0;
+    const int kvh = GEN ? vh * a.maps + head % a.maps : head / (a.n_heads / a.n_kv);
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
@@ -291,12 +320,22 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
             const int* pages = a.block_table + (size_t)a.slot_of_seq[seq] * a.table_stride;
             mbar_expect_tx(q_full, kQBytes);
 #pragma unroll
-            for (int h = 0; h < SUB; ++h) tma_load_2d(Qs + h * kTile, &qmap, head * HD + h * 64, tok0 + q0, q_full);
+            for (int h = 0; h < SUB; ++h) {
+                // (GEN: lanes by heads by tokens, so that lanes beyond the head's are zeros)
+                if (GEN) tma_load_3d(Qs + h * kTile, &qmap, h * 64, head, tok0 + q0, q_full);
+                else tma_load_2d(Qs + h * kTile, &qmap, head * HDK + h * 64, tok0 + q0, q_full);
+            }
             auto row_of = [&](int step) { return ((pages[kb_lo + step] * 2) * a.n_kv + kvh) * 64; };      // the page's keys of this kv head
             auto load_keys = [&](int step) -> bool {
                 const int ks = step % kKStages;
                 if (step >= kKStages && !mbar_wait(k_empty + ks, ((step / kKStages) - 1) & 1)) { atomicCAS(a.status, 0, TC_ATTN_FREE); return false; }
                 mbar_expect_tx(k_full + ks, kKBytes);
+                if (GEN) {
+                    const int page = pages[kb_lo + step];
+#pragma unroll
+                    for (int h = 0; h < SUB; ++h) tma_load_3d(Ks + ks * kKBytes + h * kPage, &pool_map, h * 64, kvh * 64, page, k_full + ks);
+                    return true;
+                }
                 const int krow = row_of(step);
 #pragma unroll
                 for (int h = 0; h < SUB; ++h) tma_load_2d(Ks + ks * kKBytes + h * kPage, &pool_map, h * 64, krow, k_full + ks);
@@ -307,9 +346,15 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
                 const int b = j & 1;
                 if (j >= 2 && !mbar_wait(pv_done + (j - 2) % kSRing, ((j - 2) / kSRing) & 1)) { atomicCAS(a.status, 0, TC_ATTN_FREE); break; }
                 mbar_expect_tx(v_full + b, kVBytes);
-                const int vrow = row_of(j) + a.n_kv * 64;                    // the values lie n_kv * 64 rows after the keys
+                if (GEN) {
+                    const int page = pages[kb_lo + j];
 #pragma unroll
-                for (int h = 0; h < SUB; ++h) tma_load_2d(Vs + b * kVBytes + h * kPage, &pool_map, h * 64, vrow, v_full + b);
+                    for (int h = 0; h < SUBV; ++h) tma_load_3d(Vs + b * kVBytes + h * kPage, &value_map, h * 64, vh * 64, page, v_full + b);
+                } else {
+                    const int vrow = row_of(j) + a.n_kv * 64;                // the values lie n_kv * 64 rows after the keys
+#pragma unroll
+                    for (int h = 0; h < SUBV; ++h) tma_load_2d(Vs + b * kVBytes + h * kPage, &pool_map, h * 64, vrow, v_full + b);
+                }
                 if (j + kKStages - 1 < n_blocks && !load_keys(j + kKStages - 1)) break;
             }
         }
@@ -326,10 +371,10 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
                 if (j >= kSRing && !mbar_wait(pv_done + t, ((j / kSRing) - 1) & 1)) { atomicCAS(a.status, 0, TC_ATTN_PV); break; }
                 if (!mbar_wait(k_full + ks, (j / kKStages) & 1)) { atomicCAS(a.status, 0, TC_ATTN_K); break; }
                 asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-                // HD / 16 steps of k; a step is 32 bytes along the swizzled row (+2 in the address field), the
+                // HDK / 16 steps of k; a step is 32 bytes along the swizzled row (+2 in the address field), the
                 // second half of a 128-lane head lies in the next sub-tile
 #pragma unroll
-                for (int kk = 0; kk < HD / 16; ++kk) {
+                for (int kk = 0; kk < HDK / 16; ++kk) {
                     const unsigned long long ad = q_desc + (unsigned)((kk >> 2) * (kTile >> 4) + 2 * (kk & 3));
                     const unsigned long long bd = k_desc + (unsigned)(ks * (kKBytes >> 4) + (kk >> 2) * (kPage >> 4) + 2 * (kk & 3));
                     umma(tmem_base + (unsigned)(t * BKV), ad, bd, kIdescS, kk > 0 ? 1u : 0u);
@@ -341,7 +386,7 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
     } else if (warp == 2) {
         if (lane == 0) {
             // ---------------- tensor core, values: O += P(j) V(j) ----------------
-            constexpr unsigned kIdescPV = idesc(HD, true);
+            constexpr unsigned kIdescPV = idesc(HDV, true);
             const unsigned long long v_desc = desc_mn_major(Vs, kPage);
             for (int j = 0; j < n_blocks; ++j) {
                 const int b = j & 1, t = j % kSRing;
@@ -364,7 +409,8 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
         const int r = quarter * 32 + lane;                       // row of the tile, lane of tensor memory
         const bool live = r < rows;
         const int pos = start + q0 + r;                          // this row's position: it sees keys lo .. pos
-        const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+        const int lo = first_key(pos);
+        const int warp_lo = first_key(start + q0 + quarter * 32), warp_hi_lo = first_key(start + q0 + quarter * 32 + 31);    // of the warp's first and last row
         const unsigned trow = tmem_base + ((unsigned)(quarter * 32) << 16);
         // O accumulates in tensor memory over the blocks, against a reference maximum m_run per row that only
         // moves when a block's maximum exceeds it by more than 2^kLazy: then the row of O is rescaled in tensor
@@ -381,8 +427,8 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
             // of zero without a look at the scores.
             const unsigned taddr = trow + (unsigned)(t * BKV);
             const int wpos_lo = start + q0 + quarter * 32, wpos_hi = wpos_lo + 31;
-            const bool open_block = key0 + BKV - 1 <= wpos_lo && (a.window <= 0 || key0 >= wpos_hi - a.window + 1);
-            const bool dead = key0 > wpos_hi || (a.window > 0 && key0 + BKV - 1 < wpos_lo - a.window + 1);
+            const bool open_block = key0 + BKV - 1 <= wpos_lo && key0 >= warp_hi_lo;
+            const bool dead = key0 > wpos_hi || key0 + BKV - 1 < warp_lo;
             unsigned buf[2][32];           // two loads of 32 columns: one in flight, one being worked on
             float rs4[4] = {0.f, 0.f, 0.f, 0.f};
             // An open block of a row that has its reference maximum already: ONE pass over the scores.  The
@@ -453,7 +499,7 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
                         if (!mbar_wait(pv_done + (j - 1) % kSRing, ((j - 1) / kSRing) & 1)) { if (lane == 0) atomicCAS(a.status, 0, TC_ATTN_PV); ok = false; break; }
                         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
 #pragma unroll 1
-                        for (int c = 0; c < HD / 32; ++c) {
+                        for (int c = 0; c < HDV / 32; ++c) {
                             float v[32];
                             tmem_ld32(trow + kOCol + c * 32, v);
 #pragma unroll
@@ -503,7 +549,7 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
                 if (!mbar_wait(v_full + b, (j >> 1) & 1)) { if (lane == 0) atomicCAS(a.status, 0, TC_ATTN_V); ok = false; break; }
                 if (r < BKV && key0 + r >= kv_total) {
 #pragma unroll
-                    for (int h = 0; h < SUB; ++h)
+                    for (int h = 0; h < SUBV; ++h)
 #pragma unroll
                         for (int c = 0; c < 8; ++c)
                             *reinterpret_cast<uint4*>(Vs + b * kVBytes + h * kPage + r * 128 + c * 16) = make_uint4(0u, 0u, 0u, 0u);
@@ -516,34 +562,76 @@ __global__ void __launch_bounds__(attn_tc::kThreads, 2) attn_prefill_tc_kernel(c
             if (lane == 0) mbar_arrive(p_full + t);
         }
         // the last product into O, then the row: O / l
-        float o[HD];
         if (ok) {
             if (!mbar_wait(pv_done + (n_blocks - 1) % kSRing, ((n_blocks - 1) / kSRing) & 1)) { if (lane == 0) atomicCAS(a.status, 0, TC_ATTN_PV); ok = false; }
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         }
-        if (ok) {
+        if (!GEN && ok) {
+            float o[GEN ? 1 : HDV];
 #pragma unroll
-            for (int c = 0; c < HD / 32; ++c) {
+            for (int c = 0; c < HDV / 32; ++c) {
                 float v[32];
                 tmem_ld32(trow + kOCol + c * 32, v);
 #pragma unroll
-                for (int i = 0; i < 32; ++i) o[c * 32 + i] = v[i];
+                for (int i = 0; i < 32; ++i) o[GEN ? 0 : c * 32 + i] = v[i];
             }
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
-        }
-        if (ok && live) {
-            const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
-            __nv_bfloat16* dst = a.out + (size_t)(tok0 + q0 + r) * a.n_heads * HD + (size_t)head * HD;
+            if (live) {
+                const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+                __nv_bfloat16* dst = a.out + (size_t)(tok0 + q0 + r) * a.n_heads * HDV + (size_t)head * HDV;
 #pragma unroll
-            for (int d = 0; d < HD; d += 8) {
-                unsigned pk[4];
+                for (int d = 0; d < (GEN ? 0 : HDV); d += 8) {
+                    unsigned pk[4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const __nv_bfloat162 two = __floats2bfloat162_rn(o[d + 2 * e] * inv, o[d + 2 * e + 1] * inv);
-                    pk[e] = *reinterpret_cast<const unsigned*>(&two);
+                    for (int e = 0; e < 4; ++e) {
+                        const __nv_bfloat162 two = __floats2bfloat162_rn(o[d + 2 * e] * inv, o[d + 2 * e + 1] * inv);
+                        pk[e] = *reinterpret_cast<const unsigned*>(&two);
+                    }
+                    *reinterpret_cast<uint4*>(dst + d) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
                 }
-                *reinterpret_cast<uint4*>(dst + d) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
             }
+        }
+        if (GEN && ok) {
+            const size_t n = (size_t)(tok0 + q0 + r);
+            float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+            float* part = a.partial ? a.partial + (n * a.n_heads + head) * (a.dv + 2) : nullptr;       // dv even: 8-byte aligned
+            if (live && part != nullptr) *reinterpret_cast<float2*>(part) = make_float2(0.f, 1.f);     // one share: normalised
+            if (part == nullptr) {
+                inv *= a.out_scale;
+                if (live && a.gate != nullptr && a.gate_lanes == 0) inv /= 1.0f + __expf(-a.gate[n * a.gate_stride + head]);
+            }
+            const float* gate = live && a.gate != nullptr && a.gate_lanes > 0 ? a.gate + n * a.gate_stride + (size_t)head * a.gate_lanes : nullptr;
+            __nv_bfloat16* dst = a.out + n * a.out_stride + (size_t)head * a.dv;
+#pragma unroll 1
+            for (int c = 0; c < HDV / 32 && c * 32 < a.dv; ++c) {
+                float v[32];
+                tmem_ld32(trow + kOCol + c * 32, v);
+                if (live && part != nullptr) {
+#pragma unroll
+                    for (int i = 0; i < 32; i += 2)
+                        if (c * 32 + i < a.dv) *reinterpret_cast<float2*>(part + 2 + c * 32 + i) = make_float2(v[i] * inv, v[i + 1] * inv);
+                } else if (live) {
+#pragma unroll
+                    for (int d = 0; d < 32; d += 8) {
+                        if (c * 32 + d < a.dv) {                 // dv is a multiple of 8
+                            unsigned pk[4];
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                float lo_v = v[d + 2 * e] * inv, hi_v = v[d + 2 * e + 1] * inv;
+                                if (gate != nullptr) {
+                                    lo_v = __fdividef(lo_v, 1.0f + __expf(-gate[c * 32 + d + 2 * e]));
+                                    hi_v = __fdividef(hi_v, 1.0f + __expf(-gate[c * 32 + d + 2 * e + 1]));
+                                }
+                                const __nv_bfloat162 two = __floats2bfloat162_rn(lo_v, hi_v);
+                                pk[e] = *reinterpret_cast<const unsigned*>(&two);
+                            }
+                            *reinterpret_cast<uint4*>(dst + c * 32 + d) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                        }
+                    }
+                }
+                __syncwarp();            // the warp reads its next columns of tensor memory together
+            }
+            asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
         }
     }
     // everybody meets; then the warp that took the tensor memory gives it back
@@ -559,8 +647,10 @@ typedef CUresult (*TcAttnEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuin
                                         const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                         CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-// A bf16 matrix [rows, width] with row stride ld (elements) as the TMA sees it: boxes of box_rows x 64, 128-byte swizzle.
-static bool attn_tc_map(const void* base, long long ld, long long rows, int width, int box_rows, CUtensorMap* out) {
+// bf16 numbers as the TMA sees them: up to three dimensions (the innermost contiguous), `strides` in bytes from the second
+// on, boxes of 64 x box1 x box2, 128-byte swizzle; what lies outside reads as zeros.
+static bool attn_tc_map_nd(const void* base, int rank, const cuuint64_t (&dims)[3], const cuuint64_t (&strides)[2], cuuint32_t box1, cuuint32_t box2,
+                           CUtensorMap* out) {
     static TcAttnEncodeTiledFn encode = nullptr;
     if (!encode) {
         void* fn = nullptr;
@@ -570,16 +660,14 @@ static bool attn_tc_map(const void* base, long long ld, long long rows, int widt
             return false;
         encode = (TcAttnEncodeTiledFn)fn;
     }
-    static std::map<std::tuple<const void*, long long, long long, int, int>, CUtensorMap> maps;
-    const auto key = std::make_tuple(base, ld, rows, width, box_rows);
+    static std::map<std::tuple<const void*, int, cuuint64_t, cuuint64_t, cuuint64_t, cuuint64_t, cuuint64_t, cuuint32_t, cuuint32_t>, CUtensorMap> maps;
+    const auto key = std::make_tuple(base, rank, dims[0], dims[1], dims[2], strides[0], strides[1], box1, box2);
     auto it = maps.find(key);
     if (it == maps.end()) {
         CUtensorMap m;
-        const cuuint64_t dims[2] = {(cuuint64_t)width, (cuuint64_t)rows};
-        const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
-        const cuuint32_t box[2] = {64, (cuuint32_t)box_rows};
-        const cuuint32_t estr[2] = {1, 1};
-        if (encode(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+        const cuuint32_t box[3] = {64, box1, box2};
+        const cuuint32_t estr[3] = {1, 1, 1};
+        if (encode(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank, const_cast<void*>(base), dims, strides, box, estr,
                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
             return false;
@@ -589,24 +677,30 @@ static bool attn_tc_map(const void* base, long long ld, long long rows, int widt
     *out = it->second;
     return true;
 }
+// A matrix [rows, width] with row stride ld (elements): boxes of box_rows x 64.
+static bool attn_tc_map(const void* base, long long ld, long long rows, int width, int box_rows, CUtensorMap* out) {
+    return attn_tc_map_nd(base, 2, {(cuuint64_t)width, (cuuint64_t)rows, 1}, {(cuuint64_t)ld * 2, 0}, (cuuint32_t)box_rows, 1, out);
+}
 
-template <int HD>
-static int attn_prefill_tc_launch(const AttnPrefillTcArgs& a, const CUtensorMap& qmap, const CUtensorMap& pmap, dim3 grid, cudaStream_t stream) {
-    constexpr int SUB = HD / 64;
-    const size_t smem = (size_t)SUB * 128 * 128 + (size_t)(attn_tc::key_stages(HD) + attn_tc::kVStages) * SUB * 64 * 128 + 24 * 8 + 16 + 1024;
+template <int HDK, int HDV, bool GEN>
+static int attn_prefill_tc_launch(const AttnPrefillTcArgs& a, const CUtensorMap& qmap, const CUtensorMap& pmap, const CUtensorMap& vmap, dim3 grid,
+                                  cudaStream_t stream) {
+    const size_t smem = (size_t)(HDK / 64) * 128 * 128 + (size_t)attn_tc::key_stages(HDK, HDV) * (HDK / 64) * 64 * 128 +
+                        (size_t)attn_tc::kVStages * (HDV / 64) * 64 * 128 + 24 * 8 + 16 + 1024;
+    auto kernel = attn_prefill_tc_kernel<HDK, HDV, GEN>;
     static bool opted_in = false;
     if (!opted_in) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "attention prefill (tcgen05): %s", cudaGetErrorString(e));
         opted_in = true;
     }
-    cudaError_t e = blm_launch_dependent(attn_prefill_tc_kernel<HD>, grid, dim3(attn_tc::kThreads), smem, stream, a, qmap, pmap);
+    cudaError_t e = blm_launch_dependent(kernel, grid, dim3(attn_tc::kThreads), smem, stream, a, qmap, pmap, vmap);
     if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "attention prefill (tcgen05): %s", cudaGetErrorString(e));
     return BLM_OK;
 }
 
+#ifndef BLM_ATTN_TC_GENERAL
 // BLM_OK when the kernel took the step, -1 when the shape is not its own, else an error.
 // q: the step's rows, token n's head h at q + n * q_stride + h * hd.
 static int launch_attn_prefill_tc(const AttnPrefillTcArgs& a, const void* q, long long q_stride, const void* pool, int n_pages,
@@ -617,5 +711,31 @@ static int launch_attn_prefill_tc(const AttnPrefillTcArgs& a, const void* q, lon
     if (!attn_tc_map(q, q_stride, n_tokens, a.n_heads * hd, attn_tc::BQ, &qmap) ||
         !attn_tc_map(pool, hd, (long long)n_pages * 2 * a.n_kv * 64, hd, 64, &pmap))
         return blm_fail(BLM_CUDA_ERROR, "attention prefill (tcgen05): cuTensorMapEncodeTiled failed");
-    return hd == 64 ? attn_prefill_tc_launch<64>(a, qmap, pmap, grid, stream) : attn_prefill_tc_launch<128>(a, qmap, pmap, grid, stream);
+    return hd == 64 ? attn_prefill_tc_launch<64, 64, false>(a, qmap, pmap, pmap, grid, stream)
+                    : attn_prefill_tc_launch<128, 128, false>(a, qmap, pmap, pmap, grid, stream);
 }
+#else
+// The windowed family's use of the kernel: whether it takes the sizes, and its launch (BLM_OK, or an error).  q [N, n_heads, dk]
+// contiguous; the pool's pages hold keys [n_kv, 64, dk], then values [n_kv / maps, 64, dv], page_elems in all.
+static bool attn_prefill_tc_general_takes(int dk, int dv) { return dk >= 64 && dk <= 128 && dk % 8 == 0 && dv >= 64 && dv <= 256 && dv % 8 == 0; }
+static int launch_attn_prefill_tc_general(const AttnPrefillTcArgs& a, const void* q, const void* pool, long long page_elems, int n_pages, int dk,
+                                          int n_tokens, int n_seqs, int max_q_len, cudaStream_t stream) {
+    const dim3 grid(a.n_heads, (max_q_len + attn_tc::BQ - 1) / attn_tc::BQ, n_seqs);
+    BLM_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "attention prefill (tcgen05): grid %u x %u too large", grid.y, grid.z);
+    const int n_v = a.n_kv / a.maps;
+    const __nv_bfloat16* values = (const __nv_bfloat16*)pool + (size_t)a.n_kv * 64 * dk;
+    CUtensorMap qmap, kmap, vmap;
+    if (!attn_tc_map_nd(q, 3, {(cuuint64_t)dk, (cuuint64_t)a.n_heads, (cuuint64_t)n_tokens}, {(cuuint64_t)dk * 2, (cuuint64_t)a.n_heads * dk * 2}, 1,
+                        attn_tc::BQ, &qmap) ||
+        !attn_tc_map_nd(pool, 3, {(cuuint64_t)dk, (cuuint64_t)a.n_kv * 64, (cuuint64_t)n_pages}, {(cuuint64_t)dk * 2, (cuuint64_t)page_elems * 2}, 64, 1,
+                        &kmap) ||
+        !attn_tc_map_nd(values, 3, {(cuuint64_t)a.dv, (cuuint64_t)n_v * 64, (cuuint64_t)n_pages}, {(cuuint64_t)a.dv * 2, (cuuint64_t)page_elems * 2}, 64,
+                        1, &vmap))
+        return blm_fail(BLM_CUDA_ERROR, "attention prefill (tcgen05): cuTensorMapEncodeTiled failed");
+    if (dk <= 64 && a.dv <= 64) return attn_prefill_tc_launch<64, 64, true>(a, qmap, kmap, vmap, grid, stream);
+    if (dk <= 64 && a.dv <= 128) return attn_prefill_tc_launch<64, 128, true>(a, qmap, kmap, vmap, grid, stream);
+    if (a.dv <= 128) return attn_prefill_tc_launch<128, 128, true>(a, qmap, kmap, vmap, grid, stream);
+    if (a.dv <= 192) return attn_prefill_tc_launch<128, 192, true>(a, qmap, kmap, vmap, grid, stream);
+    return attn_prefill_tc_launch<128, 256, true>(a, qmap, kmap, vmap, grid, stream);
+}
+#endif

@@ -16,6 +16,8 @@
 // The cache page of this family holds the keys [n_kv, page, dk] followed by the values [n_kv / maps, page, dv].
 // Scores, softmax and sums are fp32; q, keys and values are read in the cache's dtype.
 #include "common.cuh"
+#define BLM_ATTN_TC_GENERAL
+#include "attention_prefill_tc.cuh"
 
 BLM_API const char* blm_attention_sink_last_error() { return g_blm_error; }
 
@@ -574,6 +576,7 @@ __device__ __forceinline__ void zero_unwritten(__nv_bfloat16* buf, int n_rows, i
     }
 }
 
+constexpr int kNoWindow = 1 << 28;      // a window of this many or more is no window
 constexpr int kTileQ = 64, kTileK = 64;
 
 // The pages a query tile walks: `kept` pages from the sequence's start, then pages wp0 .. wp1.
@@ -1200,7 +1203,9 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
                                long long gate_stride, int gate_lanes, void* out, long long out_stride, float out_scale, float* partial,
                                int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, int page_size, int window,
                                int chunk, int keep_first, float scale, int sink, const float* head_scale, const float* sink_logit,
-                               float softcap, float diff_lambda, float diff_scale, float diff_eps, cudaStream_t stream) {
+                               float softcap, float diff_lambda, float diff_scale, float diff_eps, int n_pages, int* status,
+                               cudaStream_t stream) {
+    // n_pages, status: of the pool, and where a bounded wait that ran out is recorded (for the tcgen05 kernel; 0 and null: not run)
     // maps 2: n_heads and n_kv count every map, and diff_* are the difference's numbers (DiffOpts); partial is then needed
     // chunk > 0: the mask is by chunks and `window` is not looked at; gate_lanes 0: a gate per head, dv: one per lane
     // head_scale, sink_logit: float32 [n_heads] or null; softcap: 0 for none (see ScoreOpts)
@@ -1225,6 +1230,20 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
     const Mask mask{window, chunk};
     const RowOut ro{gate, gate_stride, gate_lanes, out_stride, out_scale};
     const DiffOpts df{diff_lambda, diff_scale, diff_eps};
+    if (is_prompt && max_q_len >= 64 && status != nullptr && n_pages > 0 && attn_prefill_tc_general_takes(dk, dv) && !sink && softcap == 0.f &&
+        head_scale == nullptr && keep_first == 0 && scale > 0.f && out_stride % 8 == 0 && (((size_t)out | (size_t)q | (size_t)pool) & 15) == 0) {
+        // long portions without options of the scores: the products on tcgen05, accumulators in tensor memory
+        AttnPrefillTcArgs t = {};
+        t.block_table = block_table; t.table_stride = table_stride; t.cu_seqlens = cu_seqlens; t.slot_of_seq = slot_of_seq;
+        t.start_pos = start_pos; t.out = (__nv_bfloat16*)out; t.n_heads = n_heads; t.n_kv = n_kv; t.window = window < kNoWindow ? window : 0;
+        t.scale_log2e = scale * 1.4426950408889634f; t.status = status;
+        t.chunk = chunk; t.maps = maps; t.dv = dv; t.gate = gate; t.gate_stride = gate_stride; t.gate_lanes = gate_lanes;
+        t.out_stride = out_stride; t.out_scale = out_scale; t.partial = partial;
+        const int rc = launch_attn_prefill_tc_general(t, q, pool, page_elems, n_pages, dk, n_tokens, n_seqs, max_q_len, stream);
+        if (rc != BLM_OK) return rc;
+        if (partial != nullptr) finish_shares<__nv_bfloat16>(partial, ro, out, n_tokens, n_heads, maps, dv, 1, df, stream);
+        return blm_check_launch("attention_sink (tcgen05)");
+    }
     if (is_prompt) {
 #define BLM_PROMPT(NV) launch_prompt_heads<NV>(hb, q, pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq, n_seqs, ro, \
                                          out, partial, n_tokens, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df, stream)

@@ -95,7 +95,7 @@ _protos = {
         "blm_attention_sink": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                c_void_p, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_float, c_void_p, c_int, c_int,
                                c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_float,
-                               c_float, c_float, c_float, c_void_p],
+                               c_float, c_float, c_float, c_int, c_void_p, c_void_p],
         "blm_head_norm_rope_append": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
                                       c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
                                       c_void_p, c_void_p, c_int, c_void_p],
@@ -476,7 +476,8 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
     o = a_1 - lambda a_2, out = o / sqrt(mean(o^2) + eps) * c per head; it needs `scratch` for any n_splits.
 
     `max_q_len`: the longest run of new tokens of one sequence (a bound is enough): bfloat16 steps of 8 or more run
-    the tensor-core prompt kernel, 64 query rows a block (it reads step.cu_seqlens and step.start_pos); shorter ones
+    the tensor-core prompt kernel, 64 query rows a block (it reads step.cu_seqlens and step.start_pos), and steps of 64 or
+    more without options of the scores the tcgen05 kernel (keys of 64 to 128 lanes, values of 64 to 256); shorter ones
     the tensor-core decode kernel (bfloat16, up to 16 query heads a kv head) or else the row kernel, a block per (row,
     kv head) either, whose keys `n_splits` > 1 cuts over that many blocks (it then needs `scratch`:
     attention_sink_scratch_floats(...) float32)."""
@@ -507,7 +508,8 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
           _ptr(step.start_pos if prompt else None), (cu.numel() - 1) if prompt else 0, int(max_q_len), _ptr(gate), int(gate_stride),
           int(gate_lanes), _ptr(out), c_longlong(out.stride(0)), c_float(out_scale), _ptr(scratch if need else None), int(n_splits), n, n_heads,
           n_kv, int(maps), key_dim, value_dim, PAGE, int(window), int(chunk), int(keep_first), c_float(scale), 1 if sink else 0,
-          _ptr(head_scale), _ptr(sink_logit if sink else None), c_float(softcap or 0.0), *(c_float(v) for v in difference), _stream(),
+          _ptr(head_scale), _ptr(sink_logit if sink else None), c_float(softcap or 0.0), *(c_float(v) for v in difference),
+          pool.shape[0] if prompt else 0, _ptr(status_word(q.device)) if prompt else None, _stream(),
           kernels=2 if need else 1)
 
 

@@ -227,6 +227,29 @@ def test_chunked_attention_beside_a_selective_scan(shape, schedule, dtype, tol):
     check_mixer(entry, P.parallel_mixers, 48, (200, 9), [3, 1], SCHEDULES[schedule](200, 9), dtype, tol, H + dk + chunk)
 
 
+@pytest.mark.parametrize("dk,dv", [(64, 64), (64, 128), (72, 136), (128, 128), (96, 192), (128, 256), (104, 64), (128, 200)])
+@pytest.mark.parametrize("kind", ["chunks", "maps"])
+def test_long_portions_of_large_heads(kind, dk, dv):
+    """Portions of several tiles of query rows, beside one another, that start inside chunks and pages (the tcgen05 kernel);
+    the rows of a page no key has been written to hold NaN."""
+    rng = np.random.default_rng(dk + dv)
+    if kind == "maps":
+        entry, plain = difference(2, 1, dk, dv, None, rot_dims=32, base=300.0, diff=0.2, scale=0.5 * dk ** -0.5), lambda h, w, m: P.differential_attention(h, w, m, 1e-5)
+        plan = mixer_plan(entry, 40)
+    else:
+        entry, plain = pair(4, 2, dk, dv, 150, 8, 1, 1, 1, None, rot_dims=32, base=300.0), lambda h, w, m: P.chunk_attention(h, w, m["left"])
+        plan = mixer_plan(entry, 40).spec.left
+    w = mixer_weights(plan, rng)
+    hs = [bf(rng.normal(size=(n, 40))) for n in (500, 300)]
+    part = bound(plan, w, "bfloat16")
+    prefix = "l0.mix." if kind == "maps" else "l0.mix.left."
+    for schedule in ([(500, 300)], [(290, 1), (110, 199), (100, 100)], [(64, 64), (65, 127), (371, 109)]):
+        got = run_mixer(part, OwnCache(part, "bfloat16"), hs, [2, 0], schedule, "bfloat16")
+        for g, h in zip(got, hs):
+            want = plain(h, short(w, prefix), entry["mixer"])
+            assert np.abs(g - want).max() < 4e-2 * np.abs(want).max(), schedule
+
+
 @pytest.mark.parametrize("dtype,tol", [("float32", 5e-5), ("bfloat16", 2e-2)])
 @pytest.mark.parametrize("shape", sorted(PAIR_SHAPES))
 def test_the_scan_alone_over_several_sequences(shape, dtype, tol):
