@@ -802,6 +802,19 @@ def marinex_kernels(z, pk):
     return out
 
 
+def _time_captured(fn, reps=10):
+    """As _time, the calls captured in a CUDA graph: what single tokens cost inside a captured step, without the interpreter."""
+    import torch
+    for _ in range(2):
+        fn()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for _ in range(reps):
+            fn()
+    return _time(graph.replay, 5) / reps
+
+
 def tomalix_configs(z):
     """(llama, tomalix) of one size.  The new design's layers take turns: attention with scaled frequencies (Llama's head counts
     and head size) and a dense feed-forward; differential attention (half of Llama's heads with two maps each of its head
@@ -828,7 +841,7 @@ def tomalix_configs(z):
 
 
 def tomalix_kernels(z, pk):
-    """The new design's kernels alone, CUDA events, back to back, beside the like kernel of another model: attention in chunks
+    """The new design's kernels alone, CUDA events, back to back (single tokens: captured in a graph), beside the like kernel of another model: attention in chunks
     with a gate a lane and differential attention (one 2,048-token prompt; 64 sequences of 1,088 tokens) beside the dense
     decoder's attention, what stands between projection and attention, the selective scan beside the state-space scan of the
     same channels, feed-forwards and experts with a squared relu beside the dense decoder's and the GELU experts."""
@@ -843,6 +856,8 @@ def tomalix_kernels(z, pk):
     frac_bf16 = lambda flops, ms: round(flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12), 4)
     frac_hbm = lambda nbytes, ms: round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4)
 
+    timer = lambda prompt: globals()["_time" if prompt else "_time_captured"]
+
     def step(n_seqs, new, cached):
         seq = [s for s in range(n_seqs) for _ in range(new)]
         pos = [cached + t for _ in range(n_seqs) for t in range(new)]
@@ -852,6 +867,7 @@ def tomalix_kernels(z, pk):
 
     for n_seqs, new, cached in ((1, 2048, 0), (64, 1, 1087)):
         total, prompt = cached + new, new > 1
+        _time = timer(prompt)
         pages_each = -(-total // K.PAGE)
         n = n_seqs * new
         bt = torch.arange(n_seqs * pages_each, dtype=torch.int32, device=dev).reshape(n_seqs, pages_each)
@@ -865,7 +881,8 @@ def tomalix_kernels(z, pk):
                                                     H, G, hd, hd ** -0.5, window=w, n_splits=1, max_kv_len=total))
         ms_l, ms_lw = llama(0), llama(W)
         windowed = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, hd, hd ** -0.5, W, 0, sink=False, max_q_len=new))
-        chunks = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, hd, hd ** -0.5, 1 << 30, 0, sink=False, max_q_len=new, chunk=W,
+        chunk = W if prompt else 2 * W                      # (single tokens: all keys lie in the chunk)
+        chunks = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, hd, hd ** -0.5, 1 << 30, 0, sink=False, max_q_len=new, chunk=chunk,
                                                 gate=gate, gate_stride=gate.stride(0), gate_lanes=hd))
         plain = _time(lambda: K.attention_sink(q, st, pool, bt, o, H, G, hd, hd, hd ** -0.5, 1 << 30, 0, sink=False, max_q_len=new))
         scratch = torch.empty(K.attention_sink_scratch_floats(n, H, 2 * hd, 1, 2), dtype=torch.float32, device=dev)
@@ -882,7 +899,7 @@ def tomalix_kernels(z, pk):
                      chunks_frac_bf16=frac_bf16(4.0 * H * hd * in_chunk, chunks), difference_frac_bf16=frac_bf16(6.0 * H * hd * full, diff))
         else:
             key_bytes = n * G * 2 * hd * 2.0
-            seen = (total - 1) % W + 1
+            seen = (total - 1) % chunk + 1
             r.update(keys_seen_in_the_chunk=seen, llama_frac_hbm=frac_hbm(key_bytes * total, ms_l),
                      llama_window_frac_hbm=frac_hbm(key_bytes * min(total, W), ms_lw), windowed_family_no_mask_frac_hbm=frac_hbm(key_bytes * total, plain),
                      windowed_family_window_frac_hbm=frac_hbm(key_bytes * min(total, W), windowed),
@@ -893,9 +910,10 @@ def tomalix_kernels(z, pk):
         proj = torch.randn((n, cols), dtype=torch.float32, device=dev)
         qkv = torch.randn((n, cols), dtype=bf, device=dev)
         freq = torch.tensor([500000.0 ** (-2.0 * i / hd) for i in range(hd // 2)], dtype=torch.float64, device=dev)
-        ms_new = _time(lambda: K.head_norm_rope_append(proj, st, pool, bt, q, H, G, hd, 2 * hd, freq=freq, rotary_dims=hd, halves=True, maps=2))
+        table = K.rope_table(freq, total)
+        ms_new = _time(lambda: K.head_norm_rope_append(proj, st, pool, bt, q, H, G, hd, 2 * hd, freq=freq, rotary_dims=hd, halves=True, maps=2, table=table))
         ms_llama = _time(lambda: K.rope_append(qkv, st.token_seq, st.token_pos, st.slot_of_seq, bt, freq, hd, K.PAIRS_HALVES, pool5, H, G, hd,
-                                               write_cache=True, max_position=cached + new - 1))
+                                               write_cache=True, table=table, max_position=cached + new - 1))
         out[f"between_{n_seqs}x{new}"] = {"turn_append_two_maps_ms": round(ms_new, 4), "llama_turn_append_ms": round(ms_llama, 4),
                                           "frac_hbm": frac_hbm(n * cols * 6.0, ms_new), "llama_frac_hbm": frac_hbm(n * cols * 4.0, ms_llama)}
         # the scan: rows in and out, and the states
@@ -905,8 +923,8 @@ def tomalix_kernels(z, pk):
         xz = torch.randn((n, 2 * C), dtype=torch.float32, device=dev)
         low = torch.randn((n, R + 2 * S), dtype=torch.float32, device=dev)
         a_log, one = torch.zeros((C, S), dtype=torch.float32, device=dev), torch.ones(C, dtype=torch.float32, device=dev)
-        y = torch.empty((n, C), dtype=bf, device=dev)
-        ms_scan = _time(lambda: K.selective_scan(x, low, R, S, one, a_log, one, xz[:, C:], y, st, state, 0, dt=dt))
+        y, rates = torch.empty((n, C), dtype=bf, device=dev), K.scan_rates(a_log)
+        ms_scan = _time(lambda: K.selective_scan(x, low, R, S, one, a_log, one, xz[:, C:], y, st, state, 0, dt=dt, rates=rates))
         nbytes = n * C * (3 * 4.0 + 2.0) + 4.0 * n * 2 * S + (2.0 if not prompt else 1.0) * 4 * n_seqs * C * S
         heads, groups, rows, dv = C // 64, 8, 128, 64
         floats = K.scan_state_floats(heads, rows, dv)
@@ -937,6 +955,7 @@ def tomalix_kernels(z, pk):
     up, down = torch.randn((E, each, d), dtype=bf, device=dev) * 0.02, torch.randn((E, d, each), dtype=bf, device=dev) * 0.02
     router, bias = torch.randn((E, d), dtype=torch.float32, device=dev), torch.randn(E, dtype=torch.float32, device=dev)
     for n in (2048, 64, 8):
+        _time = timer(n == 2048)
         h = torch.randn((n, d), dtype=bf, device=dev)
         ms_up = _time(lambda: w_up.activated(h, bf, K.ACT_RELU2))
         ms_gated = _time(lambda: w1.gated(h, bf))

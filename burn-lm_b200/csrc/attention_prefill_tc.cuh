@@ -602,9 +602,24 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
             }
             const float* gate = live && a.gate != nullptr && a.gate_lanes > 0 ? a.gate + n * a.gate_stride + (size_t)head * a.gate_lanes : nullptr;
             __nv_bfloat16* dst = a.out + n * a.out_stride + (size_t)head * a.dv;
+            const bool gate16 = (((size_t)a.gate & 15) | (a.gate_stride & 3) | (a.gate_lanes & 3)) == 0;
 #pragma unroll 1
             for (int c = 0; c < HDV / 32 && c * 32 < a.dv; ++c) {
-                float v[32];
+                float v[32], g[32];
+                if (gate != nullptr) {           // asked for before the wait for tensor memory
+#pragma unroll
+                    for (int i = 0; i < 32; i += 4) {
+                        if (c * 32 + i >= a.dv) continue;
+                        if (gate16) {
+                            const float4 q4 = *reinterpret_cast<const float4*>(gate + c * 32 + i);
+                            g[i] = q4.x; g[i + 1] = q4.y; g[i + 2] = q4.z; g[i + 3] = q4.w;
+                        } else {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) g[i + e] = gate[c * 32 + i + e];
+                        }
+                    }
+                }
+                __syncwarp();
                 tmem_ld32(trow + kOCol + c * 32, v);
                 if (live && part != nullptr) {
 #pragma unroll
@@ -619,8 +634,8 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
                             for (int e = 0; e < 4; ++e) {
                                 float lo_v = v[d + 2 * e] * inv, hi_v = v[d + 2 * e + 1] * inv;
                                 if (gate != nullptr) {
-                                    lo_v = __fdividef(lo_v, 1.0f + __expf(-gate[c * 32 + d + 2 * e]));
-                                    hi_v = __fdividef(hi_v, 1.0f + __expf(-gate[c * 32 + d + 2 * e + 1]));
+                                    lo_v = __fdividef(lo_v, 1.0f + __expf(-g[d + 2 * e]));
+                                    hi_v = __fdividef(hi_v, 1.0f + __expf(-g[d + 2 * e + 1]));
                                 }
                                 const __nv_bfloat162 two = __floats2bfloat162_rn(lo_v, hi_v);
                                 pk[e] = *reinterpret_cast<const unsigned*>(&two);

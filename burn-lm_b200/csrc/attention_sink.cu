@@ -483,12 +483,54 @@ __global__ void attention_difference_kernel(const float* __restrict__ partial, R
     }
 }
 
+// The same for one share a map and an even dv (prompts): pairs of lanes, both maps' loads at once.
+template <typename T>
+__global__ void attention_difference_one_kernel(const float* __restrict__ partial, RowOut ro, T* __restrict__ out, int n_rows, int n_heads, int dv,
+                                                DiffOpts df) {
+    const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= n_rows * n_heads) return;
+    const int n = item / n_heads, head = item % n_heads;
+    const float* part = partial + (size_t)item * 2 * (dv + 2);
+    const float l1 = part[1], l2 = part[dv + 3];
+    float2 a1[kMaxVRegs / 2], a2[kMaxVRegs / 2];
+#pragma unroll
+    for (int i = 0; i < kMaxVRegs / 2; ++i) {
+        const int d = 2 * (lane + 32 * i);
+        a1[i] = a2[i] = make_float2(0.f, 0.f);
+        if (d < dv) {
+            a1[i] = *reinterpret_cast<const float2*>(part + 2 + d);
+            a2[i] = *reinterpret_cast<const float2*>(part + dv + 4 + d);
+        }
+    }
+    const float w1 = l1 > 0.f ? 1.f / l1 : 0.f, w2 = l2 > 0.f ? -df.lambda / l2 : 0.f;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMaxVRegs / 2; ++i) {
+        a1[i].x = a1[i].x * w1 + a2[i].x * w2;
+        a1[i].y = a1[i].y * w1 + a2[i].y * w2;
+        ss += a1[i].x * a1[i].x + a1[i].y * a1[i].y;
+    }
+    ss = warp_sum(ss);
+    const float inv = df.c / sqrtf(ss / (float)dv + df.eps) * ro.head_gate(n, head);
+    T* dst = out + (size_t)n * ro.stride + (size_t)head * dv;
+#pragma unroll
+    for (int i = 0; i < kMaxVRegs / 2; ++i) {
+        const int d = 2 * (lane + 32 * i);
+        if (d < dv) {
+            dst[d] = from_f32<T>(a1[i].x * inv * ro.lane_gate(n, head, d));
+            dst[d + 1] = from_f32<T>(a1[i].y * inv * ro.lane_gate(n, head, d + 1));
+        }
+    }
+}
+
 // what follows the kernels that left shares: one launch either way
 template <typename T>
 static void finish_shares(const float* partial, RowOut ro, void* out, int n_tokens, int n_heads, int maps, int dv, int n_splits, DiffOpts df,
                           cudaStream_t stream) {
     const int items = n_tokens * (n_heads / maps);
-    if (maps == 2)
+    if (maps == 2 && n_splits == 1 && dv % 2 == 0)
+        attention_difference_one_kernel<T><<<(items + 7) / 8, 256, 0, stream>>>(partial, ro, (T*)out, n_tokens, n_heads / 2, dv, df);
+    else if (maps == 2)
         attention_difference_kernel<T><<<(items + 3) / 4, 128, 0, stream>>>(partial, ro, (T*)out, n_tokens, n_heads / 2, dv, n_splits, df);
     else
         attention_sink_combine_kernel<T><<<(items + 3) / 4, 128, 0, stream>>>(partial, ro, (T*)out, n_tokens, n_heads, dv, n_splits);

@@ -742,7 +742,7 @@ BLM_API int blm_gated_group_norm(const float* y, long long y_stride, const float
 // [T, C], or (dt_w) formed here from the first `rank` columns of low and dt_w [C, rank]: for single tokens, where a product
 // of its own would be a launch for a few kilobytes.  A block owns (sequence, kSelThreads / kSelLanes channels); kSelLanes lanes
 // share a channel, RN neighbouring states each in registers.  The state is stored as [channel][state].  Three kernels:
-//   selective_scan_kernel   portions, bfloat16 results: chunks of kChunk tokens; four warps walk the tokens and four serve
+//   selective_scan_kernel   portions, bfloat16 results: chunks of kChunk tokens; four warps walk the tokens and eight serve
 //                           them (rows through cp.async, what is made of them, results out), a chunk apart, so that the
 //                           walk waits for nothing but its own arithmetic; a lane leaves its share of a token's sum in
 //                           shared memory, so nothing is shuffled on the way.  The exponentials are exp2 by the special
@@ -758,6 +758,7 @@ struct SelArgs {
     const float* dt_raw; long long dt_stride;
     const void* dt_w; int dt_w_bf16, rank;
     const float* dt_bias; const float* A_log; const float* D;
+    const float* rates;      // A log2 e = -exp(A_log) log2 e, for the kernels that take exp2 of it
     const float* z; long long z_stride;
     void* out; long long out_stride; float scale;
     int channels, n_states;
@@ -881,7 +882,13 @@ __device__ __forceinline__ void load_states(float (&v)[RN], const float* p) {
     }
 }
 
-constexpr int kSelBlock = 2 * kSelThreads;      // threads of a block of the portions' kernel: four warps scan, four serve them
+// Threads that serve the four scanning warps of a block.  Measured, one prompt of 2,048 tokens and eight of 512: 4,096
+// channels of 16 states with 128 threads 156 and 194 us, with 256 112 and 163; 8,192 channels 205 and 365, 179 and 314;
+// 4,096 channels of 64 states 455 and 818, 375 and 674.
+#ifndef BLM_SEL_SERVE
+#define BLM_SEL_SERVE 256
+#endif
+constexpr int kSelServe = BLM_SEL_SERVE, kSelBlock = kSelThreads + kSelServe;      // the portions' kernel: four warps scan, the others serve them
 
 template <int RN>
 struct SelSmem {
@@ -923,7 +930,7 @@ __global__ void __launch_bounds__(kSelBlock)
             const bool in = live && n0 + r < a.n_states;
             const size_t at = (size_t)c * a.n_states + n0 + r;
             s[r] = in && sq.read ? sq.read[at] : 0.f;
-            A[r] = in ? -expf(a.A_log[at]) * 1.4426950408889634f : 0.f;
+            A[r] = in ? a.rates[at] : 0.f;
         }
         for (int turn = 0; turn < n_chunks + 2; ++turn) {
             const int k = turn - 1;                     // the chunk this turn walks
@@ -993,7 +1000,7 @@ __global__ void __launch_bounds__(kSelBlock)
         const size_t row0 = (size_t)(sq.first + t0);
         if (rows16) {
             constexpr int V = CH / 4;
-            for (int e = tid; e < nt * V; e += kSelThreads) {
+            for (int e = tid; e < nt * V; e += kSelServe) {
                 const int t = e / V, kk = (e % V) * 4;
                 if (c0 + kk < a.channels) {             // channels is a multiple of 4
                     copy_async<16>(&sm.x[buf][t][kk], a.x + (row0 + t) * a.x_stride + c0 + kk);
@@ -1002,7 +1009,7 @@ __global__ void __launch_bounds__(kSelBlock)
                 }
             }
         } else {
-            for (int t = row_of; t < nt; t += kSelThreads / CH)
+            for (int t = row_of; t < nt; t += kSelServe / CH)
                 if (mine) {
                     copy_async<4>(&sm.x[buf][t][col], a.x + (row0 + t) * a.x_stride + c0 + col);
                     copy_async<4>(&sm.dt[buf][t][col], a.dt_raw + (row0 + t) * a.dt_stride + c0 + col);
@@ -1011,7 +1018,7 @@ __global__ void __launch_bounds__(kSelBlock)
         }
         if (low16) {
             constexpr int V = NP / 4;
-            for (int e = tid; e < nt * V; e += kSelThreads) {
+            for (int e = tid; e < nt * V; e += kSelServe) {
                 const int t = e / V, n = (e % V) * 4;
                 if (n < a.n_states) {                   // n_states is a multiple of 4
                     const float* low = a.low + (row0 + t) * a.low_stride;
@@ -1020,7 +1027,7 @@ __global__ void __launch_bounds__(kSelBlock)
                 }
             }
         } else {
-            for (int e = tid; e < nt * NP; e += kSelThreads) {
+            for (int e = tid; e < nt * NP; e += kSelServe) {
                 const int t = e / NP, n = e % NP;
                 if (n < a.n_states) {
                     const float* low = a.low + (row0 + t) * a.low_stride;
@@ -1032,14 +1039,15 @@ __global__ void __launch_bounds__(kSelBlock)
     };
     fetch(0);
     asm volatile("cp.async.commit_group;\n" ::: "memory");
-    constexpr int kPasses = kChunk * CH / kSelThreads;
+    constexpr int kPasses = kChunk * CH / kSelServe;
+    static_assert(kSelServe % CH == 0 && kChunk * CH % kSelServe == 0, "every serving thread has one column and as many rows");
     for (int turn = 0; turn < n_chunks + 2; ++turn) {
         if (turn >= 2 && mine) {                        // chunk turn - 2 goes out
             const int k = turn - 2, nt = min(kChunk, sq.n_new - k * kChunk);
             __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (size_t)(sq.first + k * kChunk) * a.out_stride + c0 + col;
 #pragma unroll
             for (int i = 0; i < kPasses; ++i) {
-                const int t = row_of + i * (kSelThreads / CH);
+                const int t = row_of + i * (kSelServe / CH);
                 const float4 y = sm.y[k & 1][t][col];
                 const float2 f = sm.after[k & 1][t][col];
                 if (t < nt) out[(size_t)t * a.out_stride] = __float2bfloat16_rn(((y.x + y.y) + (y.z + y.w) + f.x) * f.y);
@@ -1048,13 +1056,13 @@ __global__ void __launch_bounds__(kSelBlock)
         if (turn < n_chunks) {
             asm volatile("cp.async.wait_group 0;\n" ::: "memory");
             // every serving thread's copies have landed when all of them have waited
-            asm volatile("bar.sync 1, %0;\n" ::"n"(kSelThreads) : "memory");
+            asm volatile("bar.sync 1, %0;\n" ::"n"(kSelServe) : "memory");
             const int k = turn, nt = min(kChunk, sq.n_new - k * kChunk), buf = k & 1;
             if (turn + 1 < n_chunks) fetch(turn + 1);
             asm volatile("cp.async.commit_group;\n" ::: "memory");
 #pragma unroll
             for (int i = 0; i < kPasses; ++i) {
-                const int t = row_of + i * (kSelThreads / CH);
+                const int t = row_of + i * (kSelServe / CH);
                 const float x = sm.x[buf][t][col], z = sm.z[buf][t][col];
                 const float dt = t < nt ? softplus_r(sm.dt[buf][t][col] + bias) : 0.f;
                 sm.made[buf][t][col] = make_float2(dt, t < nt ? dt * x : 0.f);
@@ -1066,38 +1074,68 @@ __global__ void __launch_bounds__(kSelBlock)
     }
 }
 
+// How many sequences a block of the single tokens' kernel takes (a channel's constants are read once for them).  Measured in a
+// captured graph, 64 sequences, 4,096 and 8,192 channels of 16 states: one sequence 12.4 and 23.0 us, two 12.1 and 21.9, four
+// 13.8 and 25.3; with the step sizes formed inside, 8 sequences: 4.6 and 10.3 us, 5.1 and 8.5, 6.4 and 10.0.
+#ifndef BLM_STEP_SEQS
+#define BLM_STEP_SEQS 2
+#endif
+constexpr int kStepSeqs = BLM_STEP_SEQS;
+
 template <int RN>
 __global__ void __launch_bounds__(kSelThreads)
-    selective_step_kernel(SelArgs a, int vec8, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
+    selective_step_kernel(SelArgs a, int n_seqs, int vec8, int vec4, const int* __restrict__ cu_seqlens, const int* __restrict__ slot_of_seq,
                           const int* __restrict__ start_pos, float* __restrict__ state, long long slot_stride, long long copy_stride,
                           long long state_off) {
-    // vec8: rows of dt_w are bfloat16 and can be read 16 bytes at a time
+    // vec8: rows of dt_w are bfloat16 and can be read 16 bytes at a time; vec4: so can a thread's states, rates, B and C
     extern __shared__ __align__(16) unsigned char sel_raw[];
-    float* lat = reinterpret_cast<float*>(sel_raw);      // [rank]
-    const int seq = blockIdx.x;
-    const ScanSeq sq = scan_seq(seq, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off);
-    if (sq.n_new <= 0) return;
+    float* lat = reinterpret_cast<float*>(sel_raw);      // [kStepSeqs][rank]
+    const int seq0 = blockIdx.x * kStepSeqs, many = min(kStepSeqs, n_seqs - seq0);
     const int tid = threadIdx.x, ch = tid / kSelLanes, g = tid % kSelLanes, n0 = g * RN;
     const int c = min(blockIdx.y * kSelChannels + ch, a.channels - 1);      // (lanes beyond the last channel work on it too and write nothing)
     const bool live = blockIdx.y * kSelChannels + ch < a.channels;
-    const size_t row = (size_t)sq.first;
-    const float* low = a.low + row * a.low_stride;
-    float s[RN], A[RN], b[RN], cc[RN];
+    auto get = [&](float (&v)[RN], const float* p) {     // this thread's states' numbers from a row of n_states
+        if (vec4 && RN % 4 == 0) {
 #pragma unroll
-    for (int r = 0; r < RN; ++r) {
-        const bool in = n0 + r < a.n_states;
-        const size_t at = (size_t)c * a.n_states + n0 + r;
-        s[r] = in && sq.read ? sq.read[at] : 0.f;
-        A[r] = in ? a.A_log[at] : 0.f;
-        b[r] = in ? low[a.b_col0 + n0 + r] : 0.f;
-        cc[r] = in ? low[a.c_col0 + n0 + r] : 0.f;
-    }
-    const float x = a.x[row * a.x_stride + c], z = a.z[row * a.z_stride + c];
-    float raw = a.dt_bias[c];
+            for (int r = 0; r < RN; r += 4) {
+                const float4 q = *reinterpret_cast<const float4*>(p + n0 + r);
+                v[r] = q.x; v[r + 1] = q.y; v[r + 2] = q.z; v[r + 3] = q.w;
+            }
+        } else {
+#pragma unroll
+            for (int r = 0; r < RN; ++r) v[r] = n0 + r < a.n_states ? p[n0 + r] : 0.f;
+        }
+    };
+    float A[RN], s[kStepSeqs][RN], x[kStepSeqs], z[kStepSeqs], raw[kStepSeqs];
+    float* write[kStepSeqs];
+    get(A, a.rates + (size_t)c * a.n_states);
     if (a.dt_w != nullptr) {
-        for (int k = tid; k < a.rank; k += kSelThreads) lat[k] = low[k];
+        for (int k = tid; k < many * a.rank; k += kSelThreads) {
+            const int q = k / a.rank, row = cu_seqlens[seq0 + q];
+            lat[k] = cu_seqlens[seq0 + q + 1] > row ? a.low[(size_t)row * a.low_stride + k % a.rank] : 0.f;
+        }
         __syncthreads();
-        float sum = 0.f;
+    }
+#pragma unroll
+    for (int q = 0; q < kStepSeqs; ++q) {
+        write[q] = nullptr;
+        raw[q] = x[q] = z[q] = 0.f;
+        if (q < many) {
+            const ScanSeq sq = scan_seq(seq0 + q, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride, state_off);
+            if (sq.n_new > 0) {
+                const size_t row = (size_t)sq.first;
+                write[q] = sq.write + (size_t)c * a.n_states;
+                if (sq.read) get(s[q], sq.read + (size_t)c * a.n_states);
+                else
+#pragma unroll
+                    for (int r = 0; r < RN; ++r) s[q][r] = 0.f;
+                x[q] = a.x[row * a.x_stride + c];
+                z[q] = a.z[row * a.z_stride + c];
+                if (a.dt_w == nullptr) raw[q] = a.dt_raw[row * a.dt_stride + c];
+            }
+        }
+    }
+    if (a.dt_w != nullptr) {
         if (vec8) {
             const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.dt_w) + (size_t)c * a.rank;
 #pragma unroll 4
@@ -1107,34 +1145,51 @@ __global__ void __launch_bounds__(kSelThreads)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const float2 f = __bfloat1622float2(p[e]);
-                    sum = fmaf(f.x, lat[k + 2 * e], fmaf(f.y, lat[k + 2 * e + 1], sum));
+#pragma unroll
+                    for (int q = 0; q < kStepSeqs; ++q)
+                        if (q < many) raw[q] = fmaf(f.x, lat[q * a.rank + k + 2 * e], fmaf(f.y, lat[q * a.rank + k + 2 * e + 1], raw[q]));
                 }
             }
-        } else if (a.dt_w_bf16) {
-            const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.dt_w) + (size_t)c * a.rank;
-            for (int k = g; k < a.rank; k += kSelLanes) sum = fmaf(__bfloat162float(w[k]), lat[k], sum);
         } else {
-            const float* w = reinterpret_cast<const float*>(a.dt_w) + (size_t)c * a.rank;
-            for (int k = g; k < a.rank; k += kSelLanes) sum = fmaf(w[k], lat[k], sum);
+            for (int k = g; k < a.rank; k += kSelLanes) {
+                const float w = a.dt_w_bf16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.dt_w)[(size_t)c * a.rank + k])
+                                            : reinterpret_cast<const float*>(a.dt_w)[(size_t)c * a.rank + k];
+#pragma unroll
+                for (int q = 0; q < kStepSeqs; ++q)
+                    if (q < many) raw[q] = fmaf(w, lat[q * a.rank + k], raw[q]);
+            }
         }
-        raw += group_sum<kSelLanes>(sum);
-    } else {
-        raw += a.dt_raw[row * a.dt_stride + c];
-    }
-    const float dt = softplus_r(raw), dx = dt * x;
-    float y = 0.f;
 #pragma unroll
-    for (int r = 0; r < RN; ++r) {
-        const float dec = n0 + r < a.n_states ? ex2_approx(-expf(A[r]) * 1.4426950408889634f * dt) : 0.f;
-        s[r] = fmaf(dec, s[r], dx * b[r]);
-        y = fmaf(s[r], cc[r], y);
+        for (int q = 0; q < kStepSeqs; ++q) raw[q] = group_sum<kSelLanes>(raw[q]);
     }
-    y = group_sum<kSelLanes>(y);
-    if (!live) return;
+    const float bias = a.dt_bias[c], skip = a.D[c];
 #pragma unroll
-    for (int r = 0; r < RN; ++r)
-        if (n0 + r < a.n_states) sq.write[(size_t)c * a.n_states + n0 + r] = s[r];
-    if (g == 0) reinterpret_cast<__nv_bfloat16*>(a.out)[row * a.out_stride + c] = __float2bfloat16_rn(a.scale * (y + a.D[c] * x) * silu_f(z));
+    for (int q = 0; q < kStepSeqs; ++q) {
+        if (q >= many || write[q] == nullptr) continue;      // (the same for the whole block)
+        const size_t row = (size_t)cu_seqlens[seq0 + q];
+        const float* low = a.low + row * a.low_stride;
+        float b[RN], cc[RN];
+        get(b, low + a.b_col0);
+        get(cc, low + a.c_col0);
+        const float dt = softplus_r(raw[q] + bias), dx = dt * x[q];
+        float y = 0.f;
+#pragma unroll
+        for (int r = 0; r < RN; ++r) {
+            s[q][r] = fmaf(ex2_approx(A[r] * dt), s[q][r], dx * b[r]);
+            y = fmaf(s[q][r], cc[r], y);
+        }
+        y = group_sum<kSelLanes>(y);
+        if (!live) continue;
+        if (vec4 && RN % 4 == 0) {
+#pragma unroll
+            for (int r = 0; r < RN; r += 4) *reinterpret_cast<float4*>(write[q] + n0 + r) = make_float4(s[q][r], s[q][r + 1], s[q][r + 2], s[q][r + 3]);
+        } else {
+#pragma unroll
+            for (int r = 0; r < RN; ++r)
+                if (n0 + r < a.n_states) write[q][n0 + r] = s[q][r];
+        }
+        if (g == 0) reinterpret_cast<__nv_bfloat16*>(a.out)[row * a.out_stride + c] = __float2bfloat16_rn(a.scale * (y + skip * x[q]) * silu_f(z[q]));
+    }
 }
 
 static bool aligned16(const void* p, long long stride) { return ((size_t)p & 15) == 0 && stride % 4 == 0; }
@@ -1149,9 +1204,12 @@ static int launch_selective(const SelArgs& a, int exact, int single, int n_seqs,
     }
     if (single) {
         const int vec8 = a.dt_w != nullptr && a.dt_w_bf16 && a.rank % 8 == 0 && ((size_t)a.dt_w & 15) == 0;
-        const size_t smem = a.dt_w != nullptr ? (size_t)a.rank * sizeof(float) : 0;
+        const size_t smem = a.dt_w != nullptr ? (size_t)kStepSeqs * a.rank * sizeof(float) : 0;
         BLM_REQUIRE(smem <= 48 * 1024, "selective_scan: step sizes made of %d numbers", a.rank);
-        selective_step_kernel<RN><<<grid, kSelThreads, smem, stream>>>(a, vec8, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride,
+        const int vec4 = a.n_states == RN * kSelLanes && aligned16(a.low, a.low_stride) && a.b_col0 % 4 == 0 && a.c_col0 % 4 == 0 &&
+                         aligned16(state, slot_stride) && copy_stride % 4 == 0 && state_off % 4 == 0 && ((size_t)a.rates & 15) == 0;
+        const dim3 tiles((n_seqs + kStepSeqs - 1) / kStepSeqs, grid.y);
+        selective_step_kernel<RN><<<tiles, kSelThreads, smem, stream>>>(a, n_seqs, vec8, vec4, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, copy_stride,
                                                                        state_off);
         return blm_check_launch("selective_scan (single tokens)");
     }
@@ -1167,7 +1225,7 @@ static int launch_selective(const SelArgs& a, int exact, int single, int n_seqs,
 
 BLM_API int blm_selective_scan(const float* x, long long x_stride, const float* low, long long low_stride, int b_col0, int c_col0,
                                const float* dt_raw, long long dt_stride, const void* dt_w, int dt_w_dtype, int rank, const float* dt_bias,
-                               const float* A_log, const float* D, const float* z, long long z_stride, void* out, int out_dtype,
+                               const float* A_log, const float* rates, const float* D, const float* z, long long z_stride, void* out, int out_dtype,
                                long long out_stride, float scale, int channels, int n_states, const int* cu_seqlens, const int* slot_of_seq,
                                const int* start_pos, int n_seqs, int single_tokens, float* state, long long slot_stride,
                                long long copy_stride, long long state_off, cudaStream_t stream) {
@@ -1181,9 +1239,10 @@ BLM_API int blm_selective_scan(const float* x, long long x_stride, const float* 
     SelArgs a;
     a.x = x; a.x_stride = x_stride; a.low = low; a.low_stride = low_stride; a.b_col0 = b_col0; a.c_col0 = c_col0;
     a.dt_raw = dt_raw; a.dt_stride = dt_stride; a.dt_w = dt_w; a.dt_w_bf16 = dt_w_dtype == BLM_BF16; a.rank = rank;
-    a.dt_bias = dt_bias; a.A_log = A_log; a.D = D; a.z = z; a.z_stride = z_stride;
+    a.dt_bias = dt_bias; a.A_log = A_log; a.rates = rates; a.D = D; a.z = z; a.z_stride = z_stride;
     a.out = out; a.out_stride = out_stride; a.scale = scale; a.channels = channels; a.n_states = n_states;
     BLM_REQUIRE(out_dtype == BLM_F32 || out_dtype == BLM_BF16, "selective_scan: out dtype %d", out_dtype);
+    BLM_REQUIRE(out_dtype == BLM_F32 || rates != nullptr, "selective_scan: no rates");
 #define BLM_SEL(RN)                                                                                                                      \
     if (n_states <= RN * kSelLanes)                                                                                                      \
         return launch_selective<RN>(a, out_dtype == BLM_F32, single_tokens, n_seqs, cu_seqlens, slot_of_seq, start_pos, state, slot_stride, \

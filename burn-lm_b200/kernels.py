@@ -130,7 +130,7 @@ _protos = {
                            c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_longlong,
                            c_void_p],
         "blm_selective_scan": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int,
-                               c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_float, c_int, c_int,
+                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_float, c_int, c_int,
                                c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p],
         "blm_take_cols": [c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
         "blm_gated_group_norm": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int,
@@ -1361,16 +1361,23 @@ GATE_FIRST, GATE_LAST, GATE_SILU_LAST, GATE_NONE = 0, 1, 2, 3
 SELECTIVE_STATES = 128      # states a channel the selective scan takes at most
 
 
-def selective_scan(x, low, rank, n_state, dt_bias, a_log, d_skip, z, out, step, state, state_offset, dt=None, dt_weight=None, scale=1.0):
+def scan_rates(a_log):
+    """What the selective scan's bfloat16 kernels take the exponent of: A log2 e with A = -exp(a_log)."""
+    return (a_log.to(torch.float64).exp() * -1.4426950408889634).to(torch.float32).contiguous()
+
+
+def selective_scan(x, low, rank, n_state, dt_bias, a_log, d_skip, z, out, step, state, state_offset, dt=None, dt_weight=None, scale=1.0, rates=None):
     """The selective scan per channel c with `n_state` states: S <- exp(dt A) S + dt x B, y = S C + D x, out = scale y silu(z),
     dt = softplus(. + dt_bias), A = -exp(a_log).  x float32 [N, channels]; low float32 [N, rank + 2 n_state] = [dt | B | C];
     the step sizes before bias and softplus are `dt` float32 [N, channels], or dt_weight [channels, rank] times low's first
     columns, formed by the kernel (steps of one token a sequence, and the 32-bit path); z float32 [N, channels], possibly a column range; out [N, channels] bfloat16, or float32 in
     the 32-bit path (sums in float64), possibly a column range.  The state (fp32) lies in `state` at state_offset,
-    [channels, n_state]."""
+    [channels, n_state].  `rates`: scan_rates(a_log), made here when not given."""
     channels = x.shape[1]
-    _need_cuda(x, low, dt, dt_weight, dt_bias, a_log, d_skip, state)
-    _f32(x, low, dt, dt_bias, a_log, d_skip, z)
+    if rates is None and out.dtype == torch.bfloat16:
+        rates = scan_rates(a_log)
+    _need_cuda(x, low, dt, dt_weight, dt_bias, a_log, rates, d_skip, state)
+    _f32(x, low, dt, dt_bias, a_log, rates, d_skip, z)
     n = step.n_tokens
     if n_state > SELECTIVE_STATES:
         raise KernelError(f"selective_scan: {n_state} states a channel; at most {SELECTIVE_STATES}")
@@ -1385,7 +1392,7 @@ def selective_scan(x, low, rank, n_state, dt_bias, a_log, d_skip, z, out, step, 
             raise KernelError("selective_scan: z and out are CUDA tensors [N, C] with unit stride along their rows")
     _call("recurrent", "blm_selective_scan", _ptr(x), c_longlong(x.stride(0)), _ptr(low), c_longlong(low.stride(0)), int(rank),
           int(rank + n_state), _ptr(dt), c_longlong(channels), _ptr(dt_weight), _code(dt_weight.dtype) if dt_weight is not None else F32,
-          int(rank), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), _ptr(z), c_longlong(z.stride(0)), _ptr(out), _code(out.dtype),
+          int(rank), _ptr(dt_bias), _ptr(a_log), _ptr(rates), _ptr(d_skip), _ptr(z), c_longlong(z.stride(0)), _ptr(out), _code(out.dtype),
           c_longlong(out.stride(0)), c_float(scale), channels, int(n_state), _ptr(step.cu_seqlens), _ptr(step.slot_of_seq),
           _ptr(step.start_pos), step.n_seqs, 1 if getattr(step, "max_q_len", 0) == 1 else 0, *_state_args(state, state_offset), _stream())
 

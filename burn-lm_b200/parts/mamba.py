@@ -18,7 +18,8 @@ from ..weights.loader import TensorSpec
 from .base import CacheNeed, Part
 from .linear import Linear
 
-FUSED_STEP_TOKENS = 16     # up to this many tokens the scan's kernel forms the step sizes itself
+FUSED_STEP_TOKENS = 16     # up to this many tokens the scan's kernel forms the step sizes itself,
+FUSED_STEP_RANK = 2048     # from at most so many lanes
 
 
 @dataclass(frozen=True)
@@ -70,6 +71,7 @@ class Mamba(Part):
         self.proj, self.x, self.dt, self.o = (Linear(loaded[t[r]].contiguous()) for r in ("in", "x", "dt", "o"))
         self.taps, self.conv_bias = f32(loaded[t["conv"]]), f32(loaded[t["conv_bias"]])
         self.dt_bias, self.a_log, self.d_skip = f32(loaded[t["dt_bias"]]), f32(loaded[t["A_log"]]), f32(loaded[t["D"]])
+        self.rates = K.scan_rates(self.a_log)
 
     def cache_need(self) -> CacheNeed:
         return CacheNeed("state", state_shape=(2, self.state_floats))
@@ -98,10 +100,10 @@ class Mamba(Part):
         K.causal_conv(proj, 0, s.inner, self.taps, self.conv_bias, x, 0, step, cache.state, cache.state_offset, silu=True, out_bf16=rounded)
         low = self.x(rounded if rounded is not None else x, out_dtype=torch.float32)            # [N, dt | B | C] in fp32
         dt = None
-        if n > FUSED_STEP_TOKENS or step.max_q_len > 1:
+        if n > FUSED_STEP_TOKENS or step.max_q_len > 1 or s.dt_rank > FUSED_STEP_RANK:
             latent = torch.empty((n, s.dt_rank), dtype=self.dt.weight.dtype, device=proj.device)
             K.take_cols(low, 0, latent)
             dt = self.dt(latent, out_dtype=torch.float32)
         K.selective_scan(x, low, s.dt_rank, s.state, self.dt_bias, self.a_log, self.d_skip, proj[:, s.inner: 2 * s.inner], out, step,
                          cache.state, cache.state_offset + self.hist_floats, dt=dt, dt_weight=self.dt.weight if dt is None else None,
-                         scale=scale)
+                         scale=scale, rates=self.rates)
