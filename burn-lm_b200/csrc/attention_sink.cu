@@ -250,6 +250,101 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
     }
 }
 
+// The same without norms for a bfloat16 cache, lanes (i, i + rot_dims / 2), all sizes multiples of 8 (rot_dims of 16): a thread
+// eight pairs of turning lanes, eight lanes that pass, or eight lanes of a value, in 16-byte accesses.
+__global__ void turn_append_vec_kernel(const float* __restrict__ proj, long long proj_stride, int n_heads, int n_kv, int n_v, int dk, int dv,
+                                       const double* __restrict__ freq, int rot_dims, float turn_scale, const float2* __restrict__ table,
+                                       int table_len, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ pool, long long page_elems,
+                                       int page_size, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
+                                       const int* __restrict__ slot_of_seq, const int* __restrict__ block_table, int table_stride) {
+    const int n = blockIdx.x, item = blockIdx.y * blockDim.x + threadIdx.x;
+    const int half = rot_dims >> 1, turns = half >> 3, passes = (dk - rot_dims) >> 3, vecs = dv >> 3, qk = n_heads + n_kv;
+    if (item >= qk * (turns + passes) + n_v * vecs) return;
+    const int seq = token_seq[n];
+    const bool is_v = item >= qk * (turns + passes);
+    int head, d0;                                      // of q and k together, or of v; the first of the eight lanes
+    bool turning = false;
+    if (is_v) {
+        const int j = item - qk * (turns + passes);
+        head = j / vecs;
+        d0 = (j % vecs) * 8;
+    } else if (item < qk * turns) {
+        head = item / turns;
+        d0 = (item % turns) * 8;
+        turning = true;
+    } else {
+        const int j = item - qk * turns;
+        head = j / passes;
+        d0 = rot_dims + (j % passes) * 8;
+    }
+    const bool is_q = !is_v && head < n_heads;
+    if (seq < 0 && !is_q) return;                      // a row of no sequence leaves zeros in q and reaches no cache
+    const int pos = seq >= 0 ? token_pos[n] : 0;
+    __nv_bfloat16* dst;
+    if (is_q) {
+        dst = q_out + ((size_t)n * n_heads + head) * dk + d0;
+    } else {
+        const int page = block_table[(size_t)slot_of_seq[seq] * table_stride + pos / page_size];
+        __nv_bfloat16* base = pool + (size_t)page * page_elems;
+        const int r = pos % page_size;
+        dst = is_v ? base + (size_t)n_kv * page_size * dk + ((size_t)head * page_size + r) * dv + d0
+                   : base + ((size_t)(head - n_heads) * page_size + r) * dk + d0;
+    }
+    const float* src = proj + (size_t)n * proj_stride + (is_v ? (size_t)qk * dk + (size_t)head * dv : (size_t)head * dk) + d0;
+    auto put = [](__nv_bfloat16* to, const float (&v)[8]) {
+        uint4 w;
+        unsigned* p = reinterpret_cast<unsigned*>(&w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const __nv_bfloat162 two = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+            p[e] = *reinterpret_cast<const unsigned*>(&two);
+        }
+        *reinterpret_cast<uint4*>(to) = w;
+    };
+    auto get = [](float (&v)[8], const float* from) {
+        const float4 x = *reinterpret_cast<const float4*>(from), y = *reinterpret_cast<const float4*>(from + 4);
+        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+    };
+    float a[8], b[8];
+    if (seq < 0) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] = 0.f;
+        put(dst, a);
+        if (turning) put(dst + half, a);
+        return;
+    }
+    get(a, src);
+    if (!turning) {
+        put(dst, a);
+        return;
+    }
+    get(b, src + half);
+#pragma unroll
+    for (int e = 0; e < 8; e += 2) {
+        float2 t[2];
+        if (pos < table_len) {
+            const float4 two = *reinterpret_cast<const float4*>(table + (size_t)pos * half + d0 + e);
+            t[0] = make_float2(two.x, two.y);
+            t[1] = make_float2(two.z, two.w);
+        } else {
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                double sn, cs;
+                sincos((double)pos * freq[d0 + e + u], &sn, &cs);
+                t[u] = make_float2(turn_scale * (float)cs, turn_scale * (float)sn);
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const float x = a[e + u], y = b[e + u];
+            a[e + u] = x * t[u].x - y * t[u].y;
+            b[e + u] = y * t[u].x + x * t[u].y;
+        }
+    }
+    put(dst, a);
+    put(dst + half, b);
+}
+
 BLM_API int blm_head_norm_rope_append(const float* proj, long long proj_stride, int n_tokens, int n_heads, int n_kv, int maps, int dk,
                                       int dv, const float* wq, const float* wk, float eps, int value_norm, const double* freq, int rot_dims,
                                       int halves, float turn_scale, const float* table, int table_len, void* q_out, void* pool, int dtype, long long page_elems, int page_size,
@@ -264,6 +359,14 @@ BLM_API int blm_head_norm_rope_append(const float* proj, long long proj_stride, 
     BLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || freq != nullptr),
                 "head_norm_rope_append: %d turning lanes of %d", rot_dims, dk);
     if (table == nullptr) table_len = 0;               // [table_len][rot_dims / 2] (cosine, sine), already times turn_scale
+    if (dtype == BLM_BF16 && wq == nullptr && wk == nullptr && !value_norm && (halves || rot_dims == 0) && dk % 8 == 0 && dv % 8 == 0 &&
+        rot_dims % 16 == 0 && proj_stride % 4 == 0 && (((size_t)proj | (size_t)q_out | (size_t)pool | (size_t)table) & 15) == 0) {
+        const int items = (n_heads + n_kv) * (rot_dims / 16 + (dk - rot_dims) / 8) + n_v * (dv / 8);
+        turn_append_vec_kernel<<<dim3(n_tokens, (items + 127) / 128), 128, 0, stream>>>(
+            proj, proj_stride, n_heads, n_kv, n_v, dk, dv, freq, rot_dims, turn_scale, (const float2*)table, table_len, (__nv_bfloat16*)q_out,
+            (__nv_bfloat16*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride);
+        return blm_check_launch("head_norm_rope_append (no norms)");
+    }
     const int vectors = n_heads + n_kv + n_v;
     const int threads = vectors >= 8 ? 256 : 32 * vectors;
 #define BLM_HNRA(T)                                                                                                              \
