@@ -110,7 +110,7 @@ def test_folders_hold_what_the_plain_implementation_reads(tmp_path):
 
 
 # rotations: the product's constants against the plain ones, and both against what they should do ------------------------
-@pytest.mark.parametrize("dims,base,scaling", [(48, 1e6, (4.0, 2048, 32.0, 1.0)), (24, 500000.0, (8.0, 256, 16.0, 1.0)), (16, 1000.0, (3.0, 64, 8.0, 2.0)),
+@pytest.mark.parametrize("dims,base,scaling", [(56, 2e6, (5.0, 1024, 24.0, 1.0)), (24, 500000.0, (8.0, 256, 16.0, 1.0)), (16, 1000.0, (3.0, 64, 8.0, 2.0)),
                                                (64, 1e4, (40.0, 4096, 32.0, 1.0)), (2, 1e4, (2.0, 100, 4.0, 1.0)), (128, 5e5, (1.0, 512, 1.0, 1.0))])
 def test_frequencies_scaled_by_lanes(dims, base, scaling):
     from burn_lm_b200.parts.position import RotarySpec, YarnScaling, rotary_inverse_frequencies, rotary_multiplier
