@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the Llama-3.2-1B shape with random weights on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 1b|3b|8b]
-    python bench.py --compare fobilorn|nufolix|ridopel|marinex [--size 1b-layers|8b-layers]     (another design beside this one, see run_compare)
+    python bench.py --compare fobilorn|nufolix|ridopel|marinex|tomalix [--size 1b-layers|8b-layers]     (another design beside this one, see run_compare)
 
 A "step" is one decode step of the whole batch.  The default run has the layer sizes of the 1B
 configuration (16 layers, width 2048, 32 heads on 8 kv heads of 64, inner 8192, vocabulary 128256,

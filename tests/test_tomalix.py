@@ -81,8 +81,7 @@ def test_what_the_runs_keep():
     kv, state = needs[1]
     assert (kv.kind, kv.n_kv_heads, kv.head_dim, kv.value_dim, kv.chunk) == ("kv", 2, 24, 40, 80)
     assert state.kind == "state" and state.state_shape == (2, 3 * 128 + 128 * 16)
-    assert sorted(model.kernel_modules()) == ["attention_sink", "elementwise", "gemm", "moe", "recurrent", "stream_ops"] or \
-        sorted(model.kernel_modules()) == ["attention_sink", "elementwise", "moe", "recurrent", "stream_ops"]
+    assert sorted(set(model.kernel_modules()) - {"gemm", "gemm_tc"}) == ["attention_sink", "elementwise", "moe", "recurrent", "stream_ops"]
 
 
 def test_a_chunked_line_gives_back_the_pages_of_the_chunks_before():
