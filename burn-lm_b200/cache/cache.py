@@ -34,7 +34,8 @@ class CacheView:
     writes: bool                            # False: the line belongs to an earlier run; read only
     pool: Optional[torch.Tensor] = None     # kv: [pages, 2, n_kv_heads, PAGE, head_dim]; with values of another size than
                                             # the keys [pages, n_kv_heads * PAGE * (head_dim + value_dim)], a page's keys
-                                            # [n_kv_heads, PAGE, head_dim] followed by its values [n_kv_heads, PAGE, value_dim];
+                                            # [n_kv_heads, PAGE, head_dim] followed by its values [n_kv_heads, PAGE, value_dim]
+                                            # (value_dim 0: the keys alone);
                                             # ids: int32 [pages, PAGE]; rows: [pages, PAGE, head_dim]
     block_table: Optional[torch.Tensor] = None   # kv: int32 [max_seqs, max_pages_per_seq]
     state: Optional[torch.Tensor] = None    # state: [max_seqs, *state_shape]

@@ -210,6 +210,34 @@ _PRESETS["tomalix_tiny"] = {
 }
 
 
+def _samusun_attention(heads, kv_heads, dim, scale, window, q_temp, mlp):
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale, "mask": {"size": window},
+                      "q_temp": dict(zip(("coef", "every"), q_temp))}}
+
+
+def _samusun_retention(heads, dim, vdim, decay, rot_dims, base, mlp):
+    return {"type": "retention", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay, "rot": {"dims": rot_dims, "base": base}}}
+
+
+# a small Samusun decoder that uses every branch of the design: both mixers with dense feed-forwards, experts and none, several
+# query heads a key/value head and one, windows inside a cache page and across page borders, values wider and narrower than the
+# keys of a retention head, some and all of its lanes turning, a loop over layers of both kinds
+_PRESETS["samusun_tiny"] = {
+    "architecture": "Samusun", "vocab": 272, "width": 96, "norm": {"eps": 1e-5}, "embedding": {"scale": 0.75}, "logit_scale": 1.5,
+    "logit_softcap": 20.0, "loop": {"start": 1, "stop": 4, "times": 2},
+    "layers": [
+        _samusun_retention(3, 16, 32, [0.9, 0.97, 0.995], 16, 10000.0, {"kind": "dense", "ff": 160}),
+        _samusun_attention(4, 2, 24, 0.25, 70, (0.2, 24), _tomalix_experts(6, 2, 48)),
+        _samusun_retention(2, 32, 24, [0.95, 0.99], 12, 3000.0, _tomalix_experts(5, 3, 32)),
+        _samusun_attention(6, 6, 16, 0.3, 20, (0.4, 10), {"kind": "dense", "ff": 96}),
+        _samusun_attention(3, 1, 32, 0.2, 150, (0.1, 50), None),
+        _samusun_retention(4, 16, 16, [0.8, 0.9, 0.98, 0.999], 8, 500.0, None),
+    ],
+}
+
+
 def preset_names() -> list:
     return sorted(_PRESETS)
 

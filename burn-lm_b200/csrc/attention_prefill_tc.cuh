@@ -32,7 +32,13 @@
 // values of one size, the dense decoder's use of it.  GEN true, the windowed family's: keys and values of any multiple of 8
 // lanes up to HDK and HDV (the TMA fills the lanes beyond with zeros: three-dimensional maps, lanes by rows by pages), a
 // window or chunks, two maps a head (a query head for each; their sums leave as shares for the kernel that forms the
-// difference), a gate per head or per lane, results scaled and written as columns of wider rows.
+// difference), a gate per head or per lane, results scaled and written as columns of wider rows, values that are the keys (the
+// value map is then the keys' own: a page's tile of keys by lanes is the K-major operand of the scores and the MN-major one of
+// the second product).
+//
+// BIAS (with GEN): slope_h times the distance is taken off a score.  The pages are then walked from the diagonal back: the row's
+// largest score is mostly found in the first pages, where with a bias by distance it would otherwise move in every page, and with
+// it the row of O in tensor memory.
 #pragma once
 #include <cuda.h>
 
@@ -59,6 +65,8 @@ struct AttnPrefillTcArgs {
     long long out_stride;
     float out_scale;
     float* partial;              // null, or where a row's share goes: [N][n_heads][max, sum, dv lanes]
+    const float* slope;          // BIAS: [n_heads]
+    int shared;                  // the values are the keys, and a page holds the keys alone
 };
 
 namespace attn_tc {
@@ -238,7 +246,7 @@ __device__ __forceinline__ void tmem_st32_bits(unsigned taddr, const unsigned (&
 constexpr float kLazy = 8.0f;     // the reference maximum of a row moves only when a block exceeds it by more than 2^kLazy
 }  // namespace attn_tc
 
-template <int HDK, int HDV, bool GEN>
+template <int HDK, int HDV, bool GEN, bool BIAS>
 __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
     attn_prefill_tc_kernel(const AttnPrefillTcArgs a, const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap pool_map,
                            const __grid_constant__ CUtensorMap value_map) {
@@ -285,6 +293,7 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
     };
     const int key_lo = first_key(start + q0);
     const int kb_lo = key_lo / BKV, kb_hi = key_hi / BKV, n_blocks = kb_hi - kb_lo + 1;
+    auto page_at = [&](int step) -> int { return BIAS ? kb_hi - step : kb_lo + step; };      // the page of the sequence a step works on
     const int vh = GEN ? head / a.maps / (a.n_heads / a.n_kv) : 0;
     const int kvh = GEN ? vh * a.maps + head % a.maps : head / (a.n_heads / a.n_kv);
 
@@ -325,13 +334,13 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
                 if (GEN) tma_load_3d(Qs + h * kTile, &qmap, h * 64, head, tok0 + q0, q_full);
                 else tma_load_2d(Qs + h * kTile, &qmap, head * HDK + h * 64, tok0 + q0, q_full);
             }
-            auto row_of = [&](int step) { return ((pages[kb_lo + step] * 2) * a.n_kv + kvh) * 64; };      // the page's keys of this kv head
+            auto row_of = [&](int step) { return ((pages[page_at(step)] * 2) * a.n_kv + kvh) * 64; };      // the page's keys of this kv head
             auto load_keys = [&](int step) -> bool {
                 const int ks = step % kKStages;
                 if (step >= kKStages && !mbar_wait(k_empty + ks, ((step / kKStages) - 1) & 1)) { atomicCAS(a.status, 0, TC_ATTN_FREE); return false; }
                 mbar_expect_tx(k_full + ks, kKBytes);
                 if (GEN) {
-                    const int page = pages[kb_lo + step];
+                    const int page = pages[page_at(step)];
 #pragma unroll
                     for (int h = 0; h < SUB; ++h) tma_load_3d(Ks + ks * kKBytes + h * kPage, &pool_map, h * 64, kvh * 64, page, k_full + ks);
                     return true;
@@ -347,7 +356,7 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
                 if (j >= 2 && !mbar_wait(pv_done + (j - 2) % kSRing, ((j - 2) / kSRing) & 1)) { atomicCAS(a.status, 0, TC_ATTN_FREE); break; }
                 mbar_expect_tx(v_full + b, kVBytes);
                 if (GEN) {
-                    const int page = pages[kb_lo + j];
+                    const int page = pages[page_at(j)];
 #pragma unroll
                     for (int h = 0; h < SUBV; ++h) tma_load_3d(Vs + b * kVBytes + h * kPage, &value_map, h * 64, vh * 64, page, v_full + b);
                 } else {
@@ -416,9 +425,10 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
         // moves when a block's maximum exceeds it by more than 2^kLazy: then the row of O is rescaled in tensor
         // memory (read, multiply, write back).  Otherwise probabilities may exceed one, by at most that factor.
         float m_run = -INFINITY, l_run = 0.f;
+        const float slope = BIAS ? a.slope[head] * 1.4426950408889634f : 0.f;     // in units of log 2, like the scores
         bool ok = true;
         for (int j = 0; j < n_blocks && ok; ++j) {
-            const int key0 = (kb_lo + j) * BKV;
+            const int key0 = page_at(j) * BKV;
             const int b = j & 1, t = j % kSRing;                 // which V stage, which score tile this step has
             if (!mbar_wait(s_full + t, (j / kSRing) & 1)) { if (lane == 0) atomicCAS(a.status, 0, TC_ATTN_S); ok = false; break; }
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
@@ -444,7 +454,7 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
 #pragma unroll
                 for (int i = 0; i < BKV / 2; ++i) packed[i] = 0u;
             } else if (open_block && __all_sync(0xffffffffu, m_run != -INFINITY)) {
-                const float neg_ref = -m_run;
+                const float neg_ref = BIAS ? slope * (float)(key0 - pos) - m_run : -m_run;
                 float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
                 tmem_ld32_issue(taddr, buf[0]);
 #pragma unroll
@@ -454,15 +464,18 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
                         const float s0 = __uint_as_float(buf[c & 1][i]), s1 = __uint_as_float(buf[c & 1][i + 1]);
-                        m4[(i >> 1) & 3] = fmaxf(m4[(i >> 1) & 3], fmaxf(s0, s1));
-                        const float p0 = ex2(fmaf(s0, a.scale_log2e, neg_ref)), p1 = ex2(fmaf(s1, a.scale_log2e, neg_ref));
+                        // (BIAS: the maximum is of the biased scores, above the reference)
+                        const float x0 = fmaf(s0, a.scale_log2e, BIAS ? fmaf(slope, (float)(c * 32 + i), neg_ref) : neg_ref);
+                        const float x1 = fmaf(s1, a.scale_log2e, BIAS ? fmaf(slope, (float)(c * 32 + i + 1), neg_ref) : neg_ref);
+                        m4[(i >> 1) & 3] = fmaxf(m4[(i >> 1) & 3], BIAS ? fmaxf(x0, x1) : fmaxf(s0, s1));
+                        const float p0 = ex2(x0), p1 = ex2(x1);
                         rs4[(i >> 1) & 3] += p0 + p1;
                         const __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
                         packed[c * 16 + (i >> 1)] = *reinterpret_cast<const unsigned*>(&pk);
                     }
                 }
-                const float m_one = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * a.scale_log2e;
-                done = !__any_sync(0xffffffffu, m_one > m_run + kLazy);
+                const float m_one = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+                done = !__any_sync(0xffffffffu, BIAS ? m_one > kLazy : m_one * a.scale_log2e > m_run + kLazy);
                 if (!done) { rs4[0] = 0.f; rs4[1] = 0.f; rs4[2] = 0.f; rs4[3] = 0.f; }
             }
             if (!done) {
@@ -476,7 +489,10 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
                     tmem_ld32_issue(taddr + ((c + 1) % (BKV / 32)) * 32, buf[(c + 1) & 1]);
                     float v[32];
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(buf[c & 1][i]);
+                    for (int i = 0; i < 32; ++i) {
+                        v[i] = __uint_as_float(buf[c & 1][i]);
+                        if (BIAS) v[i] = fmaf(v[i], a.scale_log2e, slope * (float)(key0 + c * 32 + i - pos));
+                    }
                     if (open_block) {
                         float m4[4] = {v[0], v[1], v[2], v[3]};
 #pragma unroll
@@ -490,7 +506,7 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
                         }
                     }
                 }
-                const float m_blk = mx * a.scale_log2e;
+                const float m_blk = BIAS ? mx : mx * a.scale_log2e;
                 const bool move = m_blk > m_run + kLazy;                     // also the first block that shows the row a key
                 if (__any_sync(0xffffffffu, move)) {
                     const float alpha = move ? (m_run == -INFINITY ? 0.f : ex2(m_run - m_blk)) : 1.0f;
@@ -520,11 +536,14 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
                     if (c + 1 < BKV / 32) tmem_ld32_issue(taddr + (c + 1) * 32, buf[(c + 1) & 1]);
                     float v[32];
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(buf[c & 1][i]);
+                    for (int i = 0; i < 32; ++i) {
+                        const float m_i = BIAS ? fmaf(slope, (float)(key0 + c * 32 + i - pos), neg_m) : neg_m;
+                        v[i] = fmaf(__uint_as_float(buf[c & 1][i]), a.scale_log2e, m_i);
+                    }
                     if (open_block) {
 #pragma unroll
                         for (int i = 0; i < 32; i += 2) {
-                            const float p0 = ex2(fmaf(v[i], a.scale_log2e, neg_m)), p1 = ex2(fmaf(v[i + 1], a.scale_log2e, neg_m));
+                            const float p0 = ex2(v[i]), p1 = ex2(v[i + 1]);
                             rs4[(i >> 1) & 3] += p0 + p1;
                             const __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
                             packed[c * 16 + (i >> 1)] = *reinterpret_cast<const unsigned*>(&pk);
@@ -533,8 +552,8 @@ __global__ void __launch_bounds__(attn_tc::kThreads, attn_tc::blocks_an_sm(HDV))
 #pragma unroll
                         for (int i = 0; i < 32; i += 2) {
                             const int key = key0 + c * 32 + i;
-                            const float p0 = (live && key >= lo && key <= pos) ? ex2(fmaf(v[i], a.scale_log2e, neg_m)) : 0.f;
-                            const float p1 = (live && key + 1 >= lo && key + 1 <= pos) ? ex2(fmaf(v[i + 1], a.scale_log2e, neg_m)) : 0.f;
+                            const float p0 = (live && key >= lo && key <= pos) ? ex2(v[i]) : 0.f;
+                            const float p1 = (live && key + 1 >= lo && key + 1 <= pos) ? ex2(v[i + 1]) : 0.f;
                             rs4[(i >> 1) & 3] += p0 + p1;
                             const __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
                             packed[c * 16 + (i >> 1)] = *reinterpret_cast<const unsigned*>(&pk);
@@ -697,12 +716,12 @@ static bool attn_tc_map(const void* base, long long ld, long long rows, int widt
     return attn_tc_map_nd(base, 2, {(cuuint64_t)width, (cuuint64_t)rows, 1}, {(cuuint64_t)ld * 2, 0}, (cuuint32_t)box_rows, 1, out);
 }
 
-template <int HDK, int HDV, bool GEN>
+template <int HDK, int HDV, bool GEN, bool BIAS = false>
 static int attn_prefill_tc_launch(const AttnPrefillTcArgs& a, const CUtensorMap& qmap, const CUtensorMap& pmap, const CUtensorMap& vmap, dim3 grid,
                                   cudaStream_t stream) {
     const size_t smem = (size_t)(HDK / 64) * 128 * 128 + (size_t)attn_tc::key_stages(HDK, HDV) * (HDK / 64) * 64 * 128 +
                         (size_t)attn_tc::kVStages * (HDV / 64) * 64 * 128 + 24 * 8 + 16 + 1024;
-    auto kernel = attn_prefill_tc_kernel<HDK, HDV, GEN>;
+    auto kernel = attn_prefill_tc_kernel<HDK, HDV, GEN, BIAS>;
     static bool opted_in = false;
     if (!opted_in) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -731,14 +750,14 @@ static int launch_attn_prefill_tc(const AttnPrefillTcArgs& a, const void* q, lon
 }
 #else
 // The windowed family's use of the kernel: whether it takes the sizes, and its launch (BLM_OK, or an error).  q [N, n_heads, dk]
-// contiguous; the pool's pages hold keys [n_kv, 64, dk], then values [n_kv / maps, 64, dv], page_elems in all.
+// contiguous; the pool's pages hold keys [n_kv, 64, dk], then (unless they are the keys) values [n_kv / maps, 64, dv], page_elems in all.
 static bool attn_prefill_tc_general_takes(int dk, int dv) { return dk >= 64 && dk <= 128 && dk % 8 == 0 && dv >= 64 && dv <= 256 && dv % 8 == 0; }
 static int launch_attn_prefill_tc_general(const AttnPrefillTcArgs& a, const void* q, const void* pool, long long page_elems, int n_pages, int dk,
                                           int n_tokens, int n_seqs, int max_q_len, cudaStream_t stream) {
     const dim3 grid(a.n_heads, (max_q_len + attn_tc::BQ - 1) / attn_tc::BQ, n_seqs);
     BLM_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "attention prefill (tcgen05): grid %u x %u too large", grid.y, grid.z);
     const int n_v = a.n_kv / a.maps;
-    const __nv_bfloat16* values = (const __nv_bfloat16*)pool + (size_t)a.n_kv * 64 * dk;
+    const __nv_bfloat16* values = (const __nv_bfloat16*)pool + (a.shared ? 0 : (size_t)a.n_kv * 64 * dk);
     CUtensorMap qmap, kmap, vmap;
     if (!attn_tc_map_nd(q, 3, {(cuuint64_t)dk, (cuuint64_t)a.n_heads, (cuuint64_t)n_tokens}, {(cuuint64_t)dk * 2, (cuuint64_t)a.n_heads * dk * 2}, 1,
                         attn_tc::BQ, &qmap) ||
@@ -747,6 +766,9 @@ static int launch_attn_prefill_tc_general(const AttnPrefillTcArgs& a, const void
         !attn_tc_map_nd(values, 3, {(cuuint64_t)a.dv, (cuuint64_t)n_v * 64, (cuuint64_t)n_pages}, {(cuuint64_t)a.dv * 2, (cuuint64_t)page_elems * 2}, 64,
                         1, &vmap))
         return blm_fail(BLM_CUDA_ERROR, "attention prefill (tcgen05): cuTensorMapEncodeTiled failed");
+    if (a.slope != nullptr)                              // (as many value lanes as key lanes: see the caller)
+        return dk <= 64 ? attn_prefill_tc_launch<64, 64, true, true>(a, qmap, kmap, vmap, grid, stream)
+                        : attn_prefill_tc_launch<128, 128, true, true>(a, qmap, kmap, vmap, grid, stream);
     if (dk <= 64 && a.dv <= 64) return attn_prefill_tc_launch<64, 64, true>(a, qmap, kmap, vmap, grid, stream);
     if (dk <= 64 && a.dv <= 128) return attn_prefill_tc_launch<64, 128, true>(a, qmap, kmap, vmap, grid, stream);
     if (a.dv <= 128) return attn_prefill_tc_launch<128, 128, true>(a, qmap, kmap, vmap, grid, stream);

@@ -6,14 +6,16 @@
 //                                                                             that carries no value; 0: plain softmax)
 //   out[n, h] = gate(n, h) * sum_j p_j v_j,  gate = sigmoid(g[n, h]) or 1
 // Options of the scores (ScoreOpts): a number per query head that multiplies its scores, s_j = scale t_h q.k_j; a cap,
-// s_j <- cap tanh(s_j / cap); and a score z_h of the sink other than 0, p_j = exp(s_j) / (exp(z_h) + sum exp(s_j)).
+// s_j <- cap tanh(s_j / cap); a bias by distance, s_j <- s_j - slope_h (i - j), after the cap; and a score z_h of the sink other
+// than 0, p_j = exp(s_j) / (exp(z_h) + sum exp(s_j)).
 // Instead of a window the mask may be a chunk: visible(i, j) = j <= i and j / chunk == i / chunk (Mask).  The gate may have a
 // number per value lane instead of one per head, and the result may be scaled and written as columns of wider rows (RowOut).
 // Differential attention (maps 2): every head has two queries and every key/value head two keys, [head][map][dk], over one
 // value; the kernels run the 2 n heads on 2 n_kv key heads and leave their sums, and a last kernel forms
 //   o = a_1 - lambda a_2,   out = o / sqrt(mean(o^2) + eps) * c   per head.
 //
-// The cache page of this family holds the keys [n_kv, page, dk] followed by the values [n_kv / maps, page, dv].
+// The cache page of this family holds the keys [n_kv, page, dk] followed by the values [n_kv / maps, page, dv].  Where the
+// values are the keys (`shared`) it holds the keys alone, and the kernels bring a key in once for both of its uses.
 // Scores, softmax and sums are fp32; q, keys and values are read in the cache's dtype.
 #include "common.cuh"
 #define BLM_ATTN_TC_GENERAL
@@ -173,17 +175,29 @@ __device__ __forceinline__ void stage_row<__nv_bfloat16>(float* dst, const __nv_
 //   the first rot_dims lanes of q_h and k_h turn by pos * freq[i]: lanes (2i, 2i + 1) when `halves` is 0, lanes
 //   (i, i + rot_dims / 2) when it is 1, cosine and sine both times `turn_scale`; the other lanes pass;
 //   v_h <- v_h / rms(v_h) when `value_norm` (no weight);
+//   before all that a bias joins (float32, over the columns of q, k and v; null: none), and at the end q is multiplied by
+//   1 + temp_coef ln(floor((pos + 1) / temp_every) + 1) when temp_every > 0; n_v 0: the values are the keys, nothing beside k is kept;
 // q goes to q_out, k and v to the token's place in the paged cache.  rms(x) = sqrt(mean(x^2) + eps).  A warp a head;
 // the angle, its sine and cosine in fp64, everything else fp32.
 // ---------------------------------------------------------------------------------------------
 // `turn`: (cosine, sine) of the token's angle for every pair of turning lanes, worked out once a token (all heads turn alike)
-__device__ __forceinline__ float turned_lane(const float* src, const float* w, float inv, int j, int rot_dims, int halves,
+// What joins the projections and what multiplies q (see above).
+struct PrepareOpts {
+    const float* bias;           // [q | k | v columns] or null
+    float temp_coef;
+    int temp_every;              // 0: q as it is
+    __device__ __forceinline__ float temperature(int pos) const {
+        return temp_every > 0 ? 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1)) : 1.0f;
+    }
+};
+__device__ __forceinline__ float turned_lane(const float* src, const float* bias, const float* w, float inv, int j, int rot_dims, int halves,
                                              const float2* __restrict__ turn) {
-    if (j >= rot_dims) return src[j] * inv * (w ? w[j] : 1.f);
+    if (j >= rot_dims) return (src[j] + (bias ? bias[j] : 0.f)) * inv * (w ? w[j] : 1.f);
     const int half = rot_dims >> 1;
     const int i = halves ? (j < half ? j : j - half) : (j >> 1);
     const int ia = halves ? i : 2 * i, ib = halves ? i + half : 2 * i + 1;
-    const float a = src[ia] * inv * (w ? w[ia] : 1.f), b = src[ib] * inv * (w ? w[ib] : 1.f), cf = turn[i].x, sf = turn[i].y;
+    const float a = (src[ia] + (bias ? bias[ia] : 0.f)) * inv * (w ? w[ia] : 1.f), b = (src[ib] + (bias ? bias[ib] : 0.f)) * inv * (w ? w[ib] : 1.f);
+    const float cf = turn[i].x, sf = turn[i].y;
     return j == ib ? b * cf + a * sf : a * cf - b * sf;
 }
 
@@ -194,7 +208,7 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
                                              const float2* __restrict__ table, int table_len, T* __restrict__ q_out, T* __restrict__ pool, long long page_elems, int page_size,
                                              const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                                              const int* __restrict__ slot_of_seq, const int* __restrict__ block_table,
-                                             int table_stride) {
+                                             int table_stride, PrepareOpts po) {
     extern __shared__ float2 turn[];                   // [rot_dims / 2]
     const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
     const float* p = proj + (size_t)n * proj_stride;
@@ -225,27 +239,33 @@ __global__ void head_norm_rope_append_kernel(const float* __restrict__ proj, lon
         const bool is_q = item < n_heads, is_k = !is_q && item < n_heads + n_kv;
         const int head = is_q ? item : (is_k ? item - n_heads : item - n_heads - n_kv);
         const int width = (is_q || is_k) ? dk : dv;
-        const float* src = p + (is_q ? (size_t)head * dk : (is_k ? (size_t)n_heads * dk + (size_t)head * dk
-                                                                  : (size_t)(n_heads + n_kv) * dk + (size_t)head * dv));
+        const size_t col = is_q ? (size_t)head * dk : (is_k ? (size_t)n_heads * dk + (size_t)head * dk
+                                                            : (size_t)(n_heads + n_kv) * dk + (size_t)head * dv);
+        const float* src = p + col;
+        const float* bias = po.bias ? po.bias + col : nullptr;
         const float* w = is_q ? wq : (is_k ? wk : nullptr);
         float inv = 1.f;
         if (w != nullptr || (!is_q && !is_k && value_norm)) {
             float ss = 0.f;
-            for (int d = lane; d < width; d += 32) ss += src[d] * src[d];
+            for (int d = lane; d < width; d += 32) {
+                const float v = src[d] + (bias ? bias[d] : 0.f);
+                ss += v * v;
+            }
             ss = warp_sum(ss);
             inv = 1.0f / sqrtf(ss / (float)width + eps);
         }
         if (is_q) {
             T* dst = q_out + ((size_t)n * n_heads + head) * dk;
-            for (int d = lane; d < dk; d += 32) dst[d] = from_f32<T>(real ? turned_lane(src, w, inv, d, rot_dims, halves, turn) : 0.f);
+            const float temp = po.temperature(pos);
+            for (int d = lane; d < dk; d += 32) dst[d] = from_f32<T>(real ? turned_lane(src, bias, w, inv, d, rot_dims, halves, turn) * temp : 0.f);
         } else if (is_k) {
             if (!real) continue;
             T* dst = kpage + ((size_t)head * page_size + r) * dk;
-            for (int d = lane; d < dk; d += 32) dst[d] = from_f32<T>(turned_lane(src, w, inv, d, rot_dims, halves, turn));
+            for (int d = lane; d < dk; d += 32) dst[d] = from_f32<T>(turned_lane(src, bias, w, inv, d, rot_dims, halves, turn));
         } else {
             if (!real) continue;
             T* dst = vpage + ((size_t)head * page_size + r) * dv;
-            for (int d = lane; d < dv; d += 32) dst[d] = from_f32<T>(src[d] * inv);
+            for (int d = lane; d < dv; d += 32) dst[d] = from_f32<T>((src[d] + (bias ? bias[d] : 0.f)) * inv);
         }
     }
 }
@@ -256,7 +276,7 @@ __global__ void turn_append_vec_kernel(const float* __restrict__ proj, long long
                                        const double* __restrict__ freq, int rot_dims, float turn_scale, const float2* __restrict__ table,
                                        int table_len, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ pool, long long page_elems,
                                        int page_size, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
-                                       const int* __restrict__ slot_of_seq, const int* __restrict__ block_table, int table_stride) {
+                                       const int* __restrict__ slot_of_seq, const int* __restrict__ block_table, int table_stride, PrepareOpts po) {
     const int n = blockIdx.x, item = blockIdx.y * blockDim.x + threadIdx.x;
     const int half = rot_dims >> 1, turns = half >> 3, passes = (dk - rot_dims) >> 3, vecs = dv >> 3, qk = n_heads + n_kv;
     if (item >= qk * (turns + passes) + n_v * vecs) return;
@@ -290,7 +310,9 @@ __global__ void turn_append_vec_kernel(const float* __restrict__ proj, long long
         dst = is_v ? base + (size_t)n_kv * page_size * dk + ((size_t)head * page_size + r) * dv + d0
                    : base + ((size_t)(head - n_heads) * page_size + r) * dk + d0;
     }
-    const float* src = proj + (size_t)n * proj_stride + (is_v ? (size_t)qk * dk + (size_t)head * dv : (size_t)head * dk) + d0;
+    const size_t col = (is_v ? (size_t)qk * dk + (size_t)head * dv : (size_t)head * dk) + d0;
+    const float* src = proj + (size_t)n * proj_stride + col;
+    const float temp = is_q ? po.temperature(pos) : 1.0f;
     auto put = [](__nv_bfloat16* to, const float (&v)[8]) {
         uint4 w;
         unsigned* p = reinterpret_cast<unsigned*>(&w);
@@ -301,9 +323,22 @@ __global__ void turn_append_vec_kernel(const float* __restrict__ proj, long long
         }
         *reinterpret_cast<uint4*>(to) = w;
     };
-    auto get = [](float (&v)[8], const float* from) {
-        const float4 x = *reinterpret_cast<const float4*>(from), y = *reinterpret_cast<const float4*>(from + 4);
-        v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+    auto get = [&](float (&v)[8], int off) {
+        auto four = [](float* to, const float* from, bool add) {
+            const float4 x = *reinterpret_cast<const float4*>(from);
+            to[0] = add ? to[0] + x.x : x.x; to[1] = add ? to[1] + x.y : x.y;
+            to[2] = add ? to[2] + x.z : x.z; to[3] = add ? to[3] + x.w : x.w;
+        };
+        four(v, src + off, false);
+        four(v + 4, src + off + 4, false);
+        if (po.bias) {
+            four(v, po.bias + col + off, true);
+            four(v + 4, po.bias + col + off + 4, true);
+        }
+        if (is_q) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] *= temp;
+        }
     };
     float a[8], b[8];
     if (seq < 0) {
@@ -313,12 +348,12 @@ __global__ void turn_append_vec_kernel(const float* __restrict__ proj, long long
         if (turning) put(dst + half, a);
         return;
     }
-    get(a, src);
+    get(a, 0);
     if (!turning) {
         put(dst, a);
         return;
     }
-    get(b, src + half);
+    get(b, half);
 #pragma unroll
     for (int e = 0; e < 8; e += 2) {
         float2 t[2];
@@ -349,29 +384,31 @@ BLM_API int blm_head_norm_rope_append(const float* proj, long long proj_stride, 
                                       int dv, const float* wq, const float* wk, float eps, int value_norm, const double* freq, int rot_dims,
                                       int halves, float turn_scale, const float* table, int table_len, void* q_out, void* pool, int dtype, long long page_elems, int page_size,
                                       const int* token_seq, const int* token_pos, const int* slot_of_seq, const int* block_table,
-                                      int table_stride, cudaStream_t stream) {
+                                      int table_stride, const float* bias, float temp_coef, int temp_every, int shared, cudaStream_t stream) {
     if (n_tokens == 0) return BLM_OK;
-    BLM_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv > 0 && dk > 0 && dv > 0 && page_size > 0, "head_norm_rope_append: bad sizes");
+    BLM_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv > 0 && dk > 0 && dv > 0 && page_size > 0 && temp_every >= 0, "head_norm_rope_append: bad sizes");
+    BLM_REQUIRE(!shared || (maps == 1 && dk == dv && !value_norm), "head_norm_rope_append: values that are the keys: %d maps, %d and %d lanes", maps, dk, dv);
+    const PrepareOpts po{bias, temp_coef, temp_every};
     BLM_REQUIRE(maps >= 1 && n_kv % maps == 0, "head_norm_rope_append: %d maps of %d key heads", maps, n_kv);
-    const int n_v = n_kv / maps;                       // n_heads and n_kv count every map
+    const int n_v = shared ? 0 : n_kv / maps;          // n_heads and n_kv count every map
     BLM_REQUIRE(page_elems == (long long)page_size * ((long long)n_kv * dk + (long long)n_v * dv),
                 "head_norm_rope_append: a page holds page * (n_kv * dk + n_kv / maps * dv) elements");
     BLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || freq != nullptr),
                 "head_norm_rope_append: %d turning lanes of %d", rot_dims, dk);
     if (table == nullptr) table_len = 0;               // [table_len][rot_dims / 2] (cosine, sine), already times turn_scale
     if (dtype == BLM_BF16 && wq == nullptr && wk == nullptr && !value_norm && (halves || rot_dims == 0) && dk % 8 == 0 && dv % 8 == 0 &&
-        rot_dims % 16 == 0 && proj_stride % 4 == 0 && (((size_t)proj | (size_t)q_out | (size_t)pool | (size_t)table) & 15) == 0) {
+        rot_dims % 16 == 0 && proj_stride % 4 == 0 && (((size_t)proj | (size_t)q_out | (size_t)pool | (size_t)table | (size_t)bias) & 15) == 0) {
         const int items = (n_heads + n_kv) * (rot_dims / 16 + (dk - rot_dims) / 8) + n_v * (dv / 8);
         turn_append_vec_kernel<<<dim3(n_tokens, (items + 127) / 128), 128, 0, stream>>>(
             proj, proj_stride, n_heads, n_kv, n_v, dk, dv, freq, rot_dims, turn_scale, (const float2*)table, table_len, (__nv_bfloat16*)q_out,
-            (__nv_bfloat16*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride);
+            (__nv_bfloat16*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride, po);
         return blm_check_launch("head_norm_rope_append (no norms)");
     }
     const int vectors = n_heads + n_kv + n_v;
     const int threads = vectors >= 8 ? 256 : 32 * vectors;
 #define BLM_HNRA(T)                                                                                                              \
     head_norm_rope_append_kernel<T><<<n_tokens, threads, (size_t)(rot_dims / 2 + 1) * sizeof(float2), stream>>>(proj, proj_stride, n_heads, n_kv, n_v, dk, dv, wq, wk, eps, value_norm, \
-        freq, rot_dims, halves, turn_scale, (const float2*)table, table_len, (T*)q_out, (T*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride)
+        freq, rot_dims, halves, turn_scale, (const float2*)table, table_len, (T*)q_out, (T*)pool, page_elems, page_size, token_seq, token_pos, slot_of_seq, block_table, table_stride, po)
     if (dtype == BLM_F32) BLM_HNRA(float);
     else if (dtype == BLM_BF16) BLM_HNRA(__nv_bfloat16);
     else return blm_fail(BLM_BAD_ARGUMENT, "head_norm_rope_append: dtype %d", dtype);
@@ -384,6 +421,7 @@ struct ScoreOpts {
     const float* head_scale;     // [n_heads]: multiplies the head's scores beside `scale`
     const float* sink_logit;     // [n_heads]: the sink's score (null: 0); read only when the softmax has a sink
     float cap;                   // > 0: s <- cap tanh(s / cap)
+    const float* slope;          // [n_heads]: slope * (query's position - key's position) is taken off the score (null: nothing is)
 };
 __device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 // The same for the tensor-core kernels, whose operands are bfloat16: tanh(x) = (1 - e) / (1 + e), e = exp(-2 |x|), by the
@@ -401,15 +439,16 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
                                            const int* __restrict__ block_table, int table_stride, const int* __restrict__ token_seq,
                                            const int* __restrict__ token_pos, const int* __restrict__ slot_of_seq,
                                            RowOut ro, T* __restrict__ out, float* __restrict__ partial, int n_heads, int n_kv, int maps,
-                                           int dk, int dv, int page_size, Mask mask, int keep_first, float scale, int sink, ScoreOpts so) {
+                                           int dk, int dv, int page_size, Mask mask, int keep_first, float scale, int sink, ScoreOpts so, int shared) {
     extern __shared__ float smem[];
     const int n = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z, n_splits = gridDim.z;
     const int group = n_heads / n_kv;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
     const int kstride = dk + 1;                        // odd row length: the lanes of a warp read one column of 32 rows
     float* ks = smem;                                  // [kChunk][dk + 1]
-    float* vs = ks + kChunk * kstride;                 // [kChunk][dv]
-    float* qs = vs + kChunk * dv;                      // [n_warps][dk]
+    float* vs = shared ? ks : ks + kChunk * kstride;   // [kChunk][dv]; the keys themselves where they are the values
+    float* qs = ks + kChunk * (kstride + (shared ? 0 : dv));      // [n_warps][dk]
+    const int vrow = shared ? kstride : dv;
     const int seq = token_seq[n];
     T* orow = out + (size_t)n * ro.stride;
     const int vh = kvh / maps;
@@ -441,7 +480,7 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
         __syncthreads();                               // the chunk buffers and qs of the heads before are done with
         if (active)
             for (int d = lane; d < dk; d += 32) qs[warp * dk + d] = to_f32(q[((size_t)n * n_heads + head) * dk + d]);
-        const float pre = scale * (active && so.head_scale ? so.head_scale[head] : 1.f);
+        const float pre = scale * (active && so.head_scale ? so.head_scale[head] : 1.f), slope = active && so.slope ? so.slope[head] : 0.f;
         float m = with_sink ? (active && so.sink_logit ? so.sink_logit[head] : 0.f) : -INFINITY, l = with_sink ? 1.f : 0.f;
         float acc[kMaxVRegs];
 #pragma unroll
@@ -456,7 +495,7 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
                     stage_row<T>(ks + row * kstride, kpage + ((size_t)kvh * page_size + j % page_size) * dk, d, kvec);
                 }
             }
-            for (int idx = threadIdx.x; idx < kChunk * (dv / vstep); idx += blockDim.x) {
+            for (int idx = threadIdx.x; !shared && idx < kChunk * (dv / vstep); idx += blockDim.x) {
                 const int row = idx / (dv / vstep), d = (idx % (dv / vstep)) * vstep, i = c0 + row;
                 if (i < c_end) {
                     const int j = i < n_first ? i : lo + (i - n_first);
@@ -473,7 +512,8 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
                     const float* kr = ks + lane * kstride;
                     const float* qr = qs + warp * dk;
                     for (int d = 0; d < dk; ++d) dot = fmaf(qr[d], kr[d], dot);
-                    s = capped(dot * pre, so.cap);
+                    const int i = c0 + lane, j = i < n_first ? i : lo + (i - n_first);
+                    s = capped(dot * pre, so.cap) - slope * (float)(pos - j);
                 }
                 const float m_new = fmaxf(m, warp_max(s));      // finite: the chunk has a key
                 const float p = mine ? expf(s - m_new) : 0.f;
@@ -488,7 +528,7 @@ __global__ void attention_sink_rows_kernel(const T* __restrict__ q, const T* __r
 #pragma unroll
                     for (int i = 0; i < kMaxVRegs; ++i) {
                         const int d = lane + 32 * i;
-                        if (d < dv) acc[i] = fmaf(pj, vs[j * dv + d], acc[i]);
+                        if (d < dv) acc[i] = fmaf(pj, vs[j * vrow + d], acc[i]);
                     }
                 }
             }
@@ -643,10 +683,10 @@ template <typename T>
 static int launch_rows(const void* q, const void* pool, long long page_elems, const int* block_table, int table_stride,
                        const int* token_seq, const int* token_pos, const int* slot_of_seq, RowOut ro, void* out, float* partial,
                        int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, int page_size, Mask mask,
-                       int keep_first, float scale, int sink, ScoreOpts so, DiffOpts df, cudaStream_t stream) {
+                       int keep_first, float scale, int sink, ScoreOpts so, int shared, DiffOpts df, cudaStream_t stream) {
     const int group = n_heads / n_kv;
     const int warps = group < 8 ? group : 8;
-    const size_t smem = ((size_t)kChunk * (dk + 1) + (size_t)kChunk * dv + (size_t)warps * dk) * sizeof(float);
+    const size_t smem = ((size_t)kChunk * (dk + 1) + (shared ? 0 : (size_t)kChunk * dv) + (size_t)warps * dk) * sizeof(float);
     if (smem > 48 * 1024) {
         BLM_REQUIRE(smem <= 200 * 1024, "attention_sink: heads of %d and %d lanes need %zu bytes of shared memory", dk, dv, smem);
         cudaError_t e = cudaFuncSetAttribute(attention_sink_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -654,7 +694,7 @@ static int launch_rows(const void* q, const void* pool, long long page_elems, co
     }
     attention_sink_rows_kernel<T><<<dim3(n_tokens, n_kv, n_splits), warps * 32, smem, stream>>>(
         (const T*)q, (const T*)pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro,
-        (T*)out, partial, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink, so);
+        (T*)out, partial, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink, so, shared);
     if (partial != nullptr) finish_shares<T>(partial, ro, out, n_tokens, n_heads, maps, dv, n_splits, df, stream);
     return blm_check_launch("attention_sink");
 }
@@ -748,14 +788,16 @@ struct GroupWalk {
 };
 
 // one page's keys and values of one kv head into a buffer pair (every thread of the block takes its share)
+template <bool SHARED>
 __device__ __forceinline__ void stage_page(__nv_bfloat16* kbuf, __nv_bfloat16* vbuf, const __nv_bfloat16* page, int n_kv, int kvh, int vh,
                                            int dk, int dv, int qstride, int vstride, int first_pos, int p_last, const GroupWalk& kw,
                                            const GroupWalk& vw, int key_rows = kTileK) {
-    // key_rows: 2 kTileK brings the keys of the next key head as well (they lie behind these)
+    // key_rows: 2 kTileK brings the keys of the next key head as well (they lie behind these).  SHARED: the keys are the values,
+    // so keys beyond the last query become zeros as well
     const __nv_bfloat16* kpage = page + (size_t)kvh * kTileK * dk;
     const __nv_bfloat16* vpage = page + (size_t)n_kv * kTileK * dk + (size_t)vh * kTileK * dv;
     for (int r = kw.r, c = kw.c; r < key_rows;) {
-        cp_async16(kbuf + r * qstride + c * 8, kpage + r * dk + c * 8, true);
+        cp_async16(kbuf + r * qstride + c * 8, kpage + r * dk + c * 8, !SHARED || first_pos + r <= p_last);
         r += kw.dr;
         c += kw.dc;
         if (c >= kw.vec) {
@@ -763,7 +805,7 @@ __device__ __forceinline__ void stage_page(__nv_bfloat16* kbuf, __nv_bfloat16* v
             ++r;
         }
     }
-    for (int r = vw.r, c = vw.c; r < kTileK;) {
+    for (int r = SHARED ? kTileK : vw.r, c = vw.c; r < kTileK;) {
         cp_async16(vbuf + r * vstride + c * 8, vpage + r * dv + c * 8, first_pos + r <= p_last);
         r += vw.dr;
         c += vw.dc;
@@ -774,7 +816,7 @@ __device__ __forceinline__ void stage_page(__nv_bfloat16* kbuf, __nv_bfloat16* v
     }
 }
 
-template <int NV, int HB>
+template <int NV, int HB, bool SHARED>
 __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool, long long page_elems,
     const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ start_pos,
@@ -785,11 +827,11 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     __shared__ int found[3];
     const int tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, hb = tid >> 7;     // hb: which of the block's heads
     const int dkp = (dk + 15) & ~15;                   // the reduction runs in steps of 16 lanes; the rest is zeros
-    const int qstride = dkp + 8;                       // rows 16 bytes apart modulo 128: ldmatrix reads eight of them at once
     constexpr int vstride = 8 * NV + 8;
+    const int qstride = SHARED ? vstride : dkp + 8;    // rows 16 bytes apart modulo 128: ldmatrix reads eight of them at once
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [HB][64][qstride]
     __nv_bfloat16* Kb = Qs + HB * kTileQ * qstride;                      // kPromptStages x [64][qstride]
-    __nv_bfloat16* Vb = Kb + kPromptStages * kTileK * qstride;           // kPromptStages x [64][vstride]
+    __nv_bfloat16* Vb = SHARED ? Kb : Kb + kPromptStages * kTileK * qstride;      // kPromptStages x [64][vstride]
     const int head = blockIdx.y * HB + hb;             // the block's heads share a kv head (HB divides the group)
     if (tid == 0) {
         int t = blockIdx.x;
@@ -829,7 +871,7 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
 #pragma unroll
     for (int i = 0; i < HB; ++i) zero_unwritten(Qs + i * kTileQ * qstride, kTileQ, qstride, rows, dk);
     zero_unwritten(Kb, kPromptStages * kTileK, qstride, kPromptStages * kTileK, dk);
-    zero_unwritten(Vb, kPromptStages * kTileK, vstride, kPromptStages * kTileK, dv);
+    if (!SHARED) zero_unwritten(Vb, kPromptStages * kTileK, vstride, kPromptStages * kTileK, dv);
     const PageWalk walk(mask.first(p0), p_last, keep_first);
     for (int idx = tid & 127; idx < rows * (dk / 8); idx += 128) {       // every group of four warps brings its head's queries
         const int r = idx / (dk / 8), c = (idx % (dk / 8)) * 8;
@@ -838,7 +880,7 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     const GroupWalk kw(dk / 8), vw(dv / 8);
     auto fetch = [&](int it) {                         // page `it` of the walk into its place in the ring
         const int pg = walk.page(it), b = it % kPromptStages;
-        stage_page(Kb + b * kTileK * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
+        stage_page<SHARED>(Kb + b * kTileK * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
                    vstride, pg * kTileK, p_last, kw, vw);
     };
 #pragma unroll
@@ -853,7 +895,8 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     // scores in units of log 2: the exponentials are exp2.  A cap (or a head's multiplier that is not positive, under which
     // the largest raw score is not the largest score) is applied to the raw scores first, which are then in natural units.
     const float pre = scale * (so.head_scale ? so.head_scale[head] : 1.f);
-    const bool shaped = so.cap > 0.f || !(pre > 0.f);
+    const float slope = so.slope ? so.slope[head] : 0.f;
+    const bool shaped = so.cap > 0.f || so.slope != nullptr || !(pre > 0.f);
     const float scale2 = (shaped ? 1.f : pre) * 1.4426950408889634f;
     const float inv_cap = so.cap > 0.f ? 1.0f / so.cap : 0.f;
     float m[2], l[2], o[NV][4];
@@ -890,7 +933,8 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
 #pragma unroll
             for (int j = 0; j < 8; ++j)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) s[j][e] = capped_fast(s[j][e] * pre, so.cap, inv_cap);
+                for (int e = 0; e < 4; ++e)
+                    s[j][e] = capped_fast(s[j][e] * pre, so.cap, inv_cap) - slope * (float)((e < 2 ? pr0 : pr1) - (pg * kTileK + 8 * j + pair + (e & 1)));
         }
         float mx0 = -INFINITY, mx1 = -INFINITY;
         // every row of this warp sees every key of the page when the page lies behind the warp's first row and inside
@@ -1005,20 +1049,21 @@ __global__ void __launch_bounds__(128 * HB) attention_sink_prompt_kernel(
     }
 }
 
-template <int NV, int HB>
+template <int NV, int HB, bool SHARED>
 static int launch_prompt(const void* q, const void* pool, long long page_elems, const int* block_table, int table_stride,
                          const int* cu_seqlens, const int* start_pos, const int* slot_of_seq, int n_seqs, RowOut ro, void* out,
                          float* partial, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, Mask mask, int keep_first,
                          float scale, int sink, ScoreOpts so, DiffOpts df, cudaStream_t stream) {
     const int dkp = (dk + 15) & ~15;
-    const size_t smem = ((size_t)(HB + kPromptStages) * kTileQ * (dkp + 8) + (size_t)kPromptStages * kTileK * (8 * NV + 8)) * sizeof(__nv_bfloat16);
+    const size_t smem = (SHARED ? (size_t)(HB + kPromptStages) * kTileQ * (8 * NV + 8)
+                                : (size_t)(HB + kPromptStages) * kTileQ * (dkp + 8) + (size_t)kPromptStages * kTileK * (8 * NV + 8)) * sizeof(__nv_bfloat16);
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(attention_sink_prompt_kernel<NV, HB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_sink_prompt_kernel<NV, HB, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "attention_sink: %s", cudaGetErrorString(e));
     }
-    cudaFuncSetAttribute(attention_sink_prompt_kernel<NV, HB>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    cudaFuncSetAttribute(attention_sink_prompt_kernel<NV, HB, SHARED>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
     const unsigned tiles = (unsigned)((n_tokens + kTileQ - 1) / kTileQ + n_seqs);     // every sequence may end in a tile that is not full
-    attention_sink_prompt_kernel<NV, HB><<<dim3(tiles, n_heads / HB), 128 * HB, smem, stream>>>(
+    attention_sink_prompt_kernel<NV, HB, SHARED><<<dim3(tiles, n_heads / HB), 128 * HB, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq,
         n_seqs, n_tokens, ro, (__nv_bfloat16*)out, partial, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so);
     if (partial != nullptr) finish_shares<__nv_bfloat16>(partial, ro, out, n_tokens, n_heads, maps, dv, 1, df, stream);
@@ -1035,7 +1080,7 @@ static int launch_prompt(const void* q, const void* pool, long long page_elems, 
 // of a page lie in shared memory and the products with either give all sixteen rows, of which each keeps its own eight.
 // Without splits the block also forms the difference (DiffOpts) itself.
 
-template <int NV, int kDecodeStages, bool PAIR>
+template <int NV, int kDecodeStages, bool PAIR, bool SHARED>
 __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pool, long long page_elems,
     const int* __restrict__ block_table, int table_stride, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
@@ -1046,12 +1091,12 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     const int n = blockIdx.x, kvh = PAIR ? 2 * blockIdx.y : blockIdx.y, split = blockIdx.z, n_splits = gridDim.z;
     const int group = n_heads / n_kv;                  // <= 16: the rows of the tile
     const int dkp = (dk + 15) & ~15;
-    const int qstride = dkp + 8;
     constexpr int vstride = 8 * NV + 8;
+    const int qstride = SHARED ? vstride : dkp + 8;
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [16][qstride]
     constexpr int kKeyRows = PAIR ? 2 * kTileK : kTileK;
     __nv_bfloat16* Kb = Qs + 16 * qstride;                               // kDecodeStages x [kKeyRows][qstride]
-    __nv_bfloat16* Vb = Kb + kDecodeStages * kKeyRows * qstride;         // kDecodeStages x [64][vstride]
+    __nv_bfloat16* Vb = SHARED ? Kb : Kb + kDecodeStages * kKeyRows * qstride;    // kDecodeStages x [64][vstride]
     const int seq = token_seq[n];
     const int vh = kvh / maps, head0 = vh * group * maps + kvh % maps;      // this key head's query heads: head0, head0 + maps, ...
     // rows of the tile that stand for a query, and its head (every map counted)
@@ -1074,7 +1119,7 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
         if (!row_used(r) || c >= dk) *reinterpret_cast<uint4*>(Qs + r * qstride + c) = make_uint4(0u, 0u, 0u, 0u);
     }
     zero_unwritten(Kb, kDecodeStages * kKeyRows, qstride, kDecodeStages * kKeyRows, dk);
-    zero_unwritten(Vb, kDecodeStages * kTileK, vstride, kDecodeStages * kTileK, dv);
+    if (!SHARED) zero_unwritten(Vb, kDecodeStages * kTileK, vstride, kDecodeStages * kTileK, dv);
     const int lo = mask.first(pos);
     const PageWalk walk(lo, pos, keep_first);
     const int per_split = (walk.n_tiles + n_splits - 1) / n_splits;
@@ -1086,7 +1131,7 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     const GroupWalk kw(dk / 8), vw(dv / 8);
     auto fetch = [&](int it) {                         // page `it` of the walk into its place in the ring
         const int pg = walk.page(it), b = (it - it_begin) % kDecodeStages;
-        stage_page(Kb + b * kKeyRows * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
+        stage_page<SHARED>(Kb + b * kKeyRows * qstride, Vb + b * kTileK * vstride, pool + (size_t)pages[pg] * page_elems, n_kv, kvh, vh, dk, dv, qstride,
                    vstride, pg * kTileK, pos, kw, vw, kKeyRows);
     };
 #pragma unroll
@@ -1098,12 +1143,13 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     const int lrow = lane & 7, lmat = lane >> 3;
     const bool with_sink = sink && split == 0 && warp == 0;      // the sink is counted once
     const float log2e = 1.4426950408889634f;                     // scores in units of log 2: the exponentials are exp2
-    float m[2], l[2], o[NV][4], pre[2];
+    float m[2], l[2], o[NV][4], pre[2], slope[2];
     const float inv_cap = so.cap > 0.f ? 1.0f / so.cap : 0.f;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {                       // this thread's two rows are two heads of the group
         const int r = quad + 8 * half;
         pre[half] = scale * (so.head_scale && row_used(r) ? so.head_scale[row_head(r)] : 1.f);
+        slope[half] = so.slope && row_used(r) ? so.slope[row_head(r)] : 0.f;
         m[half] = with_sink ? (so.sink_logit && row_used(r) ? so.sink_logit[row_head(r)] * log2e : 0.f) : -INFINITY;
         l[half] = with_sink ? 0.25f : 0.f;
     }
@@ -1147,7 +1193,7 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
             for (int e = 0; e < 4; ++e) {
                 const int key = pg * kTileK + 16 * warp + 8 * j + pair + (e & 1);
                 const bool sees = key <= pos && (key >= lo || key < keep_first);
-                s[j][e] = sees ? capped_fast(s[j][e] * pre[e >> 1], so.cap, inv_cap) * log2e : -INFINITY;
+                s[j][e] = sees ? (capped_fast(s[j][e] * pre[e >> 1], so.cap, inv_cap) - slope[e >> 1] * (float)(pos - key)) * log2e : -INFINITY;
             }
         float mx0 = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
         float mx1 = fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]));
@@ -1280,21 +1326,23 @@ __global__ void __launch_bounds__(128) attention_sink_decode_kernel(
     }
 }
 
-template <int NV, int kDecodeStages, bool PAIR>
+template <int NV, int kDecodeStages, bool PAIR, bool SHARED>
 static int launch_decode(const void* q, const void* pool, long long page_elems, const int* block_table, int table_stride,
                          const int* token_seq, const int* token_pos, const int* slot_of_seq, RowOut ro, void* out, float* partial,
                          int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, Mask mask, int keep_first,
                          float scale, int sink, ScoreOpts so, DiffOpts df, cudaStream_t stream) {
     const int dkp = (dk + 15) & ~15;
-    size_t smem = ((size_t)16 * (dkp + 8) + (size_t)kDecodeStages * kTileK * ((PAIR ? 2 : 1) * (dkp + 8) + (8 * NV + 8))) * sizeof(__nv_bfloat16);
-    const size_t merge = (size_t)16 * (dkp + 8) * sizeof(__nv_bfloat16) + (size_t)4 * 16 * (8 * NV + 2) * sizeof(float);
+    static_assert(!(PAIR && SHARED), "two maps have values of their own");
+    const int qstride = SHARED ? 8 * NV + 8 : dkp + 8;
+    size_t smem = ((size_t)16 * qstride + (size_t)kDecodeStages * kTileK * ((PAIR ? 2 : 1) * qstride + (SHARED ? 0 : 8 * NV + 8))) * sizeof(__nv_bfloat16);
+    const size_t merge = (size_t)16 * qstride * sizeof(__nv_bfloat16) + (size_t)4 * 16 * (8 * NV + 2) * sizeof(float);
     if (merge > smem) smem = merge;
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages, PAIR, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "attention_sink: %s", cudaGetErrorString(e));
     }
-    cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages, PAIR>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
-    attention_sink_decode_kernel<NV, kDecodeStages, PAIR><<<dim3(n_tokens, PAIR ? n_kv / 2 : n_kv, n_splits), 128, smem, stream>>>(
+    cudaFuncSetAttribute(attention_sink_decode_kernel<NV, kDecodeStages, PAIR, SHARED>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    attention_sink_decode_kernel<NV, kDecodeStages, PAIR, SHARED><<<dim3(n_tokens, PAIR ? n_kv / 2 : n_kv, n_splits), 128, smem, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro,
         (__nv_bfloat16*)out, partial, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df);
     if (partial != nullptr) finish_shares<__nv_bfloat16>(partial, ro, out, n_tokens, n_heads, maps, dv, n_splits, df, stream);
@@ -1310,16 +1358,16 @@ static int launch_decode(const void* q, const void* pool, long long page_elems, 
 #ifndef BLM_PROMPT_HEADS
 #define BLM_PROMPT_HEADS 1
 #endif
-template <int NV, typename... Args>
+template <int NV, bool SHARED, typename... Args>
 static int launch_prompt_heads(int hb, Args... args) {
 #if BLM_PROMPT_HEADS >= 4
-    if (hb == 4) return launch_prompt<NV, 4>(args...);
+    if (hb == 4) return launch_prompt<NV, 4, SHARED>(args...);
 #endif
 #if BLM_PROMPT_HEADS >= 2
-    if (hb >= 2) return launch_prompt<NV, 2>(args...);
+    if (hb >= 2) return launch_prompt<NV, 2, SHARED>(args...);
 #endif
     (void)hb;
-    return launch_prompt<NV, 1>(args...);
+    return launch_prompt<NV, 1, SHARED>(args...);
 }
 
 // Whether a step of this shape runs the prompt kernel (else the row kernel): bfloat16, pages of 64, sizes it takes,
@@ -1348,14 +1396,15 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
                                long long gate_stride, int gate_lanes, void* out, long long out_stride, float out_scale, float* partial,
                                int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, int page_size, int window,
                                int chunk, int keep_first, float scale, int sink, const float* head_scale, const float* sink_logit,
-                               float softcap, float diff_lambda, float diff_scale, float diff_eps, int n_pages, int* status,
+                               float softcap, const float* slope, int shared, float diff_lambda, float diff_scale, float diff_eps, int n_pages, int* status,
                                cudaStream_t stream) {
     // n_pages, status: of the pool, and where a bounded wait that ran out is recorded (for the tcgen05 kernel; 0 and null: not run)
     // maps 2: n_heads and n_kv count every map, and diff_* are the difference's numbers (DiffOpts); partial is then needed
     // chunk > 0: the mask is by chunks and `window` is not looked at; gate_lanes 0: a gate per head, dv: one per lane
-    // head_scale, sink_logit: float32 [n_heads] or null; softcap: 0 for none (see ScoreOpts)
+    // head_scale, sink_logit, slope: float32 [n_heads] or null; softcap: 0 for none (see ScoreOpts)
+    // shared: the values are the keys (dv == dk), and a page holds the keys alone
     if (n_tokens == 0) return BLM_OK;
-    const ScoreOpts so{head_scale, sink_logit, softcap};
+    const ScoreOpts so{head_scale, sink_logit, softcap, slope};
     BLM_REQUIRE(softcap >= 0.f, "attention_sink: a cap of %g", (double)softcap);
     BLM_REQUIRE(n_tokens > 0 && n_heads > 0 && n_kv > 0 && n_heads % n_kv == 0 && dk > 0 && dv > 0 && page_size > 0,
                 "attention_sink: bad sizes");
@@ -1365,8 +1414,9 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
                            blm_attention_sink_prompt_takes(dtype, dk, dv, page_size, max_q_len, n_heads) && out_stride % 2 == 0 && ((size_t)out & 3) == 0;
     const bool inside = !is_prompt && n_splits == 1 && blm_attention_sink_pairs(dtype, dk, dv, page_size, n_heads, n_kv, maps);
     BLM_REQUIRE(maps == 1 || (maps == 2 && n_kv % 2 == 0 && (inside || partial != nullptr)), "attention_sink: %d maps of %d key heads", maps, n_kv);
-    BLM_REQUIRE(page_elems == (long long)page_size * ((long long)n_kv * dk + (long long)(n_kv / maps) * dv),
-                "attention_sink: a page holds page * (n_kv * dk + n_kv / maps * dv) elements");
+    BLM_REQUIRE(!shared || (maps == 1 && dk == dv), "attention_sink: values that are the keys: %d maps, %d and %d lanes", maps, dk, dv);
+    BLM_REQUIRE(page_elems == (long long)page_size * ((long long)n_kv * dk + (shared ? 0 : (long long)(n_kv / maps) * dv)),
+                "attention_sink: a page holds page * (n_kv * dk + n_kv / maps * dv) elements, or page * n_kv * dk where the values are the keys");
     BLM_REQUIRE(gate_lanes == 0 || gate_lanes == dv, "attention_sink: a gate of %d lanes for values of %d", gate_lanes, dv);
     BLM_REQUIRE(out_stride >= (long long)(n_heads / maps) * dv, "attention_sink: output rows of %lld elements", out_stride);
     BLM_REQUIRE(n_kv <= 65535 && n_splits >= 1 && n_splits <= 65535, "attention_sink: %d kv heads, %d splits", n_kv, n_splits);
@@ -1376,21 +1426,22 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
     const RowOut ro{gate, gate_stride, gate_lanes, out_stride, out_scale};
     const DiffOpts df{diff_lambda, diff_scale, diff_eps};
     if (is_prompt && max_q_len >= 64 && status != nullptr && n_pages > 0 && attn_prefill_tc_general_takes(dk, dv) && !sink && softcap == 0.f &&
-        head_scale == nullptr && keep_first == 0 && scale > 0.f && out_stride % 8 == 0 && (((size_t)out | (size_t)q | (size_t)pool) & 15) == 0) {
+        head_scale == nullptr && keep_first == 0 && (scale > 0.f || slope != nullptr) && (slope == nullptr || dk == dv) && out_stride % 8 == 0 && (((size_t)out | (size_t)q | (size_t)pool) & 15) == 0) {
         // long portions without options of the scores: the products on tcgen05, accumulators in tensor memory
         AttnPrefillTcArgs t = {};
         t.block_table = block_table; t.table_stride = table_stride; t.cu_seqlens = cu_seqlens; t.slot_of_seq = slot_of_seq;
         t.start_pos = start_pos; t.out = (__nv_bfloat16*)out; t.n_heads = n_heads; t.n_kv = n_kv; t.window = window < kNoWindow ? window : 0;
         t.scale_log2e = scale * 1.4426950408889634f; t.status = status;
         t.chunk = chunk; t.maps = maps; t.dv = dv; t.gate = gate; t.gate_stride = gate_stride; t.gate_lanes = gate_lanes;
-        t.out_stride = out_stride; t.out_scale = out_scale; t.partial = partial;
+        t.out_stride = out_stride; t.out_scale = out_scale; t.partial = partial; t.slope = slope; t.shared = shared;
         const int rc = launch_attn_prefill_tc_general(t, q, pool, page_elems, n_pages, dk, n_tokens, n_seqs, max_q_len, stream);
         if (rc != BLM_OK) return rc;
         if (partial != nullptr) finish_shares<__nv_bfloat16>(partial, ro, out, n_tokens, n_heads, maps, dv, 1, df, stream);
         return blm_check_launch("attention_sink (tcgen05)");
     }
     if (is_prompt) {
-#define BLM_PROMPT(NV) launch_prompt_heads<NV>(hb, q, pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq, n_seqs, ro, \
+#define BLM_PROMPT(NV) (shared ? BLM_PROMPT_OF(NV, true) : BLM_PROMPT_OF(NV, false))
+#define BLM_PROMPT_OF(NV, SHARED) launch_prompt_heads<NV, SHARED>(hb, q, pool, page_elems, block_table, table_stride, cu_seqlens, start_pos, slot_of_seq, n_seqs, ro, \
                                          out, partial, n_tokens, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df, stream)
         const int group = n_heads / n_kv;
         int hb = maps == 1 && dv <= 128 ? BLM_PROMPT_HEADS : 1;
@@ -1401,30 +1452,38 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
         if (dv <= 192) return BLM_PROMPT(24);
         return BLM_PROMPT(32);
 #undef BLM_PROMPT
+#undef BLM_PROMPT_OF
     }
     if (blm_attention_sink_decode_takes(dtype, dk, dv, page_size, n_heads, n_kv)) {
-#define BLM_DECODE(NV, STAGES, PAIR) launch_decode<NV, STAGES, PAIR>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, \
+#define BLM_DECODE(NV, STAGES, PAIR, SHARED) launch_decode<NV, STAGES, PAIR, SHARED>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, \
                                          out, partial, n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, mask, keep_first, scale, sink, so, df, stream)
         if (blm_attention_sink_pairs(dtype, dk, dv, page_size, n_heads, n_kv, maps)) {
             if (n_splits == 1) partial = nullptr;
-            if (dv <= 64) return BLM_DECODE(8, 2, true);
-            if (dv <= 128) return BLM_DECODE(16, 2, true);
-            if (dv <= 192) return BLM_DECODE(24, 2, true);
-            return BLM_DECODE(32, 2, true);
+            if (dv <= 64) return BLM_DECODE(8, 2, true, false);
+            if (dv <= 128) return BLM_DECODE(16, 2, true, false);
+            if (dv <= 192) return BLM_DECODE(24, 2, true, false);
+            return BLM_DECODE(32, 2, true, false);
         }
-        if (dv <= 32) return BLM_DECODE(4, 2, false);
-        if (dv <= 64) return BLM_DECODE(8, 2, false);
-        if (dv <= 128) return BLM_DECODE(16, 3, false);
-        if (dv <= 192) return BLM_DECODE(24, 2, false);
-        return BLM_DECODE(32, 2, false);
+        if (shared) {
+            if (dv <= 32) return BLM_DECODE(4, 3, false, true);
+            if (dv <= 64) return BLM_DECODE(8, 3, false, true);
+            if (dv <= 128) return BLM_DECODE(16, 3, false, true);
+            if (dv <= 192) return BLM_DECODE(24, 2, false, true);
+            return BLM_DECODE(32, 2, false, true);
+        }
+        if (dv <= 32) return BLM_DECODE(4, 2, false, false);
+        if (dv <= 64) return BLM_DECODE(8, 2, false, false);
+        if (dv <= 128) return BLM_DECODE(16, 3, false, false);
+        if (dv <= 192) return BLM_DECODE(24, 2, false, false);
+        return BLM_DECODE(32, 2, false, false);
 #undef BLM_DECODE
     }
     if (dtype == BLM_F32)
         return launch_rows<float>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, out, partial,
-                                  n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink, so, df, stream);
+                                  n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink, so, shared, df, stream);
     if (dtype == BLM_BF16)
         return launch_rows<__nv_bfloat16>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, out,
                                           partial, n_splits, n_tokens, n_heads, n_kv, maps, dk, dv, page_size, mask, keep_first, scale, sink,
-                                          so, df, stream);
+                                          so, shared, df, stream);
     return blm_fail(BLM_BAD_ARGUMENT, "attention_sink: dtype %d", dtype);
 }

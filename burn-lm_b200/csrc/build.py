@@ -36,6 +36,7 @@ MODULES = {
     "moe": ["moe.cu"],
     "stream_ops": ["stream_ops.cu"],
     "recurrent": ["recurrent.cu"],
+    "retention": ["retention.cu"],
     "attention_sigmoid": ["attention_sigmoid.cu"],
     "attention_latent": ["attention_latent.cu"],
     "gemm": ["gemm_f32.cu"],

@@ -188,6 +188,115 @@ BLM_API int blm_add_rmsnorm(float* resid, const void* delta, int delta_dtype, co
 }
 
 // ---------------------------------------------------------------------------------------------
+// The same for a pending sum of several parts: up to two outputs (float32 or bfloat16, each its own) and up to two biases
+// (float32 [width]) join the stream, then the RMS norm.  gamma null: only the sum.  Four lanes a thread where VEC.
+// ---------------------------------------------------------------------------------------------
+struct PendingParts {
+    const void* out[2];
+    int is_f32[2];
+    const float* bias[2];
+};
+template <int N>
+__device__ __forceinline__ void pending_lanes(const PendingParts& p, size_t row, int d, float (&h)[N]) {
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        if (p.out[k] != nullptr) {
+            if (p.is_f32[k]) {
+                const float* src = reinterpret_cast<const float*>(p.out[k]) + row + d;
+                if (N == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(src);
+                    h[0] += v.x; h[1 % N] += v.y; h[2 % N] += v.z; h[3 % N] += v.w;
+                } else {
+                    h[0] += src[0];
+                }
+            } else {
+                const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.out[k]) + row + d;
+                if (N == 4) {
+                    const uint2 raw = *reinterpret_cast<const uint2*>(src);
+                    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)),
+                                 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+                    h[0] += a.x; h[1 % N] += a.y; h[2 % N] += b.x; h[3 % N] += b.y;
+                } else {
+                    h[0] += __bfloat162float(src[0]);
+                }
+            }
+        }
+        if (p.bias[k] != nullptr) {
+            const float* src = p.bias[k] + d;
+            if (N == 4) {
+                const float4 v = *reinterpret_cast<const float4*>(src);
+                h[0] += v.x; h[1 % N] += v.y; h[2 % N] += v.z; h[3 % N] += v.w;
+            } else {
+                h[0] += src[0];
+            }
+        }
+    }
+}
+template <typename TA, typename TG, int N>
+__global__ void add_rmsnorm_parts_kernel(float* __restrict__ resid, PendingParts p, const TG* __restrict__ gamma, TA* __restrict__ out,
+                                         const int* __restrict__ rows, int width, float eps) {
+    extern __shared__ float row_buf[];  // [33] for the reduction, [3] empty, [width]
+    float* keep = row_buf + 36;
+    const int src = rows ? rows[blockIdx.x] : blockIdx.x;
+    float* r = resid + (size_t)src * width;
+    float ss = 0.f;
+    for (int d = threadIdx.x * N; d < width; d += blockDim.x * N) {
+        float h[N];
+        if (N == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(r + d);
+            h[0] = v.x; h[1 % N] = v.y; h[2 % N] = v.z; h[3 % N] = v.w;
+        } else {
+            h[0] = r[d];
+        }
+        pending_lanes<N>(p, (size_t)src * width, d, h);
+        if (N == 4) {
+            const float4 v = make_float4(h[0], h[1 % N], h[2 % N], h[3 % N]);
+            if (!rows) *reinterpret_cast<float4*>(r + d) = v;
+            *reinterpret_cast<float4*>(keep + d) = v;
+        } else {
+            if (!rows) r[d] = h[0];
+            keep[d] = h[0];
+        }
+#pragma unroll
+        for (int e = 0; e < N; ++e) ss += h[e] * h[e];
+    }
+    if (gamma == nullptr) return;
+    const float total = block_sum(ss, row_buf);
+    const float inv = 1.0f / sqrtf(total / (float)width + eps);
+    TA* o = out + (size_t)blockIdx.x * width;
+    for (int d = threadIdx.x * N; d < width; d += blockDim.x * N) {
+#pragma unroll
+        for (int e = 0; e < N; ++e) o[d + e] = from_f32<TA>(keep[d + e] * inv * to_f32(gamma[d + e]));
+    }
+}
+
+BLM_API int blm_add_rmsnorm_parts(float* resid, const void* out0, int dtype0, const void* out1, int dtype1, const float* bias0, const float* bias1,
+                                  const void* gamma, int gamma_dtype, void* out, int act_dtype, const int* rows, int n_rows, int width,
+                                  float eps, cudaStream_t stream) {
+    if (n_rows == 0) return BLM_OK;
+    BLM_REQUIRE(n_rows > 0 && width > 0 && (gamma == nullptr) == (out == nullptr), "rms norm: bad sizes");
+    BLM_REQUIRE(gamma != nullptr || rows == nullptr, "rms norm: chosen rows are normed, not summed");
+    const PendingParts p{{out0, out1}, {dtype0 == BLM_F32, dtype1 == BLM_F32}, {bias0, bias1}};
+    const size_t smem = (size_t)(width + 36) * sizeof(float);
+    BLM_REQUIRE(smem <= 200 * 1024, "rms norm: width %d is beyond the 51,000 this kernel holds in shared memory", width);
+    const bool vec = width % 4 == 0 && (((size_t)resid | (size_t)out0 | (size_t)out1 | (size_t)bias0 | (size_t)bias1) & 15) == 0;
+    const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
+    auto launch = [&](auto kernel, auto* g, auto* o) -> int {
+        if (smem > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "rms norm: %s", cudaGetErrorString(e));
+        }
+        kernel<<<n_rows, threads, smem, stream>>>(resid, p, g, o, rows, width, eps);
+        return blm_check_launch("add_rmsnorm (parts)");
+    };
+#define BLM_PARTS(TA, TG) (vec ? launch(add_rmsnorm_parts_kernel<TA, TG, 4>, (const TG*)gamma, (TA*)out) : launch(add_rmsnorm_parts_kernel<TA, TG, 1>, (const TG*)gamma, (TA*)out))
+    if (act_dtype == BLM_F32) return gamma_dtype == BLM_F32 ? BLM_PARTS(float, float) : BLM_PARTS(float, __nv_bfloat16);
+    if (act_dtype == BLM_BF16) return gamma_dtype == BLM_F32 ? BLM_PARTS(__nv_bfloat16, float) : BLM_PARTS(__nv_bfloat16, __nv_bfloat16);
+#undef BLM_PARTS
+    return blm_fail(BLM_BAD_ARGUMENT, "rms norm: dtypes %d/%d", act_dtype, gamma_dtype);
+}
+
+// ---------------------------------------------------------------------------------------------
 // rotary position encoding of q and k, fused with the append of k and v to the paged cache.
 //   qkv [N, (H + 2 KV) * hd]: q heads, then k heads, then v heads of every token.
 //   q is rotated in place; rotated k and plain v go to the page that holds the token's position.
@@ -384,7 +493,7 @@ BLM_API int blm_rope_table(const double* inv_freq, float* table, int n_pos, int 
 // holds gate then up (tile == 0), or tiles of `tile` gates followed by the `tile` ups of the same outputs.
 // ---------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int inner, size_t total, int tile) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long out_stride, int inner, size_t total, int tile) {
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
          idx += (size_t)gridDim.x * blockDim.x) {
         const size_t n = idx / inner;
@@ -393,12 +502,12 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const size_t ui = tile ? gi + tile : (size_t)inner + i;
         const float g = to_f32(gu[n * 2 * inner + gi]);
         const float u = to_f32(gu[n * 2 * inner + ui]);
-        out[idx] = from_f32<T>(g / (1.0f + expf(-g)) * u);
+        out[n * out_stride + i] = from_f32<T>(g / (1.0f + expf(-g)) * u);
     }
 }
 
 // bf16, eight outputs per thread: 16-byte loads of the gates and of the ups, one 16-byte store
-__global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, int inner,
+__global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, long long out_stride, int inner,
                                      size_t total8, int tile) {
     const int per_row = inner >> 3;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total8; idx += (size_t)gridDim.x * blockDim.x) {
@@ -417,26 +526,26 @@ __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_
             const float2 g = __bfloat1622float2(gp[e]), u = __bfloat1622float2(up[e]);
             op[e] = __floats2bfloat162_rn(g.x / (1.0f + expf(-g.x)) * u.x, g.y / (1.0f + expf(-g.y)) * u.y);
         }
-        *reinterpret_cast<uint4*>(out + n * inner + i) = ov;
+        *reinterpret_cast<uint4*>(out + n * out_stride + i) = ov;
     }
 }
 
-BLM_API int blm_swiglu(const void* gu, void* out, int dtype, int n_rows, int inner, int tile, cudaStream_t stream) {
+BLM_API int blm_swiglu(const void* gu, void* out, long long out_stride, int dtype, int n_rows, int inner, int tile, cudaStream_t stream) {
     if (n_rows == 0) return BLM_OK;
     BLM_REQUIRE(tile >= 0 && (tile == 0 || inner % tile == 0), "swiglu: tiles of %d do not divide %d", tile, inner);
     const size_t total = (size_t)n_rows * inner;
     const int threads = 256;
     const int blocks = (int)((total + threads - 1) / threads < blm_sm_count() * 16 ? (total + threads - 1) / threads : blm_sm_count() * 16);
-    if (dtype == BLM_BF16 && inner % 8 == 0 && (tile == 0 || tile % 8 == 0) && ((size_t)gu & 15) == 0 && ((size_t)out & 15) == 0) {
+    if (dtype == BLM_BF16 && inner % 8 == 0 && (tile == 0 || tile % 8 == 0) && ((size_t)gu & 15) == 0 && ((size_t)out & 15) == 0 && out_stride % 8 == 0) {
         const size_t total8 = total / 8;
         const int b8 = (int)((total8 + threads - 1) / threads < blm_sm_count() * 16 ? (total8 + threads - 1) / threads : blm_sm_count() * 16);
-        swiglu_bf16x8_kernel<<<b8, threads, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, inner, total8, tile);
+        swiglu_bf16x8_kernel<<<b8, threads, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, out_stride, inner, total8, tile);
         return blm_check_launch("swiglu");
     }
     if (dtype == BLM_F32)
-        swiglu_kernel<float><<<blocks, threads, 0, stream>>>((const float*)gu, (float*)out, inner, total, tile);
+        swiglu_kernel<float><<<blocks, threads, 0, stream>>>((const float*)gu, (float*)out, out_stride, inner, total, tile);
     else if (dtype == BLM_BF16)
-        swiglu_kernel<__nv_bfloat16><<<blocks, threads, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, inner, total, tile);
+        swiglu_kernel<__nv_bfloat16><<<blocks, threads, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out, out_stride, inner, total, tile);
     else
         return blm_fail(BLM_BAD_ARGUMENT, "swiglu: dtype %d", dtype);
     return blm_check_launch("swiglu");

@@ -84,6 +84,7 @@ struct GemvArgs {
     long long ldy;
     int y_f32;
     float* acc;              // EPI_RESID_ADD: fp32 [N, M] (ld = M)
+    const float* add_bias;   // EPI_RESID_ADD: fp32 [M] that joins every row's sum, or null
     int epi;
     int n_stages;            // ring depth
     // A norm handed over by the kernel that wrote the stream: x is bf16(stream * gamma), not yet divided by
@@ -551,6 +552,18 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvArgs a,
                     const int m = tile * 16 + g + 8 * (e >> 1), b = j * 8 + 2 * t + (e & 1);
                     old[j][e] = (m < a.M && b < a.N) ? a.acc[(size_t)b * a.M + m] : 0.f;
                 }
+            if (a.add_bias != nullptr) {
+#pragma unroll
+                for (int rr = 0; rr < 2; ++rr) {
+                    const int m = tile * 16 + g + 8 * rr;
+                    const float bias = m < a.M ? a.add_bias[m] : 0.f;
+#pragma unroll
+                    for (int j = 0; j < NBT; ++j) {
+                        c[0][j][2 * rr] += bias;
+                        c[0][j][2 * rr + 1] += bias;
+                    }
+                }
+            }
             float gm[2] = {0.f, 0.f};          // the next norm's gamma of rows g and g + 8
             if (a.xg_out != nullptr) {
 #pragma unroll
@@ -786,7 +799,7 @@ static int token_map(const void* x, long long ldx, int N, int K, int nrows, int 
 
 BLM_API int blm_gemv(const void* w, long long ldw, int M, int K, const void* x, long long ldx,
                      const float* resid, const void* gamma, int gamma_f32, float eps, const int* rows, int N,
-                     void* y, long long ldy, int y_f32, float* acc, int epi, const float* ssq_in, int ssq_parts,
+                     void* y, long long ldy, int y_f32, float* acc, const float* add_bias, int epi, const float* ssq_in, int ssq_parts,
                      const void* next_gamma, int next_gamma_f32, void* xg_out, float* ssq_out, const GemvRope* rope,
                      int* status, cudaStream_t stream) {
     if (N == 0 || M == 0) return BLM_OK;
@@ -815,7 +828,7 @@ BLM_API int blm_gemv(const void* w, long long ldw, int M, int K, const void* x, 
     GemvArgs a;
     a.w = (const __nv_bfloat16*)w; a.ldw = ldw; a.M = M; a.K = K;
     a.x = (const __nv_bfloat16*)x; a.ldx = ldx; a.resid = resid; a.gamma = gamma; a.gamma_f32 = gamma_f32; a.eps = eps;
-    a.rows = rows; a.N = N; a.y = y; a.ldy = ldy; a.y_f32 = y_f32; a.acc = acc; a.epi = epi; a.status = status;
+    a.rows = rows; a.N = N; a.y = y; a.ldy = ldy; a.y_f32 = y_f32; a.acc = acc; a.add_bias = epi == EPI_RESID_ADD ? add_bias : nullptr; a.epi = epi; a.status = status;
     a.ssq_in = ssq_in; a.ssq_parts = ssq_parts; a.next_gamma = next_gamma; a.next_gamma_f32 = next_gamma_f32;
     a.xg_out = (__nv_bfloat16*)xg_out; a.ssq_out = ssq_out;
     if (epi == EPI_ROPE) a.rope = *rope;

@@ -1,0 +1,752 @@
+// Retention: linear attention with one fixed decay per head over the packed tokens of a step.  Per head,
+//   S_t = a S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   out = o / sqrt(mean(o^2) + eps) * silu(g)      (S: dk x dv)
+// with q and k turned by their position and k scaled first.  A row of the projection holds [q | k | v | g], float32.
+//
+// What a sequence carries is S of every head, float32 [head][dk][dv], twice (see recurrent.cu): a step that starts at position p
+// reads copy (p & 1) and writes copy ((p + n) & 1) for its n new tokens; one that starts at position 0 reads zeros.
+//
+// Three forms, which share that state:
+//   the scan: tokens in order, S and the sums over its rows in float64 inside a step; it serves the 32-bit path and head sizes
+//     the others do not take, and leaves o for a kernel that norms and gates it;
+//   the single token: a block a (token, head) reads S once, writes it once, and finishes the row (norm, gate);
+//   chunks of 64 tokens: (1) what every chunk adds to S by itself, sum_t a^(last - t) k_t v_t^T; (2) S in front of every chunk,
+//     from these in order; (3) a chunk's outputs, o_t = a^(t + 1) S^T q_t + sum_(s <= t) a^(t - s) (q_t . k_s) v_s, normed and
+//     gated.  All chunks of a sequence run side by side in (1) and (3).  Products on the tensor cores with float32 sums, bfloat16
+//     operands; operands that carry a decay or are S itself go in as two bfloat16 numbers, high part and rest (16 bits).
+#include "common.cuh"
+
+BLM_API const char* blm_retention_last_error() { return g_blm_error; }
+
+constexpr int kC = 64;             // tokens of a chunk
+
+// The step's projection and how its queries and keys turn: lanes (i, i + rot / 2) of the first `rot` by position * freq[i].
+struct RetIn {
+    const float* proj;
+    long long stride;
+    int heads, dk, dv;
+    float k_scale;
+    const double* freq;
+    int rot;
+    const float2* table;           // [table_len][rot / 2] (cosine, sine), or null
+    int table_len;
+    const float* powers;           // [heads][kC + 1]: the decay to the power m
+};
+struct RetSeq {
+    const int* cu_seqlens;
+    const int* slot_of_seq;
+    const int* start_pos;
+    int n_seqs;
+    float* state;
+    long long slot_stride, copy_stride, offset;
+    __device__ __forceinline__ float* copy(int seq, int pos) const {
+        return state + (size_t)slot_of_seq[seq] * slot_stride + (size_t)(pos & 1) * copy_stride + offset;
+    }
+};
+
+__device__ __forceinline__ float2 ret_turn(const RetIn& in, int pos, int i) {
+    if (pos < in.table_len) return in.table[(size_t)pos * (in.rot >> 1) + i];
+    double sn, cs;
+    sincos((double)pos * in.freq[i], &sn, &cs);
+    return make_float2((float)cs, (float)sn);
+}
+// lane d of a head's query or key (`src`: the head's first lane), turned
+__device__ __forceinline__ float ret_lane(const RetIn& in, const float* src, int pos, int d) {
+    if (d >= in.rot) return src[d];
+    const int half = in.rot >> 1;
+    if (d < half) {
+        const float2 t = ret_turn(in, pos, d);
+        return src[d] * t.x - src[d + half] * t.y;
+    }
+    const float2 t = ret_turn(in, pos, d - half);
+    return src[d] * t.x + src[d - half] * t.y;
+}
+// lanes d .. d + 3, d a multiple of 4; `vec`: rows and halves allow 16-byte loads
+__device__ __forceinline__ void ret_lanes4(const RetIn& in, const float* src, int pos, int d, bool vec, float (&v)[4]) {
+    if (!vec) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] = d + e < in.dk ? ret_lane(in, src, pos, d + e) : 0.f;
+        return;
+    }
+    const float4 a = *reinterpret_cast<const float4*>(src + d);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    if (d >= in.rot) return;
+    const int half = in.rot >> 1;
+    const bool first = d < half;
+    const float4 b = *reinterpret_cast<const float4*>(src + (first ? d + half : d - half));
+    const float o[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const float2 t = ret_turn(in, pos, (first ? d : d - half) + e);
+        v[e] = first ? v[e] * t.x - o[e] * t.y : v[e] * t.x + o[e] * t.y;
+    }
+}
+static bool ret_vec(const RetIn& in) {
+    return in.dk % 4 == 0 && in.dv % 4 == 0 && in.rot % 8 == 0 && in.stride % 4 == 0 && ((size_t)in.proj & 15) == 0;
+}
+__device__ __forceinline__ float ret_silu(float z) { return z / (1.0f + expf(-z)); }
+
+// ---------------------------------------------------------------------------------------------
+// the scan: a block per (32 value lanes, head, sequence); thread (column, row group) keeps rows rg, rg + 8, ... of its column
+// ---------------------------------------------------------------------------------------------
+constexpr int kScanTokens = 32;    // tokens staged in shared memory at a time
+
+template <int RN>
+__global__ void __launch_bounds__(256) retention_scan_kernel(RetIn in, RetSeq sq, float* __restrict__ o, long long o_stride) {
+    extern __shared__ float sm[];
+    float* qs = sm;                                    // [kScanTokens][dk]
+    float* ks = qs + kScanTokens * in.dk;
+    float* vs = ks + kScanTokens * in.dk;              // [kScanTokens][32]
+    const int head = blockIdx.y, seq = blockIdx.z, col0 = blockIdx.x * 32;
+    const int rg = threadIdx.x & 7, col = threadIdx.x >> 3, dk = in.dk, dv = in.dv;
+    const int t0 = sq.cu_seqlens[seq], len = sq.cu_seqlens[seq + 1] - t0;
+    if (len <= 0) return;
+    const int start = sq.start_pos[seq];
+    const bool mine = col0 + col < dv;
+    const float* from = sq.copy(seq, start) + (size_t)head * dk * dv + col0 + col;
+    double S[RN];
+#pragma unroll
+    for (int r = 0; r < RN; ++r) {
+        const int row = rg + 8 * r;
+        S[r] = mine && row < dk && start > 0 ? (double)from[(size_t)row * dv] : 0.0;
+    }
+    const double decay = (double)in.powers[(size_t)head * (kC + 1) + 1];
+    const int hq = head * dk, hk = in.heads * dk + hq, hv = 2 * in.heads * dk + head * dv + col0;
+    for (int c0 = 0; c0 < len; c0 += kScanTokens) {
+        const int m = min(kScanTokens, len - c0);
+        __syncthreads();
+        for (int idx = threadIdx.x; idx < m * dk; idx += 256) {
+            const int t = idx / dk, d = idx % dk, pos = start + c0 + t;
+            const float* row = in.proj + (size_t)(t0 + c0 + t) * in.stride;
+            qs[idx] = ret_lane(in, row + hq, pos, d);
+            ks[idx] = ret_lane(in, row + hk, pos, d) * in.k_scale;
+        }
+        for (int idx = threadIdx.x; idx < m * 32; idx += 256) {
+            const int t = idx >> 5, c = idx & 31;
+            vs[idx] = col0 + c < dv ? in.proj[(size_t)(t0 + c0 + t) * in.stride + hv + c] : 0.f;
+        }
+        __syncthreads();
+        for (int t = 0; t < m; ++t) {
+            const double v = (double)vs[t * 32 + col];
+            double acc = 0.0;
+#pragma unroll
+            for (int r = 0; r < RN; ++r) {
+                const int row = rg + 8 * r;
+                if (row < dk) {
+                    S[r] = decay * S[r] + (double)ks[t * dk + row] * v;
+                    acc += S[r] * (double)qs[t * dk + row];
+                }
+            }
+            acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+            acc += __shfl_xor_sync(0xffffffffu, acc, 2);
+            acc += __shfl_xor_sync(0xffffffffu, acc, 4);
+            if (rg == 0 && mine) o[(size_t)(t0 + c0 + t) * o_stride + (size_t)head * dv + col0 + col] = (float)acc;
+        }
+    }
+    float* to = sq.copy(seq, start + len) + (size_t)head * dk * dv + col0 + col;
+#pragma unroll
+    for (int r = 0; r < RN; ++r) {
+        const int row = rg + 8 * r;
+        if (mine && row < dk) to[(size_t)row * dv] = (float)S[r];
+    }
+}
+
+// ---------------------------------------------------------------------------------------------
+// the single token: a block per (head, token).  Thread (row group, column group) takes N value lanes of rows rg, rg + n_rg, ...
+// ---------------------------------------------------------------------------------------------
+constexpr int kStepThreads = 256;
+constexpr int kAhead = 8;          // rows a thread asks for before it works on the first
+
+template <typename TO, int N>
+__global__ void __launch_bounds__(kStepThreads) retention_step_kernel(RetIn in, RetSeq sq, const int* __restrict__ token_seq,
+                                                                      const int* __restrict__ token_pos, float eps, TO* __restrict__ out,
+                                                                      long long out_stride, int vec) {
+    extern __shared__ __align__(16) float sm[];
+    const int dk = in.dk, dv = in.dv, head = blockIdx.x, tid = threadIdx.x;
+    float* qs = sm;                                    // [dk]
+    float* ks = qs + ((dk + 3) & ~3);
+    float* red = ks + ((dk + 3) & ~3);                 // [36], then [n_rg][dv] partial sums
+    float* part = red + 36;
+    const size_t n = blockIdx.y;
+    TO* orow = out + n * out_stride + (size_t)head * dv;
+    const int seq = token_seq[n];
+    if (seq < 0) {                                     // a row of no sequence
+        for (int d = tid; d < dv; d += kStepThreads) orow[d] = from_f32<TO>(0.f);
+        return;
+    }
+    const int pos = token_pos[n], groups = dv / N, n_rg = kStepThreads / groups;
+    const int cg = tid % groups, rg = tid / groups, c = cg * N;
+    const bool works = rg < n_rg;
+    const float* from = sq.copy(seq, pos) + (size_t)head * dk * dv + c;
+    float* to = sq.copy(seq, pos + 1) + (size_t)head * dk * dv + c;
+    float S[kAhead][N];
+    auto fetch = [&](int row0) {
+#pragma unroll
+        for (int a = 0; a < kAhead; ++a) {
+            const int row = row0 + a * n_rg;
+            if (works && row < dk && pos > 0) {
+                if (N == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(from + (size_t)row * dv);
+                    S[a][0] = v.x; S[a][1 % N] = v.y; S[a][2 % N] = v.z; S[a][3 % N] = v.w;
+                } else {
+                    S[a][0] = from[(size_t)row * dv];
+                }
+            } else {
+#pragma unroll
+                for (int e = 0; e < N; ++e) S[a][e] = 0.f;
+            }
+        }
+    };
+    fetch(rg);                                         // the state is on its way while the token's row is prepared
+    const float* row_p = in.proj + n * in.stride;
+    const int quads = (dk + 3) / 4;
+    for (int i = tid; i < 2 * quads; i += kStepThreads) {
+        const bool is_k = i >= quads;
+        const int d = (is_k ? i - quads : i) * 4;
+        float v[4];
+        ret_lanes4(in, row_p + (is_k ? in.heads * dk : 0) + head * dk, pos, d, vec, v);
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+            if (d + e < dk) (is_k ? ks : qs)[d + e] = is_k ? v[e] * in.k_scale : v[e];
+    }
+    const float decay = in.powers[(size_t)head * (kC + 1) + 1];
+    float v[N], acc[N];
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+        v[e] = works ? row_p[2 * in.heads * dk + head * dv + c + e] : 0.f;
+        acc[e] = 0.f;
+    }
+    __syncthreads();
+    for (int row0 = rg; row0 < dk && works; row0 += kAhead * n_rg) {
+        if (row0 != rg) fetch(row0);
+#pragma unroll
+        for (int a = 0; a < kAhead; ++a) {
+            const int row = row0 + a * n_rg;
+            if (row >= dk) break;
+            const float kk = ks[row], qq = qs[row];
+#pragma unroll
+            for (int e = 0; e < N; ++e) {
+                S[a][e] = fmaf(decay, S[a][e], kk * v[e]);
+                acc[e] = fmaf(qq, S[a][e], acc[e]);
+            }
+            if (N == 4) *reinterpret_cast<float4*>(to + (size_t)row * dv) = make_float4(S[a][0], S[a][1 % N], S[a][2 % N], S[a][3 % N]);
+            else to[(size_t)row * dv] = S[a][0];
+        }
+    }
+    if (works) {
+#pragma unroll
+        for (int e = 0; e < N; ++e) part[(size_t)rg * dv + c + e] = acc[e];
+    }
+    __syncthreads();
+    // the row groups' sums in order, then the norm over the head's lanes and the gate
+    float ss = 0.f;
+    for (int d = tid; d < dv; d += kStepThreads) {
+        float s = 0.f;
+        for (int r = 0; r < n_rg; ++r) s += part[(size_t)r * dv + d];
+        part[d] = s;                                   // (only this thread reads or writes column d from here on)
+        ss += s * s;
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dv + eps);
+    const float* gate = row_p + 2 * in.heads * dk + in.heads * dv + head * dv;
+    for (int d = tid; d < dv; d += kStepThreads) orow[d] = from_f32<TO>(part[d] * inv * ret_silu(gate[d]));
+}
+
+// ---------------------------------------------------------------------------------------------
+// chunks
+// ---------------------------------------------------------------------------------------------
+__device__ __forceinline__ unsigned ret_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ret_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ret_ldsm(uint32_t (&r)[4], unsigned a) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void ret_ldsm_t(uint32_t (&r)[4], unsigned a) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ uint32_t ret_pack(float lo, float hi) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&v);
+}
+// two numbers as bfloat16 pairs: the rounded ones, and what the rounding left (rounded again)
+__device__ __forceinline__ void ret_split(float a, float b, uint32_t& hi, uint32_t& rest) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    const float2 f = __bfloat1622float2(h);
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    rest = ret_pack(a - f.x, b - f.y);
+}
+__device__ __forceinline__ void ret_put4(__nv_bfloat16* dst, const float (&v)[4]) {
+    *reinterpret_cast<uint2*>(dst) = make_uint2(ret_pack(v[0], v[1]), ret_pack(v[2], v[3]));
+}
+
+// Which chunk a block has: sequence, first token of the chunk in the sequence, tokens, and whether there is one.
+struct RetChunk {
+    int seq, t0, rows, first_row, start;
+    bool found;
+};
+__device__ __forceinline__ RetChunk ret_find(const RetSeq& sq, int block, int* shared3) {
+    if (threadIdx.x == 0) {
+        int t = block;
+        shared3[0] = -1;
+        for (int s = 0; s < sq.n_seqs; ++s) {
+            const int len = sq.cu_seqlens[s + 1] - sq.cu_seqlens[s], tiles = (len + kC - 1) / kC;
+            if (t < tiles) {
+                shared3[0] = s;
+                shared3[1] = t * kC;
+                shared3[2] = len;
+                break;
+            }
+            t -= tiles;
+        }
+    }
+    __syncthreads();
+    RetChunk c;
+    c.seq = shared3[0];
+    c.found = c.seq >= 0;
+    if (!c.found) return c;
+    c.t0 = shared3[1];
+    c.rows = min(kC, shared3[2] - c.t0);
+    c.first_row = sq.cu_seqlens[c.seq] + c.t0;
+    c.start = sq.start_pos[c.seq] + c.t0;
+    return c;
+}
+
+// a head's values of a chunk as bfloat16 [kC][vstride], zeros beyond its tokens and lanes
+__device__ __forceinline__ void ret_stage_values(const RetIn& in, const RetChunk& c, int head, __nv_bfloat16* vs, int vstride, int cols, bool vec) {
+    const int quads = cols / 4;
+    for (int idx = threadIdx.x; idx < kC * quads; idx += blockDim.x) {
+        const int t = idx / quads, d = (idx % quads) * 4;
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (t < c.rows) {
+            const float* src = in.proj + (size_t)(c.first_row + t) * in.stride + 2 * in.heads * in.dk + head * in.dv;
+            if (vec) {
+                if (d < in.dv) {
+                    const float4 f = *reinterpret_cast<const float4*>(src + d);
+                    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+                }
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (d + e < in.dv) v[e] = src[d + e];
+            }
+        }
+        ret_put4(vs + t * vstride + d, v);
+    }
+}
+
+// (1) what a chunk adds to S by itself: kv [chunk][head][dk][dv]
+__global__ void __launch_bounds__(256) retention_chunk_add_kernel(RetIn in, RetSeq sq, float* __restrict__ kv, int vec) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ int found[3];
+    const RetChunk c = ret_find(sq, blockIdx.x, found);
+    if (!c.found) return;
+    const int head = blockIdx.y, dk = in.dk, dv = in.dv;
+    const int dkp = (dk + 15) & ~15, kstride = dkp + 8, cols = (dv + 63) & ~63, vstride = cols + 8;
+    __nv_bfloat16* kh = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [kC][kstride] a^(last - t) k_t: high parts
+    __nv_bfloat16* kr = kh + kC * kstride;                               // ... and rests
+    __nv_bfloat16* vs = kr + kC * kstride;                               // [kC][vstride]
+    const float* powers = in.powers + (size_t)head * (kC + 1);
+    const int quads = dkp / 4;
+    for (int idx = threadIdx.x; idx < kC * quads; idx += blockDim.x) {
+        const int t = idx / quads, d = (idx % quads) * 4;
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (t < c.rows && d < dk) {
+            ret_lanes4(in, in.proj + (size_t)(c.first_row + t) * in.stride + (in.heads + head) * dk, c.start + t, d, vec, v);
+            const float w = powers[c.rows - 1 - t] * in.k_scale;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] *= w;
+        }
+        uint32_t h0, h1, r0, r1;
+        ret_split(v[0], v[1], h0, r0);
+        ret_split(v[2], v[3], h1, r1);
+        *reinterpret_cast<uint2*>(kh + t * kstride + d) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2*>(kr + t * kstride + d) = make_uint2(r0, r1);
+    }
+    ret_stage_values(in, c, head, vs, vstride, cols, vec);
+    __syncthreads();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const int lrow = lane & 7, lmat = lane >> 3, quad = lane >> 2, pair = (lane & 3) * 2;
+    float* dst = kv + ((size_t)blockIdx.x * in.heads + head) * dk * dv;
+    // a unit: 16 rows of S by 64 of its columns
+    const int units = (dkp / 16) * (cols / 64);
+    const bool two = dv % 2 == 0;
+    for (int u = warp; u < units; u += n_warps) {
+        const int m0 = (u % (dkp / 16)) * 16, n0 = (u / (dkp / 16)) * 64;
+        float acc[8][4];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+        // A: the keys read transposed (rows of S by tokens)
+        const unsigned ao = (unsigned)((((lmat >> 1) * 8 + lrow) * kstride + m0 + (lmat & 1) * 8) * 2);
+        const unsigned bo = ret_smem(vs) + (unsigned)((((lmat & 1) * 8 + lrow) * vstride + n0 + (lmat >> 1) * 8) * 2);
+#pragma unroll
+        for (int kk = 0; kk < kC; kk += 16) {
+            uint32_t ah[4], ar[4], b[4];
+            ret_ldsm_t(ah, ret_smem(kh) + ao + kk * kstride * 2);
+            ret_ldsm_t(ar, ret_smem(kr) + ao + kk * kstride * 2);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                ret_ldsm_t(b, bo + (kk * vstride + 16 * j) * 2);
+                ret_mma(acc[2 * j], ah, b[0], b[1]);
+                ret_mma(acc[2 * j + 1], ah, b[2], b[3]);
+                ret_mma(acc[2 * j], ar, b[0], b[1]);
+                ret_mma(acc[2 * j + 1], ar, b[2], b[3]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int row = m0 + quad + 8 * half, col = n0 + 8 * j + pair;
+                if (row >= dk || col >= dv) continue;
+                float* p = dst + (size_t)row * dv + col;
+                if (two) {
+                    *reinterpret_cast<float2*>(p) = make_float2(acc[j][2 * half], acc[j][2 * half + 1]);
+                } else {
+                    p[0] = acc[j][2 * half];
+                    if (col + 1 < dv) p[1] = acc[j][2 * half + 1];
+                }
+            }
+    }
+}
+
+// (2) S in front of every chunk, in place of what the chunk adds; S behind the last one goes to the sequence's state
+template <int N>
+__global__ void __launch_bounds__(256) retention_carry_kernel(RetIn in, RetSeq sq, float* __restrict__ kv) {
+    const int head = blockIdx.y, seq = blockIdx.z;
+    const size_t size = (size_t)in.dk * in.dv, at = ((size_t)blockIdx.x * 256 + threadIdx.x) * N;
+    const int len = sq.cu_seqlens[seq + 1] - sq.cu_seqlens[seq];
+    if (at >= size || len <= 0) return;
+    int first = 0;                                     // the sequence's first chunk
+    for (int s = 0; s < seq; ++s) first += (sq.cu_seqlens[s + 1] - sq.cu_seqlens[s] + kC - 1) / kC;
+    const int start = sq.start_pos[seq], n_chunks = (len + kC - 1) / kC;
+    const float* from = sq.copy(seq, start) + (size_t)head * size + at;
+    float S[N];
+#pragma unroll
+    for (int e = 0; e < N; ++e) S[e] = start > 0 ? from[e] : 0.f;
+    const float* powers = in.powers + (size_t)head * (kC + 1);
+    const float full = powers[kC], last = powers[len - (n_chunks - 1) * kC];
+    const size_t step = (size_t)in.heads * size;
+    float* p = kv + (size_t)first * step + (size_t)head * size + at;
+    constexpr int kRead = 4;                           // chunks read ahead of their turn
+    for (int c0 = 0; c0 < n_chunks; c0 += kRead) {
+        float add[kRead][N];
+#pragma unroll
+        for (int a = 0; a < kRead; ++a)
+            if (c0 + a < n_chunks) {
+                if (N == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(p + (size_t)(c0 + a) * step);
+                    add[a][0] = v.x; add[a][1 % N] = v.y; add[a][2 % N] = v.z; add[a][3 % N] = v.w;
+                } else {
+                    add[a][0] = p[(size_t)(c0 + a) * step];
+                }
+            }
+#pragma unroll
+        for (int a = 0; a < kRead; ++a)
+            if (c0 + a < n_chunks) {
+                float* q = p + (size_t)(c0 + a) * step;
+                if (N == 4) *reinterpret_cast<float4*>(q) = make_float4(S[0], S[1 % N], S[2 % N], S[3 % N]);
+                else q[0] = S[0];
+                const float w = c0 + a == n_chunks - 1 ? last : full;
+#pragma unroll
+                for (int e = 0; e < N; ++e) S[e] = fmaf(w, S[e], add[a][e]);
+            }
+    }
+    float* to = sq.copy(seq, start + len) + (size_t)head * size + at;
+#pragma unroll
+    for (int e = 0; e < N; ++e) to[e] = S[e];
+}
+
+// (3) a chunk's rows: four warps of 16 rows each for every 64 value lanes.  slice: rows of S in shared memory at a time.
+template <int WARPS>
+__global__ void __launch_bounds__(32 * WARPS) retention_chunk_out_kernel(RetIn in, RetSeq sq, const float* __restrict__ kv, int slice, float eps,
+                                                                   __nv_bfloat16* __restrict__ out, long long out_stride, int n_tokens, int vec) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ int found[3];
+    __shared__ float pw[kC + 1];
+    __shared__ float ssq[8][kC];
+    const RetChunk c = ret_find(sq, blockIdx.x, found);
+    const int head = blockIdx.y, dk = in.dk, dv = in.dv, tid = threadIdx.x;
+    if (!c.found) {                                    // rows after the last sequence (padding up to a captured step's size) get zeros
+        const int end = sq.cu_seqlens[sq.n_seqs];
+        for (int idx = tid; idx < (n_tokens - end) * dv; idx += blockDim.x)
+            out[(size_t)(end + idx / dv) * out_stride + (size_t)head * dv + idx % dv] = __float2bfloat16_rn(0.f);
+        return;
+    }
+    const int dkp = (dk + 15) & ~15, kstride = dkp + 8, cols = (dv + 63) & ~63, vstride = cols + 8;
+    __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [kC][kstride]
+    __nv_bfloat16* ks = qs + kC * kstride;                               // [kC][kstride]
+    __nv_bfloat16* vs = ks + kC * kstride;                               // [kC][vstride]
+    __nv_bfloat16* sh = vs + kC * vstride;                               // [slice][vstride] S: high parts
+    __nv_bfloat16* sr = sh + slice * vstride;                            // ... and rests
+    const int quads = dkp / 4;
+    for (int idx = tid; idx < 2 * kC * quads; idx += blockDim.x) {
+        const bool is_k = idx >= kC * quads;
+        const int i = is_k ? idx - kC * quads : idx, t = i / quads, d = (i % quads) * 4;
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (t < c.rows && d < dk) {
+            ret_lanes4(in, in.proj + (size_t)(c.first_row + t) * in.stride + ((is_k ? in.heads : 0) + head) * dk, c.start + t, d, vec, v);
+            if (is_k) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v[e] *= in.k_scale;
+            }
+        }
+        ret_put4((is_k ? ks : qs) + t * kstride + d, v);
+    }
+    ret_stage_values(in, c, head, vs, vstride, cols, vec);
+    for (int i = tid; i <= kC; i += blockDim.x) pw[i] = in.powers[(size_t)head * (kC + 1) + i];
+    const int lane = tid & 31, warp = tid >> 5, wr = warp & 3, wc = warp >> 2;
+    const int lrow = lane & 7, lmat = lane >> 3, quad = lane >> 2, pair = (lane & 3) * 2;
+    const int r0 = wr * 16 + quad, r1 = r0 + 8;        // this thread's two rows of the chunk
+    float acc[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    const unsigned qa = ret_smem(qs) + (unsigned)(((wr * 16 + lrow + (lmat & 1) * 8) * kstride + (lmat >> 1) * 8) * 2);
+    const unsigned vo = (unsigned)((((lmat & 1) * 8 + lrow) * vstride + wc * 64 + (lmat >> 1) * 8) * 2);
+    if (c.start > 0) {                                 // (else S is zero)
+        const float* S = kv + ((size_t)blockIdx.x * in.heads + head) * dk * dv;
+        const int vquads = cols / 4;
+        for (int s0 = 0; s0 < dkp; s0 += slice) {
+            const int m = min(slice, dkp - s0);
+            __syncthreads();
+            for (int idx = tid; idx < m * vquads; idx += blockDim.x) {
+                const int r = idx / vquads, d = (idx % vquads) * 4;
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                if (s0 + r < dk) {
+                    const float* src = S + (size_t)(s0 + r) * dv + d;
+                    if (vec) {
+                        if (d < dv) {
+                            const float4 f = *reinterpret_cast<const float4*>(src);
+                            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+                        }
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e)
+                            if (d + e < dv) v[e] = src[e];
+                    }
+                }
+                uint32_t h0, h1, x0, x1;
+                ret_split(v[0], v[1], h0, x0);
+                ret_split(v[2], v[3], h1, x1);
+                *reinterpret_cast<uint2*>(sh + r * vstride + d) = make_uint2(h0, h1);
+                *reinterpret_cast<uint2*>(sr + r * vstride + d) = make_uint2(x0, x1);
+            }
+            __syncthreads();
+            for (int kk = 0; kk < m; kk += 16) {
+                uint32_t a[4], b[4];
+                ret_ldsm(a, qa + (s0 + kk) * 2);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    ret_ldsm_t(b, ret_smem(sh) + vo + (kk * vstride + 16 * j) * 2);
+                    ret_mma(acc[2 * j], a, b[0], b[1]);
+                    ret_mma(acc[2 * j + 1], a, b[2], b[3]);
+                    ret_ldsm_t(b, ret_smem(sr) + vo + (kk * vstride + 16 * j) * 2);
+                    ret_mma(acc[2 * j], a, b[0], b[1]);
+                    ret_mma(acc[2 * j + 1], a, b[2], b[3]);
+                }
+            }
+        }
+        const float w0 = pw[r0 + 1], w1 = pw[r1 + 1];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            acc[j][0] *= w0; acc[j][1] *= w0;
+            acc[j][2] *= w1; acc[j][3] *= w1;
+        }
+    } else {
+        __syncthreads();
+    }
+    // the chunk's own tokens: (q_t . k_s) a^(t - s), then times the values
+    float s[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+    const unsigned ka = ret_smem(ks) + (unsigned)(((lrow + (lmat >> 1) * 8) * kstride + (lmat & 1) * 8) * 2);
+    for (int kk = 0; kk < dkp; kk += 16) {
+        uint32_t a[4], b[4];
+        ret_ldsm(a, qa + kk * 2);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            if (j > wr) break;                         // keys behind every row of the warp
+            ret_ldsm(b, ka + (16 * j * kstride + kk) * 2);
+            ret_mma(s[2 * j], a, b[0], b[1]);
+            ret_mma(s[2 * j + 1], a, b[2], b[3]);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int back = (e < 2 ? r0 : r1) - (8 * j + pair + (e & 1));
+            s[j][e] = back >= 0 ? s[j][e] * pw[back] : 0.f;
+        }
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) {
+        if (kk > wr) break;
+        uint32_t ah[4], ar[4], b[4];
+        ret_split(s[2 * kk][0], s[2 * kk][1], ah[0], ar[0]);
+        ret_split(s[2 * kk][2], s[2 * kk][3], ah[1], ar[1]);
+        ret_split(s[2 * kk + 1][0], s[2 * kk + 1][1], ah[2], ar[2]);
+        ret_split(s[2 * kk + 1][2], s[2 * kk + 1][3], ah[3], ar[3]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            ret_ldsm_t(b, ret_smem(vs) + vo + (16 * kk * vstride + 16 * j) * 2);
+            ret_mma(acc[2 * j], ah, b[0], b[1]);
+            ret_mma(acc[2 * j + 1], ah, b[2], b[3]);
+            ret_mma(acc[2 * j], ar, b[0], b[1]);
+            ret_mma(acc[2 * j + 1], ar, b[2], b[3]);
+        }
+    }
+    // the norm over the head's lanes: this warp's 64 of them, then the other warps' of the same rows
+    float q0 = 0.f, q1 = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+        q0 += acc[j][0] * acc[j][0] + acc[j][1] * acc[j][1];
+        q1 += acc[j][2] * acc[j][2] + acc[j][3] * acc[j][3];
+    }
+    q0 += __shfl_xor_sync(0xffffffffu, q0, 1);
+    q0 += __shfl_xor_sync(0xffffffffu, q0, 2);
+    q1 += __shfl_xor_sync(0xffffffffu, q1, 1);
+    q1 += __shfl_xor_sync(0xffffffffu, q1, 2);
+    if (pair == 0) {
+        ssq[wc][r0] = q0;
+        ssq[wc][r1] = q1;
+    }
+    __syncthreads();
+    const int n_wc = cols / 64;
+    const bool two = dv % 2 == 0 && out_stride % 2 == 0 && ((size_t)out & 3) == 0 && vec;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int r = half ? r1 : r0;
+        if (r >= c.rows) continue;
+        float ss = 0.f;
+        for (int w = 0; w < n_wc; ++w) ss += ssq[w][r];
+        const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
+        const float* gate = in.proj + (size_t)(c.first_row + r) * in.stride + 2 * in.heads * dk + (in.heads + head) * dv;
+        __nv_bfloat16* o = out + (size_t)(c.first_row + r) * out_stride + (size_t)head * dv;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const int d = wc * 64 + 8 * j + pair;
+            if (d >= dv) continue;
+            const float x0 = acc[j][2 * half] * inv, x1 = acc[j][2 * half + 1] * inv;
+            if (two) {
+                const float2 g = *reinterpret_cast<const float2*>(gate + d);
+                *reinterpret_cast<uint32_t*>(o + d) = ret_pack(x0 * ret_silu(g.x), x1 * ret_silu(g.y));
+            } else {
+                o[d] = __float2bfloat16_rn(x0 * ret_silu(gate[d]));
+                if (d + 1 < dv) o[d + 1] = __float2bfloat16_rn(x1 * ret_silu(gate[d + 1]));
+            }
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------------------------
+// entry points
+// ---------------------------------------------------------------------------------------------
+static size_t chunk_smem(int dk, int dv, int slice) {
+    const int kstride = ((dk + 15) & ~15) + 8, vstride = ((dv + 63) & ~63) + 8;
+    return ((size_t)2 * kC * kstride + (size_t)kC * vstride + (size_t)2 * slice * vstride) * sizeof(__nv_bfloat16);
+}
+// rows of S that fit beside a chunk's tokens, 0 when the chunk kernels do not take the head size
+static int chunk_slice(int dk, int dv) {
+    if (dk > 256 || dv > 512) return 0;
+    const int dkp = (dk + 15) & ~15;
+    for (int slice = dkp < 64 ? dkp : 64; slice >= 16; slice -= 16)
+        if (chunk_smem(dk, dv, slice) <= 220 * 1024) return slice;
+    return 0;
+}
+BLM_API int blm_retention_chunks_take(int dk, int dv) { return chunk_slice(dk, dv) > 0; }
+BLM_API int blm_retention_step_takes(int dk, int dv) { return dk <= 2048 && (dv % 4 == 0 ? dv <= 4 * kStepThreads : dv <= kStepThreads); }
+BLM_API int blm_retention_power_row() { return kC + 1; }
+BLM_API int blm_retention_chunks(int n_tokens, int n_seqs) { return (n_tokens + kC - 1) / kC + n_seqs; }
+
+#define RET_ARGS                                                                                                                          \
+    const float *proj, long long stride, int heads, int dk, int dv, float k_scale, const double *freq, int rot, const float *table,      \
+        int table_len, const float *powers, const int *cu_seqlens, const int *slot_of_seq, const int *start_pos, int n_seqs, float *state, \
+        long long slot_stride, long long copy_stride, long long offset
+#define RET_CHECK(what)                                                                                                                   \
+    BLM_REQUIRE(heads > 0 && heads <= 65535 && dk > 0 && dv > 0 && n_seqs >= 0 && n_seqs <= 65535, what ": bad sizes");                  \
+    BLM_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dk && (rot == 0 || freq != nullptr), what ": %d turning lanes of %d", rot, dk);       \
+    BLM_REQUIRE(stride >= (long long)heads * (2 * dk + 2 * dv) && powers != nullptr && state != nullptr, what ": rows of %lld", stride); \
+    const RetIn in{proj, stride, heads, dk, dv, k_scale, freq, rot, (const float2*)table, table ? table_len : 0, powers};                \
+    const RetSeq sq{cu_seqlens, slot_of_seq, start_pos, n_seqs, state, slot_stride, copy_stride, offset};                                \
+    const int vec = ret_vec(in) && (((size_t)state | (size_t)table) & 15) == 0 && slot_stride % 4 == 0 && copy_stride % 4 == 0 && offset % 4 == 0
+
+// o [N, heads * dv] float32, not normed yet; rows of no sequence are left alone
+BLM_API int blm_retention_scan(RET_ARGS, float* o, long long o_stride, cudaStream_t stream) {
+    if (n_seqs == 0) return BLM_OK;
+    RET_CHECK("retention_scan");
+    (void)vec;
+    BLM_REQUIRE(dk <= 512 && dv <= 65535, "retention_scan: keys of %d lanes; at most 512", dk);
+    const size_t smem = (size_t)kScanTokens * (2 * dk + 32) * sizeof(float);
+    const dim3 grid((dv + 31) / 32, heads, n_seqs);
+    auto launch = [&](auto kernel) -> int {
+        if (smem > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "retention_scan: %s", cudaGetErrorString(e));
+        }
+        kernel<<<grid, 256, smem, stream>>>(in, sq, o, o_stride);
+        return blm_check_launch("retention_scan");
+    };
+    if (dk <= 16) return launch(retention_scan_kernel<2>);
+    if (dk <= 32) return launch(retention_scan_kernel<4>);
+    if (dk <= 64) return launch(retention_scan_kernel<8>);
+    if (dk <= 128) return launch(retention_scan_kernel<16>);
+    if (dk <= 256) return launch(retention_scan_kernel<32>);
+    return launch(retention_scan_kernel<64>);
+}
+
+// out [N, heads * dv] (rows of out_stride), finished; every sequence brings one token
+BLM_API int blm_retention_step(RET_ARGS, const int* token_seq, const int* token_pos, int n_tokens, float eps, void* out, int out_dtype,
+                               long long out_stride, cudaStream_t stream) {
+    if (n_tokens == 0) return BLM_OK;
+    RET_CHECK("retention_step");
+    BLM_REQUIRE(blm_retention_step_takes(dk, dv) && n_tokens <= 65535, "retention_step: %d tokens, heads of %d and %d lanes", n_tokens, dk, dv);
+    const int n = vec ? 4 : 1;
+    BLM_REQUIRE(dv / n <= kStepThreads, "retention_step: values of %d lanes", dv);
+    const size_t smem = ((size_t)2 * ((dk + 3) & ~3) + 36 + (size_t)(kStepThreads / (dv / n)) * dv) * sizeof(float);
+    const dim3 grid(heads, n_tokens);
+#define RET_STEP(TO, N) retention_step_kernel<TO, N><<<grid, kStepThreads, smem, stream>>>(in, sq, token_seq, token_pos, eps, (TO*)out, out_stride, vec)
+    if (out_dtype == BLM_BF16) {
+        if (vec) RET_STEP(__nv_bfloat16, 4); else RET_STEP(__nv_bfloat16, 1);
+    } else if (out_dtype == BLM_F32) {
+        if (vec) RET_STEP(float, 4); else RET_STEP(float, 1);
+    } else {
+        return blm_fail(BLM_BAD_ARGUMENT, "retention_step: dtype %d", out_dtype);
+    }
+#undef RET_STEP
+    return blm_check_launch("retention_step");
+}
+
+// out bfloat16 as above, any number of tokens a sequence; kv: float32 scratch [blm_retention_chunks(...)][heads][dk][dv]
+BLM_API int blm_retention_portions(RET_ARGS, int n_tokens, float eps, float* kv, void* out, long long out_stride, cudaStream_t stream) {
+    if (n_tokens == 0) return BLM_OK;
+    RET_CHECK("retention_portions");
+    const int slice = chunk_slice(dk, dv), chunks = blm_retention_chunks(n_tokens, n_seqs);
+    BLM_REQUIRE(slice > 0 && kv != nullptr && ((size_t)kv & 15) == 0, "retention_portions: heads of %d and %d lanes", dk, dv);
+    const size_t smem1 = ((size_t)2 * kC * (((dk + 15) & ~15) + 8) + (size_t)kC * (((dv + 63) & ~63) + 8)) * sizeof(__nv_bfloat16);
+    const size_t smem3 = chunk_smem(dk, dv, slice);
+    static size_t allowed1 = 48 * 1024;
+    if (smem1 > allowed1) {
+        cudaError_t e = cudaFuncSetAttribute(retention_chunk_add_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "retention_portions: %s", cudaGetErrorString(e));
+        allowed1 = smem1;
+    }
+    const dim3 grid(chunks, heads);
+    retention_chunk_add_kernel<<<grid, 256, smem1, stream>>>(in, sq, kv, vec);
+    const size_t size = (size_t)dk * dv;
+    const bool four = size % 4 == 0 && (((size_t)state) & 15) == 0 && slot_stride % 4 == 0 && copy_stride % 4 == 0 && offset % 4 == 0;
+    if (four) retention_carry_kernel<4><<<dim3((unsigned)((size / 4 + 255) / 256), heads, n_seqs), 256, 0, stream>>>(in, sq, kv);
+    else retention_carry_kernel<1><<<dim3((unsigned)((size + 255) / 256), heads, n_seqs), 256, 0, stream>>>(in, sq, kv);
+    const int warps = 4 * ((dv + 63) / 64);
+    auto rows = [&](auto kernel) -> int {
+        if (smem3 > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+            if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "retention_portions: %s", cudaGetErrorString(e));
+        }
+        kernel<<<grid, 32 * warps, smem3, stream>>>(in, sq, kv, slice, eps, (__nv_bfloat16*)out, out_stride, n_tokens, vec);
+        return blm_check_launch("retention_portions");
+    };
+    if (warps <= 4) return rows(retention_chunk_out_kernel<4>);
+    if (warps <= 8) return rows(retention_chunk_out_kernel<8>);
+    if (warps <= 16) return rows(retention_chunk_out_kernel<16>);
+    return rows(retention_chunk_out_kernel<32>);
+}

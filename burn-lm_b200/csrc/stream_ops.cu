@@ -220,20 +220,20 @@ BLM_API int blm_pack_cols(float* src, const void* delta, int delta_dtype, void* 
 }
 
 // ---------------------------------------------------------------------------------------------
-// x <- cap * tanh(x / cap) in place (fp32): logits squashed into (-cap, cap)
+// x <- cap * tanh(scale * x / cap) in place (fp32): scaled logits squashed into (-cap, cap); cap 0: x <- scale * x
 // ---------------------------------------------------------------------------------------------
-__global__ void softcap_kernel(float* __restrict__ x, float cap, size_t total) {
+__global__ void softcap_kernel(float* __restrict__ x, float scale, float cap, size_t total) {
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
-        x[i] = cap * tanhf(x[i] / cap);
+        x[i] = cap > 0.f ? cap * tanhf(scale * x[i] / cap) : scale * x[i];
 }
 
-BLM_API int blm_softcap(float* x, float cap, size_t total, cudaStream_t stream) {
+BLM_API int blm_softcap(float* x, float scale, float cap, size_t total, cudaStream_t stream) {
     if (total == 0) return BLM_OK;
-    BLM_REQUIRE(cap > 0.f, "softcap: the cap must be positive");
+    BLM_REQUIRE(cap >= 0.f, "softcap: a cap of %g", (double)cap);
     const int threads = 256;
     const size_t want = (total + threads - 1) / threads;
     const int blocks = (int)(want < 65535u * 16u ? want : 65535u * 16u);
-    softcap_kernel<<<blocks, threads, 0, stream>>>(x, cap, total);
+    softcap_kernel<<<blocks, threads, 0, stream>>>(x, scale, cap, total);
     return blm_check_launch("softcap");
 }
 

@@ -70,15 +70,20 @@ def _need_cuda(*tensors):
             raise KernelError("kernel arguments must be contiguous")
 
 
+# the projection and its turn, then the step's sequences and their states
+_RETENTION = [c_void_p, c_longlong, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+              c_int, c_void_p, c_longlong, c_longlong, c_longlong]
 _protos = {
     "elementwise": {
         "blm_embed": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p],
         "blm_add_rmsnorm": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int,
                             c_float, c_void_p],
+        "blm_add_rmsnorm_parts": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                                  c_void_p, c_int, c_int, c_float, c_void_p],
         "blm_rope_append": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                             c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p],
         "blm_rope_table": [c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
-        "blm_swiglu": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "blm_swiglu": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p],
         "blm_convert": [c_void_p, c_int, c_void_p, c_int, c_size_t, c_void_p],
         "blm_decode_advance": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "blm_step_tables": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
@@ -95,10 +100,10 @@ _protos = {
         "blm_attention_sink": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                c_void_p, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_float, c_void_p, c_int, c_int,
                                c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_float,
-                               c_float, c_float, c_float, c_int, c_void_p, c_void_p],
+                               c_void_p, c_int, c_float, c_float, c_float, c_int, c_void_p, c_void_p],
         "blm_head_norm_rope_append": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
                                       c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
-                                      c_void_p, c_void_p, c_int, c_void_p],
+                                      c_void_p, c_void_p, c_int, c_void_p, c_float, c_int, c_int, c_void_p],
         "blm_attention_sink_prompt_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
         "blm_attention_sink_decode_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
         "blm_attention_sink_pairs": [c_int, c_int, c_int, c_int, c_int, c_int, c_int],
@@ -111,7 +116,7 @@ _protos = {
         "blm_weighted_sum": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_size_t, c_void_p],
         "blm_pack_cols": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p],
         "blm_pass_entry": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
-        "blm_softcap": [c_void_p, c_float, c_size_t, c_void_p],
+        "blm_softcap": [c_void_p, c_float, c_float, c_size_t, c_void_p],
     },
     "recurrent": {
         "blm_causal_conv": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_longlong, c_int,
@@ -135,6 +140,15 @@ _protos = {
         "blm_take_cols": [c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
         "blm_gated_group_norm": [c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                  c_float, c_void_p, c_int, c_longlong, c_int, c_void_p],
+    },
+    "retention": {
+        "blm_retention_scan": _RETENTION + [c_void_p, c_longlong, c_void_p],
+        "blm_retention_step": _RETENTION + [c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_longlong, c_void_p],
+        "blm_retention_portions": _RETENTION + [c_int, c_float, c_void_p, c_void_p, c_longlong, c_void_p],
+        "blm_retention_chunks_take": [c_int, c_int],
+        "blm_retention_step_takes": [c_int, c_int],
+        "blm_retention_power_row": [],
+        "blm_retention_chunks": [c_int, c_int],
     },
     "attention_sigmoid": {
         "blm_bias_rope_append": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
@@ -183,7 +197,7 @@ _protos = {
     },
     "gemv": {
         "blm_gemv": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int,
-                     c_float, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p, c_int,
+                     c_float, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int,
                      c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
         "blm_gemv_supported": [c_int, c_int, c_int, c_int],
     },
@@ -311,6 +325,27 @@ def add_rmsnorm(resid, delta, gamma, eps, out, rows=None):
           _code(out.dtype), _ptr(rows), n_out, d, c_float(eps), _stream())
 
 
+def add_rmsnorm_parts(resid, outputs, biases, gamma, eps, out, rows=None):
+    """add_rmsnorm for a pending sum of several parts: up to two `outputs` (float32 or bfloat16 [N, D]) and up to two `biases`
+    (float32 [D]) join the stream.  gamma and out None: only the sum."""
+    outputs, biases = list(outputs), list(biases)
+    _need_cuda(resid, gamma, out, rows, *outputs, *biases)
+    d = resid.shape[-1]
+    n_out = rows.numel() if rows is not None else resid.shape[0]
+    if len(outputs) > 2 or len(biases) > 2 or resid.dtype != torch.float32 or (gamma is None) != (out is None):
+        raise KernelError("add_rmsnorm_parts: up to two outputs and two biases; resid float32 [N, D]; gamma and out, or neither")
+    if any(o.shape != resid.shape for o in outputs) or any(b.dtype != torch.float32 or b.numel() != d for b in biases):
+        raise KernelError("add_rmsnorm_parts: outputs [N, D], biases float32 [D]")
+    if gamma is not None and (gamma.numel() != d or tuple(out.shape) != (n_out, d)):
+        raise KernelError("add_rmsnorm_parts: gamma [D], out [rows, D]")
+    if rows is not None and rows.dtype != torch.int32:
+        raise KernelError("add_rmsnorm_parts: rows must be int32")
+    os_, bs = outputs + [None] * (2 - len(outputs)), biases + [None] * (2 - len(biases))
+    code = lambda t: _code(t.dtype) if t is not None else F32
+    _call("elementwise", "blm_add_rmsnorm_parts", _ptr(resid), _ptr(os_[0]), code(os_[0]), _ptr(os_[1]), code(os_[1]), _ptr(bs[0]), _ptr(bs[1]),
+          _ptr(gamma), code(gamma), _ptr(out), code(out), _ptr(rows), n_out, d, c_float(eps), _stream())
+
+
 def embed_pairs(tokens, table, pairs, out, step, ids_pool, block_table, buckets, mul_prev, mul_cur, norm=None):
     """out[n] = table[tokens[n]] + pairs[(previous token * mul_prev + token * mul_cur) mod buckets] as fp32 (the row
     `buckets` for a sequence's first token), then, with `norm` = (weight, bias, alpha) in float32, tanh(alpha x) * weight
@@ -370,9 +405,9 @@ def kv_page_elems(n_kv, key_dim, value_dim) -> int:
     return n_kv * PAGE * (key_dim + value_dim)
 
 
-def _flat_pool(pool, n_kv, key_dim, value_dim, maps=1):
-    """Elements of a page of n_kv key heads (every map counted) and n_kv / maps value heads."""
-    elems = kv_page_elems(n_kv // maps, maps * key_dim, value_dim)
+def _flat_pool(pool, n_kv, key_dim, value_dim, maps=1, shared=False):
+    """Elements of a page of n_kv key heads (every map counted) and n_kv / maps value heads (`shared`: of the keys alone)."""
+    elems = kv_page_elems(n_kv // maps, maps * key_dim, 0 if shared else value_dim)
     if not pool.is_contiguous() or pool.numel() != pool.shape[0] * elems:
         raise KernelError(f"the cache pool must hold pages of {elems} elements ({n_kv} kv heads, keys of {key_dim}, values of {value_dim})")
     return elems
@@ -402,7 +437,8 @@ def qk_norm_append(proj, step, pool, block_table, q_out, n_heads, n_kv, key_dim,
 
 
 def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, key_dim, value_dim, q_weight=None, k_weight=None,
-                          eps=0.0, value_norm=False, freq=None, rotary_dims=0, halves=False, turn_scale=1.0, maps=1, table=None):
+                          eps=0.0, value_norm=False, freq=None, rotary_dims=0, halves=False, turn_scale=1.0, maps=1, table=None, bias=None,
+                          temperature=None, shared=False):
     """What follows a fused projection [q | k | v | ...] (float32 [N, >= (n_heads + n_kv) key_dim + n_kv value_dim]), head by
     head: every head of q is divided by its root mean square (eps inside the root) and multiplied by `q_weight` (float32
     [key_dim], the same for all heads; None: q stays as it is), every head of k likewise with `k_weight`; the first
@@ -411,15 +447,20 @@ def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, k
     of v is divided by its root mean square (no weight).  q goes to `q_out` [N, n_heads key_dim], k and v to the token's place
     in the paged cache.  `maps` 2: a head has two queries and two keys, [head][map][key_dim], over one value; n_heads and
     n_kv count every map.  `table` (from rope_table, with the same turn_scale) spares the angles of the positions it covers.
-    `proj` may be a column range of a wider tensor."""
-    _need_cuda(pool, block_table, q_out, q_weight, k_weight, freq, table)
-    _f32(proj, q_weight, k_weight, table)
+    `proj` may be a column range of a wider tensor.  `bias` (float32, a number per column of q, k and v) joins the projection
+    first; `temperature` = (coef, every) multiplies q by 1 + coef ln(floor((position + 1) / every) + 1).  `shared`: the values
+    are the keys, the projection is [q | k | ...] and a page holds the keys alone."""
+    _need_cuda(pool, block_table, q_out, q_weight, k_weight, freq, table, bias)
+    _f32(proj, q_weight, k_weight, table, bias)
     if table is not None and tuple(table.shape[1:]) != (rotary_dims // 2, 2):
         raise KernelError("head_norm_rope_append: the table is float32 [positions, rotary_dims / 2, 2]")
     if not proj.is_cuda:
         raise KernelError("burn-lm_b200 kernels run on a CUDA device only; got a CPU tensor")
     n = proj.shape[0]
-    qc, kc, vc = n_heads * key_dim, n_kv * key_dim, n_kv // maps * value_dim
+    qc, kc, vc = n_heads * key_dim, n_kv * key_dim, 0 if shared else n_kv // maps * value_dim
+    if bias is not None and bias.numel() != qc + kc + vc:
+        raise KernelError("head_norm_rope_append: the bias has a number per column of q, k and v")
+    coef, every = temperature or (0.0, 0)
     if proj.dim() != 2 or proj.shape[1] < qc + kc + vc or proj.stride(1) != 1:
         raise KernelError("head_norm_rope_append: the projection is float32 [N, q + k + v (+ more)]")
     if tuple(q_out.shape) != (n, qc) or q_out.dtype != pool.dtype or not q_out.is_contiguous():
@@ -431,8 +472,9 @@ def head_norm_rope_append(proj, step, pool, block_table, q_out, n_heads, n_kv, k
         raise KernelError("head_norm_rope_append: freq must be float64 [rotary_dims / 2]")
     _call("attention_sink", "blm_head_norm_rope_append", _ptr(proj), c_longlong(proj.stride(0)), n, n_heads, n_kv, int(maps), key_dim,
           value_dim, _ptr(q_weight), _ptr(k_weight), c_float(eps), 1 if value_norm else 0, _ptr(freq), int(rotary_dims), 1 if halves else 0,
-          c_float(turn_scale), _ptr(table), table.shape[0] if table is not None else 0, _ptr(q_out), _ptr(pool), _code(pool.dtype), c_longlong(_flat_pool(pool, n_kv, key_dim, value_dim, maps)), PAGE, _ptr(step.token_seq),
-          _ptr(step.token_pos), _ptr(step.slot_of_seq), _ptr(block_table), block_table.shape[1], _stream())
+          c_float(turn_scale), _ptr(table), table.shape[0] if table is not None else 0, _ptr(q_out), _ptr(pool), _code(pool.dtype), c_longlong(_flat_pool(pool, n_kv, key_dim, value_dim, maps, shared)), PAGE,
+          _ptr(step.token_seq), _ptr(step.token_pos), _ptr(step.slot_of_seq), _ptr(block_table), block_table.shape[1], _ptr(bias), c_float(coef),
+          int(every), 1 if shared else 0, _stream())
 
 
 def attention_sink_pairs(dtype, key_dim, value_dim, n_heads, n_kv, maps) -> bool:
@@ -459,7 +501,7 @@ def attention_sink_decode_takes(dtype, key_dim, value_dim, n_heads, n_kv) -> boo
 
 def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, value_dim, scale, window, keep_first=0, sink=True,
                    gate=None, gate_stride=0, max_q_len=1, n_splits=1, scratch=None, head_scale=None, sink_logit=None, softcap=0.0,
-                   chunk=0, gate_lanes=0, out_scale=1.0, maps=1, difference=(0.0, 1.0, 0.0)):
+                   chunk=0, gate_lanes=0, out_scale=1.0, maps=1, difference=(0.0, 1.0, 0.0), slope=None, shared=False):
     """Attention of the step's tokens over the paged cache (after the append) where the query at position i sees the
     key at j when j <= i and (i - j < window or j < keep_first); softmax with `sink` added to its denominator (one more
     entry of score 0 without a value); keys of `key_dim` and values of `value_dim` lanes; `gate`: a float32 tensor
@@ -474,6 +516,8 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
     `maps` 2, differential attention: a head has two queries and a key/value head two keys, [head][map][key_dim], over one
     value; n_heads and n_kv count every map, out is [N, n_heads / 2 value_dim], and `difference` = (lambda, c, eps) gives
     o = a_1 - lambda a_2, out = o / sqrt(mean(o^2) + eps) * c per head; it needs `scratch` for any n_splits.
+    `slope` float32 [n_heads]: slope[h] * (the query's position - the key's) is taken off head h's scores (after the cap).
+    `shared`: the values are the keys (as many lanes), and a page holds the keys alone.
 
     `max_q_len`: the longest run of new tokens of one sequence (a bound is enough): bfloat16 steps of 8 or more run
     the tensor-core prompt kernel, 64 query rows a block (it reads step.cu_seqlens and step.start_pos), and steps of 64 or
@@ -481,13 +525,13 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
     the tensor-core decode kernel (bfloat16, up to 16 query heads a kv head) or else the row kernel, a block per (row,
     kv head) either, whose keys `n_splits` > 1 cuts over that many blocks (it then needs `scratch`:
     attention_sink_scratch_floats(...) float32)."""
-    _need_cuda(q, pool, block_table, scratch, head_scale, sink_logit)
-    _f32(head_scale, sink_logit)
+    _need_cuda(q, pool, block_table, scratch, head_scale, sink_logit, slope)
+    _f32(head_scale, sink_logit, slope)
     if not out.is_cuda or out.stride(1) != 1:
         raise KernelError("attention_sink: out is a CUDA tensor with unit stride along its rows")
-    for t in (head_scale, sink_logit):
+    for t in (head_scale, sink_logit, slope):
         if t is not None and t.numel() != n_heads:
-            raise KernelError("attention_sink: head_scale and sink_logit have a number per query head")
+            raise KernelError("attention_sink: head_scale, sink_logit and slope have a number per query head")
     n = q.shape[0]
     if tuple(q.shape) != (n, n_heads * key_dim) or tuple(out.shape) != (n, n_heads // maps * value_dim) or q.dtype != pool.dtype \
             or out.dtype != pool.dtype:
@@ -503,12 +547,13 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"attention_sink: {n_splits} splits need {need} float32 of scratch")
     cu = step.cu_seqlens if prompt else None
-    _call("attention_sink", "blm_attention_sink", _ptr(q), _ptr(pool), _code(pool.dtype), _flat_pool(pool, n_kv, key_dim, value_dim, maps),
+    _call("attention_sink", "blm_attention_sink", _ptr(q), _ptr(pool), _code(pool.dtype), _flat_pool(pool, n_kv, key_dim, value_dim, maps, shared),
           _ptr(block_table), block_table.shape[1], _ptr(step.token_seq), _ptr(step.token_pos), _ptr(step.slot_of_seq), _ptr(cu),
           _ptr(step.start_pos if prompt else None), (cu.numel() - 1) if prompt else 0, int(max_q_len), _ptr(gate), int(gate_stride),
           int(gate_lanes), _ptr(out), c_longlong(out.stride(0)), c_float(out_scale), _ptr(scratch if need else None), int(n_splits), n, n_heads,
           n_kv, int(maps), key_dim, value_dim, PAGE, int(window), int(chunk), int(keep_first), c_float(scale), 1 if sink else 0,
-          _ptr(head_scale), _ptr(sink_logit if sink else None), c_float(softcap or 0.0), *(c_float(v) for v in difference),
+          _ptr(head_scale), _ptr(sink_logit if sink else None), c_float(softcap or 0.0), _ptr(slope), 1 if shared else 0,
+          *(c_float(v) for v in difference),
           pool.shape[0] if prompt else 0, _ptr(status_word(q.device)) if prompt else None, _stream(),
           kernels=2 if need else 1)
 
@@ -685,12 +730,14 @@ GATE_TILE = 8   # a fused [gate; up] weight for the skinny kernel: tiles of 8 ga
 
 def swiglu(gate_up, out, tile=0):
     """out[n, i] = silu(gate_i) * up_i.  gate_up [N, 2 I] holds all gates then all ups (tile 0), or
-    tiles of `tile` gates followed by the ups of the same outputs."""
-    _need_cuda(gate_up, out)
+    tiles of `tile` gates followed by the ups of the same outputs.  `out` may be a column range of a wider tensor."""
+    _need_cuda(gate_up)
+    if not out.is_cuda or out.stride(1) != 1:
+        raise KernelError("swiglu: out is a CUDA tensor with unit stride along its rows")
     n, two_i = gate_up.shape
     if tuple(out.shape) != (n, two_i // 2) or out.dtype != gate_up.dtype or two_i % 2:
         raise KernelError("swiglu: out must be [N, I] for gate_up [N, 2 I], same dtype")
-    _call("elementwise", "blm_swiglu", _ptr(gate_up), _ptr(out), _code(out.dtype), n, two_i // 2, tile, _stream())
+    _call("elementwise", "blm_swiglu", _ptr(gate_up), _ptr(out), c_longlong(out.stride(0)), _code(out.dtype), n, two_i // 2, tile, _stream())
 
 
 def convert(src, dst):
@@ -837,7 +884,9 @@ def gemm_tc(x, w, out=None, swiglu=False, add_into=None, relu2=False):
     rows followed by their up rows and out [M, N / 2] = silu(gate) * up, formed in the epilogue; with
     `add_into` (float32 [M, N], the residual stream) the product is added into it in the epilogue and
     nothing else is written; with `relu2` out = relu(product)^2."""
-    _need_cuda(x, w, out, add_into)
+    _need_cuda(x, w, add_into)
+    if out is not None and (not out.is_cuda or out.stride(1) != 1):
+        raise KernelError("gemm_tc: out is a CUDA tensor with unit stride along its rows")
     m, k = x.shape
     n = w.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != k:
@@ -987,7 +1036,7 @@ SQUARES_ROWS = 16     # row length of the sums of squares that go with a handed-
 
 
 def gemv(w, n_tokens, x=None, stream_rows=None, gamma=None, eps=0.0, rows=None, out=None, add_into=None, swiglu=False,
-         squares=None, hand_over=None, rope=None, relu2=False):
+         squares=None, hand_over=None, rope=None, relu2=False, add_bias=None):
     """Skinny product of n_tokens <= 16 tokens with a bfloat16 weight [M, K], with fused ends.
 
     Input: `x` bfloat16 [N, K], or the fp32 residual stream `stream_rows` [*, K] to be RMS-normalised
@@ -997,7 +1046,7 @@ def gemv(w, n_tokens, x=None, stream_rows=None, gamma=None, eps=0.0, rows=None, 
     Output: `out` [N, M] bfloat16 or float32 (with `relu2`: relu of the product, squared);
     with `swiglu` the weight is [2 I, K] in tiles of GATE_TILE gate rows followed by the up rows of the
     same outputs, and out [N, I] = silu(gate) * up; with
-    `add_into` (fp32 [N, M]) the product is added into it and nothing else is written, unless
+    `add_into` (fp32 [N, M]) the product (and `add_bias`, fp32 [M]) is added into it and nothing else is written, unless
     `hand_over` = (gamma, scaled, squares) asks for the next norm's input as well: scaled
     (bfloat16 [N, M]) = the new stream times gamma, squares (fp32 [ceil(M / 16), SQUARES_ROWS]) its
     sums of squares by tiles of 16 lanes.
@@ -1006,7 +1055,10 @@ def gemv(w, n_tokens, x=None, stream_rows=None, gamma=None, eps=0.0, rows=None, 
     write_cache) whose q and k heads have their rows in tiled_pair_order(): q and k are rotated by their
     token's position, q goes to `out` [N, n_heads * head_dim] (lanes in that order), the rotated k and the
     v to the token's place in `pool`."""
-    _need_cuda(w, x, stream_rows, gamma, rows, out, add_into, squares)
+    for t in (x, out):                 # rows of wider tensors: a column range of 16-byte aligned rows
+        if t is not None and (not t.is_cuda or t.dim() != 2 or t.stride(1) != 1):
+            raise KernelError("gemv: x and out are CUDA tensors with unit stride along their rows")
+    _need_cuda(w, stream_rows, gamma, rows, add_into, squares, add_bias)
     m_rows, k = w.shape
     if w.dtype != torch.bfloat16:
         raise KernelError("gemv: the weight must be bfloat16")
@@ -1055,6 +1107,8 @@ def gemv(w, n_tokens, x=None, stream_rows=None, gamma=None, eps=0.0, rows=None, 
     if epi == EPI_RESID_ADD:
         if add_into.dtype != torch.float32 or tuple(add_into.shape) != (n_tokens, m):
             raise KernelError("gemv: add_into must be float32 [N, M]")
+        if add_bias is not None and (add_bias.dtype != torch.float32 or add_bias.numel() != m):
+            raise KernelError("gemv: add_bias must be float32 [M]")
     elif epi == EPI_ROPE:
         pass
     elif out is None or tuple(out.shape) != (n_tokens, m) or out.dtype not in (torch.bfloat16, torch.float32) \
@@ -1063,7 +1117,7 @@ def gemv(w, n_tokens, x=None, stream_rows=None, gamma=None, eps=0.0, rows=None, 
     _call("gemv", "blm_gemv", _ptr(w), w.stride(0), m, k, _ptr(x), x.stride(0) if x is not None else 0,
           _ptr(stream_rows), _ptr(gamma), 1 if (gamma is not None and gamma.dtype == torch.float32) else 0, c_float(eps),
           _ptr(rows), n_tokens, _ptr(out), out.stride(0) if out is not None else 0,
-          1 if (out is not None and out.dtype == torch.float32) else 0, _ptr(add_into), epi,
+          1 if (out is not None and out.dtype == torch.float32) else 0, _ptr(add_into), _ptr(add_bias), epi,
           _ptr(squares), squares.shape[0] if squares is not None else 0,
           _ptr(next_gamma), 1 if (next_gamma is not None and next_gamma.dtype == torch.float32) else 0,
           _ptr(scaled), _ptr(squares_out), ctypes.byref(rope_arg) if rope_arg is not None else None,
@@ -1411,14 +1465,85 @@ def gated_group_norm(y, gate, gate_col0, weight, group, mode, eps, out):
     weight; GATE_LAST: out = y / rms(y) * weight * sigmoid(gate); GATE_SILU_LAST: ... * silu(gate); GATE_NONE: no gate
     (`gate` None).  weight float32 of a row's or of a group's size (then
     shared by the groups); y float32 [N, C]; the gate a column range of a float32 tensor; out [N, C]."""
-    _need_cuda(y, weight, out)
+    _need_cuda(y, weight)
     _f32(y, weight)
     n, c = y.shape
-    if c % group or weight.numel() not in (c, group) or tuple(out.shape) != (n, c) or not y.is_contiguous() or not out.is_contiguous():
+    if c % group or weight.numel() not in (c, group) or tuple(out.shape) != (n, c) or not y.is_contiguous() or not out.is_cuda or out.stride(1) != 1:
         raise KernelError("gated_group_norm: groups must divide the row; weight of a row's or a group's size")
     gp, gs, gc = _cols(gate, gate_col0, c) if gate is not None else (c_void_p(0), c_longlong(0), 0)
     _call("recurrent", "blm_gated_group_norm", _ptr(y), c_longlong(y.stride(0)), gp, gs, gc, _ptr(weight), weight.numel(), group,
           c // group, int(mode), c_float(eps), _ptr(out), _code(out.dtype), c_longlong(out.stride(0)), n, _stream())
+
+
+# ------------------------------------------------------------------------------------------------
+# retention
+# ------------------------------------------------------------------------------------------------
+RETENTION_CHUNK = 64        # tokens of a chunk of the portions' kernels
+
+
+def retention_powers(decay) -> torch.Tensor:
+    """float32 [heads, RETENTION_CHUNK + 1]: every head's decay to the powers 0, 1, ..., worked out in float64."""
+    d = torch.tensor(list(decay), dtype=torch.float64).reshape(-1, 1)
+    return torch.pow(d, torch.arange(RETENTION_CHUNK + 1, dtype=torch.float64)).to(torch.float32).contiguous()
+
+
+def _retention_args(what, proj, step, state, state_offset, heads, key_dim, value_dim, k_scale, powers, freq, rotary_dims, table):
+    _need_cuda(powers, freq, table, state)
+    _f32(proj, powers, table)
+    if not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1 or proj.shape[1] < 2 * heads * (key_dim + value_dim):
+        raise KernelError(f"{what}: the projection is float32 [N, q | k | v | g] on a CUDA device")
+    if tuple(powers.shape) != (heads, RETENTION_CHUNK + 1):
+        raise KernelError(f"{what}: powers are retention_powers(decay)")
+    if rotary_dims and (freq is None or freq.dtype != torch.float64 or freq.numel() != rotary_dims // 2):
+        raise KernelError(f"{what}: freq must be float64 [rotary_dims / 2]")
+    if table is not None and tuple(table.shape[1:]) != (rotary_dims // 2, 2):
+        raise KernelError(f"{what}: the table is float32 [positions, rotary_dims / 2, 2]")
+    ptr, slot_stride, copy_stride, offset = _state_args(state, state_offset)
+    if state_offset + heads * key_dim * value_dim > state.shape[2]:
+        raise KernelError(f"{what}: a state copy of {state.shape[2]} floats is too small")
+    return [_ptr(proj), c_longlong(proj.stride(0)), heads, key_dim, value_dim, c_float(k_scale), _ptr(freq), int(rotary_dims), _ptr(table),
+            table.shape[0] if table is not None else 0, _ptr(powers), _ptr(step.cu_seqlens), _ptr(step.slot_of_seq), _ptr(step.start_pos),
+            step.n_seqs, ptr, slot_stride, copy_stride, offset]
+
+
+def retention_chunks_take(key_dim, value_dim) -> bool:
+    """Whether portions with heads of these sizes run by chunks on the tensor cores (bfloat16; else the scan)."""
+    return bool(_lib("retention").blm_retention_chunks_take(key_dim, value_dim))
+
+
+def retention_step_takes(key_dim, value_dim) -> bool:
+    return bool(_lib("retention").blm_retention_step_takes(key_dim, value_dim))
+
+
+def retention_scan(proj, step, state, state_offset, heads, key_dim, value_dim, k_scale, powers, o, freq=None, rotary_dims=0, table=None):
+    """Retention over the step's tokens, in order, sums in float64 inside the step: per head S <- a S + k v^T, o = S^T q, with q
+    and k turned (lanes (i, i + rotary_dims / 2) by position * freq[i]) and k times k_scale.  proj float32 [N, q | k | v | g];
+    o float32 [N, heads * value_dim], not normed (rows of no sequence are left alone); S in `state` (float32 [slots, 2, floats])
+    at state_offset, [head][key_dim][value_dim]."""
+    args = _retention_args("retention_scan", proj, step, state, state_offset, heads, key_dim, value_dim, k_scale, powers, freq, rotary_dims, table)
+    _need_cuda(o)
+    if o.dtype != torch.float32 or tuple(o.shape) != (proj.shape[0], heads * value_dim):
+        raise KernelError("retention_scan: o is float32 [N, heads * value_dim]")
+    _call("retention", "blm_retention_scan", *args, _ptr(o), c_longlong(o.stride(0)), _stream())
+
+
+def retention(proj, step, state, state_offset, heads, key_dim, value_dim, k_scale, powers, eps, out, freq=None, rotary_dims=0, table=None):
+    """Retention as above, finished: out [N, heads * value_dim] (may be a column range) = o / sqrt(mean(o^2) + eps) * silu(g) head
+    by head.  Steps in which every sequence brings one token (step.max_q_len == 1) run one kernel; other steps run by chunks of
+    RETENTION_CHUNK tokens (bfloat16 out only)."""
+    args = _retention_args("retention", proj, step, state, state_offset, heads, key_dim, value_dim, k_scale, powers, freq, rotary_dims, table)
+    n = proj.shape[0]
+    if not out.is_cuda or tuple(out.shape) != (n, heads * value_dim) or out.stride(1) != 1:
+        raise KernelError("retention: out is a CUDA tensor [N, heads * value_dim] with unit stride along its rows")
+    if step.max_q_len == 1:
+        _call("retention", "blm_retention_step", *args, _ptr(step.token_seq), _ptr(step.token_pos), n, c_float(eps), _ptr(out), _code(out.dtype),
+              c_longlong(out.stride(0)), _stream())
+        return
+    if out.dtype != torch.bfloat16:
+        raise KernelError("retention: portions by chunks write bfloat16")
+    chunks = int(_lib("retention").blm_retention_chunks(n, step.n_seqs))
+    kv = torch.empty(chunks * heads * key_dim * value_dim, dtype=torch.float32, device=proj.device)
+    _call("retention", "blm_retention_portions", *args, n, c_float(eps), _ptr(kv), _ptr(out), c_longlong(out.stride(0)), _stream(), kernels=3)
 
 
 # ------------------------------------------------------------------------------------------------
@@ -1606,11 +1731,11 @@ def pack_cols(src, delta, dst, col0):
           _code(dst.dtype), c_longlong(dst.stride(0)), int(col0), n, d, _stream())
 
 
-def softcap(x, cap: float):
-    """x <- cap * tanh(x / cap) in place; x float32."""
+def softcap(x, cap: float = 0.0, scale: float = 1.0):
+    """x <- cap * tanh(scale * x / cap) in place (cap 0: scale * x); x float32."""
     _need_cuda(x)
     _f32(x)
-    _call("stream_ops", "blm_softcap", _ptr(x), c_float(cap), c_size_t(x.numel()), _stream())
+    _call("stream_ops", "blm_softcap", _ptr(x), c_float(scale), c_float(cap), c_size_t(x.numel()), _stream())
 
 
 def pass_entry(resid, delta, embedded, step):

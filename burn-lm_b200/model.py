@@ -99,6 +99,9 @@ class Model:
     def bind(self, loaded: dict):
         for p in self.parts():
             p.bind(loaded)
+        for layer in self.layers:
+            if hasattr(layer.block, "bound"):
+                layer.block.bound()                # a block may join its parts' weights
         # a run that reads another run's cache line must agree with its writer on how the entries lie there
         for run, e in enumerate(self.plan.schedule):
             if e.cache_of is not None:
@@ -164,8 +167,12 @@ class Model:
         delta = None
         for run, entry in enumerate(schedule):
             if entry.before is not None:
-                resid = self.stream_parts[entry.before].forward(resid, delta, embedded, step)
-                delta = None
+                part = self.stream_parts[entry.before]
+                if getattr(part, "passes_pending", False):
+                    delta = part.join(delta)
+                else:
+                    resid = part.forward(resid, delta, embedded, step)
+                    delta = None
                 if step.handoff is not None:
                     step.handoff.expect(None)      # nothing left for a norm fits the new stream
             block = self.layers[entry.layer].block
@@ -173,6 +180,9 @@ class Model:
                 # the norm that reads the stream after this block: the next run's first, or the last norm
                 after = self.layers[schedule[run + 1].layer].block if run + 1 < len(schedule) else None
                 next_norm = self.final_norm if after is None else (after.first_norm() if hasattr(after, "first_norm") else None)
+                before = schedule[run + 1].before if after is not None else None
+                if before is not None and not getattr(self.stream_parts[before], "passes_pending", False):
+                    next_norm = None               # a stream part rewrites the stream first
                 delta = block.forward(resid, delta, step, cache.view(run), next_norm=next_norm)
             else:
                 delta = block.forward(resid, delta, step, cache.view(run))

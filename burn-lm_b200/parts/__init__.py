@@ -2,7 +2,7 @@
 embedding and head.  Importing this package registers the built-in kinds."""
 from .base import CacheNeed, Part, Runtime, StepContext
 from .linear import Linear
-from .norm import DynamicTanh, DynamicTanhSpec, PostNormed, PostRMSNorm, PostRMSNormSpec, RMSNorm, RMSNormSpec
+from .norm import DynamicTanh, DynamicTanhSpec, PendingSum, PostNormed, PostRMSNorm, PostRMSNormSpec, RMSNorm, RMSNormSpec
 from .position import LinearScaling, Llama3Scaling, NoPosition, NoPositionSpec, YarnScaling, rotary_multiplier, Rotary, RotarySpec, rotary_inverse_frequencies
 from .attention import Attention, AttentionSpec
 from .feed_forward import MLP, MLPSpec, BiasedMLP, BiasedMLPSpec, SwiGLU, SwiGLUSpec
@@ -21,6 +21,7 @@ from .hgrn2 import Hgrn2, Hgrn2Spec
 from .wkv import Wkv, WkvSpec
 from .stream import ConcatProjection, ConcatProjectionSpec, PassEntry, PassEntrySpec
 from .normed_attention import NormedAttention, NormedAttentionSpec
+from .retention import Retention, RetentionSpec
 
 __all__ = ["CacheNeed", "Part", "Runtime", "StepContext", "Linear", "RMSNorm", "RMSNormSpec", "Llama3Scaling",
            "NoPosition", "NoPositionSpec", "Rotary", "RotarySpec", "rotary_inverse_frequencies", "Attention",
@@ -31,4 +32,4 @@ __all__ = ["CacheNeed", "Part", "Runtime", "StepContext", "Linear", "RMSNorm", "
            "ParallelMixers", "ParallelMixersSpec", "ShortConv", "ShortConvSpec", "LatentAttention", "LatentAttentionSpec", "Hgrn2",
            "Hgrn2Spec", "Wkv", "WkvSpec", "ConcatProjection", "ConcatProjectionSpec", "NormedAttention", "NormedAttentionSpec",
            "PostNormBlock", "Mamba", "MambaSpec", "PassEntry", "PassEntrySpec", "LinearScaling", "YarnScaling", "rotary_multiplier", "MLP",
-           "MLPSpec"]
+           "MLPSpec", "Retention", "RetentionSpec", "PendingSum"]

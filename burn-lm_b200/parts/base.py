@@ -47,7 +47,7 @@ class CacheNeed:
     """What one run of a mixer keeps per sequence.
 
     kind "kv":    keys and values per position: n_kv_heads x head_dim each (values of `value_dim` lanes when
-                  that is set and differs); `window` None keeps all positions, a number keeps that many of the
+                  that is set and differs; 0: the values are the keys, nothing is kept beside them); `window` None keeps all positions, a number keeps that many of the
                   latest, and beside them the first `keep_first` positions of the sequence; `chunk`: a position looks back to the
                   start of its own chunk of that many positions, counted from the sequence's start.
     kind "rows":  one row of `head_dim` lanes per position in the compute dtype, shared by all heads (a latent that keys

@@ -8,9 +8,12 @@ the block before it (`delta`) and returns its own.
 """
 from __future__ import annotations
 
+import torch
+
 from .. import kernels as K
 from ..registry import register_part
-from .linear import NormHandoff
+from .linear import FUSED_NORM_TOKENS, Linear, NormedStream, NormHandoff
+from .norm import PendingSum
 
 
 def _add_norm(norm, resid, delta, lazy, handoff):
@@ -64,8 +67,14 @@ class PreNormBlock:
 @register_part("block", "parallel")
 class ParallelBlock:
     """h = norm(x); x <- x + (mixer(h) + feed_forward(h)): one norm, and both parts read its output.  The layer
-    may have no feed-forward.  What the parts return is handed, as a tuple, to the norm that reads the stream next
-    when that norm adds several outputs at once (`takes_several`); else it is added into the stream here."""
+    may have no feed-forward.  What the parts return is handed to the norm that reads the stream next when that norm adds several
+    outputs at once (a tuple for one that `takes_several`, a parts.norm.PendingSum for one that `takes_pending_sum`); else it is
+    added into the stream here.
+
+    A mixer and a feed-forward that both offer `before_output`, `output_weight` and `output_bias` run in front of ONE last product:
+    what the two output products would read stands side by side, W_mixer a + W_ff b = [W_mixer | W_ff] [a; b].  For a few tokens
+    that product adds into the stream itself and leaves the next norm's input beside the sum; the norm in front of such a pair may
+    be pending, and each part's first product normalises on the fly."""
     family = "block"
     graph_safe = True
 
@@ -75,33 +84,67 @@ class ParallelBlock:
         if not {"norm", "mixer"} <= set(parts) <= set(self.NAMES):
             raise ValueError(f"the parallel block arranges parts named {self.NAMES} (the last may be absent); the layer has {sorted(parts)}")
         self.norm, self.mixer, self.feed_forward = parts["norm"], parts["mixer"], parts.get("feed_forward")
+        self.joint = self.joint_bias = None
 
     def first_norm(self):
         return self.norm
 
-    def forward(self, resid, delta, step, cache_view, next_norm=None):
-        if getattr(step, "handoff", None) is not None:
-            step.handoff.expect(None)          # no product of this block prepares a norm's input
-        h = self.norm.add_norm(resid, delta)
-        if not isinstance(h, type(resid)):
-            h = h.materialize()                # both parts read it
-        pending = []
-        mixer, ff = self.mixer, self.feed_forward
-        a = mixer.forward(h, step, cache_view, stream=resid) if getattr(mixer, "adds_to_stream", False) else mixer.forward(h, step, cache_view)
-        if a is not None:
-            pending.append(a)
-        if ff is not None:
-            f = ff.forward(h, step, stream=resid) if getattr(ff, "adds_to_stream", False) else ff.forward(h, step)
-            if f is not None:
-                pending.append(f)
-        if not pending:
-            return None
-        if len(pending) == 1:
-            return pending[0]
-        if getattr(next_norm, "takes_several", False):
-            return tuple(pending)
-        K.add_dyt(resid, pending, None, None, None, None)     # only the sum into the stream
+    def bound(self) -> None:
+        """Called when the parts have their weights."""
+        pair = (self.mixer, self.feed_forward)
+        if not all(hasattr(p, "before_output") and hasattr(p, "output_weight") for p in pair):
+            return
+        weights = [p.output_weight() for p in pair]
+        if weights[0].dtype != weights[1].dtype:
+            return
+        self.joint = Linear(torch.cat(weights, dim=1).contiguous())
+        self.border = weights[0].shape[1]
+        biases = [p.output_bias() for p in pair if p.output_bias() is not None]
+        self.joint_bias = sum(biases[1:], biases[0]).contiguous() if biases else None
+
+    @staticmethod
+    def _hand_on(resid, pending, next_norm):
+        """What is pending, as the norm that reads the stream next takes it; added here where it takes nothing of the kind."""
+        simple = pending.simplest()
+        if simple is None or isinstance(simple, torch.Tensor):
+            return simple
+        if getattr(next_norm, "takes_pending_sum", False) and pending.fits():
+            return pending
+        if getattr(next_norm, "takes_several", False) and not pending.biases:
+            return pending.outputs
+        pending.add(resid)
         return None
+
+    def forward(self, resid, delta, step, cache_view, next_norm=None):
+        mixer, ff = self.mixer, self.feed_forward
+        if step.handoff is None:
+            step.handoff = NormHandoff()
+        handoff = step.handoff
+        if self.joint is not None:
+            h = _add_norm(self.norm, resid, delta, True, handoff)
+            if isinstance(h, NormedStream) and h.n_tokens > FUSED_NORM_TOKENS:
+                h = h.materialize()                # both parts read it
+            n = step.n_tokens
+            both = torch.empty((n, self.joint.in_features), dtype=mixer.runtime.dtype, device=resid.device)
+            mixer.before_output(h, step, cache_view, both[:, : self.border])
+            ff.before_output(h, step, both[:, self.border:])
+            handoff.expect(next_norm)
+            y = self.joint.into_stream(both, resid, torch.float32, handoff=handoff, bias=self.joint_bias)
+            if y is None:
+                return None
+            return self._hand_on(resid, PendingSum((y,), (self.joint_bias,) if self.joint_bias is not None else ()), next_norm)
+        lone = ff is None and getattr(mixer, "takes_pending_norm", False)
+        h = _add_norm(self.norm, resid, delta, lone, handoff)
+        if not lone and not isinstance(h, torch.Tensor):
+            h = h.materialize()                    # both parts read it
+        # a mixer that adds into the stream leaves the norm behind it only where nothing else joins the stream first
+        handoff.expect(next_norm if ff is None else None)
+        adds = getattr(mixer, "adds_to_stream", False)
+        pending = PendingSum.of(mixer.forward(h, step, cache_view, stream=resid) if adds else mixer.forward(h, step, cache_view))
+        if ff is not None:
+            handoff.expect(None)
+            pending = pending.and_(ff.forward(h, step, stream=resid) if getattr(ff, "adds_to_stream", False) else ff.forward(h, step))
+        return self._hand_on(resid, pending, next_norm)
 
 
 @register_part("block", "sandwich")

@@ -188,15 +188,16 @@ class CappedHeadSpec:
     vocab_size: int
     hidden_size: int
     cap: Optional[float] = None        # logits <- cap * tanh(logits / cap); None: as they are
+    scale: float = 1.0                 # multiplies the logits before that
 
 
 @register_part("head", "capped_linear")
 class CappedHead(Head):
-    """logits = x W^T in fp32, then squashed into (-cap, cap)."""
+    """logits = scale * x W^T in fp32, then squashed into (-cap, cap)."""
     kernel_modules = ("elementwise", "stream_ops")
 
     def forward(self, x):
         logits = self.linear(x, out_dtype=torch.float32)
-        if self.spec.cap:
-            K.softcap(logits, self.spec.cap)
+        if self.spec.cap or self.spec.scale != 1.0:
+            K.softcap(logits, self.spec.cap or 0.0, self.spec.scale)
         return logits

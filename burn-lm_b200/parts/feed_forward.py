@@ -57,6 +57,17 @@ class SwiGLU(Part):
         act = self.gate_up.gated(x, rt.dtype)
         return self.down.into_stream(act, stream, rt.dtype, handoff=getattr(step, "handoff", None))
 
+    # for a block that runs this part's last product and a mixer's as one (parts.block.ParallelBlock)
+    def output_weight(self):
+        return self.down.weight
+
+    def output_bias(self):
+        return None
+
+    def before_output(self, x, step, out):
+        """What the last product reads, into `out` [N, inner] in the compute dtype (it may be a column range)."""
+        self.gate_up.gated(x, self.runtime.dtype, out=out)
+
 
 @dataclass(frozen=True)
 class BiasedMLPSpec:

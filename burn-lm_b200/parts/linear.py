@@ -171,10 +171,12 @@ class Linear:
             x = x.materialize()
         return self._library(x, out_dtype or x.dtype)
 
-    def into_stream(self, x, stream: Optional[torch.Tensor], out_dtype: torch.dtype, handoff: Optional[NormHandoff] = None):
+    def into_stream(self, x, stream: Optional[torch.Tensor], out_dtype: torch.dtype, handoff: Optional[NormHandoff] = None,
+                    bias: Optional[torch.Tensor] = None):
         """The product added into the fp32 residual stream when the skinny kernel can do that itself
         (returns None); otherwise the product, for the next norm to add.  With a `handoff` that expects a
-        norm, the kernel also leaves that norm's input there."""
+        norm, the kernel also leaves that norm's input there.  `bias` (float32) joins the stream with the product; a product that
+        is handed back comes without it."""
         n = self._tokens(x)
         if stream is not None and self._skinny(n, self.out_features, x):
             hand_over = None
@@ -184,11 +186,11 @@ class Linear:
                                     torch.empty(((self.out_features + 15) // 16, K.SQUARES_ROWS), dtype=torch.float32,
                                                 device=stream.device))
                 hand_over = (norm.gamma, handed.scaled, handed.squares)
-            K.gemv(self.weight, n, add_into=stream, hand_over=hand_over, **self._source(x))
+            K.gemv(self.weight, n, add_into=stream, hand_over=hand_over, add_bias=bias, **self._source(x))
             if hand_over is not None:
                 handoff.leave(stream, norm.gamma, handed)
             return None
-        if stream is not None and self._sk(n):
+        if stream is not None and bias is None and self._sk(n):
             hand_over = None
             norm = handoff.wanted if handoff is not None else None
             if norm is not None and n <= K.SK_SQUARES_ROWS and norm.gamma.numel() == self.out_features:
@@ -200,7 +202,7 @@ class Linear:
             if hand_over is not None:
                 handoff.leave(stream, norm.gamma, handed)
             return None
-        if (OWN_PRODUCTS and stream is not None and self.weight.dtype == torch.bfloat16 and n >= OWN_PRODUCTS_TOKENS
+        if (OWN_PRODUCTS and stream is not None and bias is None and self.weight.dtype == torch.bfloat16 and n >= OWN_PRODUCTS_TOKENS
                 and K.gemm_tc_supported(n, self.out_features, self.in_features)):
             if isinstance(x, NormedStream):
                 x = x.materialize()
@@ -225,19 +227,20 @@ class Linear:
             return "cluster"
         return ""
 
-    def gated(self, x, out_dtype: torch.dtype) -> torch.Tensor:
-        """silu(x Wgate^T) * (x Wup^T) for a fused [gate; up] weight."""
+    def gated(self, x, out_dtype: torch.dtype, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """silu(x Wgate^T) * (x Wup^T) for a fused [gate; up] weight; into `out` (it may be a column range) when given."""
         n = self._tokens(x)
         inner = self.out_features // 2
-        act = torch.empty((n, inner), dtype=out_dtype, device=self.weight.device)
+        act = out if out is not None else torch.empty((n, inner), dtype=out_dtype, device=self.weight.device)
+        aligned = act.data_ptr() % 16 == 0 and act.stride(0) % 8 == 0
         if out_dtype == torch.bfloat16 and self.gate_tile == K.GATE_TILE and self._skinny(n, inner, x):
             K.gemv(self.weight, n, out=act, swiglu=True, **self._source(x))
             return act
-        if out_dtype == torch.bfloat16 and self.gate_tile == K.GATE_TILE and self._sk(n):
+        if out_dtype == torch.bfloat16 and self.gate_tile == K.GATE_TILE and out is None and self._sk(n):
             K.gemm_sk(self.weight, out=act, swiglu=True, **self._sk_source(x))
             return act
         if (out_dtype == torch.bfloat16 and self.gate_tile == K.GATE_TILE and self.weight.dtype == torch.bfloat16
-                and n >= TENSOR_CORE_TOKENS and K.gemm_tc_supported(n, self.out_features, self.in_features)):
+                and aligned and n >= TENSOR_CORE_TOKENS and K.gemm_tc_supported(n, self.out_features, self.in_features)):
             # prompts: the tcgen05 product with the gated activation in its epilogue
             if isinstance(x, NormedStream):
                 x = x.materialize()

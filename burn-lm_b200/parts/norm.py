@@ -40,6 +40,42 @@ class PostNormed:
                                             # scale_b * output_b (two mixers side by side), summed by the same kernel
 
 
+@dataclass
+class PendingSum:
+    """Outputs and biases (one or two of each) that are still to be added to the stream.  The norm that reads the stream next adds
+    them in its own kernel (a norm with `takes_pending_sum`), or `add` does it alone."""
+    outputs: tuple = ()           # of [N, D] float32 or the compute dtype
+    biases: tuple = ()            # of float32 [D]
+
+    def fits(self) -> bool:
+        return len(self.outputs) <= 2 and len(self.biases) <= 2
+
+    def add(self, resid) -> None:
+        outputs, biases = list(self.outputs), list(self.biases)
+        while outputs or biases:
+            K.add_rmsnorm_parts(resid, outputs[:2], biases[:2], None, 0.0, None)
+            outputs, biases = outputs[2:], biases[2:]
+
+    @staticmethod
+    def of(delta) -> "PendingSum":
+        """A part's result (None, a tensor, a tuple of tensors, or a PendingSum) as a PendingSum."""
+        if isinstance(delta, PendingSum):
+            return delta
+        if delta is None:
+            return PendingSum()
+        return PendingSum(tuple(delta) if isinstance(delta, (tuple, list)) else (delta,))
+
+    def and_(self, other) -> "PendingSum":
+        other = PendingSum.of(other)
+        return PendingSum(self.outputs + other.outputs, self.biases + other.biases)
+
+    def simplest(self):
+        """None when nothing is pending, the output itself when it is one alone, else this."""
+        if not self.biases and len(self.outputs) <= 1:
+            return self.outputs[0] if self.outputs else None
+        return self
+
+
 @register_part("norm", "rmsnorm")
 class RMSNorm(Part):
     family = "norm"
@@ -56,12 +92,20 @@ class RMSNorm(Part):
 
     takes_handed_norm = True      # a product that writes the stream may leave this norm's input (parts.linear.NormHandoff)
     takes_post_normed = True      # `delta` may be a PostNormed: normed, scaled and added by this norm's kernel
+    takes_pending_sum = True      # `delta` may be a PendingSum: up to two outputs and two biases, added by this norm's kernel
 
     def add_norm(self, resid, delta, rows=None, lazy=False, handoff=None, out_dtype=None):
         """`lazy`: the caller can take a norm that is not computed yet (parts.linear.NormedStream);
         it gets one when nothing has to be added into the stream first.  `handoff`: where the writer of
         the stream may have left this norm's input.  `out_dtype` float32: the normed rows unrounded, for a reader
         that works on them before a product does (`delta` is then float32 or None)."""
+        if isinstance(delta, PendingSum):
+            if handoff is not None:
+                handoff.claim(resid, self.gamma)
+            n = rows.numel() if rows is not None else resid.shape[0]
+            out = torch.empty((n, self.spec.size), dtype=out_dtype or self.runtime.dtype, device=resid.device)
+            K.add_rmsnorm_parts(resid, delta.outputs, delta.biases, self.gamma, self.spec.eps, out, rows)
+            return out
         if out_dtype is not None and out_dtype != self.runtime.dtype:
             if handoff is not None:
                 handoff.claim(resid, self.gamma)

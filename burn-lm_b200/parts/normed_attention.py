@@ -1,8 +1,8 @@
 """Grouped-query attention with options on its queries, keys, values, scores, mask and output: normed heads, a turn of some
 lanes, a number per head on the scores, capped scores, a sink in the softmax, a window or chunks, two maps a head whose
-difference is taken, a gate on every lane.
+difference is taken, a gate on every lane, values that are the keys, a bias by distance, queries scaled by their position.
 
-q = Wq h, k = Wk h, v = Wv h without biases.  With `qk_norm` every head of q and of k is divided by its root mean square and
+q = Wq h, k = Wk h, v = Wv h, without biases or with (`projection_bias`).  With `qk_norm` every head of q and of k is divided by its root mean square and
 multiplied by a weight of the head's size that all heads share; the first `rotary_dims` lanes of every q and k head then turn
 by position * f_i, f_i = base^(-2i / rotary_dims) or scaled as `rotary_scaling` says (parts.position), lanes (2i, 2i + 1)
 together (`rotary_halves`: lanes (i, i + rotary_dims / 2)); with `value_norm` every head of v is divided by its root mean
@@ -10,7 +10,11 @@ square and cached so.  Query head h reads key/value head h // (heads / kv heads)
 s = scale * t_h * q.k (`head_temperature`: t a stored number per query head), then s <- cap tanh(s / cap) (`softcap`);
 position i sees j <= i, or only 0 <= i - j < window, or only the j of its own chunk of the sequence; p_j = exp(s_j) / (sink +
 sum exp(s_j)) with `sink` one more entry of score 0 that carries no value.  With `output_gate` every lane of the heads' outputs
-is multiplied by sigmoid(Wg h).  The heads' outputs are concatenated and projected by Wo.
+is multiplied by sigmoid(Wg h).  The heads' outputs are concatenated and projected by Wo (plus a bias with `output_bias`).
+
+`values_are_keys`: v is k as projected (bias included); there is no Wv and the cache keeps one line for both.
+`query_temperature` (coef, every): q is multiplied by 1 + coef ln(floor((position + 1) / every) + 1).  `slopes` (a number per
+query head): slope_h * (i - j) is taken off a score, after the cap.
 
 `diff` makes it differential attention: q has two queries and k two keys a head, [head][map][head_dim], each pair an attention
 of its own over the head's one value; with lambda = exp(lq1.lk1) - exp(lq2.lk2) + diff the head's output is a_1 - lambda a_2,
@@ -33,6 +37,7 @@ from ..registry import register_part
 from ..weights.loader import TensorSpec
 from .base import CacheNeed, Part
 from .linear import Linear
+from .norm import PendingSum
 from .position import RotarySpec, rotary_inverse_frequencies, rotary_multiplier
 
 BLOCKS_PER_SM = 4          # blocks of the single-token kernels a step should offer every multiprocessor
@@ -62,13 +67,18 @@ class NormedAttentionSpec:
     rotary_scaling: object = None     # parts.position.LinearScaling, YarnScaling or Llama3Scaling
     output_gate: bool = False         # sigmoid(Wg h) on every lane of the heads' outputs
     diff: Optional[float] = None      # two maps a head, and this constant in the weight of the second
+    values_are_keys: bool = False
+    projection_bias: bool = False     # biases on q, k and v
+    output_bias: bool = False
+    query_temperature: Optional[tuple] = None    # (coef, every)
+    slopes: Optional[tuple] = None    # a number per query head: what a position of distance takes off its scores
 
 
 @register_part("mixer", "normed_attention")
 class NormedAttention(Part):
     family = "mixer"
     graph_safe = True
-    roles = ("q", "k", "v", "o", "g", "q_norm", "k_norm", "temperature", "lq1", "lk1", "lq2", "lk2")
+    roles = ("q", "k", "v", "o", "g", "q_bias", "k_bias", "v_bias", "o_bias", "q_norm", "k_norm", "temperature", "lq1", "lk1", "lq2", "lk2")
     kernel_modules = ("elementwise", "attention_sink")
 
     def __init__(self, spec, tensors, runtime):
@@ -83,9 +93,16 @@ class NormedAttention(Part):
             raise ValueError(f"a window of {spec.window}")
         if spec.chunk is not None and (spec.chunk < 1 or spec.window is not None):
             raise ValueError(f"chunks of {spec.chunk} with a window of {spec.window}: one of the two, at least 1")
+        if spec.values_are_keys and (spec.value_dim != spec.head_dim or spec.value_norm or spec.diff is not None):
+            raise ValueError(f"values that are the keys have their {spec.head_dim} lanes, no norm of their own and one map a head")
+        if spec.slopes is not None and (len(spec.slopes) != spec.n_heads or spec.diff is not None):
+            raise ValueError(f"{len(spec.slopes)} slopes for {spec.n_heads} heads of one map")
+        if spec.query_temperature is not None and (spec.query_temperature[1] < 1 or spec.query_temperature[1] != int(spec.query_temperature[1])):
+            raise ValueError(f"a query temperature that steps every {spec.query_temperature[1]} positions")
         self.maps = 1 if spec.diff is None else 2
         self.q_cols, self.k_cols = self.maps * spec.n_heads * spec.head_dim, self.maps * spec.n_kv_heads * spec.head_dim
-        self.v_cols = spec.n_kv_heads * spec.value_dim
+        self.v_cols = 0 if spec.values_are_keys else spec.n_kv_heads * spec.value_dim
+        self.bias_roles = [r for r in ("q", "k", "v") if spec.projection_bias and not (r == "v" and spec.values_are_keys)]
         self.out_width = spec.n_heads * spec.value_dim
         self.proj_width = self.q_cols + self.k_cols + self.v_cols + (self.out_width if spec.output_gate else 0)
 
@@ -93,8 +110,13 @@ class NormedAttention(Part):
         s, t = self.spec, self.tensor_names
         specs = [TensorSpec(t["q"], (self.q_cols, s.hidden_size)),
                  TensorSpec(t["k"], (self.k_cols, s.hidden_size)),
-                 TensorSpec(t["v"], (self.v_cols, s.hidden_size)),
                  TensorSpec(t["o"], (s.hidden_size, self.out_width))]
+        if not s.values_are_keys:
+            specs.insert(2, TensorSpec(t["v"], (self.v_cols, s.hidden_size)))
+        cols = {"q": self.q_cols, "k": self.k_cols, "v": self.v_cols}
+        specs += [TensorSpec(t[r + "_bias"], (cols[r],), init="normal:0.1") for r in self.bias_roles]
+        if s.output_bias:
+            specs.append(TensorSpec(t["o_bias"], (s.hidden_size,), init="normal:0.1"))
         if s.output_gate:
             specs.append(TensorSpec(t["g"], (self.out_width, s.hidden_size)))
         if s.diff is not None:
@@ -108,7 +130,7 @@ class NormedAttention(Part):
 
     def bind(self, loaded):
         s, t = self.spec, self.tensor_names
-        ws = [loaded[t[r]] for r in (("q", "k", "v", "g") if s.output_gate else ("q", "k", "v"))]
+        ws = [loaded[t[r]] for r in ("q", "k", "v", "g") if not (r == "v" and s.values_are_keys) and (r != "g" or s.output_gate)]
         if len({w.dtype for w in ws}) != 1:
             raise ValueError(f"the projections of {t['q']} and its neighbours are stored in different dtypes")
         self.proj = Linear(torch.cat(ws, dim=0).contiguous())
@@ -117,6 +139,9 @@ class NormedAttention(Part):
         self.q_weight = f32(loaded[t["q_norm"]]) if s.qk_norm else None
         self.k_weight = f32(loaded[t["k_norm"]]) if s.qk_norm else None
         self.temperature = f32(loaded[t["temperature"]]) if s.head_temperature else None
+        self.bias = torch.cat([f32(loaded[t[r + "_bias"]]) for r in self.bias_roles]).contiguous() if self.bias_roles else None
+        self.o_bias = f32(loaded[t["o_bias"]]) if s.output_bias else None
+        self.slopes = torch.tensor(s.slopes, dtype=torch.float64).to(torch.float32).to(self.o.weight.device) if s.slopes is not None else None
         self.freq, self.turn_scale, self.table = None, 1.0, None
         if s.rotary_dims:
             rot = RotarySpec(s.head_dim, s.rotary_base, rotary_dim=s.rotary_dims, scaling=s.rotary_scaling)
@@ -137,8 +162,8 @@ class NormedAttention(Part):
 
     def cache_need(self) -> CacheNeed:
         s = self.spec
-        return CacheNeed("kv", n_kv_heads=s.n_kv_heads, head_dim=self.maps * s.head_dim, window=s.window, value_dim=s.value_dim,
-                         chunk=s.chunk)
+        return CacheNeed("kv", n_kv_heads=s.n_kv_heads, head_dim=self.maps * s.head_dim, window=s.window,
+                         value_dim=0 if s.values_are_keys else s.value_dim, chunk=s.chunk)
 
     def _splits(self, step) -> int:
         """Over how many blocks the single-token kernels cut a row's keys: a few tokens with many keys leave most of the
@@ -165,7 +190,16 @@ class NormedAttention(Part):
         proj = self.proj(x, out_dtype=torch.float32)            # [N, q | k | v (| g)] in fp32
         out = torch.empty((step.n_tokens, self.out_width), dtype=rt.dtype, device=proj.device)
         self.core(proj, step, cache, out)
-        return self.o.into_stream(out, stream, torch.float32, handoff=getattr(step, "handoff", None) if stream is not None else None)
+        y = self.o.into_stream(out, stream, torch.float32, handoff=getattr(step, "handoff", None) if stream is not None else None, bias=self.o_bias)
+        return y if y is None or self.o_bias is None else PendingSum((y,), (self.o_bias,))
+
+    # for a block that runs this part's last product and a feed-forward's as one (parts.block.ParallelBlock)
+    def output_bias(self):
+        return self.o_bias
+
+    def before_output(self, x, step, cache, out):
+        """What the output product reads, into `out` [N, out_width] in the compute dtype (it may be a column range)."""
+        self.core(self.proj(x, out_dtype=torch.float32), step, cache, out)
 
     # what two mixers that run side by side with one product in front and one behind ask for (parts.parallel_mixers)
     def input_weight(self):
@@ -184,7 +218,8 @@ class NormedAttention(Part):
         q = torch.empty((n, self.q_cols), dtype=rt.dtype, device=proj.device)
         K.head_norm_rope_append(proj, step, cache.pool, cache.block_table, q, heads, kv_heads, s.head_dim, s.value_dim,
                                 q_weight=self.q_weight, k_weight=self.k_weight, eps=s.eps, value_norm=s.value_norm, freq=self.freq,
-                                rotary_dims=s.rotary_dims, halves=s.rotary_halves, turn_scale=self.turn_scale, maps=maps, table=self.table)
+                                rotary_dims=s.rotary_dims, halves=s.rotary_halves, turn_scale=self.turn_scale, maps=maps, table=self.table,
+                                bias=self.bias, temperature=s.query_temperature, shared=s.values_are_keys)
         n_splits = self._splits(step)
         prompt = K.attention_sink_prompt_takes(rt.dtype, s.head_dim, s.value_dim, step.max_q_len, heads)
         inside = maps == 2 and not prompt and K.attention_sink_pairs(rt.dtype, s.head_dim, s.value_dim, heads, kv_heads, maps)
@@ -198,4 +233,5 @@ class NormedAttention(Part):
         K.attention_sink(q, step, cache.pool, cache.block_table, out, heads, kv_heads, s.head_dim, s.value_dim, s.scale,
                          s.window or NO_WINDOW, 0, sink=s.sink, gate=gate, gate_stride=proj.stride(0), max_q_len=step.max_q_len,
                          n_splits=n_splits, scratch=scratch, head_scale=self.temperature, softcap=s.softcap or 0.0, chunk=s.chunk or 0,
-                         gate_lanes=s.value_dim if s.output_gate else 0, out_scale=scale, maps=maps, difference=self.difference)
+                         gate_lanes=s.value_dim if s.output_gate else 0, out_scale=scale, maps=maps, difference=self.difference,
+                         slope=self.slopes, shared=s.values_are_keys)
