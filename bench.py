@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the Llama-3.2-1B shape with random weights on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 1b|3b|8b]
-    python bench.py --compare fobilorn|nufolix|ridopel|marinex|tomalix [--size 1b-layers|8b-layers]     (another design beside this one, see run_compare)
+    python bench.py --compare fobilorn|nufolix|ridopel|marinex|tomalix|samusun [--size 1b-layers|8b-layers]     (another design beside this one, see run_compare)
 
 A "step" is one decode step of the whole batch.  The default run has the layer sizes of the 1B
 configuration (16 layers, width 2048, 32 heads on 8 kv heads of 64, inner 8192, vocabulary 128256,
@@ -975,10 +975,154 @@ def tomalix_kernels(z, pk):
     return out
 
 
+def samusun_configs(z):
+    """(llama, samusun) of one size.  The new design's layers take turns: attention over a window of 1,024 with Llama's head counts
+    and head size (keys that are their own values) and a dense feed-forward of Llama's inner size; retention with Llama's query
+    heads for keys and values and 8 experts of which a token uses 2, whose inner sizes make Llama's together; then either mixer
+    with the other feed-forward."""
+    llama = compare_configs(z)["llama"]
+    hd, d, H, G = z["hd"], z["width"], z["heads"], z["kv"]
+    dense = {"kind": "dense", "ff": z["inner"]}
+    moe = {"kind": "moe", "expert": {"ff": z["inner"] // z["top"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    attention = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": z["window"]},
+                 "q_temp": {"coef": 0.1, "every": 512}}
+    retention = {"heads": H, "dim": hd, "vdim": hd, "decay": [1.0 - 2.0 ** (-5.0 - 4.0 * h / H) for h in range(H)],
+                 "rot": {"dims": hd, "base": 500000.0}}
+    turn = [("attention", attention, dense), ("retention", retention, moe), ("attention", attention, moe), ("retention", retention, dense)]
+    sam = {"architecture": "Samusun", "vocab": z["vocab"], "width": d, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "logit_scale": 1.0,
+           "logit_softcap": 30.0, "layers": [dict(zip(("type", "mixer", "mlp"), turn[i % 4])) for i in range(z["layers"])]}
+    return {"llama": llama, "samusun": sam}
+
+
+def samusun_kernels(z, pk):
+    """The new design's kernels alone, CUDA events, back to back (single tokens: captured in a graph), beside the like kernel of
+    another model: attention whose keys are its values with a bias by distance beside the dense decoder's, what stands between
+    projection and attention, retention beside the two scans with matrix states, the norm with what joins the stream in front of
+    it, the one product behind both sublayers beside two, and the experts."""
+    import torch
+    from types import SimpleNamespace
+    from burn_lm_b200 import kernels as K
+    from burn_lm_b200.architectures.samusun import head_slopes
+    from burn_lm_b200.parts.attention import streaming_splits
+    from burn_lm_b200.parts.normed_attention import STREAM_PAGES
+    from burn_lm_b200.parts.linear import Linear
+    dev, bf, f32 = "cuda", torch.bfloat16, torch.float32
+    H, G, hd, d, W, inner = z["heads"], z["kv"], z["hd"], z["width"], z["window"], z["inner"]
+    out = {}
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rnd = lambda *shape, dtype=f32: torch.randn(shape, dtype=dtype, device=dev)
+    frac_bf16 = lambda flops, ms: round(flops / (ms / 1e3) / (pk["bf16_tflops"] * 1e12), 4)
+    frac_hbm = lambda nbytes, ms: round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4)
+
+    def step(n_seqs, new, cached):
+        seq = [s for s in range(n_seqs) for _ in range(new)]
+        pos = [cached + t for _ in range(n_seqs) for t in range(new)]
+        return SimpleNamespace(token_seq=i32(seq), token_pos=i32(pos), slot_of_seq=i32(list(range(n_seqs))),
+                               cu_seqlens=i32([new * s for s in range(n_seqs + 1)]), start_pos=i32([cached] * n_seqs),
+                               n_tokens=n_seqs * new, n_seqs=n_seqs, max_q_len=new, max_kv_len=cached + new)
+
+    slope = torch.tensor(head_slopes(H), dtype=f32, device=dev)
+    for n_seqs, new, cached in ((1, 2048, 0), (64, 1, 1087), (8, 1, 1087)):
+        total, prompt = cached + new, new > 1
+        _time = globals()["_time" if prompt else "_time_captured"]
+        pages_each = -(-total // K.PAGE)
+        n = n_seqs * new
+        bt = torch.arange(n_seqs * pages_each, dtype=torch.int32, device=dev).reshape(n_seqs, pages_each)
+        st = step(n_seqs, new, cached)
+        pool5 = rnd(n_seqs * pages_each, 2, G, K.PAGE, hd, dtype=bf)
+        keys = pool5[:, 0].reshape(n_seqs * pages_each, -1).contiguous()
+        q = rnd(n, H * hd, dtype=bf)
+        o = torch.empty_like(q)
+        splits = 1 if prompt else streaming_splits(n_seqs, G, pages_each, STREAM_PAGES, dev)
+        scratch = torch.empty(max(1, K.attention_sink_scratch_floats(n, H, hd, splits)), dtype=f32, device=dev)
+        llama_splits = 1 if n_seqs * G >= K.sm_count() else 2
+        lscratch = torch.empty(max(1, K.attention_scratch_floats(n, H, hd, llama_splits)), dtype=f32, device=dev)
+        llama = lambda w: _time(lambda: K.attention(q, q.shape[1], pool5, bt, st.cu_seqlens, st.slot_of_seq, st.start_pos, o, n, n_seqs, new,
+                                                    H, G, hd, hd ** -0.5, window=w, n_splits=1 if prompt else llama_splits, scratch=lscratch, max_kv_len=total))
+        shared = lambda w: _time(lambda: K.attention_sink(q, st, keys, bt, o, H, G, hd, hd, hd ** -0.5, w, 0, sink=False, max_q_len=new, slope=slope,
+                                                          shared=True, n_splits=splits, scratch=scratch))
+        ms_l, ms_lw, ms, ms_w = llama(0), llama(W), shared(1 << 30), shared(W)
+        r = {"llama_ms": round(ms_l, 4), "llama_window_ms": round(ms_lw, 4), "shared_ms": round(ms, 4), "shared_window_ms": round(ms_w, 4)}
+        if prompt:
+            full, win = new * (new + 1) / 2, sum(min(t + 1, W) for t in range(new))
+            r.update(llama_frac_bf16=frac_bf16(4.0 * H * hd * full, ms_l), llama_window_frac_bf16=frac_bf16(4.0 * H * hd * win, ms_lw),
+                     shared_frac_bf16=frac_bf16(4.0 * H * hd * full, ms), shared_window_frac_bf16=frac_bf16(4.0 * H * hd * win, ms_w))
+        else:                                                # (a key is read once for both of its uses)
+            line = n * G * hd * 2.0
+            r.update(llama_frac_hbm=frac_hbm(2 * line * total, ms_l), llama_window_frac_hbm=frac_hbm(2 * line * min(total, W), ms_lw),
+                     shared_frac_hbm=frac_hbm(line * total, ms), shared_window_frac_hbm=frac_hbm(line * min(total, W), ms_w))
+        out[f"attention_{n_seqs}x{new}"] = r
+        # between the projection and the attention
+        cols, lcols = (H + G) * hd, (H + 2 * G) * hd
+        proj, bias, qkv = rnd(n, cols), rnd(cols), rnd(n, lcols, dtype=bf)
+        freq = torch.tensor([500000.0 ** (-2.0 * i / hd) for i in range(hd // 2)], dtype=torch.float64, device=dev)
+        table = K.rope_table(freq, total)
+        ms_new = _time(lambda: K.head_norm_rope_append(proj, st, keys, bt, q, H, G, hd, hd, bias=bias, temperature=(0.1, 512), shared=True))
+        ms_llama = _time(lambda: K.rope_append(qkv, st.token_seq, st.token_pos, st.slot_of_seq, bt, freq, hd, K.PAIRS_HALVES, pool5, H, G, hd,
+                                               write_cache=True, table=table, max_position=total - 1))
+        out[f"between_{n_seqs}x{new}"] = {"bias_append_ms": round(ms_new, 4), "llama_turn_append_ms": round(ms_llama, 4),
+                                          "frac_hbm": frac_hbm(n * cols * 6.0, ms_new), "llama_frac_hbm": frac_hbm(n * lcols * 4.0, ms_llama)}
+        # retention: rows in and out, and the states
+        decay = [1.0 - 2.0 ** (-5.0 - 4.0 * h / H) for h in range(H)]
+        powers = K.retention_powers(decay).to(dev)
+        rows = rnd(n, 4 * H * hd)
+        state = torch.zeros((n_seqs, 2, H * hd * hd), dtype=f32, device=dev)
+        y = torch.empty((n, H * hd), dtype=bf, device=dev)
+        ms_r = _time(lambda: K.retention(rows, st, state, 0, H, hd, hd, hd ** -0.5, powers, 1e-6, y, freq=freq, rotary_dims=hd, table=table))
+        r_bytes = n * H * hd * (4 * 4.0 + 2.0) + (2.0 if not prompt else 1.0) * 4 * n_seqs * H * hd * hd
+        floats = K.scan_state_floats(H, hd, hd)
+        state2 = torch.zeros((n_seqs, 2, floats), dtype=f32, device=dev)
+        zeros, zk, y2 = torch.zeros(H, dtype=f32, device=dev), torch.zeros(H * hd, dtype=f32, device=dev), torch.zeros((n, H * hd), dtype=f32, device=dev)
+        dth = rnd(n, H)
+        ms_ssm = _time(lambda: K.ssm_scan(rows, 0, H * hd, 2 * H * hd, dth, 0, zeros, zeros, zeros, y2, H, H, hd, hd, st, state2, 0), reps=3)
+        ms_decay = _time(lambda: K.decay_scan(rows, 0, rows, H * hd, rows, 2 * H * hd, rows, 3 * H * hd, zk, None, y2, H, hd, hd, K.DECAY_EXP_EXP, False, st,
+                                              state2, 0), reps=3)
+        ssm_bytes = 4.0 * n * (4 * H * hd + H) + (2.0 if not prompt else 1.0) * 4 * n_seqs * floats
+        decay_bytes = 4.0 * n * 5 * H * hd + (2.0 if not prompt else 1.0) * 4 * n_seqs * floats
+        out[f"retention_{n_seqs}x{new}"] = {"retention_ms": round(ms_r, 4), "retention_frac_hbm": frac_hbm(r_bytes, ms_r), "state_space_ms": round(ms_ssm, 4),
+                                            "state_space_frac_hbm": frac_hbm(ssm_bytes, ms_ssm), "decay_scan_ms": round(ms_decay, 4),
+                                            "decay_scan_frac_hbm": frac_hbm(decay_bytes, ms_decay)}
+        # the stream and the norm in front of a layer
+        resid, delta, gamma, xo, vec = rnd(n, d), rnd(n, d), torch.ones(d, dtype=f32, device=dev), torch.empty((n, d), dtype=bf, device=dev), rnd(d)
+        ms_parts = _time(lambda: K.add_rmsnorm_parts(resid, [delta, delta], [vec], gamma, 1e-6, xo))
+        ms_one = _time(lambda: K.add_rmsnorm_parts(resid, [delta], [vec], gamma, 1e-6, xo))
+        ms_norm = _time(lambda: K.add_rmsnorm(resid, delta, gamma, 1e-6, xo))
+        out[f"stream_{n_seqs}x{new}"] = {"two_outputs_norm_ms": round(ms_parts, 4), "two_outputs_frac_hbm": frac_hbm(n * d * 18.0, ms_parts),
+                                         "one_output_norm_ms": round(ms_one, 4), "one_output_frac_hbm": frac_hbm(n * d * 14.0, ms_one),
+                                         "add_norm_ms": round(ms_norm, 4), "add_norm_frac_hbm": frac_hbm(n * d * 14.0, ms_norm)}
+    # the products behind both sublayers, and the experts
+    E, top = z["experts"], z["top"]
+    each = inner // top
+    wo, wd = Linear(rnd(d, H * hd, dtype=bf) * 0.02), Linear(rnd(d, inner, dtype=bf) * 0.02)
+    joint = Linear(torch.cat([wo.weight, wd.weight], dim=1).contiguous())
+    gate_up, down = rnd(E, 2 * each, d, dtype=bf) * 0.02, rnd(E, d, each, dtype=bf) * 0.02
+    w1 = Linear(rnd(2 * inner, d, dtype=bf) * 0.02, gate_tile=K.GATE_TILE)
+    router, bias = rnd(E, d), rnd(d)
+    for n in (2048, 64, 8):
+        _time = globals()["_time" if n == 2048 else "_time_captured"]
+        both, h, stream = rnd(n, H * hd + inner, dtype=bf), rnd(n, d, dtype=bf), rnd(n, d)
+        a, b = both[:, : H * hd].contiguous(), both[:, H * hd:].contiguous()
+        ms_joint = _time(lambda: joint.into_stream(both, stream, f32, bias=bias))
+        ms_two = _time(lambda: (wo.into_stream(a, stream, bf), wd.into_stream(b, stream, bf)))
+        ms_dense = _time(lambda: wd(w1.gated(h, bf)))
+        ms_route = _time(lambda: K.moe_route(h, router, top, scores=K.SCORES_SOFTMAX))
+        ids, weights = K.moe_route(h, router, top, scores=K.SCORES_SOFTMAX)
+        run = lambda clamp: _time(lambda: K.moe_experts(h, ids, weights, gate_up, down, weight_on_input=False, out_dtype=f32, clamp_limit=clamp))
+        ms_moe, ms_clamped = run(0.0), run(7.0)
+        wbytes = 2.0 * 3 * each * d * min(E, n * top)
+        out[f"products_{n}_tokens"] = {
+            "one_product_ms": round(ms_joint, 4), "two_products_ms": round(ms_two, 4), "llama_mlp_ms": round(ms_dense, 4), "route_ms": round(ms_route, 4),
+            "llama_mlp_frac_bf16": frac_bf16(6.0 * n * inner * d, ms_dense),
+            "experts_ms": round(ms_moe, 4), "experts_clamped_ms": round(ms_clamped, 4), "experts_frac_bf16": frac_bf16(6.0 * n * top * each * d, ms_moe),
+            "experts_frac_hbm": frac_hbm(wbytes, ms_moe), "one_product_frac_bf16": frac_bf16(2.0 * n * (H * hd + inner) * d, ms_joint),
+            "one_product_frac_hbm": frac_hbm(2.0 * (H * hd + inner) * d, ms_joint)}
+    return out
+
+
 def run_compare(args):
     """One JSON line per size and model: prefill of one 2,048-token prompt and decode at batch 8 and 64 after 512-token
     prompts, for the dense Llama decoder and the named design (Fobilorn with dense feed-forwards and with experts, Nufolix,
-    Ridopel, Marinex, Tomalix) at equal layer sizes with random weights; then a line with the kernels alone."""
+    Ridopel, Marinex, Tomalix, Samusun) at equal layer sizes with random weights; then a line with the kernels alone."""
     import torch
     import burn_lm_b200 as blm
     if not torch.cuda.is_available():
@@ -988,12 +1132,14 @@ def run_compare(args):
     for size, z in COMPARE_SIZES.items():
         if args.size and size != args.size:
             continue
-        if args.compare in ("ridopel", "marinex", "tomalix"):
+        if args.compare in ("ridopel", "marinex", "tomalix", "samusun"):
             z = dict(z, experts=8)          # 8 experts of half the dense inner size each: four times the dense layer's weights
         if args.compare == "tomalix":
             z = dict(z, layers=3)           # one layer of every kind
+        if args.compare == "samusun":
+            z = dict(z, layers=4)           # either mixer with either feed-forward
         configs = {"nufolix": nufolix_configs, "ridopel": ridopel_configs, "marinex": marinex_configs,
-                   "tomalix": tomalix_configs}.get(args.compare, compare_configs)(z)
+                   "tomalix": tomalix_configs, "samusun": samusun_configs}.get(args.compare, compare_configs)(z)
         for name, cfg in configs.items():
             vocab = z["vocab"]
             lm = blm.load_random(cfg, seed=0, dtype="bfloat16", max_seq_len=4096, max_batch=64, max_tokens=64 * 1024)
@@ -1011,7 +1157,7 @@ def run_compare(args):
             del lm, engine
             torch.cuda.empty_cache()
         alone = {"nufolix": nufolix_kernels, "ridopel": ridopel_kernels, "marinex": marinex_kernels,
-                 "tomalix": tomalix_kernels}.get(args.compare, compare_kernels)(z, pk)
+                 "tomalix": tomalix_kernels, "samusun": samusun_kernels}.get(args.compare, compare_kernels)(z, pk)
         print(json.dumps({"compare": size, "kernels": alone, "peaks": pk["source"]}), flush=True)
     return 0
 
@@ -1126,7 +1272,7 @@ def main():
     ap.add_argument("--only", default=None, choices=["decode", "prefill", "sweep"],
                     help="run one workload briefly (for profilers), or a sweep over batch sizes and context lengths")
     ap.add_argument("--prompt-tokens", type=int, default=0, help="with --only prefill: one prompt of this many tokens instead of the workload's")
-    ap.add_argument("--compare", default=None, choices=["fobilorn", "nufolix", "ridopel", "marinex", "tomalix"],
+    ap.add_argument("--compare", default=None, choices=["fobilorn", "nufolix", "ridopel", "marinex", "tomalix", "samusun"],
                     help="instead of the workload: the named design beside the dense Llama decoder at equal layer sizes "
                          "(prefill and decode throughput, then its kernels alone), one JSON line each")
     ap.add_argument("--size", default=None, choices=sorted(COMPARE_SIZES), help="with --compare: one of the sizes only")

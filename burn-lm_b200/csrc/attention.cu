@@ -349,6 +349,7 @@ BLM_API int blm_attention(const void* q, long long q_stride, const void* pool, i
         d.q = (const __nv_bfloat16*)q; d.q_stride = q_stride; d.pool = (const __nv_bfloat16*)pool;
         d.block_table = block_table; d.table_stride = table_stride; d.seq_table = seq_table; d.cu_seqlens = cu_seqlens;
         d.slot_of_seq = slot_of_seq; d.start_pos = start_pos; d.out = (__nv_bfloat16*)out;
+        d.out_stride = (long long)n_heads * hd; d.slope = nullptr;
         d.part_acc = scratch;
         d.part_ml = scratch ? scratch + (size_t)n_tokens * n_heads * n_splits * hd : nullptr;
         d.n_heads = n_heads; d.n_kv = n_kv; d.window = window; d.n_splits = n_splits;
@@ -358,7 +359,7 @@ BLM_API int blm_attention(const void* q, long long q_stride, const void* pool, i
         BLM_REQUIRE(status != nullptr, "attention: no status word");
         BLM_REQUIRE(n_splits <= 64, "attention: at most 64 splits, got %d", n_splits);
         BLM_REQUIRE(n_pages > 0 && ((size_t)pool & 15) == 0, "attention: the pool's page count is needed");
-        if (launch_attn_decode(d, hd, group, n_seqs, n_pages, max_kv_len, stream)) return blm_check_launch("attention decode");
+        if (launch_attn_decode<false>(d, hd, group, n_seqs, n_pages, max_kv_len, stream)) return blm_check_launch("attention decode");
     }
     if (dtype == BLM_BF16 && max_q_len >= 16 && (hd == 64 || hd == 128) && !general_only) {
         // prompts: the tensor-core kernel

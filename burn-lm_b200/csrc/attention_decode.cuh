@@ -9,6 +9,10 @@
 // an SM.  Warps and groups keep their own running (max, sum, output) and merge at the end; splits of a
 // long sequence are merged by a second kernel.  Waits on mbarriers are bounded; one that runs out is
 // recorded in the status word.
+//
+// SHARED: the values are the keys and a page holds the keys alone: a stage of the ring is one operand, read once for the scores
+// and once, transposed, for the sums, so that a walk is half the bytes.  With it a head may have a slope: slope times the
+// distance is taken off a score.
 #pragma once
 #include <cuda.h>
 
@@ -20,14 +24,16 @@
 struct AttnDecodeArgs {
     const __nv_bfloat16* q;      // token n, head h at q + n * q_stride + h * HD
     long long q_stride;
-    const __nv_bfloat16* pool;   // [pages][2][n_kv][64][HD]
+    const __nv_bfloat16* pool;   // [pages][2][n_kv][64][HD]; SHARED: [pages][n_kv][64][HD]
     const int* block_table;
     int table_stride;
     const int* seq_table;        // optional: the block table's rows in the order of the step's sequences
     const int* cu_seqlens;
     const int* slot_of_seq;
     const int* start_pos;
-    __nv_bfloat16* out;          // [N, n_heads * HD]
+    __nv_bfloat16* out;          // [N, n_heads * HD], rows of out_stride
+    long long out_stride;
+    const float* slope;          // SHARED: [n_heads] or null
     float* part_acc;             // [N, n_heads, n_splits, HD]
     float* part_ml;              // [N, n_heads, n_splits, 2]: (max in natural-log units, sum)
     int n_heads, n_kv, window, n_splits;
@@ -91,8 +97,8 @@ __device__ __forceinline__ void bulk_copy(void* dst, const void* src, unsigned b
 // pages in flight at once, up to what shared memory takes; with many blocks the rings are short, so that
 // all blocks are resident at once (at batch 64, 512 blocks: two pages a ring and six blocks an SM measured
 // best, ahead of three or four pages).
-static inline int attn_decode_stages(int hd, int blocks, int pages_per_block) {
-    const int page_kb = 2 * 64 * hd * 2 / 1024;                    // keys and values of a page of one kv head
+static inline int attn_decode_stages(int hd, int blocks, int pages_per_block, bool shared = false) {
+    const int page_kb = (shared ? 1 : 2) * 64 * hd * 2 / 1024;     // keys and values of a page of one kv head
     const int sms = blm_sm_count();
     const int room_kb = blocks <= sms ? 192 : (blocks <= 2 * sms ? 96 : 32);
     int s = room_kb / page_kb;
@@ -130,7 +136,7 @@ __device__ __forceinline__ void dec_mma(float (&c)[4], const unsigned (&a)[4], u
 // instead of hundreds.  A page arrives as TMA boxes of 64 keys x 64 lanes with the 128-byte swizzle, which
 // ldmatrix reads without bank conflicts; the four consumer warps take 16 keys of every page each and keep
 // their own running (max, sum, output), merged at the end.
-template <int HD, int NG>
+template <int HD, int NG, bool SHARED>
 __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const AttnDecodeArgs a, const __grid_constant__ CUtensorMap pool_map) {
     using namespace attn_decode;
     const int G = a.group;
@@ -141,11 +147,12 @@ __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const At
     constexpr int DT = HD / 8;         // 8-wide output tiles
     constexpr unsigned BOX = 64 * 64 * 2;          // bytes of one box
     constexpr unsigned PB = SUB * BOX;             // bytes of the keys (or of the values) of one page of one kv head
+    constexpr unsigned STAGE = (SHARED ? 1 : 2) * PB;
     constexpr float LN2 = 0.6931471805599453f;
     extern __shared__ __align__(1024) unsigned char smem_dec_raw[];
     unsigned char* smem_dec = smem_dec_raw + ((1024u - (smem_u32(smem_dec_raw) & 1023u)) & 1023u);
     unsigned char* ring = smem_dec;                                                         // [S][k | v][SUB][64 x 128 bytes]
-    float* sm_acc = reinterpret_cast<float*>(smem_dec + (size_t)S * 2 * PB);                // [WARPS][G][HD]
+    float* sm_acc = reinterpret_cast<float*>(smem_dec + (size_t)S * STAGE);                // [WARPS][G][HD]
     float* sm_m = sm_acc + WARPS * G * HD;                                                  // [WARPS][G]
     float* sm_l = sm_m + WARPS * G;
     unsigned long long* full = reinterpret_cast<unsigned long long*>(sm_l + WARPS * G);
@@ -203,15 +210,16 @@ __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const At
                     continue;
                 }
                 // rows of the pool seen as a matrix [pages * 2 * n_kv * 64, HD]: keys, then values, of a page
-                const int krow = ((page * 2) * a.n_kv + kvh) * 64, vrow = krow + a.n_kv * 64;
-                mbar_expect_tx(full + s, 2 * PB);
-                unsigned char* dst = ring + (size_t)s * 2 * PB;
+                const int krow = ((SHARED ? page : page * 2) * a.n_kv + kvh) * 64, vrow = krow + a.n_kv * 64;
+                mbar_expect_tx(full + s, STAGE);
+                unsigned char* dst = ring + (size_t)s * STAGE;
 #pragma unroll
                 for (int h = 0; h < SUB; ++h) {
                     asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];\n" ::"r"(
                                      smem_u32(dst + h * BOX)),
                                  "l"(&pool_map), "r"(h * 64), "r"(krow), "r"(smem_u32(full + s))
                                  : "memory");
+                    if (SHARED) continue;
                     asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];\n" ::"r"(
                                      smem_u32(dst + PB + h * BOX)),
                                  "l"(&pool_map), "r"(h * 64), "r"(vrow), "r"(smem_u32(full + s))
@@ -240,6 +248,7 @@ __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const At
 #pragma unroll
             for (int e = 0; e < 4; ++e) o[d][e] = 0.f;
         float m_run = -INFINITY, l_run = 0.f;        // of row g (head g); every lane of a quad holds the same max
+        const float slope = SHARED && a.slope != nullptr && g < G ? a.slope[kvh * G + g] * 1.4426950408889634f : 0.f;     // in units of log 2
         auto swz = [](int row, int chunk) { return row * 128 + ((chunk ^ (row & 7)) << 4); };   // byte offset in a box
 
         // This warp's group takes every NG-th page; the ring's depth is a multiple of NG, so a stage always
@@ -255,8 +264,8 @@ __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const At
                 break;
             }
             if (i == 0) blm_trace(0x430);
-            const unsigned char* Kt = ring + (size_t)s * 2 * PB;
-            const unsigned char* Vt = Kt + PB;
+            const unsigned char* Kt = ring + (size_t)s * STAGE;
+            const unsigned char* Vt = SHARED ? Kt : Kt + PB;
             // scores of this warp's 16 keys: two tiles of 8 keys
             float sc[2][4];
 #pragma unroll
@@ -279,7 +288,8 @@ __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const At
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = pg * 64 + quarter * 16 + nt * 8 + 2 * t + e;
-                    const float v = (key >= key_lo && key < kv_len) ? sc[nt][e] * a.scale_log2e : -INFINITY;
+                    const float raw = SHARED ? fmaf(sc[nt][e], a.scale_log2e, slope * (float)(key - pos)) : sc[nt][e] * a.scale_log2e;
+                    const float v = (key >= key_lo && key < kv_len) ? raw : -INFINITY;
                     sc[nt][e] = v;
                     mx = fmaxf(mx, v);
                 }
@@ -312,7 +322,8 @@ __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const At
                 o[d][1] *= alpha;
             }
             // A masked key has weight zero, but 0 x NaN is NaN: rows of the value tile that hold no key of
-            // this sequence (a page's unwritten tail, keys before the window) are cleared before they are read.
+            // this sequence (a page's unwritten tail, keys before the window) are cleared before they are read.  (SHARED: these
+            // are the warp's own keys, whose scores are formed.)
             if (pg * 64 + quarter * 16 + 15 >= kv_len || pg * 64 + quarter * 16 < key_lo) {
                 const int row = quarter * 16 + (lane >> 1), key = pg * 64 + row;
                 if (key >= kv_len || key < key_lo)
@@ -360,7 +371,7 @@ __global__ void __launch_bounds__((4 * NG + 1) * 32) attn_decode_kernel(const At
         }
         const int head = kvh * G + gg;
         if (active == 1) {
-            a.out[(size_t)tok * a.n_heads * HD + (size_t)head * HD + d] = __float2bfloat16_rn(L > 0.f ? ov / L : 0.f);
+            a.out[(size_t)tok * a.out_stride + (size_t)head * HD + d] = __float2bfloat16_rn(L > 0.f ? ov / L : 0.f);
         } else {
             const size_t pi = ((size_t)tok * a.n_heads + head) * a.n_splits + split;
             a.part_acc[pi * HD + d] = ov;
@@ -410,16 +421,16 @@ __global__ void __launch_bounds__(128) attn_decode_combine_kernel(const AttnDeco
     }
     const float inv = L > 0.f ? 1.0f / L : 0.f;
 #pragma unroll
-    for (int e = 0; e < DPL; ++e) a.out[(size_t)row * HD + e * 32 + lane] = __float2bfloat16_rn(o[e] * inv);
+    for (int e = 0; e < DPL; ++e) a.out[(size_t)tok * a.out_stride + (size_t)(row % a.n_heads) * HD + e * 32 + lane] = __float2bfloat16_rn(o[e] * inv);
 }
 
 typedef CUresult (*DecEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
                                      const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                      CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-// The TMA's view of one cache line's pool [pages][2][n_kv][64][HD]: a matrix of pages * 2 * n_kv * 64 rows
+// The TMA's view of one cache line's pool [pages][operands][n_kv][64][HD]: a matrix of pages * operands * n_kv * 64 rows
 // of HD lanes; boxes of 64 rows x 64 lanes with the 128-byte swizzle.
-static bool attn_decode_pool_map(const void* pool, int n_pages, int n_kv, int hd, CUtensorMap* out) {
+static bool attn_decode_pool_map(const void* pool, int n_pages, int n_kv, int hd, int operands, CUtensorMap* out) {
     static DecEncodeTiledFn encode = nullptr;
     if (!encode) {
         void* fn = nullptr;
@@ -429,12 +440,12 @@ static bool attn_decode_pool_map(const void* pool, int n_pages, int n_kv, int hd
             return false;
         encode = (DecEncodeTiledFn)fn;
     }
-    static std::map<std::tuple<const void*, int, int, int>, CUtensorMap> maps;
-    const auto key = std::make_tuple(pool, n_pages, n_kv, hd);
+    static std::map<std::tuple<const void*, int, int, int, int>, CUtensorMap> maps;
+    const auto key = std::make_tuple(pool, n_pages, n_kv, hd, operands);
     auto it = maps.find(key);
     if (it == maps.end()) {
         CUtensorMap m;
-        const cuuint64_t dims[2] = {(cuuint64_t)hd, (cuuint64_t)n_pages * 2 * n_kv * 64};
+        const cuuint64_t dims[2] = {(cuuint64_t)hd, (cuuint64_t)n_pages * operands * n_kv * 64};
         const cuuint64_t strides[1] = {(cuuint64_t)hd * 2};
         const cuuint32_t box[2] = {64, 64};
         const cuuint32_t estr[2] = {1, 1};
@@ -449,37 +460,38 @@ static bool attn_decode_pool_map(const void* pool, int n_pages, int n_kv, int hd
     return true;
 }
 
-template <int HD, int NG>
+template <int HD, int NG, bool SHARED>
 static bool attn_decode_launch_ng(AttnDecodeArgs a, dim3 grid, int n_pages, cudaStream_t stream) {
     const int G = a.group;
     auto bytes = [&](int stages) {
-        return (size_t)stages * 2 * 64 * HD * 2 + (size_t)4 * a.n_groups * G * (HD + 2) * 4 + 2 * stages * 8 + 16 + 1024;
+        return (size_t)stages * (SHARED ? 1 : 2) * 64 * HD * 2 + (size_t)4 * a.n_groups * G * (HD + 2) * 4 + 2 * stages * 8 + 16 + 1024;
     };
     while (bytes(a.n_stages) > 220 * 1024 && a.n_stages > a.n_groups) a.n_stages -= a.n_groups;   // the warps' results need room too
     if (bytes(a.n_stages) > 220 * 1024) return false;
     const size_t smem = bytes(a.n_stages);
     CUtensorMap map;
-    if (!attn_decode_pool_map(a.pool, n_pages, a.n_kv, HD, &map)) return false;
+    if (!attn_decode_pool_map(a.pool, n_pages, a.n_kv, HD, SHARED ? 1 : 2, &map)) return false;
     static bool opted_in = false;
     if (!opted_in) {
-        if (cudaFuncSetAttribute(attn_decode_kernel<HD, NG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return false;
+        if (cudaFuncSetAttribute(attn_decode_kernel<HD, NG, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return false;
         opted_in = true;
     }
-    return blm_launch_dependent(attn_decode_kernel<HD, NG>, grid, dim3((4 * NG + 1) * 32), smem, stream, a, map) == cudaSuccess;
+    return blm_launch_dependent(attn_decode_kernel<HD, NG, SHARED>, grid, dim3((4 * NG + 1) * 32), smem, stream, a, map) == cudaSuccess;
 }
 
-template <int HD>
+template <int HD, bool SHARED>
 static bool launch_attn_decode_g(const AttnDecodeArgs& a, dim3 grid, int n_pages, cudaStream_t stream) {
     if (a.group < 1 || a.group > 8) return false;
     switch (a.n_groups) {
-        case 1: return attn_decode_launch_ng<HD, 1>(a, grid, n_pages, stream);
-        case 2: return attn_decode_launch_ng<HD, 2>(a, grid, n_pages, stream);
-        case 4: return attn_decode_launch_ng<HD, 4>(a, grid, n_pages, stream);
+        case 1: return attn_decode_launch_ng<HD, 1, SHARED>(a, grid, n_pages, stream);
+        case 2: return attn_decode_launch_ng<HD, 2, SHARED>(a, grid, n_pages, stream);
+        case 4: return attn_decode_launch_ng<HD, 4, SHARED>(a, grid, n_pages, stream);
         default: return false;
     }
 }
 
 // true when the specialised kernels were launched; false: the shape is left to the general kernel
+template <bool SHARED>
 static bool launch_attn_decode(AttnDecodeArgs a, int hd, int group, int n_seqs, int n_pages, int max_kv_len, cudaStream_t stream) {
     const dim3 grid(a.n_splits, a.n_kv, n_seqs);
     a.group = group;
@@ -493,17 +505,17 @@ static bool launch_attn_decode(AttnDecodeArgs a, int hd, int group, int n_seqs, 
     // 0.840 ms a step against 0.860).
     a.pages_per_split = (max_kv_len > 0 && blocks > 2 * blm_sm_count()) ? pages_per_block : 1;
     if (a.pages_per_split < 1) a.pages_per_split = 1;
-    a.n_stages = attn_decode_stages(hd, blocks, pages_per_block);
+    a.n_stages = attn_decode_stages(hd, blocks, pages_per_block, SHARED);
     a.n_groups = attn_decode_groups(blocks, pages_per_block, a.n_stages, hd);
     a.n_stages -= a.n_stages % a.n_groups;
     const int n_rows = n_seqs * a.n_heads;
     if (hd == 64) {
-        if (!launch_attn_decode_g<64>(a, grid, n_pages, stream)) return false;
+        if (!launch_attn_decode_g<64, SHARED>(a, grid, n_pages, stream)) return false;
         if (a.n_splits > 1) blm_launch_dependent(attn_decode_combine_kernel<64>, dim3((n_rows + 3) / 4), dim3(128), 0, stream, a, n_rows);
         return true;
     }
     if (hd == 128) {
-        if (!launch_attn_decode_g<128>(a, grid, n_pages, stream)) return false;
+        if (!launch_attn_decode_g<128, SHARED>(a, grid, n_pages, stream)) return false;
         if (a.n_splits > 1) blm_launch_dependent(attn_decode_combine_kernel<128>, dim3((n_rows + 3) / 4), dim3(128), 0, stream, a, n_rows);
         return true;
     }

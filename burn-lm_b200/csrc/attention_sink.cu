@@ -19,6 +19,7 @@
 // Scores, softmax and sums are fp32; q, keys and values are read in the cache's dtype.
 #include "common.cuh"
 #define BLM_ATTN_TC_GENERAL
+#include "attention_decode.cuh"
 #include "attention_prefill_tc.cuh"
 
 BLM_API const char* blm_attention_sink_last_error() { return g_blm_error; }
@@ -1390,15 +1391,22 @@ BLM_API int blm_attention_sink_pairs(int dtype, int dk, int dv, int page_size, i
     return maps == 2 && blm_attention_sink_decode_takes(dtype, dk, dv, page_size, n_heads, n_kv) && n_heads / n_kv <= 8 && dk <= 128;
 }
 
+// Whether single tokens of this shape run the dense decoder's streaming kernel: values that are the keys, heads of 64 or 128
+// lanes, up to 8 query heads a key/value head (and no other option than a window and slopes).
+BLM_API int blm_attention_sink_streams(int dtype, int dk, int page_size, int n_heads, int n_kv) {
+    return dtype == BLM_BF16 && page_size == kTileK && (dk == 64 || dk == 128) && n_kv > 0 && n_heads % n_kv == 0 && n_heads / n_kv <= 8;
+}
+
 BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long long page_elems, const int* block_table,
                                int table_stride, const int* token_seq, const int* token_pos, const int* slot_of_seq,
                                const int* cu_seqlens, const int* start_pos, int n_seqs, int max_q_len, const float* gate,
                                long long gate_stride, int gate_lanes, void* out, long long out_stride, float out_scale, float* partial,
                                int n_splits, int n_tokens, int n_heads, int n_kv, int maps, int dk, int dv, int page_size, int window,
                                int chunk, int keep_first, float scale, int sink, const float* head_scale, const float* sink_logit,
-                               float softcap, const float* slope, int shared, float diff_lambda, float diff_scale, float diff_eps, int n_pages, int* status,
+                               float softcap, const float* slope, int shared, float diff_lambda, float diff_scale, float diff_eps, int n_pages, int max_kv_len, int* status,
                                cudaStream_t stream) {
-    // n_pages, status: of the pool, and where a bounded wait that ran out is recorded (for the tcgen05 kernel; 0 and null: not run)
+    // n_pages, status: of the pool, and where a bounded wait that ran out is recorded (for the tcgen05 and the streaming kernel; 0
+    // and null: not run); max_kv_len: the longest sequence the step may hold (0: not known)
     // maps 2: n_heads and n_kv count every map, and diff_* are the difference's numbers (DiffOpts); partial is then needed
     // chunk > 0: the mask is by chunks and `window` is not looked at; gate_lanes 0: a gate per head, dv: one per lane
     // head_scale, sink_logit, slope: float32 [n_heads] or null; softcap: 0 for none (see ScoreOpts)
@@ -1453,6 +1461,19 @@ BLM_API int blm_attention_sink(const void* q, const void* pool, int dtype, long 
         return BLM_PROMPT(32);
 #undef BLM_PROMPT
 #undef BLM_PROMPT_OF
+    }
+    if (shared && max_q_len == 1 && n_seqs == n_tokens && start_pos != nullptr && status != nullptr && n_pages > 0 && gate == nullptr &&
+        out_scale == 1.f && chunk == 0 && !sink && softcap == 0.f && head_scale == nullptr && keep_first == 0 && n_splits <= 64 &&
+        ((size_t)pool & 15) == 0 && blm_attention_sink_streams(dtype, dk, page_size, n_heads, n_kv)) {
+        AttnDecodeArgs d = {};
+        d.q = (const __nv_bfloat16*)q; d.q_stride = (long long)n_heads * dk; d.pool = (const __nv_bfloat16*)pool;
+        d.block_table = block_table; d.table_stride = table_stride; d.slot_of_seq = slot_of_seq; d.start_pos = start_pos;
+        d.out = (__nv_bfloat16*)out; d.out_stride = out_stride; d.slope = slope;
+        d.part_acc = partial; d.part_ml = partial ? partial + (size_t)n_tokens * n_heads * n_splits * dk : nullptr;
+        d.n_heads = n_heads; d.n_kv = n_kv; d.window = window < kNoWindow ? window : 0; d.n_splits = n_splits;
+        d.scale_log2e = scale * 1.4426950408889634f; d.status = status;
+        const int most = d.window > 0 && max_kv_len > d.window + kTileK - 1 ? d.window + kTileK - 1 : max_kv_len;
+        if (launch_attn_decode<true>(d, dk, n_heads / n_kv, n_seqs, n_pages, most, stream)) return blm_check_launch("attention_sink (streaming)");
     }
     if (blm_attention_sink_decode_takes(dtype, dk, dv, page_size, n_heads, n_kv)) {
 #define BLM_DECODE(NV, STAGES, PAIR, SHARED) launch_decode<NV, STAGES, PAIR, SHARED>(q, pool, page_elems, block_table, table_stride, token_seq, token_pos, slot_of_seq, ro, \

@@ -21,7 +21,9 @@
 // ([experts x N, K]).  A table on the device names the expert of every tile of 128 rows (-1: a tile no expert owns); a block
 // looks its tile's expert up and fetches W's tiles from that expert's rows.  The tensor maps cover the whole buffers, so they
 // depend on sizes and addresses only and a step can be captured.  Its epilogues: the exact GELU or the squared relu (an expert without a gate),
-// and fp32 sums stored as they are.
+// a gated unit, and fp32 sums stored as they are.  A gated expert's rows are its gate rows and then its up rows; a five-dimensional
+// map (lanes, eight rows, gate or up, groups of eight, expert) brings them into shared memory as tiles of eight gate rows and
+// their eight up rows, so that the epilogue finds both halves of an output in one row of the accumulator.
 //
 // Every mbarrier wait is bounded; a wait that runs out records a code in the caller's status word and
 // the block goes on to its end, where the tensor memory is given back.
@@ -43,7 +45,7 @@ constexpr int kTmemCols = 512;                  // two fp32 accumulators of 256 
 constexpr unsigned kABytes = BM * BK * 2, kBBytes = BN * BK * 2;
 constexpr unsigned kSpinLimit = 1u << 22;
 
-enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESID_ADD = 2, EPI_GELU = 3, EPI_STORE_F32 = 4, EPI_RELU2 = 5 };
+enum { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESID_ADD = 2, EPI_GELU = 3, EPI_STORE_F32 = 4, EPI_RELU2 = 5, EPI_GATED_EXPERTS = 6 };
 enum { TC_OK = 0, TC_TIMEOUT_FULL = 11, TC_TIMEOUT_EMPTY = 12, TC_TIMEOUT_ACCUM = 13, TC_TIMEOUT_DRAIN = 14 };
 
 struct TcArgs {
@@ -55,6 +57,7 @@ struct TcArgs {
     int* status;
     const int* tile_expert;     // grouped form: the expert of every tile of BM rows (-1: none); null: one weight for all rows
     int expert_rows;            // grouped form: rows of W an expert (the next expert's rows follow)
+    float limit, alpha;         // EPI_GATED_EXPERTS: limit > 0: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1)
 };
 
 __device__ __forceinline__ unsigned smem_u32(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -97,6 +100,12 @@ __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, i
     asm volatile(
         "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];\n" ::"r"(smem_u32(dst)),
         "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar))
+        : "memory");
+}
+__device__ __forceinline__ void tma_load_5d(void* dst, const CUtensorMap* map, int x, int t, int e, unsigned long long* bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.5d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %3, %4, %5}], [%6];\n" ::"r"(smem_u32(dst)),
+        "l"(map), "r"(x), "r"(0), "r"(t), "r"(e), "r"(smem_u32(bar))
         : "memory");
 }
 // shared-memory operand descriptor: K-major tile of rows of 128 bytes, 128-byte swizzle; 8-row groups
@@ -170,14 +179,23 @@ __device__ __forceinline__ void store_columns(const TcArgs& a, const float (&v)[
         }
         return;
     }
-    if (EPI == EPI_SWIGLU) {
+    if (EPI == EPI_SWIGLU || EPI == EPI_GATED_EXPERTS) {
         const int inner = a.N >> 1, o0 = (n0 >> 1) + j * 8;
         if (o0 >= inner) return;
         unsigned packed[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const float g0 = v[2 * e], g1 = v[2 * e + 1], u0 = v[8 + 2 * e], u1 = v[8 + 2 * e + 1];
-            const __nv_bfloat162 p = __floats2bfloat162_rn(g0 / (1.0f + expf(-g0)) * u0, g1 / (1.0f + expf(-g1)) * u1);
+            float y0, y1;
+            if (EPI == EPI_GATED_EXPERTS && a.limit > 0.f) {
+                const float c0 = fminf(g0, a.limit), c1 = fminf(g1, a.limit);
+                y0 = c0 / (1.0f + expf(-a.alpha * c0)) * (fminf(fmaxf(u0, -a.limit), a.limit) + 1.0f);
+                y1 = c1 / (1.0f + expf(-a.alpha * c1)) * (fminf(fmaxf(u1, -a.limit), a.limit) + 1.0f);
+            } else {
+                y0 = g0 / (1.0f + expf(-g0)) * u0;
+                y1 = g1 / (1.0f + expf(-g1)) * u1;
+            }
+            const __nv_bfloat162 p = __floats2bfloat162_rn(y0, y1);
             packed[e] = *reinterpret_cast<const unsigned*>(&p);
         }
         __nv_bfloat16* dst = a.y + (size_t)row * a.ldy + o0;
@@ -264,11 +282,12 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const TcArgs a, co
             bool ok = true;
             for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
                 const int m0 = (tile % m_tiles) * BM, n0 = (tile / m_tiles) * BN;
-                int w0 = n0;                 // W's first row of the tile
+                int w0 = n0, expert = 0;     // W's first row of the tile
                 if (a.tile_expert != nullptr) {
                     const int e = a.tile_expert[tile % m_tiles];
                     if (e < 0) continue;     // a tile of rows no expert owns: every role of the block passes it by
                     w0 += e * a.expert_rows;
+                    expert = e;
                 }
                 for (int k = 0; k < k_iters; ++k, ++it) {
                     const int s = it % kStages;
@@ -279,7 +298,8 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tc_kernel(const TcArgs a, co
                     }
                     mbar_expect_tx(full + s, kABytes + kBBytes);
                     tma_load_2d(As + s * kABytes, &xmap, k * BK, m0, full + s);
-                    tma_load_2d(Bs + s * kBBytes, &wmap, k * BK, w0, full + s);
+                    if (EPI == EPI_GATED_EXPERTS) tma_load_5d(Bs + s * kBBytes, &wmap, k * BK, n0 / 16, expert, full + s);
+                    else tma_load_2d(Bs + s * kBBytes, &wmap, k * BK, w0, full + s);
                 }
             }
         }
@@ -359,6 +379,9 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
+// gated experts' weights [n_experts][gate rows | up rows][K]: boxes of 64 lanes x 8 rows x (gate, up) x BN / 16 groups of one expert
+int make_gated_map(const void* base, long long ld, int n_experts, int inner, int K, CUtensorMap* out);
+
 // The TMA's view of a K-major bf16 matrix [rows, K] (row stride ld): boxes of box_rows x 64, 128-byte swizzle.
 int make_map(const void* base, long long ld, int rows, int K, int box_rows, bool cache, CUtensorMap* out) {
     static EncodeTiledFn encode = nullptr;
@@ -394,6 +417,28 @@ int make_map(const void* base, long long ld, int rows, int K, int box_rows, bool
     return BLM_OK;
 }
 
+int make_gated_map(const void* base, long long ld, int n_experts, int inner, int K, CUtensorMap* out) {
+    static EncodeTiledFn encode = nullptr;
+    if (!encode) {
+        void* fn = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q);
+        if (e != cudaSuccess || q != cudaDriverEntryPointSuccess || !fn)
+            return blm_fail(BLM_CUDA_ERROR, "gemm_tc: the driver has no cuTensorMapEncodeTiled");
+        encode = (EncodeTiledFn)fn;
+    }
+    const cuuint64_t row = (cuuint64_t)ld * 2;
+    const cuuint64_t dims[5] = {(cuuint64_t)K, 8, 2, (cuuint64_t)(inner / 8), (cuuint64_t)n_experts};
+    const cuuint64_t strides[4] = {row, row * inner, row * 8, row * 2 * inner};
+    const cuuint32_t box[5] = {(cuuint32_t)BK, 8, 2, BN / 16, 1};
+    const cuuint32_t estr[5] = {1, 1, 1, 1, 1};
+    CUresult r = encode(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 5, const_cast<void*>(base), dims, strides, box, estr,
+                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) return blm_fail(BLM_CUDA_ERROR, "gemm_tc: cuTensorMapEncodeTiled failed for gated experts (%d)", (int)r);
+    return BLM_OK;
+}
+
 }  // namespace
 
 // 1 when blm_gemm_tc takes the shape
@@ -418,7 +463,7 @@ BLM_API int blm_gemm_tc(const void* x, long long ldx, const void* w, long long l
     if (rc != BLM_OK) return rc;
     TcArgs a;
     a.y = (__nv_bfloat16*)y; a.acc = (float*)y; a.ldy = ldy; a.M = M; a.N = N; a.K = K; a.epi = epi; a.status = status;
-    a.tile_expert = nullptr; a.expert_rows = 0;
+    a.tile_expert = nullptr; a.expert_rows = 0; a.limit = a.alpha = 0.f;
     const size_t smem = (size_t)kStages * (kABytes + kBBytes) + (2 * kStages + 4) * 8 + 16 + 1024;
     static bool opted_in = false;
     if (!opted_in) {
@@ -442,29 +487,33 @@ BLM_API int blm_gemm_tc(const void* x, long long ldx, const void* w, long long l
 // The grouped form.  x bfloat16 [M, K] (row stride ldx): the pairs' rows expert by expert, every expert's share starting at a
 // multiple of 128 rows, M a multiple of 128 (rows no pair owns hold zeros); w bfloat16 [n_experts x N, K] (row stride ldw);
 // tile_expert int32 [M / 128] on the device: the expert of every tile of rows, -1 for a tile no expert owns.
-// epi 3: y bfloat16 [M, N] = gelu(x . w_e^T), the exact form; epi 5: relu(x . w_e^T)^2; epi 4: y float32 [M, N] = x . w_e^T.
+// epi 3: y bfloat16 [M, N] = gelu(x . w_e^T), the exact form; epi 5: relu(x . w_e^T)^2; epi 4: y float32 [M, N] = x . w_e^T;
+// epi 6: an expert's N rows are N / 2 gate rows and then their up rows (N / 2 a multiple of 8), y bfloat16 [M, N / 2] =
+// silu(gate) * up, or the clamped unit (limit > 0, see TcArgs).
 BLM_API int blm_gemm_tc_grouped(const void* x, long long ldx, const void* w, long long ldw, void* y, long long ldy, int M, int N, int K,
-                                int n_experts, const int* tile_expert, int epi, int* status, cudaStream_t stream) {
+                                int n_experts, const int* tile_expert, int epi, float limit, float alpha, int* status, cudaStream_t stream) {
     if (M == 0 || N == 0) return BLM_OK;
     BLM_REQUIRE(blm_gemm_tc_supported(M, N, K) && M % BM == 0 && n_experts >= 1, "gemm_tc_grouped: shape %d x %d x %d, %d experts", M, N, K, n_experts);
     BLM_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0 && ((size_t)x & 15) == 0 && ((size_t)w & 15) == 0,
                 "gemm_tc_grouped: operand rows must be 16-byte aligned");
-    BLM_REQUIRE(epi == EPI_GELU || epi == EPI_RELU2 || epi == EPI_STORE_F32, "gemm_tc_grouped: epilogue %d", epi);
+    BLM_REQUIRE(epi == EPI_GELU || epi == EPI_RELU2 || epi == EPI_STORE_F32 || epi == EPI_GATED_EXPERTS, "gemm_tc_grouped: epilogue %d", epi);
+    BLM_REQUIRE(epi != EPI_GATED_EXPERTS || N % 16 == 0, "gemm_tc_grouped: gated experts of %d rows", N);
     BLM_REQUIRE(status != nullptr && tile_expert != nullptr, "gemm_tc_grouped: no status word or no table of tiles");
     BLM_REQUIRE((long long)n_experts * N < (1ll << 31), "gemm_tc_grouped: %d experts of %d rows", n_experts, N);
     CUtensorMap xmap, wmap;
     int rc = make_map(x, ldx, M, K, BM, false, &xmap);
     if (rc != BLM_OK) return rc;
-    rc = make_map(w, ldw, n_experts * N, K, BN, true, &wmap);
+    rc = epi == EPI_GATED_EXPERTS ? make_gated_map(w, ldw, n_experts, N / 2, K, &wmap) : make_map(w, ldw, n_experts * N, K, BN, true, &wmap);
     if (rc != BLM_OK) return rc;
     TcArgs a;
     a.y = (__nv_bfloat16*)y; a.acc = (float*)y; a.ldy = ldy; a.M = M; a.N = N; a.K = K; a.epi = epi; a.status = status;
-    a.tile_expert = tile_expert; a.expert_rows = N;
+    a.tile_expert = tile_expert; a.expert_rows = N; a.limit = limit; a.alpha = alpha;
     const size_t smem = (size_t)kStages * (kABytes + kBBytes) + (2 * kStages + 4) * 8 + 16 + 1024;
     static bool opted_in = false;
     if (!opted_in) {
         cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_GELU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_RELU2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_GATED_EXPERTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tc_kernel<EPI_STORE_F32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "gemm_tc_grouped: %s", cudaGetErrorString(e));
         opted_in = true;
@@ -473,6 +522,7 @@ BLM_API int blm_gemm_tc_grouped(const void* x, long long ldx, const void* w, lon
     const int grid = (int)(tiles < blm_sm_count() ? tiles : blm_sm_count());        // persistent: one block per SM
     if (epi == EPI_GELU) gemm_tc_kernel<EPI_GELU><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     else if (epi == EPI_RELU2) gemm_tc_kernel<EPI_RELU2><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
+    else if (epi == EPI_GATED_EXPERTS) gemm_tc_kernel<EPI_GATED_EXPERTS><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     else gemm_tc_kernel<EPI_STORE_F32><<<grid, kThreads, smem, stream>>>(a, xmap, wmap);
     return blm_check_launch("gemm_tc_grouped");
 }

@@ -100,12 +100,13 @@ _protos = {
         "blm_attention_sink": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                c_void_p, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_float, c_void_p, c_int, c_int,
                                c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_float,
-                               c_void_p, c_int, c_float, c_float, c_float, c_int, c_void_p, c_void_p],
+                               c_void_p, c_int, c_float, c_float, c_float, c_int, c_int, c_void_p, c_void_p],
         "blm_head_norm_rope_append": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
                                       c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
                                       c_void_p, c_void_p, c_int, c_void_p, c_float, c_int, c_int, c_void_p],
         "blm_attention_sink_prompt_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
         "blm_attention_sink_decode_takes": [c_int, c_int, c_int, c_int, c_int, c_int],
+        "blm_attention_sink_streams": [c_int, c_int, c_int, c_int, c_int],
         "blm_attention_sink_pairs": [c_int, c_int, c_int, c_int, c_int, c_int, c_int],
     },
     "stream_ops": {
@@ -211,7 +212,7 @@ _protos = {
                         c_void_p, c_void_p],
         "blm_gemm_tc_supported": [c_int, c_int, c_int],
         "blm_gemm_tc_grouped": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p,
-                                c_int, c_void_p, c_void_p],
+                                c_int, c_float, c_float, c_void_p, c_void_p],
     },
     "gemm_sk": {
         "blm_gemm_sk": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_int, c_void_p, c_int,
@@ -499,6 +500,12 @@ def attention_sink_decode_takes(dtype, key_dim, value_dim, n_heads, n_kv) -> boo
     return bool(_lib("attention_sink").blm_attention_sink_decode_takes(_code(dtype), key_dim, value_dim, PAGE, n_heads, n_kv))
 
 
+def attention_sink_streams(dtype, key_dim, n_heads, n_kv) -> bool:
+    """Whether single tokens whose values are the keys run the dense decoder's streaming kernel (with no other option than a window
+    and slopes); its splits are then cut as that mixer's are."""
+    return bool(_lib("attention_sink").blm_attention_sink_streams(_code(dtype), key_dim, PAGE, n_heads, n_kv))
+
+
 def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, value_dim, scale, window, keep_first=0, sink=True,
                    gate=None, gate_stride=0, max_q_len=1, n_splits=1, scratch=None, head_scale=None, sink_logit=None, softcap=0.0,
                    chunk=0, gate_lanes=0, out_scale=1.0, maps=1, difference=(0.0, 1.0, 0.0), slope=None, shared=False):
@@ -546,15 +553,17 @@ def attention_sink(q, step, pool, block_table, out, n_heads, n_kv, key_dim, valu
     if need:
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need:
             raise KernelError(f"attention_sink: {n_splits} splits need {need} float32 of scratch")
-    cu = step.cu_seqlens if prompt else None
+    cu = getattr(step, "cu_seqlens", None)
+    if cu is None or not (prompt or shared):
+        cu = None
     _call("attention_sink", "blm_attention_sink", _ptr(q), _ptr(pool), _code(pool.dtype), _flat_pool(pool, n_kv, key_dim, value_dim, maps, shared),
           _ptr(block_table), block_table.shape[1], _ptr(step.token_seq), _ptr(step.token_pos), _ptr(step.slot_of_seq), _ptr(cu),
-          _ptr(step.start_pos if prompt else None), (cu.numel() - 1) if prompt else 0, int(max_q_len), _ptr(gate), int(gate_stride),
+          _ptr(step.start_pos if cu is not None else None), (cu.numel() - 1) if cu is not None else 0, int(max_q_len), _ptr(gate), int(gate_stride),
           int(gate_lanes), _ptr(out), c_longlong(out.stride(0)), c_float(out_scale), _ptr(scratch if need else None), int(n_splits), n, n_heads,
           n_kv, int(maps), key_dim, value_dim, PAGE, int(window), int(chunk), int(keep_first), c_float(scale), 1 if sink else 0,
           _ptr(head_scale), _ptr(sink_logit if sink else None), c_float(softcap or 0.0), _ptr(slope), 1 if shared else 0,
           *(c_float(v) for v in difference),
-          pool.shape[0] if prompt else 0, _ptr(status_word(q.device)) if prompt else None, _stream(),
+          pool.shape[0] if cu is not None else 0, int(getattr(step, "max_kv_len", 0)), _ptr(status_word(q.device)) if cu is not None else None, _stream(),
           kernels=2 if need else 1)
 
 
@@ -590,7 +599,7 @@ def moe_route(h, router, top, softmax=False, correction=None, renormalise=False,
 
 # an expert's unit: gated (silu or clamped); W_down gelu(W_up x), exact or tanh form; W_down relu(W_up x)^2
 UNIT_GATED, UNIT_GELU, UNIT_GELU_TANH, UNIT_RELU2 = 0, 1, 2, 3
-MOE_TC_UNITS = {UNIT_GELU: 3, UNIT_RELU2: 5}         # units the grouped tcgen05 product takes, and its epilogue for each
+MOE_TC_UNITS = {UNIT_GATED: 6, UNIT_GELU: 3, UNIT_RELU2: 5}         # units the grouped tcgen05 product takes, and its epilogue for each
 
 
 def moe_experts(h, ids, weights, gate_up, down, extra=None, weight_on_input=True, clamp_limit=0.0, clamp_alpha=1.702, out_dtype=None,
@@ -616,8 +625,8 @@ def moe_experts(h, ids, weights, gate_up, down, extra=None, weight_on_input=True
     dev = h.device
     pairs = n * top
     if (unit in MOE_TC_UNITS and not weight_on_input and h.dtype == torch.bfloat16 and pairs >= MOE_TC_PAIRS * e and d % 8 == 0 and ff % 8 == 0
-            and d >= 64 and ff >= 64 and e * max(d, ff) < (1 << 31)):
-        return _moe_experts_tc(h, ids, weights, gate_up, down, extra, out_dtype or h.dtype, unit)
+            and d >= 64 and ff >= 64 and e * max(d, 2 * ff) < (1 << 31)):
+        return _moe_experts_tc(h, ids, weights, gate_up, down, extra, out_dtype or h.dtype, unit, clamp_limit, clamp_alpha)
     offsets = torch.empty(e + 1, dtype=torch.int32, device=dev)
     order = torch.empty(pairs, dtype=torch.int32, device=dev)
     place_of = torch.empty(pairs, dtype=torch.int32, device=dev)
@@ -635,20 +644,21 @@ def moe_experts(h, ids, weights, gate_up, down, extra=None, weight_on_input=True
     return out
 
 
-# from this many (token, expert) pairs an expert on average, experts without a gate run on tcgen05 (BURN_LM_B200_MOE_TC_PAIRS=n
+# from this many (token, expert) pairs an expert on average, experts run on tcgen05 (BURN_LM_B200_MOE_TC_PAIRS=n
 # to measure another border)
 MOE_TC_PAIRS = int(os.environ.get("BURN_LM_B200_MOE_TC_PAIRS", "16"))
 MOE_TC_ROWS = 128       # rows of a tile of the tcgen05 product: an expert's share of the pairs starts at a multiple of it
 
 
-def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype, unit=UNIT_GELU):
-    """Experts without a gate for prompts, both products on the tcgen05 tensor cores: the pairs' token rows are gathered expert
+def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype, unit=UNIT_GELU, clamp_limit=0.0, clamp_alpha=1.702):
+    """Experts for prompts, both products on the tcgen05 tensor cores: the pairs' token rows are gathered expert
     by expert, every expert's share starting at a multiple of 128 places (a place no pair owns holds zeros), and one grouped
     product runs over all experts at once (kernels of gemm_tc.cu: a table names the expert of every tile of places); the
     first product's epilogue applies the unit's activation, the second leaves fp32 sums, and the sum over a token's experts weighs
     them as ever.  Everything is sized by the token count alone, so a step can be captured."""
     n, d = h.shape
-    e, ff, _ = up.shape
+    e, rows, _ = up.shape
+    ff = down.shape[2]
     top = ids.shape[1]
     pairs, dev, stream = n * top, h.device, _stream()
     tiles = int(_lib("moe").blm_moe_padded_tiles(pairs, e, MOE_TC_ROWS))
@@ -663,10 +673,10 @@ def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype, unit=UNIT_GELU)
     status = status_word(dev)
     _call("moe", "blm_moe_group_padded", _ptr(ids), pairs, e, MOE_TC_ROWS, _ptr(place_of), _ptr(pair_of_place), _ptr(tile_expert), stream)
     _call("moe", "blm_moe_gather_rows", _ptr(h), _ptr(pair_of_place), _ptr(xs), places, d, top, stream)
-    _call("gemm_tc", "blm_gemm_tc_grouped", _ptr(xs), c_longlong(d), _ptr(up), c_longlong(d), _ptr(act), c_longlong(ff), places, ff, d, e,
-          _ptr(tile_expert), MOE_TC_UNITS[unit], _ptr(status), stream)
+    _call("gemm_tc", "blm_gemm_tc_grouped", _ptr(xs), c_longlong(d), _ptr(up), c_longlong(d), _ptr(act), c_longlong(ff), places, rows, d, e,
+          _ptr(tile_expert), MOE_TC_UNITS[unit], c_float(clamp_limit), c_float(clamp_alpha), _ptr(status), stream)
     _call("gemm_tc", "blm_gemm_tc_grouped", _ptr(act), c_longlong(ff), _ptr(down), c_longlong(ff), _ptr(y), c_longlong(d), places, d, ff, e,
-          _ptr(tile_expert), 4, _ptr(status), stream)
+          _ptr(tile_expert), 4, c_float(0.0), c_float(0.0), _ptr(status), stream)
     _call("moe", "blm_moe_combine", _ptr(y), _ptr(place_of), _ptr(weights), _ptr(extra), _ptr(out), _code(h.dtype), n, d, top,
           1, _code(out.dtype), 1, stream)
     return out

@@ -23,6 +23,19 @@ from .base import CacheNeed, Part
 from .linear import Linear
 
 BLOCKS_PER_SM = 2     # blocks a decode step should offer every multiprocessor
+
+
+def streaming_splits(n_seqs: int, n_kv_heads: int, pages: int, ring_pages: int, device) -> int:
+    """Over how many blocks the streaming decode kernel cuts a sequence's pages.  One block walks all pages of a (sequence, kv
+    head) while they fit its ring (`ring_pages`, and some more still stream well): its groups of warps work on several pages at
+    once and nothing is combined (measured best at batch 1, 8 and 64 with 9 pages).  Longer sequences are cut into a ring's worth
+    per block, as far as that still helps to fill the SMs about twice."""
+    by_length = (pages + ring_pages - 1) // ring_pages
+    want = BLOCKS_PER_SM * K.sm_count(device)
+    to_fill = (want + n_seqs * n_kv_heads - 1) // (n_seqs * n_kv_heads)
+    return max(1, min(by_length, to_fill, pages, 64))
+
+
 TUNED_HEADS = (64, 128)   # head sizes with kernels of their own (tcgen05 prompts, streaming decode); the others run the general one
 
 
@@ -108,14 +121,7 @@ class Attention(Part):
         group = s.n_heads // s.n_kv_heads
         pages = (step.max_kv_len + K.PAGE - 1) // K.PAGE
         if K.attention_decode_is_specialised(self.runtime.dtype, s.head_dim, group):
-            # One block walks all pages of a (sequence, kv head) while they fit its ring of about twelve
-            # pages (sixteen still stream well): its groups of warps work on several pages at once and nothing is combined
-            # (measured best at batch 1, 8 and 64 with 9 pages).  Longer sequences are cut into a ring's
-            # worth per block, as far as that still helps to fill the SMs about twice.
-            by_length = (pages + 15) // 16
-            want = BLOCKS_PER_SM * K.sm_count(self.runtime.device)
-            to_fill = (want + step.n_seqs * s.n_kv_heads - 1) // (step.n_seqs * s.n_kv_heads)
-            return max(1, min(by_length, to_fill, pages, 64))
+            return streaming_splits(step.n_seqs, s.n_kv_heads, pages, 16, self.runtime.device)     # (a ring holds about twelve pages)
         blocks = step.n_seqs * s.n_kv_heads * ((group + 31) // 32)
         return max(1, min(pages, (BLOCKS_PER_SM * K.sm_count(self.runtime.device) + blocks - 1) // blocks, 64))
 

@@ -35,6 +35,7 @@ import torch
 from .. import kernels as K
 from ..registry import register_part
 from ..weights.loader import TensorSpec
+from .attention import streaming_splits
 from .base import CacheNeed, Part
 from .linear import Linear
 from .norm import PendingSum
@@ -42,6 +43,7 @@ from .position import RotarySpec, rotary_inverse_frequencies, rotary_multiplier
 
 BLOCKS_PER_SM = 4          # blocks of the single-token kernels a step should offer every multiprocessor
 TABLE_BYTES = 64 << 20     # a layer's table of cosines and sines at most
+STREAM_PAGES = 20          # pages a block of the streaming kernel walks before a sequence's keys are cut
 NO_WINDOW = 1 << 30        # what the kernels take for "every earlier key"
 
 
@@ -147,6 +149,8 @@ class NormedAttention(Part):
             rot = RotarySpec(s.head_dim, s.rotary_base, rotary_dim=s.rotary_dims, scaling=s.rotary_scaling)
             self.freq = torch.tensor(rotary_inverse_frequencies(rot), dtype=torch.float64).to(self.o.weight.device)
             self.turn_scale = rotary_multiplier(rot)
+        self.streams = (s.values_are_keys and self.o.weight.is_cuda and not (s.sink or s.softcap or s.head_temperature or s.output_gate or s.chunk)
+                        and K.attention_sink_streams(self.runtime.dtype, s.head_dim, s.n_heads, s.n_kv_heads))
         self.difference = (0.0, 1.0, 0.0)
         if s.diff is not None:
             lq1, lk1, lq2, lk2 = (loaded[t[r]].to(torch.float64) for r in ("lq1", "lk1", "lq2", "lk2"))
@@ -172,6 +176,8 @@ class NormedAttention(Part):
         if K.attention_sink_prompt_takes(self.runtime.dtype, s.head_dim, s.value_dim, step.max_q_len, self.maps * s.n_heads):
             return 1
         seen = min(step.max_kv_len, s.window or s.chunk or step.max_kv_len)
+        if self.streams and step.max_q_len == 1 and step.n_tokens == step.n_seqs:
+            return streaming_splits(step.n_seqs, s.n_kv_heads, (seen + 2 * K.PAGE - 2) // K.PAGE, STREAM_PAGES, self.runtime.device)
         blocks = step.n_tokens * self.maps * s.n_kv_heads
         if self.maps == 2 and K.attention_sink_pairs(self.runtime.dtype, s.head_dim, s.value_dim, 2 * s.n_heads, 2 * s.n_kv_heads, 2):
             blocks //= 2                                     # both maps of a head share a block
