@@ -1042,7 +1042,8 @@ BLM_API int blm_moe_experts(const void* h, int dtype, const float* weights, cons
 // ---------------------------------------------------------------------------------------------
 // For the grouped product on tcgen05 (gemm_tc.cu): the pairs laid out expert by expert with every expert's share starting at
 // a multiple of `tile_rows` places.  place_of[pair] = its place; pair_of_place[place] = the pair, -1 for a place no pair
-// owns; tile_expert[tile] = the expert that owns the tile of places, -1 for none.  One block.
+// owns; tile_expert[tile] = the expert that owns the tile of places (-1 for none; such tiles come last), and behind the table
+// the number of tiles that have one.  One block.
 // ---------------------------------------------------------------------------------------------
 __global__ void moe_group_padded_kernel(const int* __restrict__ ids, int n_pairs, int n_experts, int tile_rows, int max_tiles,
                                         int* __restrict__ place_of, int* __restrict__ pair_of_place, int* __restrict__ tile_expert) {
@@ -1062,6 +1063,7 @@ __global__ void moe_group_padded_kernel(const int* __restrict__ ids, int n_pairs
             for (int t = 0; t < tiles && tile + t < max_tiles; ++t) tile_expert[tile + t] = e;
             tile += tiles;
         }
+        tile_expert[max_tiles] = min(tile, max_tiles);
     }
     __syncthreads();
     for (int a = threadIdx.x; a < n_pairs; a += blockDim.x) {

@@ -43,11 +43,35 @@ struct RetSeq {
     }
 };
 
+// (a call of its own: inlined, it would cost every kernel its registers)
+__device__ __noinline__ float2 ret_angle(double angle) {
+    double sn, cs;
+    sincos(angle, &sn, &cs);
+    return make_float2((float)cs, (float)sn);
+}
 __device__ __forceinline__ float2 ret_turn(const RetIn& in, int pos, int i) {
     if (pos < in.table_len) return in.table[(size_t)pos * (in.rot >> 1) + i];
-    double sn, cs;
-    sincos((double)pos * in.freq[i], &sn, &cs);
-    return make_float2((float)cs, (float)sn);
+    return ret_angle((double)pos * in.freq[i]);
+}
+// (cosine, sine) of pairs i .. i + 3, i a multiple of 4
+__device__ __forceinline__ void ret_turn4(const RetIn& in, int pos, int i, float4& lo, float4& hi) {
+    if (pos < in.table_len) {
+        const float4* t = reinterpret_cast<const float4*>(in.table + (size_t)pos * (in.rot >> 1) + i);
+        lo = t[0];
+        hi = t[1];
+        return;
+    }
+    float2 a = ret_angle((double)pos * in.freq[i]), b = ret_angle((double)pos * in.freq[i + 1]);
+    lo = make_float4(a.x, a.y, b.x, b.y);
+    a = ret_angle((double)pos * in.freq[i + 2]);
+    b = ret_angle((double)pos * in.freq[i + 3]);
+    hi = make_float4(a.x, a.y, b.x, b.y);
+}
+// lanes d .. d + 3 of the first half (a) and of the second (b), turned together
+__device__ __forceinline__ void ret_turn_pairs(float4& a, float4& b, const float4& lo, const float4& hi) {
+    const float4 u = a, v = b;
+    a = make_float4(u.x * lo.x - v.x * lo.y, u.y * lo.z - v.y * lo.w, u.z * hi.x - v.z * hi.y, u.w * hi.z - v.w * hi.w);
+    b = make_float4(v.x * lo.x + u.x * lo.y, v.y * lo.z + u.y * lo.w, v.z * hi.x + u.z * hi.y, v.w * hi.z + u.w * hi.w);
 }
 // lane d of a head's query or key (`src`: the head's first lane), turned
 __device__ __forceinline__ float ret_lane(const RetIn& in, const float* src, int pos, int d) {
@@ -154,10 +178,10 @@ __global__ void __launch_bounds__(256) retention_scan_kernel(RetIn in, RetSeq sq
 // the single token: a block per (head, token).  Thread (row group, column group) takes N value lanes of rows rg, rg + n_rg, ...
 // ---------------------------------------------------------------------------------------------
 constexpr int kStepThreads = 256;
-constexpr int kAhead = 8;          // rows a thread asks for before it works on the first
 
-template <typename TO, int N>
-__global__ void __launch_bounds__(kStepThreads) retention_step_kernel(RetIn in, RetSeq sq, const int* __restrict__ token_seq,
+// kAhead: rows a thread asks for before it works on the first
+template <typename TO, int N, int kAhead>
+__global__ void __launch_bounds__(kStepThreads, kAhead > 4 ? 3 : 4) retention_step_kernel(RetIn in, RetSeq sq, const int* __restrict__ token_seq,
                                                                       const int* __restrict__ token_pos, float eps, TO* __restrict__ out,
                                                                       long long out_stride, int vec) {
     extern __shared__ __align__(16) float sm[];
@@ -312,26 +336,141 @@ __device__ __forceinline__ RetChunk ret_find(const RetSeq& sq, int block, int* s
     return c;
 }
 
+// How a block's threads share out [rows][per] items: thread (ty, tx) takes item tx of rows ty, ty + step, ...
+struct RetShare {
+    int tx, ty, step;
+    bool works;
+    __device__ __forceinline__ explicit RetShare(int per) {
+        tx = threadIdx.x % per;
+        ty = threadIdx.x / per;
+        step = blockDim.x / per;
+        works = ty < step;
+    }
+};
+__device__ __forceinline__ float4 ret_zero4() { return make_float4(0.f, 0.f, 0.f, 0.f); }
+__device__ __forceinline__ void ret_put4(__nv_bfloat16* dst, const float4& v) {
+    *reinterpret_cast<uint2*>(dst) = make_uint2(ret_pack(v.x, v.y), ret_pack(v.z, v.w));
+}
+__device__ __forceinline__ void ret_split4(__nv_bfloat16* hi, __nv_bfloat16* rest, const float4& v) {
+    uint32_t h0, h1, r0, r1;
+    ret_split(v.x, v.y, h0, r0);
+    ret_split(v.z, v.w, h1, r1);
+    *reinterpret_cast<uint2*>(hi) = make_uint2(h0, h1);
+    *reinterpret_cast<uint2*>(rest) = make_uint2(r0, r1);
+}
+
 // a head's values of a chunk as bfloat16 [kC][vstride], zeros beyond its tokens and lanes
 __device__ __forceinline__ void ret_stage_values(const RetIn& in, const RetChunk& c, int head, __nv_bfloat16* vs, int vstride, int cols, bool vec) {
-    const int quads = cols / 4;
-    for (int idx = threadIdx.x; idx < kC * quads; idx += blockDim.x) {
-        const int t = idx / quads, d = (idx % quads) * 4;
-        float v[4] = {0.f, 0.f, 0.f, 0.f};
-        if (t < c.rows) {
-            const float* src = in.proj + (size_t)(c.first_row + t) * in.stride + 2 * in.heads * in.dk + head * in.dv;
-            if (vec) {
-                if (d < in.dv) {
-                    const float4 f = *reinterpret_cast<const float4*>(src + d);
-                    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-                }
-            } else {
+    const float* src = in.proj + (size_t)c.first_row * in.stride + 2 * in.heads * in.dk + head * in.dv;
+    if (vec) {
+        const RetShare sh(cols / 4);
+        const int d = sh.tx * 4;
+        for (int t = sh.ty; t < kC && sh.works; t += 4 * sh.step) {
+            float4 v[4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e)
-                    if (d + e < in.dv) v[e] = src[d + e];
+            for (int u = 0; u < 4; ++u) {
+                const int r = t + u * sh.step;
+                v[u] = r < c.rows && d < in.dv ? *reinterpret_cast<const float4*>(src + (size_t)r * in.stride + d) : ret_zero4();
+            }
+#pragma unroll
+            for (int u = 0; u < 4; ++u)
+                if (t + u * sh.step < kC) ret_put4(vs + (t + u * sh.step) * vstride + d, v[u]);
+        }
+        return;
+    }
+    for (int idx = threadIdx.x; idx < kC * cols; idx += blockDim.x) {
+        const int t = idx / cols, d = idx % cols;
+        vs[t * vstride + d] = __float2bfloat16_rn(t < c.rows && d < in.dv ? src[(size_t)t * in.stride + d] : 0.f);
+    }
+}
+
+// a head's turned keys (and queries, where QUERIES) of a chunk: put(is_query, token, first of four lanes, values), every token of
+// kC and every four lanes of dkp, zeros beyond the chunk's tokens and the head's lanes.  Keys come times k_scale.
+template <bool QUERIES, typename Put>
+__device__ __forceinline__ void ret_stage_rows(const RetIn& in, const RetChunk& c, int head, int dkp, bool vec, Put put) {
+    const float* kp = in.proj + (size_t)c.first_row * in.stride + (in.heads + head) * in.dk;
+    const float* qp = in.proj + (size_t)c.first_row * in.stride + head * in.dk;
+    if (vec) {
+        // an item: four lanes of the first half with their partners in the second, or four lanes that pass
+        const int half = in.rot >> 1, pairs = half / 4, per = pairs + (dkp - in.rot) / 4;
+        const RetShare sh(per);
+        const bool turns = sh.tx < pairs;
+        const int d = turns ? sh.tx * 4 : in.rot + (sh.tx - pairs) * 4;
+        for (int t0 = sh.ty; t0 < kC && sh.works; t0 += 2 * sh.step) {
+            float4 k[2][2], q[2][2], lo[2], hi[2];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int t = t0 + u * sh.step;
+                const bool there = t < c.rows && d < in.dk;
+                const size_t at = (size_t)t * in.stride + d;
+                k[u][0] = there ? *reinterpret_cast<const float4*>(kp + at) : ret_zero4();
+                k[u][1] = there && turns ? *reinterpret_cast<const float4*>(kp + at + half) : ret_zero4();
+                if (QUERIES) {
+                    q[u][0] = there ? *reinterpret_cast<const float4*>(qp + at) : ret_zero4();
+                    q[u][1] = there && turns ? *reinterpret_cast<const float4*>(qp + at + half) : ret_zero4();
+                }
+                if (there && turns) ret_turn4(in, c.start + t, d, lo[u], hi[u]);
+                else lo[u] = hi[u] = make_float4(1.f, 0.f, 1.f, 0.f);
+            }
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int t = t0 + u * sh.step;
+                if (t >= kC) continue;
+                if (turns) ret_turn_pairs(k[u][0], k[u][1], lo[u], hi[u]);
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    if (e == 1 && !turns) continue;
+                    float4& v = k[u][e];
+                    v.x *= in.k_scale; v.y *= in.k_scale; v.z *= in.k_scale; v.w *= in.k_scale;
+                    put(false, t, d + e * half, v);
+                }
+                if (QUERIES) {
+                    if (turns) ret_turn_pairs(q[u][0], q[u][1], lo[u], hi[u]);
+                    put(true, t, d, q[u][0]);
+                    if (turns) put(true, t, d + half, q[u][1]);
+                }
             }
         }
-        ret_put4(vs + t * vstride + d, v);
+        return;
+    }
+    const int quads = dkp / 4;
+    for (int idx = threadIdx.x; idx < (QUERIES ? 2 : 1) * kC * quads; idx += blockDim.x) {
+        const bool is_q = idx >= kC * quads;
+        const int i = is_q ? idx - kC * quads : idx, t = i / quads, d = (i % quads) * 4;
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (t < c.rows && d < in.dk) ret_lanes4(in, (is_q ? qp : kp) + (size_t)t * in.stride, c.start + t, d, false, v);
+        const float w = is_q ? 1.f : in.k_scale;
+        put(is_q, t, d, make_float4(v[0] * w, v[1] * w, v[2] * w, v[3] * w));
+    }
+}
+
+// rows s0 .. s0 + m - 1 of S as high parts and rests [m][vstride], zeros beyond its rows and columns
+__device__ __forceinline__ void ret_stage_state(const RetIn& in, const float* S, int s0, int m, __nv_bfloat16* sh, __nv_bfloat16* sr, int vstride, int cols,
+                                                bool vec) {
+    const RetShare share(cols / 4);
+    const int d = share.tx * 4;
+    for (int r0 = share.ty; r0 < m && share.works; r0 += 4 * share.step) {
+        float4 v[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int r = r0 + u * share.step;
+            v[u] = ret_zero4();
+            if (r >= m || s0 + r >= in.dk || d >= in.dv) continue;
+            const float* src = S + (size_t)(s0 + r) * in.dv + d;
+            if (vec) {
+                v[u] = *reinterpret_cast<const float4*>(src);
+            } else {
+                v[u].x = src[0];
+                if (d + 1 < in.dv) v[u].y = src[1];
+                if (d + 2 < in.dv) v[u].z = src[2];
+                if (d + 3 < in.dv) v[u].w = src[3];
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int r = r0 + u * share.step;
+            if (r < m) ret_split4(sh + r * vstride + d, sr + r * vstride + d, v[u]);
+        }
     }
 }
 
@@ -347,35 +486,24 @@ __global__ void __launch_bounds__(256) retention_chunk_add_kernel(RetIn in, RetS
     __nv_bfloat16* kr = kh + kC * kstride;                               // ... and rests
     __nv_bfloat16* vs = kr + kC * kstride;                               // [kC][vstride]
     const float* powers = in.powers + (size_t)head * (kC + 1);
-    const int quads = dkp / 4;
-    for (int idx = threadIdx.x; idx < kC * quads; idx += blockDim.x) {
-        const int t = idx / quads, d = (idx % quads) * 4;
-        float v[4] = {0.f, 0.f, 0.f, 0.f};
-        if (t < c.rows && d < dk) {
-            ret_lanes4(in, in.proj + (size_t)(c.first_row + t) * in.stride + (in.heads + head) * dk, c.start + t, d, vec, v);
-            const float w = powers[c.rows - 1 - t] * in.k_scale;
-#pragma unroll
-            for (int e = 0; e < 4; ++e) v[e] *= w;
-        }
-        uint32_t h0, h1, r0, r1;
-        ret_split(v[0], v[1], h0, r0);
-        ret_split(v[2], v[3], h1, r1);
-        *reinterpret_cast<uint2*>(kh + t * kstride + d) = make_uint2(h0, h1);
-        *reinterpret_cast<uint2*>(kr + t * kstride + d) = make_uint2(r0, r1);
-    }
+    ret_stage_rows<false>(in, c, head, dkp, vec, [&](bool, int t, int d, float4 v) {
+        const float w = t < c.rows ? powers[c.rows - 1 - t] : 0.f;
+        v.x *= w; v.y *= w; v.z *= w; v.w *= w;
+        ret_split4(kh + t * kstride + d, kr + t * kstride + d, v);
+    });
     ret_stage_values(in, c, head, vs, vstride, cols, vec);
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
     const int lrow = lane & 7, lmat = lane >> 3, quad = lane >> 2, pair = (lane & 3) * 2;
     float* dst = kv + ((size_t)blockIdx.x * in.heads + head) * dk * dv;
-    // a unit: 16 rows of S by 64 of its columns
-    const int units = (dkp / 16) * (cols / 64);
+    // a unit: 16 rows of S by 32 of its columns
+    const int units = (dkp / 16) * (cols / 32);
     const bool two = dv % 2 == 0;
     for (int u = warp; u < units; u += n_warps) {
-        const int m0 = (u % (dkp / 16)) * 16, n0 = (u / (dkp / 16)) * 64;
-        float acc[8][4];
+        const int m0 = (u % (dkp / 16)) * 16, n0 = (u / (dkp / 16)) * 32;
+        float acc[4][4];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+        for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
         // A: the keys read transposed (rows of S by tokens)
         const unsigned ao = (unsigned)((((lmat >> 1) * 8 + lrow) * kstride + m0 + (lmat & 1) * 8) * 2);
         const unsigned bo = ret_smem(vs) + (unsigned)((((lmat & 1) * 8 + lrow) * vstride + n0 + (lmat >> 1) * 8) * 2);
@@ -385,7 +513,7 @@ __global__ void __launch_bounds__(256) retention_chunk_add_kernel(RetIn in, RetS
             ret_ldsm_t(ah, ret_smem(kh) + ao + kk * kstride * 2);
             ret_ldsm_t(ar, ret_smem(kr) + ao + kk * kstride * 2);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
+            for (int j = 0; j < 2; ++j) {
                 ret_ldsm_t(b, bo + (kk * vstride + 16 * j) * 2);
                 ret_mma(acc[2 * j], ah, b[0], b[1]);
                 ret_mma(acc[2 * j + 1], ah, b[2], b[3]);
@@ -394,7 +522,7 @@ __global__ void __launch_bounds__(256) retention_chunk_add_kernel(RetIn in, RetS
             }
         }
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
+        for (int j = 0; j < 4; ++j)
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
                 const int row = m0 + quad + 8 * half, col = n0 + 8 * j + pair;
@@ -411,55 +539,38 @@ __global__ void __launch_bounds__(256) retention_chunk_add_kernel(RetIn in, RetS
 }
 
 // (2) S in front of every chunk, in place of what the chunk adds; S behind the last one goes to the sequence's state
-template <int N>
-__global__ void __launch_bounds__(256) retention_carry_kernel(RetIn in, RetSeq sq, float* __restrict__ kv) {
+__global__ void __launch_bounds__(256, 6) retention_carry_kernel(RetIn in, RetSeq sq, float* __restrict__ kv) {
     const int head = blockIdx.y, seq = blockIdx.z;
-    const size_t size = (size_t)in.dk * in.dv, at = ((size_t)blockIdx.x * 256 + threadIdx.x) * N;
+    const size_t size = (size_t)in.dk * in.dv, at = (size_t)blockIdx.x * 256 + threadIdx.x;
     const int len = sq.cu_seqlens[seq + 1] - sq.cu_seqlens[seq];
     if (at >= size || len <= 0) return;
     int first = 0;                                     // the sequence's first chunk
     for (int s = 0; s < seq; ++s) first += (sq.cu_seqlens[s + 1] - sq.cu_seqlens[s] + kC - 1) / kC;
     const int start = sq.start_pos[seq], n_chunks = (len + kC - 1) / kC;
-    const float* from = sq.copy(seq, start) + (size_t)head * size + at;
-    float S[N];
-#pragma unroll
-    for (int e = 0; e < N; ++e) S[e] = start > 0 ? from[e] : 0.f;
+    float S = start > 0 ? sq.copy(seq, start)[(size_t)head * size + at] : 0.f;
     const float* powers = in.powers + (size_t)head * (kC + 1);
     const float full = powers[kC], last = powers[len - (n_chunks - 1) * kC];
     const size_t step = (size_t)in.heads * size;
     float* p = kv + (size_t)first * step + (size_t)head * size + at;
-    constexpr int kRead = 4;                           // chunks read ahead of their turn
+    constexpr int kRead = 8;                           // chunks read ahead of their turn
     for (int c0 = 0; c0 < n_chunks; c0 += kRead) {
-        float add[kRead][N];
+        float add[kRead];
+#pragma unroll
+        for (int a = 0; a < kRead; ++a)
+            if (c0 + a < n_chunks) add[a] = p[(size_t)(c0 + a) * step];
 #pragma unroll
         for (int a = 0; a < kRead; ++a)
             if (c0 + a < n_chunks) {
-                if (N == 4) {
-                    const float4 v = *reinterpret_cast<const float4*>(p + (size_t)(c0 + a) * step);
-                    add[a][0] = v.x; add[a][1 % N] = v.y; add[a][2 % N] = v.z; add[a][3 % N] = v.w;
-                } else {
-                    add[a][0] = p[(size_t)(c0 + a) * step];
-                }
-            }
-#pragma unroll
-        for (int a = 0; a < kRead; ++a)
-            if (c0 + a < n_chunks) {
-                float* q = p + (size_t)(c0 + a) * step;
-                if (N == 4) *reinterpret_cast<float4*>(q) = make_float4(S[0], S[1 % N], S[2 % N], S[3 % N]);
-                else q[0] = S[0];
-                const float w = c0 + a == n_chunks - 1 ? last : full;
-#pragma unroll
-                for (int e = 0; e < N; ++e) S[e] = fmaf(w, S[e], add[a][e]);
+                p[(size_t)(c0 + a) * step] = S;
+                S = fmaf(c0 + a == n_chunks - 1 ? last : full, S, add[a]);
             }
     }
-    float* to = sq.copy(seq, start + len) + (size_t)head * size + at;
-#pragma unroll
-    for (int e = 0; e < N; ++e) to[e] = S[e];
+    sq.copy(seq, start + len)[(size_t)head * size + at] = S;
 }
 
-// (3) a chunk's rows: four warps of 16 rows each for every 64 value lanes.  slice: rows of S in shared memory at a time.
-template <int WARPS>
-__global__ void __launch_bounds__(32 * WARPS) retention_chunk_out_kernel(RetIn in, RetSeq sq, const float* __restrict__ kv, int slice, float eps,
+// (3) a chunk's rows: four warps of 16 rows each for every 8 NV value lanes.  slice: rows of S in shared memory at a time.
+template <int WARPS, int NV>
+__global__ void __launch_bounds__(32 * WARPS, NV == 4 ? 32 / WARPS : 1) retention_chunk_out_kernel(RetIn in, RetSeq sq, const float* __restrict__ kv, int slice, float eps,
                                                                    __nv_bfloat16* __restrict__ out, long long out_stride, int n_tokens, int vec) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ int found[3];
@@ -479,64 +590,33 @@ __global__ void __launch_bounds__(32 * WARPS) retention_chunk_out_kernel(RetIn i
     __nv_bfloat16* vs = ks + kC * kstride;                               // [kC][vstride]
     __nv_bfloat16* sh = vs + kC * vstride;                               // [slice][vstride] S: high parts
     __nv_bfloat16* sr = sh + slice * vstride;                            // ... and rests
-    const int quads = dkp / 4;
-    for (int idx = tid; idx < 2 * kC * quads; idx += blockDim.x) {
-        const bool is_k = idx >= kC * quads;
-        const int i = is_k ? idx - kC * quads : idx, t = i / quads, d = (i % quads) * 4;
-        float v[4] = {0.f, 0.f, 0.f, 0.f};
-        if (t < c.rows && d < dk) {
-            ret_lanes4(in, in.proj + (size_t)(c.first_row + t) * in.stride + ((is_k ? in.heads : 0) + head) * dk, c.start + t, d, vec, v);
-            if (is_k) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) v[e] *= in.k_scale;
-            }
-        }
-        ret_put4((is_k ? ks : qs) + t * kstride + d, v);
-    }
+    const float* S = kv + ((size_t)blockIdx.x * in.heads + head) * dk * dv;
+    ret_stage_rows<true>(in, c, head, dkp, vec, [&](bool is_q, int t, int d, const float4& v) { ret_put4((is_q ? qs : ks) + t * kstride + d, v); });
     ret_stage_values(in, c, head, vs, vstride, cols, vec);
+    if (c.start > 0) ret_stage_state(in, S, 0, min(slice, dkp), sh, sr, vstride, cols, vec);      // (else S is zero)
     for (int i = tid; i <= kC; i += blockDim.x) pw[i] = in.powers[(size_t)head * (kC + 1) + i];
     const int lane = tid & 31, warp = tid >> 5, wr = warp & 3, wc = warp >> 2;
     const int lrow = lane & 7, lmat = lane >> 3, quad = lane >> 2, pair = (lane & 3) * 2;
     const int r0 = wr * 16 + quad, r1 = r0 + 8;        // this thread's two rows of the chunk
-    float acc[8][4];
+    float acc[NV][4];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    for (int j = 0; j < NV; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
     const unsigned qa = ret_smem(qs) + (unsigned)(((wr * 16 + lrow + (lmat & 1) * 8) * kstride + (lmat >> 1) * 8) * 2);
-    const unsigned vo = (unsigned)((((lmat & 1) * 8 + lrow) * vstride + wc * 64 + (lmat >> 1) * 8) * 2);
-    if (c.start > 0) {                                 // (else S is zero)
-        const float* S = kv + ((size_t)blockIdx.x * in.heads + head) * dk * dv;
-        const int vquads = cols / 4;
+    const unsigned vo = (unsigned)((((lmat & 1) * 8 + lrow) * vstride + wc * 8 * NV + (lmat >> 1) * 8) * 2);
+    __syncthreads();
+    if (c.start > 0) {
         for (int s0 = 0; s0 < dkp; s0 += slice) {
             const int m = min(slice, dkp - s0);
-            __syncthreads();
-            for (int idx = tid; idx < m * vquads; idx += blockDim.x) {
-                const int r = idx / vquads, d = (idx % vquads) * 4;
-                float v[4] = {0.f, 0.f, 0.f, 0.f};
-                if (s0 + r < dk) {
-                    const float* src = S + (size_t)(s0 + r) * dv + d;
-                    if (vec) {
-                        if (d < dv) {
-                            const float4 f = *reinterpret_cast<const float4*>(src);
-                            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-                        }
-                    } else {
-#pragma unroll
-                        for (int e = 0; e < 4; ++e)
-                            if (d + e < dv) v[e] = src[e];
-                    }
-                }
-                uint32_t h0, h1, x0, x1;
-                ret_split(v[0], v[1], h0, x0);
-                ret_split(v[2], v[3], h1, x1);
-                *reinterpret_cast<uint2*>(sh + r * vstride + d) = make_uint2(h0, h1);
-                *reinterpret_cast<uint2*>(sr + r * vstride + d) = make_uint2(x0, x1);
+            if (s0 > 0) {
+                __syncthreads();
+                ret_stage_state(in, S, s0, m, sh, sr, vstride, cols, vec);
+                __syncthreads();
             }
-            __syncthreads();
             for (int kk = 0; kk < m; kk += 16) {
                 uint32_t a[4], b[4];
                 ret_ldsm(a, qa + (s0 + kk) * 2);
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
+                for (int j = 0; j < NV / 2; ++j) {
                     ret_ldsm_t(b, ret_smem(sh) + vo + (kk * vstride + 16 * j) * 2);
                     ret_mma(acc[2 * j], a, b[0], b[1]);
                     ret_mma(acc[2 * j + 1], a, b[2], b[3]);
@@ -548,57 +628,50 @@ __global__ void __launch_bounds__(32 * WARPS) retention_chunk_out_kernel(RetIn i
         }
         const float w0 = pw[r0 + 1], w1 = pw[r1 + 1];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+        for (int j = 0; j < NV; ++j) {
             acc[j][0] *= w0; acc[j][1] *= w0;
             acc[j][2] *= w1; acc[j][3] *= w1;
         }
-    } else {
-        __syncthreads();
     }
-    // the chunk's own tokens: (q_t . k_s) a^(t - s), then times the values
-    float s[8][4];
-#pragma unroll
-    for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+    // the chunk's own tokens, 16 keys at a time: (q_t . k_s) a^(t - s), then times the values; keys behind every row of the warp
+    // are passed by
     const unsigned ka = ret_smem(ks) + (unsigned)(((lrow + (lmat >> 1) * 8) * kstride + (lmat & 1) * 8) * 2);
-    for (int kk = 0; kk < dkp; kk += 16) {
-        uint32_t a[4], b[4];
-        ret_ldsm(a, qa + kk * 2);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            if (j > wr) break;                         // keys behind every row of the warp
-            ret_ldsm(b, ka + (16 * j * kstride + kk) * 2);
-            ret_mma(s[2 * j], a, b[0], b[1]);
-            ret_mma(s[2 * j + 1], a, b[2], b[3]);
-        }
-    }
-#pragma unroll
-    for (int j = 0; j < 8; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int back = (e < 2 ? r0 : r1) - (8 * j + pair + (e & 1));
-            s[j][e] = back >= 0 ? s[j][e] * pw[back] : 0.f;
+#pragma unroll 1
+    for (int j16 = 0; j16 <= wr; ++j16) {
+        float s[2][4];
+        s[0][0] = s[0][1] = s[0][2] = s[0][3] = s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.f;
+        for (int kk = 0; kk < dkp; kk += 16) {
+            uint32_t a[4], b[4];
+            ret_ldsm(a, qa + kk * 2);
+            ret_ldsm(b, ka + (16 * j16 * kstride + kk) * 2);
+            ret_mma(s[0], a, b[0], b[1]);
+            ret_mma(s[1], a, b[2], b[3]);
         }
 #pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-        if (kk > wr) break;
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int back = (e < 2 ? r0 : r1) - (16 * j16 + 8 * j + pair + (e & 1));
+                s[j][e] = back >= 0 ? s[j][e] * pw[back] : 0.f;
+            }
         uint32_t ah[4], ar[4], b[4];
-        ret_split(s[2 * kk][0], s[2 * kk][1], ah[0], ar[0]);
-        ret_split(s[2 * kk][2], s[2 * kk][3], ah[1], ar[1]);
-        ret_split(s[2 * kk + 1][0], s[2 * kk + 1][1], ah[2], ar[2]);
-        ret_split(s[2 * kk + 1][2], s[2 * kk + 1][3], ah[3], ar[3]);
+        ret_split(s[0][0], s[0][1], ah[0], ar[0]);
+        ret_split(s[0][2], s[0][3], ah[1], ar[1]);
+        ret_split(s[1][0], s[1][1], ah[2], ar[2]);
+        ret_split(s[1][2], s[1][3], ah[3], ar[3]);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            ret_ldsm_t(b, ret_smem(vs) + vo + (16 * kk * vstride + 16 * j) * 2);
+        for (int j = 0; j < NV / 2; ++j) {
+            ret_ldsm_t(b, ret_smem(vs) + vo + (16 * j16 * vstride + 16 * j) * 2);
             ret_mma(acc[2 * j], ah, b[0], b[1]);
             ret_mma(acc[2 * j + 1], ah, b[2], b[3]);
             ret_mma(acc[2 * j], ar, b[0], b[1]);
             ret_mma(acc[2 * j + 1], ar, b[2], b[3]);
         }
     }
-    // the norm over the head's lanes: this warp's 64 of them, then the other warps' of the same rows
+    // the norm over the head's lanes: this warp's of them, then the other warps' of the same rows
     float q0 = 0.f, q1 = 0.f;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
+    for (int j = 0; j < NV; ++j) {
         q0 += acc[j][0] * acc[j][0] + acc[j][1] * acc[j][1];
         q1 += acc[j][2] * acc[j][2] + acc[j][3] * acc[j][3];
     }
@@ -611,7 +684,7 @@ __global__ void __launch_bounds__(32 * WARPS) retention_chunk_out_kernel(RetIn i
         ssq[wc][r1] = q1;
     }
     __syncthreads();
-    const int n_wc = cols / 64;
+    const int n_wc = WARPS / 4;
     const bool two = dv % 2 == 0 && out_stride % 2 == 0 && ((size_t)out & 3) == 0 && vec;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
@@ -623,8 +696,8 @@ __global__ void __launch_bounds__(32 * WARPS) retention_chunk_out_kernel(RetIn i
         const float* gate = in.proj + (size_t)(c.first_row + r) * in.stride + 2 * in.heads * dk + (in.heads + head) * dv;
         __nv_bfloat16* o = out + (size_t)(c.first_row + r) * out_stride + (size_t)head * dv;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const int d = wc * 64 + 8 * j + pair;
+        for (int j = 0; j < NV; ++j) {
+            const int d = wc * 8 * NV + 8 * j + pair;
             if (d >= dv) continue;
             const float x0 = acc[j][2 * half] * inv, x1 = acc[j][2 * half + 1] * inv;
             if (two) {
@@ -704,7 +777,9 @@ BLM_API int blm_retention_step(RET_ARGS, const int* token_seq, const int* token_
     BLM_REQUIRE(dv / n <= kStepThreads, "retention_step: values of %d lanes", dv);
     const size_t smem = ((size_t)2 * ((dk + 3) & ~3) + 36 + (size_t)(kStepThreads / (dv / n)) * dv) * sizeof(float);
     const dim3 grid(heads, n_tokens);
-#define RET_STEP(TO, N) retention_step_kernel<TO, N><<<grid, kStepThreads, smem, stream>>>(in, sq, token_seq, token_pos, eps, (TO*)out, out_stride, vec)
+    const bool few = dk <= 4 * (kStepThreads / (dv / n));
+#define RET_STEP_OF(TO, N, A) retention_step_kernel<TO, N, A><<<grid, kStepThreads, smem, stream>>>(in, sq, token_seq, token_pos, eps, (TO*)out, out_stride, vec)
+#define RET_STEP(TO, N) do { if (few) RET_STEP_OF(TO, N, 4); else RET_STEP_OF(TO, N, 8); } while (0)
     if (out_dtype == BLM_BF16) {
         if (vec) RET_STEP(__nv_bfloat16, 4); else RET_STEP(__nv_bfloat16, 1);
     } else if (out_dtype == BLM_F32) {
@@ -713,6 +788,7 @@ BLM_API int blm_retention_step(RET_ARGS, const int* token_seq, const int* token_
         return blm_fail(BLM_BAD_ARGUMENT, "retention_step: dtype %d", out_dtype);
     }
 #undef RET_STEP
+#undef RET_STEP_OF
     return blm_check_launch("retention_step");
 }
 
@@ -733,20 +809,17 @@ BLM_API int blm_retention_portions(RET_ARGS, int n_tokens, float eps, float* kv,
     const dim3 grid(chunks, heads);
     retention_chunk_add_kernel<<<grid, 256, smem1, stream>>>(in, sq, kv, vec);
     const size_t size = (size_t)dk * dv;
-    const bool four = size % 4 == 0 && (((size_t)state) & 15) == 0 && slot_stride % 4 == 0 && copy_stride % 4 == 0 && offset % 4 == 0;
-    if (four) retention_carry_kernel<4><<<dim3((unsigned)((size / 4 + 255) / 256), heads, n_seqs), 256, 0, stream>>>(in, sq, kv);
-    else retention_carry_kernel<1><<<dim3((unsigned)((size + 255) / 256), heads, n_seqs), 256, 0, stream>>>(in, sq, kv);
-    const int warps = 4 * ((dv + 63) / 64);
-    auto rows = [&](auto kernel) -> int {
+    retention_carry_kernel<<<dim3((unsigned)((size + 255) / 256), heads, n_seqs), 256, 0, stream>>>(in, sq, kv);
+    auto rows = [&](auto kernel, int threads) -> int {
         if (smem3 > 48 * 1024) {
             cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
             if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "retention_portions: %s", cudaGetErrorString(e));
         }
-        kernel<<<grid, 32 * warps, smem3, stream>>>(in, sq, kv, slice, eps, (__nv_bfloat16*)out, out_stride, n_tokens, vec);
+        kernel<<<grid, threads, smem3, stream>>>(in, sq, kv, slice, eps, (__nv_bfloat16*)out, out_stride, n_tokens, vec);
         return blm_check_launch("retention_portions");
     };
-    if (warps <= 4) return rows(retention_chunk_out_kernel<4>);
-    if (warps <= 8) return rows(retention_chunk_out_kernel<8>);
-    if (warps <= 16) return rows(retention_chunk_out_kernel<16>);
-    return rows(retention_chunk_out_kernel<32>);
+    if (dv <= 64) return rows(retention_chunk_out_kernel<8, 4>, 256);
+    if (dv <= 128) return rows(retention_chunk_out_kernel<16, 4>, 512);
+    if (dv <= 256) return rows(retention_chunk_out_kernel<16, 8>, 512);
+    return rows(retention_chunk_out_kernel<32, 8>, 1024);
 }

@@ -665,7 +665,7 @@ def _moe_experts_tc(h, ids, weights, up, down, extra, out_dtype, unit=UNIT_GELU,
     places = tiles * MOE_TC_ROWS
     place_of = torch.empty(pairs, dtype=torch.int32, device=dev)
     pair_of_place = torch.empty(places, dtype=torch.int32, device=dev)
-    tile_expert = torch.empty(tiles, dtype=torch.int32, device=dev)
+    tile_expert = torch.empty(tiles + 1, dtype=torch.int32, device=dev)      # and how many tiles have an expert
     xs = torch.empty((places, d), dtype=torch.bfloat16, device=dev)
     act = torch.empty((places, ff), dtype=torch.bfloat16, device=dev)
     y = torch.empty((places, d), dtype=torch.float32, device=dev)
