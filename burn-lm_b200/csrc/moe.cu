@@ -23,45 +23,79 @@
 BLM_API const char* blm_moe_last_error() { return g_blm_error; }
 
 // ---------------------------------------------------------------------------------------------
-// router: one block per token
+// router: a block per TOK tokens (several where there are many: the router's rows are then read once for all of them; the sums
+// are the same).  The logits are dot products of a warp each; then a warp a token makes the scores and the choice.
 // ---------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, int TOK>
 __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, int width, int n_experts, int top,
                                  int* __restrict__ ids, float* __restrict__ weights, int scores, const float* __restrict__ bias,
-                                 const float* __restrict__ correction, int renorm, int n_groups, int keep_groups) {
+                                 const float* __restrict__ correction, int renorm, int n_groups, int keep_groups, int n_tokens) {
     const bool softmax = scores == 1, by_logit = scores == 2;      // else sigmoids
     extern __shared__ __align__(16) float smem[];
-    float* x = smem;                     // [width]
-    float* score = smem + width;         // [n_experts]: what a chosen expert is weighted by
-    float* choice = score + n_experts;   // [n_experts]: what the choice looks at (the score, plus the correction)
-    float* mark = choice + n_experts;    // [n_groups]: the groups' marks
-    const int n = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
-    for (int d = threadIdx.x; d < width; d += blockDim.x) x[d] = to_f32(h[(size_t)n * width + d]);
+    const int first_token = blockIdx.x * TOK, live = min(TOK, n_tokens - first_token);
+    float* x = smem;                     // [TOK][width]
+    float* marks = smem + (size_t)TOK * width;           // a token's [n_experts] scores, [n_experts] choices, [n_groups] marks
+    const int per_token = 2 * n_experts + n_groups;
+    const T* rows = h + (size_t)first_token * width;
+    if (sizeof(T) == 2 && (width & 7) == 0 && ((size_t)h & 15) == 0) {
+        for (int i = threadIdx.x; i < live * (width / 8); i += blockDim.x) {
+            const uint4 raw = reinterpret_cast<const uint4*>(rows)[i];
+            const __nv_bfloat162* two = reinterpret_cast<const __nv_bfloat162*>(&raw);
+            const float2 a = __bfloat1622float2(two[0]), b = __bfloat1622float2(two[1]), c = __bfloat1622float2(two[2]), d = __bfloat1622float2(two[3]);
+            reinterpret_cast<float4*>(x)[2 * i] = make_float4(a.x, a.y, b.x, b.y);
+            reinterpret_cast<float4*>(x)[2 * i + 1] = make_float4(c.x, c.y, d.x, d.y);
+        }
+    } else {
+        for (int d = threadIdx.x; d < live * width; d += blockDim.x) x[d] = to_f32(rows[d]);
+    }
+    if (TOK > 1)
+        for (int d = live * width + threadIdx.x; d < TOK * width; d += blockDim.x) x[d] = 0.f;
     __syncthreads();
     for (int e = warp; e < n_experts; e += n_warps) {
         const float* w = router + (size_t)e * width;
-        float z = 0.f;
+        float z[TOK];
         if ((width & 127) == 0) {            // four loads of 16 bytes on their way at once, four sums: the loop waits for memory, not for itself
             const float4* w4 = reinterpret_cast<const float4*>(w);
             const float4* x4 = reinterpret_cast<const float4*>(x);
-            float z0 = 0.f, z1 = 0.f, z2 = 0.f, z3 = 0.f;
+            float z4[TOK][4];
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) z4[t][0] = z4[t][1] = z4[t][2] = z4[t][3] = 0.f;
 #pragma unroll 8
             for (int d = lane; d < width / 4; d += 32) {
-                const float4 a = __ldg(w4 + d), c = x4[d];
-                z0 = fmaf(a.x, c.x, z0); z1 = fmaf(a.y, c.y, z1); z2 = fmaf(a.z, c.z, z2); z3 = fmaf(a.w, c.w, z3);
+                const float4 a = __ldg(w4 + d);
+#pragma unroll
+                for (int t = 0; t < TOK; ++t) {
+                    const float4 c = x4[t * (width / 4) + d];
+                    z4[t][0] = fmaf(a.x, c.x, z4[t][0]); z4[t][1] = fmaf(a.y, c.y, z4[t][1]);
+                    z4[t][2] = fmaf(a.z, c.z, z4[t][2]); z4[t][3] = fmaf(a.w, c.w, z4[t][3]);
+                }
             }
-            z = (z0 + z1) + (z2 + z3);
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) z[t] = (z4[t][0] + z4[t][1]) + (z4[t][2] + z4[t][3]);
         } else {
-            for (int d = lane; d < width; d += 32) z = fmaf(w[d], x[d], z);
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) z[t] = 0.f;
+            for (int d = lane; d < width; d += 32) {
+                const float a = w[d];
+#pragma unroll
+                for (int t = 0; t < TOK; ++t) z[t] = fmaf(a, x[t * width + d], z[t]);
+            }
         }
-        z = warp_sum(z);
-        if (bias) z += bias[e];
-        // (a row of no sequence may hold anything, a NaN too: its score is 0, so that it still names experts that exist)
-        if (lane == 0) score[e] = softmax || by_logit ? (z == z ? z : 0.f) : (z == z ? 1.0f / (1.0f + expf(-z)) : 0.f);
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) {
+            float v = warp_sum(z[t]);
+            if (bias) v += bias[e];
+            // (a row of no sequence may hold anything, a NaN too: its score is 0, so that it still names experts that exist)
+            if (lane == 0) marks[t * per_token + e] = softmax || by_logit ? (v == v ? v : 0.f) : (v == v ? 1.0f / (1.0f + expf(-v)) : 0.f);
+        }
     }
     __syncthreads();
-    if (warp == 0) {
+    if (warp < live) {
+        const int n = first_token + warp;
+        float* score = marks + warp * per_token;         // [n_experts]: what a chosen expert is weighted by
+        float* choice = score + n_experts;               // [n_experts]: what the choice looks at (the score, plus the correction)
+        float* mark = choice + n_experts;                // [n_groups]: the groups' marks
         if (softmax) {
             float m = -INFINITY;
             for (int e = lane; e < n_experts; e += 32) m = fmaxf(m, score[e]);
@@ -145,19 +179,25 @@ BLM_API int blm_moe_route(const void* h, int dtype, const float* router, int n_t
     BLM_REQUIRE(n_experts % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups &&
                 (long long)keep_groups * (n_experts / n_groups) >= top,
                 "moe_route: %d experts in %d groups of which %d are kept, for %d chosen", n_experts, n_groups, keep_groups, top);
-    const size_t smem = ((size_t)width + 2 * n_experts + n_groups) * sizeof(float);
-    BLM_REQUIRE(smem <= 48 * 1024, "moe_route: width %d and %d experts need %zu bytes of shared memory", width, n_experts, smem);
+    const size_t one = ((size_t)width + 2 * n_experts + n_groups) * sizeof(float);
+    BLM_REQUIRE(one <= 200 * 1024, "moe_route: width %d and %d experts need %zu bytes of shared memory", width, n_experts, one);
+    const bool many = n_tokens >= 4 * blm_sm_count() && 4 * one <= 100 * 1024;
+    const size_t smem = many ? 4 * one : one;
     // a warp an expert where the experts are few (the warps' dot products wait for memory side by side), sixteen warps at most
-    const int threads = n_experts <= 4 ? 128 : (n_experts >= 16 ? 512 : 32 * n_experts);
-    if (dtype == BLM_F32)
-        moe_route_kernel<float><<<n_tokens, threads, smem, stream>>>((const float*)h, router, width, n_experts, top, ids, weights, scores, bias,
-                                                                 correction, renorm, n_groups, keep_groups);
-    else if (dtype == BLM_BF16)
-        moe_route_kernel<__nv_bfloat16><<<n_tokens, threads, smem, stream>>>((const __nv_bfloat16*)h, router, width, n_experts, top, ids,
-                                                                         weights, scores, bias, correction, renorm, n_groups, keep_groups);
-    else
-        return blm_fail(BLM_BAD_ARGUMENT, "moe_route: dtype %d", dtype);
-    return blm_check_launch("moe_route");
+    const int threads = many || n_experts <= 4 ? (many ? 256 : 128) : (n_experts >= 16 ? 512 : 32 * n_experts);
+    auto launch = [&](auto kernel, auto* rows) -> int {
+        if (smem > 48 * 1024) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return blm_fail(BLM_CUDA_ERROR, "moe_route: %s", cudaGetErrorString(e));
+        }
+        kernel<<<many ? (n_tokens + 3) / 4 : n_tokens, threads, smem, stream>>>(rows, router, width, n_experts, top, ids, weights, scores, bias,
+                                                                                correction, renorm, n_groups, keep_groups, n_tokens);
+        return blm_check_launch("moe_route");
+    };
+    if (dtype == BLM_F32) return many ? launch(moe_route_kernel<float, 4>, (const float*)h) : launch(moe_route_kernel<float, 1>, (const float*)h);
+    if (dtype == BLM_BF16)
+        return many ? launch(moe_route_kernel<__nv_bfloat16, 4>, (const __nv_bfloat16*)h) : launch(moe_route_kernel<__nv_bfloat16, 1>, (const __nv_bfloat16*)h);
+    return blm_fail(BLM_BAD_ARGUMENT, "moe_route: dtype %d", dtype);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -1113,6 +1153,18 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
                                    const T* __restrict__ extra, TO* __restrict__ out, int width, int top, int scale_output, int n_planes,
                                    long long plane) {
     const int n = blockIdx.x;
+    if (n_planes == 1 && extra == nullptr && sizeof(TO) == 4 && (width & 3) == 0) {       // four lanes a thread
+        for (int d = (blockIdx.y * blockDim.x + threadIdx.x) * 4; d < width; d += gridDim.y * blockDim.x * 4) {
+            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int k = 0; k < top; ++k) {
+                const float4 v = *reinterpret_cast<const float4*>(y + (size_t)place_of[(size_t)n * top + k] * width + d);
+                const float w = scale_output ? weights[(size_t)n * top + k] : 1.f;
+                s.x += w * v.x; s.y += w * v.y; s.z += w * v.z; s.w += w * v.w;
+            }
+            *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + (size_t)n * width + d) = s;
+        }
+        return;
+    }
     for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < width; d += gridDim.y * blockDim.x) {
         float s = 0.f;
         for (int k = 0; k < top; ++k) {
