@@ -1007,6 +1007,7 @@ def samusun_kernels(z, pk):
     from burn_lm_b200.parts.normed_attention import STREAM_PAGES
     from burn_lm_b200.parts.linear import Linear
     dev, bf, f32 = "cuda", torch.bfloat16, torch.float32
+    torch.manual_seed(0)          # (how evenly the experts are chosen decides how full their tiles are)
     H, G, hd, d, W, inner = z["heads"], z["kv"], z["hd"], z["width"], z["window"], z["inner"]
     out = {}
     i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)

@@ -57,8 +57,8 @@ __device__ __forceinline__ float2 ret_turn(const RetIn& in, int pos, int i) {
 __device__ __forceinline__ void ret_turn4(const RetIn& in, int pos, int i, float4& lo, float4& hi) {
     if (pos < in.table_len) {
         const float4* t = reinterpret_cast<const float4*>(in.table + (size_t)pos * (in.rot >> 1) + i);
-        lo = t[0];
-        hi = t[1];
+        lo = __ldg(t);
+        hi = __ldg(t + 1);
         return;
     }
     float2 a = ret_angle((double)pos * in.freq[i]), b = ret_angle((double)pos * in.freq[i + 1]);
@@ -370,7 +370,7 @@ __device__ __forceinline__ void ret_stage_values(const RetIn& in, const RetChunk
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
                 const int r = t + u * sh.step;
-                v[u] = r < c.rows && d < in.dv ? *reinterpret_cast<const float4*>(src + (size_t)r * in.stride + d) : ret_zero4();
+                v[u] = r < c.rows && d < in.dv ? __ldg(reinterpret_cast<const float4*>(src + (size_t)r * in.stride + d)) : ret_zero4();
             }
 #pragma unroll
             for (int u = 0; u < 4; ++u)
@@ -403,11 +403,11 @@ __device__ __forceinline__ void ret_stage_rows(const RetIn& in, const RetChunk& 
                 const int t = t0 + u * sh.step;
                 const bool there = t < c.rows && d < in.dk;
                 const size_t at = (size_t)t * in.stride + d;
-                k[u][0] = there ? *reinterpret_cast<const float4*>(kp + at) : ret_zero4();
-                k[u][1] = there && turns ? *reinterpret_cast<const float4*>(kp + at + half) : ret_zero4();
+                k[u][0] = there ? __ldg(reinterpret_cast<const float4*>(kp + at)) : ret_zero4();
+                k[u][1] = there && turns ? __ldg(reinterpret_cast<const float4*>(kp + at + half)) : ret_zero4();
                 if (QUERIES) {
-                    q[u][0] = there ? *reinterpret_cast<const float4*>(qp + at) : ret_zero4();
-                    q[u][1] = there && turns ? *reinterpret_cast<const float4*>(qp + at + half) : ret_zero4();
+                    q[u][0] = there ? __ldg(reinterpret_cast<const float4*>(qp + at)) : ret_zero4();
+                    q[u][1] = there && turns ? __ldg(reinterpret_cast<const float4*>(qp + at + half)) : ret_zero4();
                 }
                 if (there && turns) ret_turn4(in, c.start + t, d, lo[u], hi[u]);
                 else lo[u] = hi[u] = make_float4(1.f, 0.f, 1.f, 0.f);
@@ -458,7 +458,7 @@ __device__ __forceinline__ void ret_stage_state(const RetIn& in, const float* S,
             if (r >= m || s0 + r >= in.dk || d >= in.dv) continue;
             const float* src = S + (size_t)(s0 + r) * in.dv + d;
             if (vec) {
-                v[u] = *reinterpret_cast<const float4*>(src);
+                v[u] = __ldg(reinterpret_cast<const float4*>(src));
             } else {
                 v[u].x = src[0];
                 if (d + 1 < in.dv) v[u].y = src[1];
@@ -539,7 +539,7 @@ __global__ void __launch_bounds__(256) retention_chunk_add_kernel(RetIn in, RetS
 }
 
 // (2) S in front of every chunk, in place of what the chunk adds; S behind the last one goes to the sequence's state
-__global__ void __launch_bounds__(256, 6) retention_carry_kernel(RetIn in, RetSeq sq, float* __restrict__ kv) {
+__global__ void __launch_bounds__(256) retention_carry_kernel(RetIn in, RetSeq sq, float* __restrict__ kv) {
     const int head = blockIdx.y, seq = blockIdx.z;
     const size_t size = (size_t)in.dk * in.dv, at = (size_t)blockIdx.x * 256 + threadIdx.x;
     const int len = sq.cu_seqlens[seq + 1] - sq.cu_seqlens[seq];
@@ -552,7 +552,7 @@ __global__ void __launch_bounds__(256, 6) retention_carry_kernel(RetIn in, RetSe
     const float full = powers[kC], last = powers[len - (n_chunks - 1) * kC];
     const size_t step = (size_t)in.heads * size;
     float* p = kv + (size_t)first * step + (size_t)head * size + at;
-    constexpr int kRead = 8;                           // chunks read ahead of their turn
+    constexpr int kRead = 16;                          // chunks read ahead of their turn
     for (int c0 = 0; c0 < n_chunks; c0 += kRead) {
         float add[kRead];
 #pragma unroll
