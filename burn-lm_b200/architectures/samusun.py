@@ -2,7 +2,7 @@
 
 A scaled token embedding; layers whose mixer and feed-forward read one norm's output side by side; a mixer per layer that is
 attention over a sliding window in which the keys are their own values (biased projections, no rotation, a bias by distance per
-head, queries scaled by a number that grows with their position), or retention (linear attention with a fixed decay per head,
+head, queries scaled by a number that grows with their position), or retention (a matrix of decayed key-value products per head,
 rotated queries and keys, a norm and a gate on every head's output); a dense gated feed-forward, a mixture of gated experts
 whose weights are softmax scores over all experts as they are, or none; a last norm, the output projection, scaled and capped
 logits.  A span of the layers may run several times in a row with the same weights, every pass with a cache line or state of

@@ -36,7 +36,7 @@ class SharedAttentionConfig:
     kv_heads: int
     dim: int            # lanes of a head's query, key and value
     scale: float
-    window: Optional[int] = None             # a position sees itself and the window - 1 tokens before it
+    window: Optional[int] = None             # how many of the latest keys, its own included, a position sees
     q_temp: Optional[TemperatureConfig] = None
 
 

@@ -1,4 +1,4 @@
-// Retention: linear attention with one fixed decay per head over the packed tokens of a step.  Per head,
+// Retention over the packed tokens of a step.  Per head, with a decay a of its own,
 //   S_t = a S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   out = o / sqrt(mean(o^2) + eps) * silu(g)      (S: dk x dv)
 // with q and k turned by their position and k scaled first.  A row of the projection holds [q | k | v | g], float32.
 //

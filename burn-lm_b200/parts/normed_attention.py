@@ -12,7 +12,7 @@ position i sees j <= i, or only 0 <= i - j < window, or only the j of its own ch
 sum exp(s_j)) with `sink` one more entry of score 0 that carries no value.  With `output_gate` every lane of the heads' outputs
 is multiplied by sigmoid(Wg h).  The heads' outputs are concatenated and projected by Wo (plus a bias with `output_bias`).
 
-`values_are_keys`: v is k as projected (bias included); there is no Wv and the cache keeps one line for both.
+`values_are_keys`: one projection (with its bias) serves as key and as value, Wv does not exist and the cache keeps one line.
 `query_temperature` (coef, every): q is multiplied by 1 + coef ln(floor((position + 1) / every) + 1).  `slopes` (a number per
 query head): slope_h * (i - j) is taken off a score, after the cap.
 

@@ -1,9 +1,9 @@
-"""The retention mixer: linear attention with one fixed decay per head, no softmax and no denominator.
+"""The retention mixer: a matrix of decayed key-value products per head, read by the query; nothing is normalised over the keys.
 
 q = Wq h and k = Wk h (heads x key_dim), v = Wv h (heads x value_dim), without biases.  The first `rotary_dims` lanes of every q
 and k head turn by position * base^(-2i / rotary_dims), lanes (i, i + rotary_dims / 2) together; then k is multiplied by
-key_dim^(-1/2).  Per head, S [key_dim x value_dim]: S <- decay_h S + k v^T, o = S^T q.  Every head's o is divided by its root mean
-square (no weight), the heads are concatenated, multiplied by silu(Wg h) and projected by Wo.
+key_dim^(-1/2).  Per head, S [key_dim x value_dim] with a decay of its own that no token changes: S <- decay_h S + k v^T,
+o = S^T q.  y = Wo (silu(Wg h) * [o_1 / rms(o_1); o_2 / rms(o_2); ...]), the unit norms without a weight.
 
 The four projections run as one product with a fused [q; k; v; g] weight whose result stays in fp32.  S is fp32 and carried per
 sequence, two copies by position as the other recurrences'.  In bfloat16, single tokens run one kernel from the projection to the

@@ -67,7 +67,7 @@ def slopes(n_heads):
 
 
 def sliding_window(T, size):
-    """[T, T]: position i sees itself and the size - 1 before it."""
+    """[T, T]: which of the keys j a query i sees: the latest `size` up to its own."""
     i = np.arange(T)
     back = i[:, None] - i[None, :]
     return (back >= 0) & (back < size)
@@ -107,7 +107,7 @@ def attention(h, w, m):
 # retention
 # --------------------------------------------------------------------------------------------
 def rotate_halves(x, positions, dims, base):
-    """x [T, ..., d]: lanes i and i + dims / 2 turn together by position * base^(-2i / dims); lanes from dims on pass."""
+    """x [T, ..., d]: a turn of lanes (i, i + dims / 2) by position * base^(-2i / dims); lanes from dims on stay."""
     if dims == 0:
         return x.copy()
     half = dims // 2
